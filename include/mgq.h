@@ -31,6 +31,7 @@ extern "C" {
 #define MGQ_FMT_F16 1
 #define MGQ_FMT_Q4  2
 #define MGQ_FMT_Q8  3
+#define MGQ_FMT_BF16 4      /* bf16 linear weights, caches and operands (no reference counterpart) */
 
 /* Activation dtype of the A operand. */
 #define MGQ_A_F32  0
@@ -77,6 +78,10 @@ const char *mgq_version(void);
  *                               src/optimize.rs:776-879), 2 every such group, e.g. q|k|v (default)
  *   "session.fuse_rope_cache"   1 (default): RoPE(q), RoPE(k), CacheWrite(k), CacheWrite(v) of a decode
  *                               layer run as one launch; 0: four dispatches like the reference
+ *   "session.fuse_mixer"        1 (default): in graphs with bf16 linear layers biases, residual adds, clamped
+ *                               GLUs, head gates and row picks run inside their producers, and independent
+ *                               linear layers of one K as one launch; 0: one launch per node
+ *   "linear.force_tiled"        1: bf16 linear layers never use the tcgen05 kernel
  *   "session.fuse_exchange"     1 (default): in a column-sharded session a single-row GEMV whose output
  *                               feeds an all_gather stores its columns into the ranks' gathered vectors
  *                               itself; 0: the all_gather does */
@@ -359,6 +364,20 @@ typedef struct mgq_session mgq_session;
 #define MGQ_SHADER_ROPE_CACHE_WRITE  12   /* RoPEDynamic x2 + CacheWrite x2 merged (no reference entry) */
 #define MGQ_SHADER_ALL_GATHER        13   /* column-sharded sessions: slice -> whole vector over peer memory (no reference entry) */
 #define MGQ_SHADER_MATMUL_GEMV_BT    14
+/* operators of decoders with recurrent and latent-attention mixers (no reference entries) */
+#define MGQ_SHADER_LINEAR            15   /* one or several bf16 linear layers (+ bias, + addend) in one launch */
+#define MGQ_SHADER_LINEAR_GLU        16   /* gate and up layers with the clamped GLU as epilogue */
+#define MGQ_SHADER_BIAS_ADD          17
+#define MGQ_SHADER_PICK_ROWS         18
+#define MGQ_SHADER_NORM              19
+#define MGQ_SHADER_TOKEN_SHIFT       20
+#define MGQ_SHADER_DECAY             21
+#define MGQ_SHADER_WKV               22   /* alone, or with the decay and head gate around it */
+#define MGQ_SHADER_MLSTM             23   /* alone, or with the head gate behind it */
+#define MGQ_SHADER_HEAD_GATE         24
+#define MGQ_SHADER_LATENT_CACHE_WRITE 25
+#define MGQ_SHADER_LATENT_ATTENTION  26   /* alone, or with the output gate behind it */
+#define MGQ_SHADER_CLAMPED_GLU       27
 
 mgq_graph *mgq_graph_new(void);
 void mgq_graph_free(mgq_graph *g);
@@ -396,6 +415,61 @@ int mgq_graph_all_gather(mgq_graph *g, int x, uint32_t world);
 /* Columns [first, first + count) of a [1, n] f32 node, without a copy (first % 4 == 0): the part of
  * a whole vector that belongs to this rank, e.g. the residual a sharded projection adds to. */
 int mgq_graph_slice_columns(mgq_graph *g, int x, uint32_t first, uint32_t count);
+
+/* ---- row-dynamic graphs and the operators of decoders with recurrent and latent-attention mixers
+ * (no reference counterpart).
+ *
+ * mgq_graph_input_u32_rows declares a u32 input of up to `capacity` rows whose count is set per step
+ * (mgq_session_set_rows): MGQ_ROWS_TOKENS for the tokens of a step, MGQ_ROWS_PICKED for the rows whose
+ * logits are wanted (may be 0: everything behind the pick is then skipped).  Nodes computed from it
+ * have `capacity` as leading dimension and run with the current count.
+ *
+ * Operand dtype: MGQ_FMT_F32, or MGQ_FMT_BF16 for the activations that only feed bf16 linear layers.
+ *
+ * matmul_bt with a parameter_bf16 [N, K]  linear layer, any number of rows, f32 accumulation and output
+ * bias_add            x[r, c] + bias[c]
+ * embedding_scaled    table[id] * scale, table f32 or bf16
+ * pick_rows           x[index[r], :]
+ * norm                x / sqrt(mean(x^2) + eps) * (weight_offset + weight)
+ * clamped_glu         g = min(gate, limit), u = clamp(up, +-limit): g sigmoid(alpha g) (u + 1)
+ * token_shift         `count` mixes h_t + (h_(t-1) - h_t) * mu_i as a [count, rows, width] node (take one
+ *                     with slot); state: zero-filled f32 parameter [2, width], row 0 the previous
+ *                     portion's last h, row 1 the pending one that wkv commits
+ * lora_decay          exp(-exp(tanh(low) . w2^T + w0)), low [rows, rank], w2 bf16 [channels, rank]
+ * wkv                 per head: o_t = (S + diag(u) k_t v_t^T)^T r_t, then S = diag(w_t) S + k_t v_t^T;
+ *                     state: f32 parameter of mgq_wkv_state_elements
+ * mlstm               matrix memory with running maximum m (zero at the start), capped log gates
+ *                     i = cap tanh(gate_i / cap), f = logsigmoid(cap tanh(gate_f / cap)), q scaled by
+ *                     dim^-1/2, o = S^T q / (max(|n . q|, exp(-m)) + 1e-6); state: f32 parameter of
+ *                     mgq_mlstm_state_elements
+ * head_gate           per head o / rms(o) * weight * act(gate); weight -1: o * act(gate) without the norm
+ * latent_cache_write  ring cache row pos % slots = [norm(down[:rank]) * weight | rotated down[rank:]]
+ * latent_attention    softmax over the last `window` positions of
+ *                     (q_nope . W_uk c + rotate(q_rot) . k_rot) * scale, values W_uv c; q is laid out head
+ *                     by head as [dim, rot_dim]; `cache` may be the cache parameter of another layer
+ * Rotations pair dimension i with i + rot_dim / 2, angle = position * rot_base^(-2i / rot_dim). */
+#define MGQ_ROWS_TOKENS 1
+#define MGQ_ROWS_PICKED 2
+#define MGQ_GATE_SIGMOID 0
+#define MGQ_GATE_SILU    1
+int mgq_graph_input_u32_rows(mgq_graph *g, const char *name, size_t capacity, int which);
+int mgq_graph_parameter_bf16(mgq_graph *g, const char *name, const size_t *shape, size_t rank);
+int mgq_graph_embedding_scaled(mgq_graph *g, int indices, int table, float scale);
+int mgq_graph_pick_rows(mgq_graph *g, int x, int index);
+int mgq_graph_norm(mgq_graph *g, int x, int weight, float eps, float weight_offset, int out_dtype);
+int mgq_graph_bias_add(mgq_graph *g, int x, int bias);
+int mgq_graph_clamped_glu(mgq_graph *g, int gate, int up, float limit, float alpha, int out_dtype);
+int mgq_graph_token_shift(mgq_graph *g, int h, const int *mu, size_t count, int state, int out_dtype);
+int mgq_graph_slot(mgq_graph *g, int x, uint32_t index);
+size_t mgq_wkv_state_elements(uint32_t heads, uint32_t dim);
+size_t mgq_mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim);
+int mgq_graph_lora_decay(mgq_graph *g, int low, int w2, int w0);
+int mgq_graph_wkv(mgq_graph *g, int r, int k, int v, int decay, int u, int state, int shift_state, uint32_t heads);
+int mgq_graph_mlstm(mgq_graph *g, int q, int k, int v, int gate_i, int gate_f, int state, uint32_t heads, float gate_cap);
+int mgq_graph_head_gate(mgq_graph *g, int o, int weight, int gate, uint32_t heads, float eps, int act, int out_dtype);
+int mgq_graph_latent_cache_write(mgq_graph *g, int down, int weight, int cache, int pos, uint32_t rot_dim, float rot_base, float eps);
+int mgq_graph_latent_attention(mgq_graph *g, int q, int cache, int uk, int uv, int pos, uint32_t heads, uint32_t dim, uint32_t rot_dim,
+                               uint32_t vdim, uint32_t window, float scale, float rot_base);
 int mgq_graph_set_outputs(mgq_graph *g, const int *ids, size_t count);
 
 /* build_inference_session (src/train.rs:380-389): fuse, lower, allocate zero-filled buffers. */
@@ -414,6 +488,11 @@ int mgq_session_set_input(mgq_session *s, const char *name, const float *data, s
 int mgq_session_save_checkpoint(mgq_session *s, const char *path);
 int mgq_session_load_checkpoint(mgq_session *s, const char *path);
 int mgq_session_set_input_u32(mgq_session *s, const char *name, const uint32_t *data, size_t len);
+/* Row-dynamic sessions: rows of the following steps (1 of each set after the build).  A captured CUDA
+ * graph is replayed when the counts are the ones it was captured with; other steps enqueue their launches. */
+int mgq_session_set_rows(mgq_session *s, int which, uint32_t count);
+/* Clears every recurrent state and latent cache: the next step starts a new sequence. */
+int mgq_session_reset_state(mgq_session *s);
 int mgq_session_step(mgq_session *s);
 /* No reference counterpart (the reference re-records its command buffer every step,
  * src/runtime.rs:2843-2881): captures the dispatch list once into a CUDA graph; later steps replay

@@ -12,7 +12,9 @@ import os
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "csrc", "libmgq.so")
 
-FMT_F32, FMT_F16, FMT_Q4, FMT_Q8 = 0, 1, 2, 3
+FMT_F32, FMT_F16, FMT_Q4, FMT_Q8, FMT_BF16 = 0, 1, 2, 3, 4
+ROWS_TOKENS, ROWS_PICKED = 1, 2
+GATE_SIGMOID, GATE_SILU = 0, 1
 A_F32, A_BF16 = 0, 1
 GEMV_MAX_M = 16
 
@@ -107,6 +109,25 @@ SIGNATURES = {
     "mgq_graph_swiglu_concat": (_int, [_vp, _int]),
     "mgq_graph_all_gather": (_int, [_vp, _int, _u32]),
     "mgq_graph_slice_columns": (_int, [_vp, _int, _u32, _u32]),
+    "mgq_graph_input_u32_rows": (_int, [_vp, ctypes.c_char_p, _sz, _int]),
+    "mgq_graph_parameter_bf16": (_int, [_vp, ctypes.c_char_p, _szp, _sz]),
+    "mgq_graph_embedding_scaled": (_int, [_vp, _int, _int, ctypes.c_float]),
+    "mgq_graph_pick_rows": (_int, [_vp, _int, _int]),
+    "mgq_graph_norm": (_int, [_vp, _int, _int, ctypes.c_float, ctypes.c_float, _int]),
+    "mgq_graph_bias_add": (_int, [_vp, _int, _int]),
+    "mgq_graph_clamped_glu": (_int, [_vp, _int, _int, ctypes.c_float, ctypes.c_float, _int]),
+    "mgq_graph_token_shift": (_int, [_vp, _int, ctypes.POINTER(_int), _sz, _int, _int]),
+    "mgq_graph_slot": (_int, [_vp, _int, _u32]),
+    "mgq_wkv_state_elements": (_sz, [_u32, _u32]),
+    "mgq_mlstm_state_elements": (_sz, [_u32, _u32, _u32]),
+    "mgq_graph_lora_decay": (_int, [_vp, _int, _int, _int]),
+    "mgq_graph_wkv": (_int, [_vp, _int, _int, _int, _int, _int, _int, _int, _u32]),
+    "mgq_graph_mlstm": (_int, [_vp, _int, _int, _int, _int, _int, _int, _u32, ctypes.c_float]),
+    "mgq_graph_head_gate": (_int, [_vp, _int, _int, _int, _u32, ctypes.c_float, _int, _int]),
+    "mgq_graph_latent_cache_write": (_int, [_vp, _int, _int, _int, _int, _u32, ctypes.c_float, ctypes.c_float]),
+    "mgq_graph_latent_attention": (_int, [_vp, _int, _int, _int, _int, _int, _u32, _u32, _u32, _u32, _u32, ctypes.c_float, ctypes.c_float]),
+    "mgq_session_set_rows": (_int, [_vp, _int, _u32]),
+    "mgq_session_reset_state": (_int, [_vp]),
     "mgq_graph_set_outputs": (_int, [_vp, ctypes.POINTER(_int), _sz]),
     "mgq_build_inference_session": (_int, [_vp, ctypes.POINTER(_vp)]),
     "mgq_session_free": (None, [_vp]),

@@ -73,6 +73,7 @@ int mgq_set_option(const char *name, long value)
     if (!name) return fail(MGQ_ERR_NULL, "null option name");
     if (!std::strncmp(name, "plan.", 5)) return set_plan_option(name, value);
     if (!std::strncmp(name, "gemm.", 5)) return set_gemm_option(name, value);
+    if (!std::strncmp(name, "linear.", 7)) return set_linear_option(name, value);
     if (!std::strncmp(name, "session.", 8)) return set_session_option(name, value);
     return set_gemv_option(name, value);
 }
@@ -154,7 +155,7 @@ int mgq_argmax(const float *logits, uint32_t n, void *workspace, uint32_t *out_t
 {
     if (!logits || !out_token) return fail(MGQ_ERR_NULL, "argmax: null pointer");
     if (n == 0) return fail(MGQ_ERR_SHAPE, "argmax: empty vector");
-    return launch_argmax(logits, n, workspace, out_token, next_token, kv_pos, history, history_cap, stream);
+    return launch_argmax(logits, n, workspace, out_token, next_token, kv_pos, history, history_cap, 1, stream);
 }
 
 int mgq_gemv_f16(const float *x, const void *w_f16, const float *addend, float *y, uint32_t m, uint32_t k, uint32_t n, void *stream)

@@ -16,37 +16,10 @@
 #include <cfloat>
 #include <cstdint>
 
-#include "mgq_internal.h"
+#include "mgq_launch.cuh"
 
 namespace mgq {
 namespace {
-
-__device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;\n" ::: "memory"); }
-__device__ __forceinline__ void pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory"); }
-
-template <typename... Args>
-int launch(void (*kernel)(Args...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args... args)
-{
-    cudaLaunchConfig_t lc{};
-    lc.gridDim = grid;
-    lc.blockDim = block;
-    lc.dynamicSmemBytes = smem;
-    lc.stream = stream;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    lc.attrs = attr;
-    lc.numAttrs = 1;
-    MGQ_CUDA(cudaLaunchKernelEx(&lc, kernel, args...));
-    return MGQ_OK;
-}
-
-__device__ __forceinline__ float warp_sum(float v)
-{
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
 
 // ---------------------------------------------------------------- embedding (embedding.wgsl)
 __global__ void embedding_kernel(const uint32_t *ids, const float *table, float *out, uint32_t seq, uint32_t hidden,
@@ -425,7 +398,7 @@ __global__ void __launch_bounds__(128) cached_attention_kernel(const float *q, c
 // feeds it back: *next_token = winner, *kv_pos += 1.
 __global__ void __launch_bounds__(256) argmax_kernel(const float *logits, uint32_t n, float *part_val, uint32_t *part_idx,
                                                      unsigned int *counter, uint32_t *out_token, uint32_t *next_token,
-                                                     uint32_t *kv_pos, uint32_t *history, uint32_t history_cap)
+                                                     uint32_t *kv_pos, uint32_t *history, uint32_t history_cap, uint32_t advance)
 {
     __shared__ float s_val[8];
     __shared__ uint32_t s_idx[8];
@@ -474,9 +447,10 @@ __global__ void __launch_bounds__(256) argmax_kernel(const float *logits, uint32
     if (t != 0) return;
     if (best_i == 0xFFFFFFFFu) best_i = 0;                   // every logit was NaN
     *out_token = best_i;
-    if (history && kv_pos && kv_pos[0] < history_cap) history[kv_pos[0]] = best_i;
+    const uint32_t at = kv_pos ? kv_pos[0] + advance - 1u : 0u;          // position of the step's last token
+    if (history && kv_pos && at < history_cap) history[at] = best_i;
     if (next_token) *next_token = best_i;
-    if (kv_pos && next_token) kv_pos[0] += 1;
+    if (kv_pos && next_token) kv_pos[0] = at + 1u;
 }
 
 }  // namespace
@@ -569,7 +543,7 @@ int launch_cached_attention(const float *q, const float *k_cache, const float *v
 size_t argmax_workspace_bytes() { return 256 + 2 * 256 * sizeof(float); }
 
 int launch_argmax(const float *logits, uint32_t n, void *workspace, uint32_t *out_token, uint32_t *next_token, uint32_t *kv_pos,
-                  uint32_t *history, uint32_t history_cap, void *stream)
+                  uint32_t *history, uint32_t history_cap, uint32_t advance, void *stream)
 {
     if (!workspace) return fail(MGQ_ERR_NULL, "argmax needs its workspace");
     unsigned int *counter = static_cast<unsigned int *>(workspace);
@@ -579,7 +553,7 @@ int launch_argmax(const float *logits, uint32_t n, void *workspace, uint32_t *ou
     if (grid > 256) grid = 256;
     if (grid < 1) grid = 1;
     return launch(argmax_kernel, dim3(grid), dim3(256), 0, static_cast<cudaStream_t>(stream), logits, n, part_val, part_idx, counter,
-                  out_token, next_token, kv_pos, history, history_cap);
+                  out_token, next_token, kv_pos, history, history_cap, advance);
 }
 
 }  // namespace mgq

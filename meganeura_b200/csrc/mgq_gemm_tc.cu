@@ -31,7 +31,7 @@
 
 #include <mutex>
 
-#include "mgq_internal.h"
+#include "mgq_tcgen05.cuh"
 
 namespace mgq {
 namespace {
@@ -43,7 +43,6 @@ constexpr uint32_t kSubA = 128 * 128;              // activation sub-tile: 128 r
 constexpr uint32_t kSubB = TN * 128;               // weight sub-tile: 112 rows x 128 B, 14 KB (a 1024-byte multiple)
 constexpr uint32_t kStageBytes = kSlabs * kSubA + 2 * kSubB;   // A0..A3 | Bhi | Blo
 constexpr uint32_t kTmemCols = 512;
-constexpr uint32_t kWaitLimit = 1u << 20;          // try_wait calls before a wait gives up (each may sleep for a short hardware quantum)
 constexpr int kThreads = 320;                      // TMA warp, MMA warp, 8 dequant/epilogue warps
 
 __device__ unsigned int g_tc_error = 0;
@@ -62,85 +61,6 @@ struct __align__(8) TcShared {
     uint32_t tmem_base;
     volatile int failed;
 };
-
-__device__ __forceinline__ uint32_t smem_u32(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-
-__device__ __forceinline__ void mbar_init(unsigned long long *bar, uint32_t count)
-{
-    asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(bar)), "r"(count) : "memory");
-}
-__device__ __forceinline__ void mbar_arrive(unsigned long long *bar)
-{
-    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void mbar_arrive_expect_tx(unsigned long long *bar, uint32_t bytes)
-{
-    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(bar)), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ bool mbar_try_wait(unsigned long long *bar, uint32_t parity)
-{
-    uint32_t ok;
-    asm volatile("{\n\t.reg .pred p;\n\t"
-                 "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-                 "selp.u32 %0, 1, 0, p;\n\t}"
-                 : "=r"(ok) : "r"(smem_u32(bar)), "r"(parity) : "memory");
-    return ok != 0;
-}
-// Bounded wait: false when the limit ran out or another role of this CTA already gave up.
-__device__ __forceinline__ bool mbar_wait(unsigned long long *bar, uint32_t parity, TcShared *sh)
-{
-    for (uint32_t i = 0; i < kWaitLimit; i++) {
-        if (mbar_try_wait(bar, parity)) return true;
-        if (sh->failed) return false;
-    }
-    sh->failed = 1;
-    atomicExch(&g_tc_error, 1u);
-    return false;
-}
-
-__device__ __forceinline__ void tma_load_2d(void *dst, const CUtensorMap *map, int x, int y, unsigned long long *bar)
-{
-    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
-                 ::"r"(smem_u32(dst)), "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y) : "memory");
-}
-
-// K-major, 128-byte swizzle: rows are 128 B apart, 8-row groups 1024 B apart (SBO), version 1.
-__device__ __forceinline__ uint64_t umma_desc(uint32_t smem_addr)
-{
-    uint64_t d = 0;
-    d |= (uint64_t)((smem_addr & 0x3FFFFu) >> 4);          // start address, 16-byte units
-    d |= (uint64_t)1 << 16;                                // leading byte offset (unused for swizzled K-major)
-    d |= (uint64_t)(1024 >> 4) << 32;                      // stride byte offset
-    d |= (uint64_t)1 << 46;                                // descriptor version (Blackwell)
-    d |= (uint64_t)2 << 61;                                // SWIZZLE_128B
-    return d;
-}
-// kind::f16: D f32, A bf16, B bf16, both K-major, N = 112, M = 128.
-constexpr uint32_t kInstrDesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(TN >> 3) << 17) | ((uint32_t)(TM >> 4) << 24);
-
-__device__ __forceinline__ void umma_f16(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t accumulate)
-{
-    asm volatile("{\n\t.reg .pred p;\n\t"
-                 "setp.ne.b32 p, %4, 0;\n\t"
-                 "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
-                 ::"r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(kInstrDesc), "r"(accumulate), "r"(0u) : "memory");
-}
-__device__ __forceinline__ void umma_commit(unsigned long long *bar)
-{
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-
-__device__ __forceinline__ void tmem_ld16(uint32_t addr, uint32_t (&r)[16])
-{
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 "
-                 "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
-                   "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-                 : "r"(addr) : "memory");
-    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-}
 
 // words[off + 9*blk] for blk in 0..3 with compile-time off: register selects instead of a dynamic index.
 __device__ __forceinline__ uint32_t pick4(const uint32_t *words, int off, uint32_t blk)
@@ -187,8 +107,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_tc_kernel(const __grid_const
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     if (warp == 1) {            // TMEM: 128 lanes x 512 columns of f32 (4 accumulators of 112 columns)
-        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&sh.tmem_base)), "r"(kTmemCols) : "memory");
-        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+        tmem_alloc(&sh.tmem_base, kTmemCols);
     }
     tc_fence_before();
     __syncthreads();
@@ -201,7 +120,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_tc_kernel(const __grid_const
             int armed = -1;
             for (uint32_t kc = 0; kc < nk; kc++) {
                 const uint32_t s = kc % kTcStages, ph = (kc / kTcStages) & 1u;
-                if (!mbar_wait(&sh.empty[s], ph ^ 1u, &sh)) break;
+                if (!mbar_wait(&sh.empty[s], ph ^ 1u, &sh.failed, &g_tc_error)) break;
                 uint8_t *st = tiles + s * kStageBytes;
                 mbar_arrive_expect_tx(&sh.full_a[s], slabs * kSubA);
                 for (uint32_t i = 0; i < slabs; i++)
@@ -219,7 +138,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_tc_kernel(const __grid_const
             bool ok = true;
             for (uint32_t kc = 0; kc < nk && ok; kc++) {
                 const uint32_t s = kc % kTcStages, ph = (kc / kTcStages) & 1u;
-                ok = mbar_wait(&sh.full_a[s], ph, &sh) && mbar_wait(&sh.full_b[s], ph, &sh);
+                ok = mbar_wait(&sh.full_a[s], ph, &sh.failed, &g_tc_error) && mbar_wait(&sh.full_b[s], ph, &sh.failed, &g_tc_error);
                 if (!ok) break;
                 tc_fence_after();
                 const uint32_t base = smem_u32(tiles + s * kStageBytes);
@@ -229,8 +148,8 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_tc_kernel(const __grid_const
                     const uint64_t dh = umma_desc(b_hi + j * 32u), dl = umma_desc(b_lo + j * 32u);
                     for (uint32_t i = 0; i < slabs; i++) {
                         const uint64_t da = umma_desc(base + i * kSubA + j * 32u);
-                        umma_f16(tmem + i * TN, da, dh, (kc | j) != 0 ? 1u : 0u);
-                        umma_f16(tmem + i * TN, da, dl, 1u);
+                        umma_f16(tmem + i * TN, da, dh, umma_instr(TM, TN), (kc | j) != 0 ? 1u : 0u);
+                        umma_f16(tmem + i * TN, da, dl, umma_instr(TM, TN), 1u);
                     }
                 }
                 umma_commit(&sh.empty[s]);                               // stage reusable once these MMAs retire
@@ -267,7 +186,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_tc_kernel(const __grid_const
             fetch(1, raw_next);
             for (uint32_t kc = 0; kc < nk; kc++) {
                 const uint32_t s = kc % kTcStages, ph = (kc / kTcStages) & 1u;
-                if (!mbar_wait(&sh.empty[s], ph ^ 1u, &sh)) { ok = false; break; }
+                if (!mbar_wait(&sh.empty[s], ph ^ 1u, &sh.failed, &g_tc_error)) { ok = false; break; }
                 uint8_t *st = tiles + s * kStageBytes;
                 uint8_t *sub_hi = st + kSlabs * kSubA, *sub_lo = sub_hi + kSubB;
                 const uint32_t *words = reinterpret_cast<const uint32_t *>(raw);
@@ -319,7 +238,7 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_tc_kernel(const __grid_const
             }
         }
         // epilogue: TMEM lane = token row; this warp may touch lanes 32*(warp%4) .. +31
-        ok = ok && mbar_wait(&sh.acc_full, 0, &sh);
+        ok = ok && mbar_wait(&sh.acc_full, 0, &sh.failed, &g_tc_error);
         ok = __all_sync(0xffffffffu, ok);                                // tcgen05.ld is warp-collective
         if (ok) {
             tc_fence_after();
@@ -362,13 +281,11 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_tc_kernel(const __grid_const
     if (warp == 1) {
         __syncwarp();
         tc_fence_after();
-        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kTmemCols) : "memory");
+        tmem_free(tmem, kTmemCols);
     }
 }
 
-using EncodeTiledFn = CUresult (*)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *,
-                                  const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+}  // namespace
 
 int encode_fn(EncodeTiledFn &out)
 {
@@ -385,8 +302,6 @@ int encode_fn(EncodeTiledFn &out)
     out = cached;
     return MGQ_OK;
 }
-
-}  // namespace
 
 bool gemm_tc_eligible(int a_dtype, uint32_t m, uint32_t k, uint32_t n, const void *a)
 {
@@ -443,7 +358,7 @@ int tc_device_status()
         MGQ_CUDA(cudaMemcpyToSymbol(g_tc_error, &zero, sizeof zero));
         return fail(MGQ_ERR_TIMEOUT, "a bounded wait inside the tensor-core GEMM ran out");
     }
-    return MGQ_OK;
+    return linear_tc_status();
 }
 
 }  // namespace mgq

@@ -41,6 +41,7 @@ int launch_all_gather(const float *slice, const void *push_dev, const void *loca
                       uint32_t pitch, uint32_t world, const unsigned long long *epoch, unsigned int *error, void *stream);
 int set_gemv_option(const char *name, long value);
 int set_plan_option(const char *name, long value);
+int set_linear_option(const char *name, long value);
 int set_gemm_option(const char *name, long value);
 int set_session_option(const char *name, long value);
 bool force_tiled();
@@ -52,6 +53,7 @@ bool gemm_tc_eligible(int a_dtype, uint32_t m, uint32_t k, uint32_t n, const voi
 int launch_gemm_tc(int fmt, const void *a, const void *w, const float *addend, float *c,
                    uint32_t m, uint32_t k, uint32_t n, void *stream);
 int tc_device_status();
+int linear_tc_status();               // mgq_linear_tc.cu
 
 // Decode-step operators (mgq_decode_ops.cu).
 int launch_embedding(const uint32_t *ids, const float *table, float *out, uint32_t seq, uint32_t hidden, uint32_t vocab, void *stream);
@@ -69,7 +71,7 @@ int launch_cached_attention(const float *q, const float *k_cache, const float *v
                             void *stream);
 size_t argmax_workspace_bytes();
 int launch_argmax(const float *logits, uint32_t n, void *workspace, uint32_t *out_token, uint32_t *next_token, uint32_t *kv_pos,
-                  uint32_t *history, uint32_t history_cap, void *stream);
+                  uint32_t *history, uint32_t history_cap, uint32_t advance, void *stream);
 
 }  // namespace mgq
 

@@ -1,0 +1,87 @@
+// Device and host helpers shared by the operator kernels: programmatic dependent launch, warp
+// reductions, f32 <-> bf16 element access.
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+
+#include <cstdint>
+
+#include "mgq_internal.h"
+
+namespace mgq {
+
+__device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;\n" ::: "memory"); }
+__device__ __forceinline__ void pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory"); }
+
+template <typename... Params, typename... Args>
+int launch(void (*kernel)(Params...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args... args)
+{
+    cudaLaunchConfig_t lc{};
+    lc.gridDim = grid;
+    lc.blockDim = block;
+    lc.dynamicSmemBytes = smem;
+    lc.stream = stream;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    lc.attrs = attr;
+    lc.numAttrs = 1;
+    MGQ_CUDA(cudaLaunchKernelEx(&lc, kernel, static_cast<Params>(args)...));
+    return MGQ_OK;
+}
+
+// Opts a kernel into more than 48 KB of dynamic shared memory (a no-op for the driver when repeated).
+template <typename K>
+int allow_smem(K *kernel, size_t bytes)
+{
+    if (bytes <= 48 * 1024) return MGQ_OK;
+    MGQ_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes));
+    return MGQ_OK;
+}
+
+__device__ __forceinline__ float warp_sum(float v)
+{
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+__device__ __forceinline__ float warp_max(float v)
+{
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
+    return v;
+}
+
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f32(float v);
+template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+// 8 consecutive elements, 16-byte aligned source.
+__device__ __forceinline__ void unpack8(const uint4 &q, float (&f)[8])
+{
+    const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        f[2 * i] = __uint_as_float(w[i] << 16);
+        f[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
+    }
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16 *p, float (&f)[8]) { unpack8(__ldg(reinterpret_cast<const uint4 *>(p)), f); }
+__device__ __forceinline__ void load8(const float *p, float (&f)[8])
+{
+    const float4 a = __ldg(reinterpret_cast<const float4 *>(p)), b = __ldg(reinterpret_cast<const float4 *>(p) + 1);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// g = min(gate, limit), u = clamp(up, +-limit):  g sigmoid(alpha g) (u + 1)
+__device__ __forceinline__ float clamped_glu_f(float gate, float up, float limit, float alpha)
+{
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g * sigmoid_f(alpha * g) * (u + 1.0f);
+}
+
+}  // namespace mgq

@@ -1,0 +1,29 @@
+// A group of linear layers that one launch computes (mgq_linear.cu, mgq_linear_tc.cu).
+#pragma once
+#include "mgq_launch.cuh"
+
+namespace mgq {
+
+constexpr uint32_t kMaxSegments = 8;
+
+struct LinearSegment {
+    const void *a;                // [m, k] activations, f32 or bf16
+    const void *w, *w2;           // [n, k] bf16; w2: the up projection of a GLU pair (w is the gate)
+    const float *bias, *bias2;    // [n] or null
+    const float *addend;          // [m, n] f32 or null
+    void *out;                    // [m, n] f32 (GLU: f32 or bf16)
+    uint32_t n;
+};
+
+struct LinearGroup {
+    LinearSegment seg[kMaxSegments];
+    uint32_t count, m, k;
+    uint32_t a_bf16, glu, out_bf16;
+    float limit, alpha;           // clamped GLU
+};
+
+int launch_linear_group(const LinearGroup &g, void *stream);
+// tcgen05 path: bf16 activations, k % 8 == 0, 16-byte aligned operands.
+int launch_linear_tc(const LinearGroup &g, void *stream);
+
+}  // namespace mgq

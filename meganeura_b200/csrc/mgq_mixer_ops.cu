@@ -1,0 +1,626 @@
+// Norms, token shift, recurrences (RWKV-style time mixing, mLSTM matrix memory), per-head output
+// gates and the clamped GLU.  All statistics, gates, decays and recurrent state are f32; only the
+// operands of the next projection may be stored as bf16.
+//
+// The two recurrences share one schedule.  A head's state is kept value-major, [value][key], and a
+// thread owns RPT keys of one value column (8 threads per column), so a token step is register
+// arithmetic plus a 3-step shuffle; keys beyond `dim` are zero.
+//   scan_kernel  several tokens: CTA = head x 16 value columns, state in registers over the whole
+//                portion, the tokens' vectors staged through a double-buffered cp.async ring.
+//   step_kernel  one token: CTA = head; the decay projection (or the gates), the recurrence, the
+//                per-head norm and the output gate in one launch, state streamed once.
+#include "mgq_mixer.cuh"
+
+namespace mgq {
+namespace {
+
+__device__ __forceinline__ float block_sum(float v, float *s_part)
+{
+    v = warp_sum(v);
+    __syncthreads();
+    if ((threadIdx.x & 31u) == 0) s_part[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float total = 0.f;
+    for (uint32_t i = 0; i < blockDim.x / 32; i++) total += s_part[i];
+    return total;
+}
+
+// ---------------------------------------------------------------- embedding, rows, element-wise
+template <typename T>
+__global__ void embedding_scaled_kernel(const uint32_t *ids, const T *table, float *out, uint32_t rows, uint32_t width, uint32_t vocab, float scale)
+{
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (i >= (size_t)rows * width) return;
+    const uint32_t row = (uint32_t)(i / width), col = (uint32_t)(i - (size_t)row * width);
+    out[i] = to_f32(table[(size_t)min(ids[row], vocab - 1u) * width + col]) * scale;
+}
+
+__global__ void pick_rows_kernel(const float *x, const uint32_t *index, float *out, uint32_t rows, uint32_t src_rows, uint32_t cols)
+{
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (i >= (size_t)rows * cols) return;
+    const uint32_t row = (uint32_t)(i / cols);
+    out[i] = x[(size_t)min(index[row], src_rows - 1u) * cols + (i - (size_t)row * cols)];
+}
+
+__global__ void bias_add_kernel(const float *x, const float *bias, float *out, size_t len, uint32_t cols)
+{
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (i < len) out[i] = x[i] + bias[i % cols];
+}
+
+template <typename OT>
+__global__ void clamped_glu_kernel(const float *gate, const float *up, OT *out, size_t len, float limit, float alpha)
+{
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (i < len) out[i] = from_f32<OT>(clamped_glu_f(gate[i], up[i], limit, alpha));
+}
+
+// ---------------------------------------------------------------- RMS norm with a weight offset, optional row index
+template <typename OT>
+__global__ void __launch_bounds__(256) norm_kernel(const float *x, const float *weight, const uint32_t *index, OT *out, uint32_t src_rows,
+                                                   uint32_t cols, float eps, float offset)
+{
+    constexpr int HOLD = 16;                     // values a thread keeps between the two passes
+    __shared__ float s_part[8];
+    const uint32_t t = threadIdx.x;
+    float w[HOLD], v[HOLD];
+    pdl_launch_dependents();
+#pragma unroll
+    for (int i = 0; i < HOLD; i++) w[i] = t + 256u * i < cols ? offset + __ldg(weight + t + 256u * i) : 0.f;
+    pdl_wait();
+    const uint32_t row = index ? min(index[blockIdx.x], src_rows - 1u) : blockIdx.x;
+    const float *src = x + (size_t)row * cols;
+    OT *dst = out + (size_t)blockIdx.x * cols;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < HOLD; i++) {
+        v[i] = t + 256u * i < cols ? src[t + 256u * i] : 0.f;
+        ss = fmaf(v[i], v[i], ss);
+    }
+    for (uint32_t j = t + 256u * HOLD; j < cols; j += 256) ss = fmaf(src[j], src[j], ss);
+    const float r = 1.0f / sqrtf(block_sum(ss, s_part) / (float)cols + eps);
+#pragma unroll
+    for (int i = 0; i < HOLD; i++)
+        if (t + 256u * i < cols) dst[t + 256u * i] = from_f32<OT>(v[i] * r * w[i]);
+    for (uint32_t j = t + 256u * HOLD; j < cols; j += 256) dst[j] = from_f32<OT>(src[j] * r * (offset + weight[j]));
+}
+
+// ---------------------------------------------------------------- token shift (with the norm in front of it)
+template <typename OT>
+__global__ void __launch_bounds__(256) token_shift_kernel(const __grid_constant__ TokenShift a)
+{
+    __shared__ float s_part[8];
+    const uint32_t t = threadIdx.x, row = blockIdx.x, width = a.width;
+    pdl_launch_dependents();
+    pdl_wait();
+    const float *cur = a.x + (size_t)row * width, *before = row ? cur - width : a.state;
+    float r_cur = 1.f, r_before = 1.f;
+    if (a.norm_weight) {
+        float s0 = 0.f, s1 = 0.f;
+        for (uint32_t j = t; j < width; j += 256) {
+            s0 = fmaf(cur[j], cur[j], s0);
+            if (row) s1 = fmaf(before[j], before[j], s1);
+        }
+        r_cur = 1.0f / sqrtf(block_sum(s0, s_part) / (float)width + a.eps);
+        if (row) r_before = 1.0f / sqrtf(block_sum(s1, s_part) / (float)width + a.eps);
+    }
+    const bool last = row + 1 == a.rows;
+    OT *out = static_cast<OT *>(a.out) + (size_t)row * width;
+    for (uint32_t j = t; j < width; j += 256) {
+        const float g = a.norm_weight ? a.offset + a.norm_weight[j] : 1.f;
+        const float h = a.norm_weight ? cur[j] * r_cur * g : cur[j];
+        const float hp = row && a.norm_weight ? before[j] * r_before * g : before[j];        // the state already holds a normed h
+        for (uint32_t s = 0; s < a.slots; s++) out[s * a.slot_stride + j] = from_f32<OT>(fmaf(hp - h, a.mu[s][j], h));
+        if (last) a.state[width + j] = h;
+    }
+}
+
+// ---------------------------------------------------------------- per-head norm and gate: one warp per (row, head)
+template <typename OT>
+__global__ void __launch_bounds__(256) head_gate_kernel(const float *o, const __grid_constant__ HeadGate hg, uint32_t total, uint32_t heads, uint32_t dim)
+{
+    constexpr int HOLD = 8;
+    const uint32_t lane = threadIdx.x & 31u, unit = blockIdx.x * 8u + (threadIdx.x >> 5);
+    pdl_launch_dependents();
+    pdl_wait();
+    if (unit >= total) return;
+    const size_t base = (size_t)unit * dim;
+    const uint32_t wbase = (unit % heads) * dim;
+    float v[HOLD], ss = 0.f, r = 1.f;
+#pragma unroll
+    for (int i = 0; i < HOLD; i++) {
+        v[i] = lane + 32u * i < dim ? o[base + lane + 32u * i] : 0.f;
+        ss = fmaf(v[i], v[i], ss);
+    }
+    for (uint32_t j = lane + 32u * HOLD; j < dim; j += 32) ss = fmaf(o[base + j], o[base + j], ss);
+    if (hg.weight) r = 1.0f / sqrtf(warp_sum(ss) / (float)dim + hg.eps);
+    OT *out = static_cast<OT *>(hg.out);
+    auto put = [&](uint32_t j, float val) {
+        const float g = hg.gate[base + j], s = sigmoid_f(g);
+        out[base + j] = from_f32<OT>(val * r * (hg.weight ? hg.weight[wbase + j] : 1.f) * (hg.silu ? g * s : s));
+    };
+#pragma unroll
+    for (int i = 0; i < HOLD; i++)
+        if (lane + 32u * i < dim) put(lane + 32u * i, v[i]);
+    for (uint32_t j = lane + 32u * HOLD; j < dim; j += 32) put(j, o[base + j]);
+}
+
+// ---------------------------------------------------------------- decay: exp(-exp(tanh(low) . w2^T + w0)), 8 rows per CTA
+constexpr uint32_t kDecayRows = 8;
+__global__ void __launch_bounds__(128) decay_kernel(const __grid_constant__ Wkv a)
+{
+    extern __shared__ float s_low[];                     // [8][rank]
+    const uint32_t ch = blockIdx.x * 128u + threadIdx.x, row0 = blockIdx.y * kDecayRows, channels = a.heads * a.dim;
+    const uint32_t rows = min(kDecayRows, a.rows - row0);
+    pdl_launch_dependents();
+    pdl_wait();
+    for (uint32_t i = threadIdx.x; i < kDecayRows * a.rank; i += 128)
+        s_low[i] = i < rows * a.rank ? tanhf(a.low[(size_t)row0 * a.rank + i]) : 0.f;
+    __syncthreads();
+    if (ch >= channels) return;
+    const __nv_bfloat16 *w = static_cast<const __nv_bfloat16 *>(a.w2) + (size_t)ch * a.rank;
+    const float w0 = a.w0[ch];
+    float acc[kDecayRows];
+#pragma unroll
+    for (int r = 0; r < (int)kDecayRows; r++) acc[r] = 0.f;
+    for (uint32_t j = 0; j < a.rank; j++) {
+        const float wv = __bfloat162float(w[j]);
+#pragma unroll
+        for (int r = 0; r < (int)kDecayRows; r++) acc[r] = fmaf(s_low[r * a.rank + j], wv, acc[r]);
+    }
+    for (uint32_t r = 0; r < rows; r++) a.decay[(size_t)(row0 + r) * channels + ch] = expf(-expf(acc[r] + w0));
+}
+
+// ---------------------------------------------------------------- recurrences
+__device__ __forceinline__ void cp_async4(void *smem, const void *gmem)
+{
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((unsigned)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void cp_async16(void *smem, const void *gmem)
+{
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((unsigned)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
+
+enum { kWkv = 0, kMlstm = 1 };
+
+struct Scan {
+    const float *q, *k, *v, *w;          // wkv: r, k, v, decay;  mlstm: q, k, v, -
+    const float *u;                      // wkv bonus [heads, dim]
+    const float *gi, *gf;                // mlstm gate pre-activations [rows, heads]
+    float *o, *state, *shift_state;
+    uint32_t rows, heads, dim, vdim, shift_width;
+    float cap, qscale;
+};
+
+__host__ __device__ inline uint32_t pad4(uint32_t d) { return (d + 3u) & ~3u; }
+template <int RPT> __host__ __device__ constexpr int chunk_tokens() { return RPT <= 8 ? 32 : RPT == 16 ? 16 : 8; }
+
+__device__ __forceinline__ float log_sigmoid(float z) { return z < 0.f ? z - log1pf(expf(z)) : -log1pf(expf(-z)); }
+
+// One token of one value column for the RPT keys this thread owns; returns the partial dot products.
+template <int MODE, int RPT>
+__device__ __forceinline__ void token_step(const float *q, const float *k, const float *w, const float (&u)[RPT], float v, float a, float b,
+                                           float (&S)[RPT], float (&n)[RPT], float &out, float &den)
+{
+    float o[2] = {0.f, 0.f}, d[2] = {0.f, 0.f};
+    if (MODE == kMlstm) v *= b;
+#pragma unroll
+    for (int i = 0; i < RPT; i += 4) {
+        const float4 q4 = *reinterpret_cast<const float4 *>(q + i * 8), k4 = *reinterpret_cast<const float4 *>(k + i * 8);
+        const float qv[4] = {q4.x, q4.y, q4.z, q4.w}, kv[4] = {k4.x, k4.y, k4.z, k4.w};
+        if (MODE == kWkv) {
+            const float4 w4 = *reinterpret_cast<const float4 *>(w + i * 8);
+            const float wv[4] = {w4.x, w4.y, w4.z, w4.w};
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const float x = kv[j] * v;
+                o[j & 1] = fmaf(qv[j], fmaf(u[i + j], x, S[i + j]), o[j & 1]);
+                S[i + j] = fmaf(wv[j], S[i + j], x);
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                S[i + j] = fmaf(kv[j], v, a * S[i + j]);
+                n[i + j] = fmaf(kv[j], b, a * n[i + j]);
+                o[j & 1] = fmaf(qv[j], S[i + j], o[j & 1]);
+                d[j & 1] = fmaf(qv[j], n[i + j], d[j & 1]);
+            }
+        }
+    }
+    out = o[0] + o[1];
+    den = d[0] + d[1];
+#pragma unroll
+    for (int off = 4; off > 0; off >>= 1) {
+        out += __shfl_xor_sync(0xffffffffu, out, off);
+        if (MODE == kMlstm) den += __shfl_xor_sync(0xffffffffu, den, off);
+    }
+}
+
+__device__ __forceinline__ float mlstm_out(float out, float den, float qscale, float floor_)
+{
+    return out * qscale / (fmaxf(fabsf(den * qscale), floor_) + 1e-6f);
+}
+
+// Keys owned by thread ks of a column: (i * 8 + ks) * 4 + j for i < RPT / 4, j < 4.
+template <int RPT>
+__device__ __forceinline__ void load_keys(const float *row, uint32_t ks, uint32_t kp, float (&x)[RPT])
+{
+#pragma unroll
+    for (int i = 0; i < RPT; i += 4) {
+        const uint32_t at = (i * 2u + ks) * 4u;              // (i / 4 * 8 + ks) * 4
+        const float4 v = at < kp ? *reinterpret_cast<const float4 *>(row + at) : make_float4(0.f, 0.f, 0.f, 0.f);
+        x[i] = v.x; x[i + 1] = v.y; x[i + 2] = v.z; x[i + 3] = v.w;
+    }
+}
+template <int RPT>
+__device__ __forceinline__ void store_keys(float *row, uint32_t ks, uint32_t kp, const float (&x)[RPT])
+{
+#pragma unroll
+    for (int i = 0; i < RPT; i += 4) {
+        const uint32_t at = (i * 2u + ks) * 4u;
+        if (at < kp) *reinterpret_cast<float4 *>(row + at) = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
+    }
+}
+
+constexpr uint32_t kScanThreads = 128, kScanCols = 16;
+
+// mLSTM: n [pad4(dim)] and m of a head, one copy per block of 16 value columns (every CTA of a head
+// advances its own, so no CTA reads what another one writes).
+__host__ __device__ inline uint32_t value_blocks(uint32_t vdim) { return (vdim + kScanCols - 1) / kScanCols; }
+__device__ __forceinline__ float *normalizer(const Scan &p, uint32_t head, uint32_t block)
+{
+    const uint32_t kp = pad4(p.dim);
+    return p.state + (size_t)p.heads * p.vdim * kp + (size_t)(head * value_blocks(p.vdim) + block) * (kp + 4u);
+}
+
+template <int MODE, int RPT>
+__global__ void __launch_bounds__(kScanThreads) scan_kernel(const __grid_constant__ Scan p)
+{
+    constexpr int TC = chunk_tokens<RPT>(), KS = RPT * 8, NA = MODE == kWkv ? 3 : 2;
+    extern __shared__ __align__(16) float smem[];
+    // per buffer: NA x [TC][KS] key vectors, [TC][16] values
+    constexpr int kBuf = NA * TC * KS + TC * (int)kScanCols;
+    __shared__ float s_gate[2][3][32];                   // mlstm: keep, write, exp(-m) per token of a chunk
+    const uint32_t t = threadIdx.x, head = blockIdx.x, col0 = blockIdx.y * kScanCols, col = col0 + t / 8, ks = t & 7u;
+    const uint32_t dim = p.dim, vdim = p.vdim, kp = pad4(dim), kpitch = p.heads * dim, vpitch = p.heads * vdim;
+    const bool live = col < vdim;
+    const uint32_t chunks = (p.rows + TC - 1) / TC;
+    for (uint32_t i = t; i < 2u * kBuf; i += kScanThreads) smem[i] = 0.f;          // keys beyond dim stay zero
+    float S[RPT], n[RPT], u[RPT];
+#pragma unroll
+    for (int i = 0; i < RPT; i++) { S[i] = 0.f; n[i] = 0.f; u[i] = 0.f; }
+    if (MODE == kWkv) {
+#pragma unroll
+        for (int i = 0; i < RPT; i++) {
+            const uint32_t key = (i / 4 * 8 + ks) * 4 + i % 4;
+            if (key < dim) u[i] = __ldg(p.u + head * dim + key);
+        }
+    }
+    pdl_launch_dependents();
+    pdl_wait();
+    __syncthreads();
+    float *srow = p.state + ((size_t)head * vdim + col) * kp;
+    float *nrow = normalizer(p, head, blockIdx.y), *mrow = nrow + kp;
+    if (live) load_keys<RPT>(srow, ks, kp, S);
+    if (MODE == kMlstm) load_keys<RPT>(nrow, ks, kp, n);
+    const bool vec = dim % 4 == 0 && (reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.w)) % 16 == 0;
+
+    auto stage = [&](uint32_t c, uint32_t buf) {
+        float *base = smem + buf * kBuf;
+        const uint32_t r0 = c * TC, cnt = min((uint32_t)TC, p.rows - r0);
+#pragma unroll
+        for (int arr = 0; arr < NA; arr++) {
+            const float *src = (arr == 0 ? p.q : arr == 1 ? p.k : p.w) + (size_t)r0 * kpitch + head * dim;
+            float *dst = base + arr * TC * KS;
+            if (vec) {
+                const uint32_t per = dim / 4;
+                for (uint32_t i = t; i < cnt * per; i += kScanThreads) {
+                    const uint32_t r = i / per, j = (i - r * per) * 4;
+                    cp_async16(dst + r * KS + j, src + (size_t)r * kpitch + j);
+                }
+            } else {
+                for (uint32_t i = t; i < cnt * dim; i += kScanThreads) {
+                    const uint32_t r = i / dim, j = i - r * dim;
+                    cp_async4(dst + r * KS + j, src + (size_t)r * kpitch + j);
+                }
+            }
+        }
+        float *dv = base + NA * TC * KS;
+        const float *sv = p.v + (size_t)r0 * vpitch + head * vdim + col0;
+        for (uint32_t i = t; i < cnt * kScanCols; i += kScanThreads) {
+            const uint32_t r = i / kScanCols, j = i % kScanCols;
+            if (col0 + j < vdim) cp_async4(dv + i, sv + (size_t)r * vpitch + j);
+        }
+        cp_commit();
+    };
+    // mlstm gates of a chunk by one warp: m_t = max(f_t + m_{t-1}, i_t) is a scan of (sum f, max) pairs
+    float m_carry = 0.f;
+    auto gates = [&](uint32_t c, uint32_t buf) {
+        const uint32_t lane = t, row = c * TC + lane;
+        const bool in = lane < (uint32_t)TC && row < p.rows;
+        const float xi = in ? p.gi[(size_t)row * p.heads + head] : 0.f, xf = in ? p.gf[(size_t)row * p.heads + head] : 0.f;
+        const float li = p.cap * tanhf(xi / p.cap), lf = in ? log_sigmoid(p.cap * tanhf(xf / p.cap)) : 0.f;
+        float F = lf, M = in ? li : -INFINITY;
+#pragma unroll
+        for (int off = 1; off < 32; off <<= 1) {
+            const float Fp = __shfl_up_sync(0xffffffffu, F, off), Mp = __shfl_up_sync(0xffffffffu, M, off);
+            if (lane >= (uint32_t)off) { M = fmaxf(M, F + Mp); F += Fp; }
+        }
+        const float m = fmaxf(F + m_carry, M);
+        float prev = __shfl_up_sync(0xffffffffu, m, 1);
+        if (lane == 0) prev = m_carry;
+        s_gate[buf][0][lane] = expf(lf + prev - m);
+        s_gate[buf][1][lane] = in ? expf(li - m) : 0.f;
+        s_gate[buf][2][lane] = expf(-m);
+        const uint32_t cnt = min((uint32_t)TC, p.rows - c * TC);
+        m_carry = __shfl_sync(0xffffffffu, m, cnt - 1);
+    };
+    if (MODE == kMlstm && t < 32) { m_carry = *mrow; gates(0, 0); }
+    stage(0, 0);
+    for (uint32_t c = 0; c < chunks; c++) {
+        const uint32_t buf = c & 1u;
+        if (c + 1 < chunks) { stage(c + 1, buf ^ 1u); cp_wait<1>(); } else { cp_wait<0>(); }
+        __syncthreads();
+        const float *base = smem + buf * kBuf, *sq = base + ks * 4, *sk = sq + TC * KS, *sw = sk + (NA == 3 ? TC * KS : 0);
+        const float *sv = base + NA * TC * KS + t / 8;
+        const uint32_t r0 = c * TC, cnt = min((uint32_t)TC, p.rows - r0);
+        float *dst = p.o + (size_t)r0 * vpitch + head * vdim + col;
+#pragma unroll 2
+        for (uint32_t r = 0; r < cnt; r++) {
+            float out, den, a = 0.f, b = 0.f;
+            if (MODE == kMlstm) { a = s_gate[buf][0][r]; b = s_gate[buf][1][r]; }
+            token_step<MODE, RPT>(sq + r * KS, sk + r * KS, sw + r * KS, u, sv[r * kScanCols], a, b, S, n, out, den);
+            if (ks == 0 && live) dst[(size_t)r * vpitch] = MODE == kMlstm ? mlstm_out(out, den, p.qscale, s_gate[buf][2][r]) : out;
+        }
+        if (MODE == kMlstm && t < 32 && c + 1 < chunks) gates(c + 1, buf ^ 1u);
+        __syncthreads();
+    }
+    if (live) store_keys<RPT>(srow, ks, kp, S);
+    if (MODE == kMlstm) {
+        if (t < 8) store_keys<RPT>(nrow, ks, kp, n);
+        if (t == 0) *mrow = m_carry;
+    }
+    if (MODE == kWkv && p.shift_state && blockIdx.y == 0) {
+        for (uint32_t j = head * kScanThreads + t; j < p.shift_width; j += p.heads * kScanThreads) p.shift_state[j] = p.shift_state[p.shift_width + j];
+    }
+}
+
+// ---------------------------------------------------------------- one token: decay / gates, recurrence, head norm, gate
+constexpr uint32_t kStepThreads = 512, kStepCols = kStepThreads / 8;
+
+template <int MODE, int RPT, typename OT>
+__global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constant__ Scan p, const __grid_constant__ HeadGate hg, const float *low,
+                                                            const __nv_bfloat16 *w2, const float *w0, uint32_t rank)
+{
+    constexpr int KS = RPT * 8;
+    extern __shared__ __align__(16) float smem[];        // q, k, w [KS] each; o [vdim]; tanh(low) [rank]
+    __shared__ float s_part[kStepThreads / 32], s_gate[3];
+    const uint32_t t = threadIdx.x, head = blockIdx.x, ks = t & 7u, dim = p.dim, vdim = p.vdim, kp = pad4(dim);
+    float *sq = smem, *sk = sq + KS, *sw = sk + KS, *so = sw + KS, *s_low = so + vdim;
+    float u[RPT], n[RPT];
+#pragma unroll
+    for (int i = 0; i < RPT; i++) {
+        const uint32_t key = (i / 4 * 8 + ks) * 4 + i % 4;
+        u[i] = MODE == kWkv && key < dim ? __ldg(p.u + head * dim + key) : 0.f;
+        n[i] = 0.f;
+    }
+    pdl_launch_dependents();
+    pdl_wait();
+    for (uint32_t i = t; i < (uint32_t)KS; i += kStepThreads) {
+        sq[i] = i < dim ? p.q[head * dim + i] : 0.f;
+        sk[i] = i < dim ? p.k[head * dim + i] : 0.f;
+        sw[i] = 0.f;
+    }
+    float *nrow = normalizer(p, head, 0);
+    if (MODE == kWkv) {
+        for (uint32_t i = t; i < rank; i += kStepThreads) s_low[i] = tanhf(low[i]);
+        __syncthreads();
+        for (uint32_t ch = t / 8; ch < ((dim + 3u) & ~3u); ch += kStepCols) {       // a warp covers 4 channels: uniform trip count
+            float acc = 0.f;
+            if (ch < dim)
+                for (uint32_t j = ks; j < rank; j += 8) acc = fmaf(s_low[j], __bfloat162float(w2[(size_t)(head * dim + ch) * rank + j]), acc);
+#pragma unroll
+            for (int off = 4; off > 0; off >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
+            if (ks == 0 && ch < dim) sw[ch] = expf(-expf(acc + w0[head * dim + ch]));
+        }
+    } else {
+        load_keys<RPT>(nrow, ks, kp, n);
+        if (t == 0) {
+            const float m0 = nrow[kp], li = p.cap * tanhf(p.gi[head] / p.cap), lf = log_sigmoid(p.cap * tanhf(p.gf[head] / p.cap));
+            const float m = fmaxf(lf + m0, li);
+            s_gate[0] = expf(lf + m0 - m);
+            s_gate[1] = expf(li - m);
+            s_gate[2] = m;
+        }
+    }
+    __syncthreads();
+    const float a = MODE == kMlstm ? s_gate[0] : 0.f, b = MODE == kMlstm ? s_gate[1] : 0.f, m_new = MODE == kMlstm ? s_gate[2] : 0.f;
+    float ss = 0.f, n_out[RPT];
+#pragma unroll
+    for (int i = 0; i < RPT; i++) n_out[i] = 0.f;
+    for (uint32_t col = t / 8; col < (vdim + kStepCols - 1) / kStepCols * kStepCols; col += kStepCols) {
+        const bool live = col < vdim;
+        float *srow = p.state + ((size_t)head * vdim + (live ? col : 0)) * kp;
+        float S[RPT], nn[RPT], out, den;
+        load_keys<RPT>(srow, ks, kp, S);
+#pragma unroll
+        for (int i = 0; i < RPT; i++) nn[i] = n[i];
+        const float v = live ? p.v[head * vdim + col] : 0.f;
+        token_step<MODE, RPT>(sq + ks * 4, sk + ks * 4, sw + ks * 4, u, v, a, b, S, nn, out, den);
+        if (MODE == kMlstm) {
+            out = mlstm_out(out, den, p.qscale, expf(-m_new));
+#pragma unroll
+            for (int i = 0; i < RPT; i++) n_out[i] = nn[i];
+        }
+        if (live) {
+            store_keys<RPT>(srow, ks, kp, S);
+            if (ks == 0) { so[col] = out; ss = fmaf(out, out, ss); }
+        }
+    }
+    const float r = 1.0f / sqrtf(block_sum(ss, s_part) / (float)vdim + hg.eps);     // its barriers also publish so[] and order the reads of n and m
+    OT *dst = static_cast<OT *>(hg.out) + head * vdim;
+    for (uint32_t j = t; j < vdim; j += kStepThreads) {
+        const float g = hg.gate[head * vdim + j], s = sigmoid_f(g);
+        dst[j] = from_f32<OT>(so[j] * r * hg.weight[head * vdim + j] * (hg.silu ? g * s : s));
+    }
+    if (MODE == kMlstm) {
+        for (uint32_t blk = t / 8; blk < value_blocks(vdim); blk += kStepCols) {
+            store_keys<RPT>(normalizer(p, head, blk), ks, kp, n_out);
+            if (ks == 0) normalizer(p, head, blk)[kp] = m_new;
+        }
+    } else if (p.shift_state) {
+        for (uint32_t j = head * kStepThreads + t; j < p.shift_width; j += p.heads * kStepThreads) p.shift_state[j] = p.shift_state[p.shift_width + j];
+    }
+}
+
+template <int MODE, int RPT>
+int launch_scan_rpt(const Scan &p, cudaStream_t stream)
+{
+    constexpr int NA = MODE == kWkv ? 3 : 2, TC = chunk_tokens<RPT>();
+    const size_t smem = (size_t)2 * (NA * TC * RPT * 8 + TC * kScanCols) * sizeof(float);
+    if (int rc = allow_smem(scan_kernel<MODE, RPT>, smem)) return rc;
+    return launch(scan_kernel<MODE, RPT>, dim3(p.heads, value_blocks(p.vdim)), dim3(kScanThreads), smem, stream, p);
+}
+
+template <int MODE>
+int launch_scan(const Scan &p, cudaStream_t stream)
+{
+    if (p.dim <= 32) return launch_scan_rpt<MODE, 4>(p, stream);
+    if (p.dim <= 64) return launch_scan_rpt<MODE, 8>(p, stream);
+    if (p.dim <= 128) return launch_scan_rpt<MODE, 16>(p, stream);
+    if (p.dim <= kMaxStateDim) return launch_scan_rpt<MODE, 32>(p, stream);
+    return fail(MGQ_ERR_SHAPE, "recurrent heads of %u key dimensions (at most %u)", p.dim, kMaxStateDim);
+}
+
+template <int MODE, int RPT>
+int launch_step_rpt(const Scan &p, const HeadGate &hg, const float *low, const void *w2, const float *w0, uint32_t rank, cudaStream_t stream)
+{
+    const size_t smem = (size_t)(3 * RPT * 8 + p.vdim + rank) * sizeof(float);
+    const __nv_bfloat16 *w2b = static_cast<const __nv_bfloat16 *>(w2);
+    if (hg.out_bf16) {
+        if (int rc = allow_smem(step_kernel<MODE, RPT, __nv_bfloat16>, smem)) return rc;
+        return launch(step_kernel<MODE, RPT, __nv_bfloat16>, dim3(p.heads), dim3(kStepThreads), smem, stream, p, hg, low, w2b, w0, rank);
+    }
+    if (int rc = allow_smem(step_kernel<MODE, RPT, float>, smem)) return rc;
+    return launch(step_kernel<MODE, RPT, float>, dim3(p.heads), dim3(kStepThreads), smem, stream, p, hg, low, w2b, w0, rank);
+}
+
+template <int MODE>
+int launch_step(const Scan &p, const HeadGate &hg, const float *low, const void *w2, const float *w0, uint32_t rank, cudaStream_t stream)
+{
+    if (p.dim <= 32) return launch_step_rpt<MODE, 4>(p, hg, low, w2, w0, rank, stream);
+    if (p.dim <= 64) return launch_step_rpt<MODE, 8>(p, hg, low, w2, w0, rank, stream);
+    if (p.dim <= 128) return launch_step_rpt<MODE, 16>(p, hg, low, w2, w0, rank, stream);
+    if (p.dim <= kMaxStateDim) return launch_step_rpt<MODE, 32>(p, hg, low, w2, w0, rank, stream);
+    return fail(MGQ_ERR_SHAPE, "recurrent heads of %u key dimensions (at most %u)", p.dim, kMaxStateDim);
+}
+
+Scan wkv_args(const Wkv &a)
+{
+    Scan p{};
+    p.q = a.r; p.k = a.k; p.v = a.v; p.w = a.decay; p.u = a.u; p.o = a.o; p.state = a.state; p.shift_state = a.shift_state;
+    p.rows = a.rows; p.heads = a.heads; p.dim = a.dim; p.vdim = a.dim; p.shift_width = a.shift_width;
+    p.cap = 1.f; p.qscale = 1.f;
+    return p;
+}
+Scan mlstm_args(const Mlstm &a)
+{
+    Scan p{};
+    p.q = a.q; p.k = a.k; p.v = a.v; p.gi = a.gi; p.gf = a.gf; p.o = a.o; p.state = a.state;
+    p.rows = a.rows; p.heads = a.heads; p.dim = a.dim; p.vdim = a.vdim;
+    p.cap = a.cap; p.qscale = (float)(1.0 / sqrt((double)a.dim));
+    return p;
+}
+
+inline uint32_t blocks_for(size_t n) { return (uint32_t)((n + 255) / 256); }
+
+}  // namespace
+
+int launch_embedding_scaled(const uint32_t *ids, const void *table, bool table_bf16, float *out, uint32_t rows, uint32_t width, uint32_t vocab,
+                            float scale, void *stream)
+{
+    const dim3 grid(blocks_for((size_t)rows * width));
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (table_bf16) return launch(embedding_scaled_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, ids, static_cast<const __nv_bfloat16 *>(table), out, rows, width, vocab, scale);
+    return launch(embedding_scaled_kernel<float>, grid, dim3(256), 0, st, ids, static_cast<const float *>(table), out, rows, width, vocab, scale);
+}
+
+int launch_norm(const float *x, const float *weight, const uint32_t *index, void *out, bool out_bf16, uint32_t rows, uint32_t src_rows,
+                uint32_t cols, float eps, float offset, void *stream)
+{
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (out_bf16) return launch(norm_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, st, x, weight, index, static_cast<__nv_bfloat16 *>(out), src_rows, cols, eps, offset);
+    return launch(norm_kernel<float>, dim3(rows), dim3(256), 0, st, x, weight, index, static_cast<float *>(out), src_rows, cols, eps, offset);
+}
+
+int launch_pick_rows(const float *x, const uint32_t *index, float *out, uint32_t rows, uint32_t src_rows, uint32_t cols, void *stream)
+{
+    return launch(pick_rows_kernel, dim3(blocks_for((size_t)rows * cols)), dim3(256), 0, static_cast<cudaStream_t>(stream), x, index, out, rows, src_rows, cols);
+}
+
+int launch_bias_add(const float *x, const float *bias, float *out, uint32_t rows, uint32_t cols, void *stream)
+{
+    const size_t len = (size_t)rows * cols;
+    return launch(bias_add_kernel, dim3(blocks_for(len)), dim3(256), 0, static_cast<cudaStream_t>(stream), x, bias, out, len, cols);
+}
+
+int launch_clamped_glu(const float *gate, const float *up, void *out, bool out_bf16, size_t len, float limit, float alpha, void *stream)
+{
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (out_bf16) return launch(clamped_glu_kernel<__nv_bfloat16>, dim3(blocks_for(len)), dim3(256), 0, st, gate, up, static_cast<__nv_bfloat16 *>(out), len, limit, alpha);
+    return launch(clamped_glu_kernel<float>, dim3(blocks_for(len)), dim3(256), 0, st, gate, up, static_cast<float *>(out), len, limit, alpha);
+}
+
+int launch_token_shift(const TokenShift &a, void *stream)
+{
+    if (a.slots == 0 || a.slots > kMaxShifts) return fail(MGQ_ERR_SHAPE, "token_shift: %u mixes (1..%d)", a.slots, kMaxShifts);
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (a.out_bf16) return launch(token_shift_kernel<__nv_bfloat16>, dim3(a.rows), dim3(256), 0, st, a);
+    return launch(token_shift_kernel<float>, dim3(a.rows), dim3(256), 0, st, a);
+}
+
+int launch_head_gate(const float *o, const HeadGate &hg, uint32_t rows, uint32_t heads, uint32_t dim, void *stream)
+{
+    const uint32_t total = rows * heads;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (hg.out_bf16) return launch(head_gate_kernel<__nv_bfloat16>, dim3((total + 7) / 8), dim3(256), 0, st, o, hg, total, heads, dim);
+    return launch(head_gate_kernel<float>, dim3((total + 7) / 8), dim3(256), 0, st, o, hg, total, heads, dim);
+}
+
+size_t wkv_state_elements(uint32_t heads, uint32_t dim) { return (size_t)heads * dim * pad4(dim); }
+size_t mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim)
+{
+    return (size_t)heads * vdim * pad4(dim) + (size_t)heads * value_blocks(vdim) * (pad4(dim) + 4u);
+}
+
+int launch_decay(const Wkv &a, void *stream)
+{
+    const size_t smem = (size_t)kDecayRows * a.rank * sizeof(float);
+    if (int rc = allow_smem(decay_kernel, smem)) return rc;
+    return launch(decay_kernel, dim3((a.heads * a.dim + 127) / 128, (a.rows + kDecayRows - 1) / kDecayRows), dim3(128), smem,
+                  static_cast<cudaStream_t>(stream), a);
+}
+
+int launch_wkv_scan(const Wkv &a, void *stream) { return launch_scan<kWkv>(wkv_args(a), static_cast<cudaStream_t>(stream)); }
+int launch_mlstm_scan(const Mlstm &a, void *stream) { return launch_scan<kMlstm>(mlstm_args(a), static_cast<cudaStream_t>(stream)); }
+int launch_wkv_step(const Wkv &a, const HeadGate &hg, void *stream)
+{
+    return launch_step<kWkv>(wkv_args(a), hg, a.low, a.w2, a.w0, a.rank, static_cast<cudaStream_t>(stream));
+}
+int launch_mlstm_step(const Mlstm &a, const HeadGate &hg, void *stream)
+{
+    return launch_step<kMlstm>(mlstm_args(a), hg, nullptr, nullptr, nullptr, 0, static_cast<cudaStream_t>(stream));
+}
+
+}  // namespace mgq

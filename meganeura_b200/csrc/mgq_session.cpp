@@ -22,18 +22,25 @@
 // gate|up only); the original results are views into its output.  (2) The dispatch list can be
 // captured once into a CUDA graph and replayed per step.  (3) A greedy pick can run on the device
 // after the dispatches and feed the next token and position back, so consecutive decode steps need
-// no host round trip.
+// no host round trip.  (4) Row-dynamic graphs: activations whose leading dimension is a capacity
+// (input_u32_rows) run with the row count set by mgq_session_set_rows, so one session serves both a
+// prompt's portions and single-token steps; a captured CUDA graph is replayed for the row counts it
+// was captured with.  (5) Recurrent mixers (token shift, RWKV-style time mixing, mLSTM), latent
+// attention over a ring cache, clamped GLUs and bf16 linear layers, with their state in zero-filled
+// parameters that mgq_session_reset_state clears.
 #include <cuda_runtime.h>
 #include <nvtx3/nvToolsExt.h>
 
 #include <algorithm>
+#include <cmath>
 #include <cstdio>
 #include <cstring>
 #include <map>
 #include <string>
 #include <vector>
 
-#include "mgq_internal.h"
+#include "mgq_linear.cuh"
+#include "mgq_mixer.cuh"
 
 namespace {
 
@@ -41,7 +48,8 @@ constexpr int kU32 = 100;         // node dtype of input_u32 (not a weight forma
 
 enum class Op {
     Input, Parameter, MatMul, Add, FusedMatMulAdd, Embedding, RmsNorm, RoPE, CacheWrite, CachedAttention,
-    SwiGLU, SwiGLUConcat, AllGather, MatMulBT, View, Nop
+    SwiGLU, SwiGLUConcat, AllGather, MatMulBT, View, Nop,
+    BiasAdd, PickRows, Norm, TokenShift, Slot, Decay, Wkv, Mlstm, HeadGate, LatentCacheWrite, LatentAttention, ClampedGlu, LinearGlu
 };
 
 struct Node {
@@ -51,6 +59,10 @@ struct Node {
     int dtype;                    // MGQ_FMT_F32 / Q4 / Q8, or kU32
     std::vector<int> inputs;
     float f0 = 0.f;               // eps (RmsNorm), theta (RoPE)
+    float f1 = 0.f, f2 = 0.f;
+    int rows = 0;                 // leading dimension: 0 fixed, MGQ_ROWS_TOKENS / MGQ_ROWS_PICKED: set per step
+    std::vector<uint32_t> at;     // integer attributes of the recurrent and latent operators
+    bool absorbed = false;        // runs inside the dispatch of its consumer (keeps its buffer)
     uint32_t u0 = 0, u1 = 0, u2 = 0;   // head_dim (RoPE); num_heads, num_kv_heads, head_dim (CachedAttention); column offset (View)
     size_t elements() const { size_t e = 1; for (size_t s : shape) e *= s; return e; }
 };
@@ -65,6 +77,7 @@ struct Dispatch {
     int weight_format;
     float f0;
     void *workspace;
+    std::vector<int> members;     // linear group: the node of each layer
     int exchange = -1;            // all_gather: which exchange; GEMV: the exchange it pushes its columns to (-1: none)
     bool push_done = false;       // all_gather: the producing GEMV has pushed the slice already
     std::string label;
@@ -106,12 +119,26 @@ const char *shader_name(int s)
         case MGQ_SHADER_ROPE_CACHE_WRITE: return "RoPEDynamic+CacheWrite";
         case MGQ_SHADER_ALL_GATHER: return "AllGather";
         case MGQ_SHADER_MATMUL_GEMV_BT: return "MatMulGemvBT";
+        case MGQ_SHADER_LINEAR: return "Linear";
+        case MGQ_SHADER_LINEAR_GLU: return "LinearGLU";
+        case MGQ_SHADER_BIAS_ADD: return "BiasAdd";
+        case MGQ_SHADER_PICK_ROWS: return "PickRows";
+        case MGQ_SHADER_NORM: return "Norm";
+        case MGQ_SHADER_TOKEN_SHIFT: return "TokenShift";
+        case MGQ_SHADER_DECAY: return "Decay";
+        case MGQ_SHADER_WKV: return "Wkv";
+        case MGQ_SHADER_MLSTM: return "Mlstm";
+        case MGQ_SHADER_HEAD_GATE: return "HeadGate";
+        case MGQ_SHADER_LATENT_CACHE_WRITE: return "LatentCacheWrite";
+        case MGQ_SHADER_LATENT_ATTENTION: return "LatentAttention";
+        case MGQ_SHADER_CLAMPED_GLU: return "ClampedGLU";
     }
     return "?";
 }
 
 int g_fuse_rope_cache = 1;        // "session.fuse_rope_cache"
 int g_horizontal_fusion = 2;      // "session.horizontal_fusion": 0 none, 1 gate|up only (the reference's), 2 every same-input GEMV group
+int g_fuse_mixer = 1;             // "session.fuse_mixer": biases, residuals, GLUs, gates, norms and same-shape linear layers merge
 int g_fuse_exchange = 1;          // "session.fuse_exchange": a GEMV that feeds an all_gather pushes its columns itself
 
 // One all_gather of a column-sharded session: what the caller bound to it.
@@ -139,6 +166,10 @@ int set_session_option(const char *name, long value)
         g_fuse_exchange = value ? 1 : 0;
         return MGQ_OK;
     }
+    if (!std::strcmp(name, "session.fuse_mixer")) {
+        g_fuse_mixer = value ? 1 : 0;
+        return MGQ_OK;
+    }
     return fail(MGQ_ERR_NAME, "unknown option: %s", name);
 }
 }  // namespace mgq
@@ -164,6 +195,9 @@ struct mgq_session {
     cudaGraphExec_t graph_exec = nullptr;
     uint64_t launches = 0;
     int device = 0;
+    // row-dynamic graphs: capacity and current count per MGQ_ROWS_* index; counts of the captured graph
+    uint32_t row_cap[3] = {0, 0, 0}, row_count[3] = {0, 1, 1}, graph_rows[3] = {0, 0, 0};
+    std::vector<int> states;                   // parameters that mgq_session_reset_state clears
     // per-dispatch timing (set_profiling): one event before every dispatch and one after the last
     bool profiling = false, profiled = false;
     std::vector<cudaEvent_t> events;
@@ -183,6 +217,12 @@ struct mgq_session {
         const int b = node_buffer[node];
         return b < 0 ? nullptr : static_cast<uint8_t *>(buffers[b].dev) + node_offset[node];
     }
+    uint32_t rows_of(int node) const
+    {
+        const Node &nd = nodes[node];
+        return nd.rows ? row_count[nd.rows] : (uint32_t)nd.shape[0];
+    }
+    bool bf16(int node) const { return nodes[node].dtype == MGQ_FMT_BF16; }
 };
 
 using mgq::fail;
@@ -191,7 +231,7 @@ using mgq::fail;
 static size_t node_bytes(const Node &nd)
 {
     if (mgq::is_quant(nd.dtype)) return mgq_packed_bytes(nd.dtype, nd.shape[0], nd.shape[1]);
-    return nd.elements() * (nd.dtype == MGQ_FMT_F16 ? 2 : 4);
+    return nd.elements() * (nd.dtype == MGQ_FMT_F16 || nd.dtype == MGQ_FMT_BF16 ? 2 : 4);
 }
 
 static int add_leaf(mgq_graph *g, Op op, const char *name, const size_t *shape, size_t rank, int dtype)
@@ -233,6 +273,15 @@ int mgq_graph_parameter_q8(mgq_graph *g, const char *name, const size_t *shape, 
 { return add_leaf(g, Op::Parameter, name, shape, rank, MGQ_FMT_Q8); }
 int mgq_graph_parameter_f16(mgq_graph *g, const char *name, const size_t *shape, size_t rank)
 { return add_leaf(g, Op::Parameter, name, shape, rank, MGQ_FMT_F16); }
+int mgq_graph_parameter_bf16(mgq_graph *g, const char *name, const size_t *shape, size_t rank)
+{ return add_leaf(g, Op::Parameter, name, shape, rank, MGQ_FMT_BF16); }
+int mgq_graph_input_u32_rows(mgq_graph *g, const char *name, size_t capacity, int which)
+{
+    if (which != MGQ_ROWS_TOKENS && which != MGQ_ROWS_PICKED) return -fail(MGQ_ERR_SHAPE, "input_u32_rows: unknown row set %d", which);
+    const int id = add_leaf(g, Op::Input, name, &capacity, 1, kU32);
+    if (id >= 0) g->nodes[id].rows = which;
+    return id;
+}
 
 int mgq_graph_matmul(mgq_graph *g, int a, int b)
 {
@@ -252,7 +301,13 @@ int mgq_graph_matmul_bt(mgq_graph *g, int a, int b)
     const Node &na = g->nodes[a], &nb = g->nodes[b];
     if (na.shape.size() != 2 || nb.shape.size() != 2) return -fail(MGQ_ERR_SHAPE, "matmul_bt requires 2D tensors");
     if (na.shape[1] != nb.shape[1]) return -fail(MGQ_ERR_SHAPE, "MatMulBT: K dimensions must match (%zu vs %zu)", na.shape[1], nb.shape[1]);
-    if (na.dtype != MGQ_FMT_F32 || nb.dtype != MGQ_FMT_F32) return -fail(MGQ_ERR_FORMAT, "matmul_bt: both operands must be f32");
+    if (nb.dtype == MGQ_FMT_BF16 && nb.op == Op::Parameter) {            // linear layer over a bf16 weight
+        if (na.dtype != MGQ_FMT_F32 && na.dtype != MGQ_FMT_BF16) return -fail(MGQ_ERR_FORMAT, "matmul_bt: activations must be f32 or bf16");
+        Node nd{Op::MatMulBT, "", {na.shape[0], nb.shape[0]}, MGQ_FMT_F32, {a, b, -1, -1}};
+        nd.rows = na.rows;
+        return push_node(g, std::move(nd));
+    }
+    if (na.dtype != MGQ_FMT_F32 || nb.dtype != MGQ_FMT_F32) return -fail(MGQ_ERR_FORMAT, "matmul_bt: the weight must be f32, or a bf16 parameter");
     return push_node(g, Node{Op::MatMulBT, "", {na.shape[0], nb.shape[0]}, MGQ_FMT_F32, {a, b}});
 }
 
@@ -263,7 +318,10 @@ int mgq_graph_add(mgq_graph *g, int a, int b)
     const Node &na = g->nodes[a], &nb = g->nodes[b];
     if (na.shape != nb.shape) return -fail(MGQ_ERR_SHAPE, "add: shapes differ");
     if (na.dtype != MGQ_FMT_F32 || nb.dtype != MGQ_FMT_F32) return -fail(MGQ_ERR_FORMAT, "add: operands must be f32");
-    return push_node(g, Node{Op::Add, "", na.shape, MGQ_FMT_F32, {a, b}});
+    if (na.rows != nb.rows) return -fail(MGQ_ERR_SHAPE, "add: row sets differ");
+    Node nd{Op::Add, "", na.shape, MGQ_FMT_F32, {a, b}};
+    nd.rows = na.rows;
+    return push_node(g, std::move(nd));
 }
 
 int mgq_graph_embedding(mgq_graph *g, int indices, int table)
@@ -382,6 +440,239 @@ int mgq_graph_all_gather(mgq_graph *g, int x, uint32_t world)
     if (world < 1 || world > MGQ_MAX_PEERS) return -fail(MGQ_ERR_SHAPE, "all_gather: world must be 1..%d", MGQ_MAX_PEERS);
     Node nd{Op::AllGather, "", {1, nx.shape[1] * world}, MGQ_FMT_F32, {x}};
     nd.u0 = world;
+    return push_node(g, std::move(nd));
+}
+
+}  // extern "C"
+
+// ---- operators of decoders with recurrent and latent-attention mixers
+namespace {
+
+bool is_param(const mgq_graph *g, int id, int dtype, size_t elements)
+{
+    const Node &n = g->nodes[id];
+    return n.op == Op::Parameter && n.dtype == dtype && (elements == 0 || n.elements() == elements);
+}
+bool is_act(const mgq_graph *g, int id, size_t rows, size_t cols, int row_set)       // f32 [rows, cols]
+{
+    const Node &n = g->nodes[id];
+    return n.dtype == MGQ_FMT_F32 && n.shape.size() == 2 && n.shape[0] == rows && n.shape[1] == cols && n.rows == row_set;
+}
+bool operand_dtype(int dtype) { return dtype == MGQ_FMT_F32 || dtype == MGQ_FMT_BF16; }
+bool all_valid(const mgq_graph *g, std::initializer_list<int> ids)
+{
+    for (int id : ids)
+        if (!valid(g, id)) return false;
+    return true;
+}
+
+}  // namespace
+
+extern "C" {
+
+int mgq_graph_embedding_scaled(mgq_graph *g, int indices, int table, float scale)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {indices, table})) return -fail(MGQ_ERR_NAME, "embedding: node id out of range");
+    const Node &ni = g->nodes[indices], &nt = g->nodes[table];
+    if (ni.dtype != kU32 || ni.shape.size() != 1) return -fail(MGQ_ERR_FORMAT, "embedding indices must be 1D U32");
+    if (nt.shape.size() != 2 || !operand_dtype(nt.dtype)) return -fail(MGQ_ERR_SHAPE, "embedding table must be 2D f32 or bf16");
+    Node nd{Op::Embedding, "", {ni.shape[0], nt.shape[1]}, MGQ_FMT_F32, {indices, table}};
+    nd.f0 = scale;
+    nd.u0 = 1;                            // scaled form
+    nd.rows = ni.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_pick_rows(mgq_graph *g, int x, int index)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {x, index})) return -fail(MGQ_ERR_NAME, "pick_rows: node id out of range");
+    const Node &nx = g->nodes[x], &ni = g->nodes[index];
+    if (nx.shape.size() != 2 || nx.dtype != MGQ_FMT_F32) return -fail(MGQ_ERR_SHAPE, "pick_rows takes a 2D f32 tensor");
+    if (ni.dtype != kU32 || ni.shape.size() != 1) return -fail(MGQ_ERR_FORMAT, "pick_rows indices must be 1D U32");
+    Node nd{Op::PickRows, "", {ni.shape[0], nx.shape[1]}, MGQ_FMT_F32, {x, index}};
+    nd.rows = ni.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_norm(mgq_graph *g, int x, int weight, float eps, float weight_offset, int out_dtype)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {x, weight})) return -fail(MGQ_ERR_NAME, "norm: node id out of range");
+    const Node &nx = g->nodes[x];
+    if (nx.shape.size() != 2 || nx.dtype != MGQ_FMT_F32) return -fail(MGQ_ERR_SHAPE, "norm takes a 2D f32 tensor");
+    if (!is_param(g, weight, MGQ_FMT_F32, nx.shape[1])) return -fail(MGQ_ERR_SHAPE, "norm weight must be an f32 parameter of %zu elements", nx.shape[1]);
+    if (!operand_dtype(out_dtype)) return -fail(MGQ_ERR_FORMAT, "norm: output must be f32 or bf16");
+    Node nd{Op::Norm, "", nx.shape, out_dtype, {x, weight, -1}};
+    nd.f0 = eps; nd.f1 = weight_offset;
+    nd.rows = nx.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_bias_add(mgq_graph *g, int x, int bias)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {x, bias})) return -fail(MGQ_ERR_NAME, "bias_add: node id out of range");
+    const Node &nx = g->nodes[x];
+    if (nx.shape.size() != 2 || nx.dtype != MGQ_FMT_F32) return -fail(MGQ_ERR_SHAPE, "bias_add takes a 2D f32 tensor");
+    if (!is_param(g, bias, MGQ_FMT_F32, nx.shape[1])) return -fail(MGQ_ERR_SHAPE, "bias must be an f32 parameter of %zu elements", nx.shape[1]);
+    Node nd{Op::BiasAdd, "", nx.shape, MGQ_FMT_F32, {x, bias}};
+    nd.rows = nx.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_clamped_glu(mgq_graph *g, int gate, int up, float limit, float alpha, int out_dtype)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {gate, up})) return -fail(MGQ_ERR_NAME, "clamped_glu: node id out of range");
+    const Node &ng = g->nodes[gate], &nu = g->nodes[up];
+    if (ng.shape.size() != 2 || ng.shape != nu.shape || ng.rows != nu.rows) return -fail(MGQ_ERR_SHAPE, "clamped_glu: shapes differ");
+    if (ng.dtype != MGQ_FMT_F32 || nu.dtype != MGQ_FMT_F32 || !operand_dtype(out_dtype)) return -fail(MGQ_ERR_FORMAT, "clamped_glu: f32 operands, f32 or bf16 output");
+    Node nd{Op::ClampedGlu, "", ng.shape, out_dtype, {gate, up}};
+    nd.f0 = limit; nd.f1 = alpha;
+    nd.rows = ng.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_token_shift(mgq_graph *g, int h, const int *mu, size_t count, int state, int out_dtype)
+{
+    if (!g || !mu) return -fail(MGQ_ERR_NULL, "null argument");
+    if (count == 0 || count > (size_t)mgq::kMaxShifts) return -fail(MGQ_ERR_SHAPE, "token_shift: %zu mixes (1..%d)", count, mgq::kMaxShifts);
+    if (!all_valid(g, {h, state})) return -fail(MGQ_ERR_NAME, "token_shift: node id out of range");
+    const Node &nh = g->nodes[h];
+    if (nh.shape.size() != 2 || nh.dtype != MGQ_FMT_F32 || !operand_dtype(out_dtype)) return -fail(MGQ_ERR_SHAPE, "token_shift takes a 2D f32 tensor");
+    const size_t width = nh.shape[1];
+    if (!is_param(g, state, MGQ_FMT_F32, 2 * width)) return -fail(MGQ_ERR_SHAPE, "token_shift state must be an f32 parameter [2, %zu]", width);
+    Node nd{Op::TokenShift, "", {count, nh.shape[0], width}, out_dtype, {h, state, -1}};
+    for (size_t i = 0; i < count; i++) {
+        if (!valid(g, mu[i]) || !is_param(g, mu[i], MGQ_FMT_F32, width)) return -fail(MGQ_ERR_SHAPE, "token_shift: mix %zu must be an f32 parameter of %zu elements", i, width);
+        nd.inputs.push_back(mu[i]);
+    }
+    nd.rows = nh.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_slot(mgq_graph *g, int x, uint32_t index)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!valid(g, x)) return -fail(MGQ_ERR_NAME, "slot: node id out of range");
+    const Node &nx = g->nodes[x];
+    if (nx.shape.size() != 3 || index >= nx.shape[0]) return -fail(MGQ_ERR_SHAPE, "slot %u of a tensor without that many matrices", index);
+    Node nd{Op::Slot, "", {nx.shape[1], nx.shape[2]}, nx.dtype, {x}};
+    nd.u0 = index;
+    nd.rows = nx.rows;
+    return push_node(g, std::move(nd));
+}
+
+size_t mgq_wkv_state_elements(uint32_t heads, uint32_t dim) { return mgq::wkv_state_elements(heads, dim); }
+size_t mgq_mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim) { return mgq::mlstm_state_elements(heads, dim, vdim); }
+
+int mgq_graph_lora_decay(mgq_graph *g, int low, int w2, int w0)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {low, w2, w0})) return -fail(MGQ_ERR_NAME, "lora_decay: node id out of range");
+    const Node &nl = g->nodes[low], &nw = g->nodes[w2];
+    if (nl.shape.size() != 2 || nl.dtype != MGQ_FMT_F32) return -fail(MGQ_ERR_SHAPE, "lora_decay takes a 2D f32 tensor");
+    if (nw.op != Op::Parameter || nw.dtype != MGQ_FMT_BF16 || nw.shape.size() != 2 || nw.shape[1] != nl.shape[1]) return -fail(MGQ_ERR_SHAPE, "lora_decay: w2 must be a bf16 parameter [channels, %zu]", nl.shape[1]);
+    if (!is_param(g, w0, MGQ_FMT_F32, nw.shape[0])) return -fail(MGQ_ERR_SHAPE, "lora_decay: w0 must be an f32 parameter of %zu elements", nw.shape[0]);
+    Node nd{Op::Decay, "", {nl.shape[0], nw.shape[0]}, MGQ_FMT_F32, {low, w2, w0}};
+    nd.rows = nl.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_wkv(mgq_graph *g, int r, int k, int v, int decay, int u, int state, int shift_state, uint32_t heads)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {r, k, v, decay, u, state}) || (shift_state >= 0 && !valid(g, shift_state))) return -fail(MGQ_ERR_NAME, "wkv: node id out of range");
+    const Node &nr = g->nodes[r];
+    if (nr.shape.size() != 2 || heads == 0 || nr.shape[1] % heads) return -fail(MGQ_ERR_SHAPE, "wkv: width does not divide over %u heads", heads);
+    const uint32_t dim = (uint32_t)(nr.shape[1] / heads);
+    if (dim > mgq::kMaxStateDim) return -fail(MGQ_ERR_SHAPE, "wkv: heads of %u dimensions (at most %u)", dim, mgq::kMaxStateDim);
+    for (int id : {r, k, v, decay})
+        if (!is_act(g, id, nr.shape[0], nr.shape[1], nr.rows)) return -fail(MGQ_ERR_SHAPE, "wkv: r, k, v and the decay must be f32 of one shape");
+    if (!is_param(g, u, MGQ_FMT_F32, nr.shape[1])) return -fail(MGQ_ERR_SHAPE, "wkv: u must be an f32 parameter of %zu elements", nr.shape[1]);
+    if (!is_param(g, state, MGQ_FMT_F32, mgq::wkv_state_elements(heads, dim))) return -fail(MGQ_ERR_SHAPE, "wkv: state must be an f32 parameter of %zu elements", mgq::wkv_state_elements(heads, dim));
+    if (shift_state >= 0 && !is_param(g, shift_state, MGQ_FMT_F32, 0)) return -fail(MGQ_ERR_SHAPE, "wkv: the shift state must be an f32 parameter");
+    Node nd{Op::Wkv, "", nr.shape, MGQ_FMT_F32, {r, k, v, decay, u, state, shift_state}};
+    nd.at = {heads, dim};
+    nd.rows = nr.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_mlstm(mgq_graph *g, int q, int k, int v, int gate_i, int gate_f, int state, uint32_t heads, float gate_cap)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {q, k, v, gate_i, gate_f, state})) return -fail(MGQ_ERR_NAME, "mlstm: node id out of range");
+    const Node &nq = g->nodes[q], &nv = g->nodes[v];
+    if (nq.shape.size() != 2 || nv.shape.size() != 2 || heads == 0 || nq.shape[1] % heads || nv.shape[1] % heads) return -fail(MGQ_ERR_SHAPE, "mlstm: widths do not divide over %u heads", heads);
+    const uint32_t dim = (uint32_t)(nq.shape[1] / heads), vdim = (uint32_t)(nv.shape[1] / heads);
+    if (dim > mgq::kMaxStateDim) return -fail(MGQ_ERR_SHAPE, "mlstm: heads of %u key dimensions (at most %u)", dim, mgq::kMaxStateDim);
+    if (!is_act(g, q, nq.shape[0], nq.shape[1], nq.rows) || !is_act(g, k, nq.shape[0], nq.shape[1], nq.rows) ||
+        !is_act(g, v, nq.shape[0], nv.shape[1], nq.rows) || !is_act(g, gate_i, nq.shape[0], heads, nq.rows) || !is_act(g, gate_f, nq.shape[0], heads, nq.rows))
+        return -fail(MGQ_ERR_SHAPE, "mlstm: q, k, v and the gates must be f32 rows of matching shapes");
+    if (!(gate_cap > 0.f)) return -fail(MGQ_ERR_SHAPE, "mlstm: the gate cap must be positive");
+    if (!is_param(g, state, MGQ_FMT_F32, mgq::mlstm_state_elements(heads, dim, vdim))) return -fail(MGQ_ERR_SHAPE, "mlstm: state must be an f32 parameter of %zu elements", mgq::mlstm_state_elements(heads, dim, vdim));
+    Node nd{Op::Mlstm, "", nv.shape, MGQ_FMT_F32, {q, k, v, gate_i, gate_f, state}};
+    nd.f0 = gate_cap;
+    nd.at = {heads, dim, vdim};
+    nd.rows = nq.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_head_gate(mgq_graph *g, int o, int weight, int gate, uint32_t heads, float eps, int act, int out_dtype)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {o, gate}) || (weight >= 0 && !valid(g, weight))) return -fail(MGQ_ERR_NAME, "head_gate: node id out of range");
+    const Node &no = g->nodes[o];
+    if (no.shape.size() != 2 || heads == 0 || no.shape[1] % heads) return -fail(MGQ_ERR_SHAPE, "head_gate: width does not divide over %u heads", heads);
+    if (!is_act(g, o, no.shape[0], no.shape[1], no.rows) || !is_act(g, gate, no.shape[0], no.shape[1], no.rows)) return -fail(MGQ_ERR_SHAPE, "head_gate: the gate must have the shape of its input");
+    if (weight >= 0 && !is_param(g, weight, MGQ_FMT_F32, no.shape[1])) return -fail(MGQ_ERR_SHAPE, "head_gate: weight must be an f32 parameter of %zu elements", no.shape[1]);
+    if (act != MGQ_GATE_SIGMOID && act != MGQ_GATE_SILU) return -fail(MGQ_ERR_FORMAT, "head_gate: unknown activation %d", act);
+    if (!operand_dtype(out_dtype)) return -fail(MGQ_ERR_FORMAT, "head_gate: output must be f32 or bf16");
+    Node nd{Op::HeadGate, "", no.shape, out_dtype, {o, gate, weight}};
+    nd.f0 = eps;
+    nd.at = {heads, (uint32_t)act};
+    nd.rows = no.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_latent_cache_write(mgq_graph *g, int down, int weight, int cache, int pos, uint32_t rot_dim, float rot_base, float eps)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {down, weight, cache, pos})) return -fail(MGQ_ERR_NAME, "latent_cache_write: node id out of range");
+    const Node &nd_ = g->nodes[down], &nc = g->nodes[cache];
+    if (nd_.shape.size() != 2 || nd_.dtype != MGQ_FMT_F32 || rot_dim % 2 || nd_.shape[1] <= rot_dim) return -fail(MGQ_ERR_SHAPE, "latent_cache_write: rows of rank + rot_dim f32 elements, rot_dim even");
+    if (nc.op != Op::Parameter || !operand_dtype(nc.dtype) || nc.shape.size() != 2 || nc.shape[1] != nd_.shape[1]) return -fail(MGQ_ERR_SHAPE, "latent_cache_write: the cache must be an f32 or bf16 parameter [slots, %zu]", nd_.shape[1]);
+    if (nc.shape[0] < nd_.shape[0]) return -fail(MGQ_ERR_SHAPE, "latent_cache_write: %zu cache rows for %zu tokens", nc.shape[0], nd_.shape[0]);
+    const size_t rank = nd_.shape[1] - rot_dim;
+    if (!is_param(g, weight, MGQ_FMT_F32, rank)) return -fail(MGQ_ERR_SHAPE, "latent_cache_write: weight must be an f32 parameter of %zu elements", rank);
+    if (g->nodes[pos].dtype != kU32) return -fail(MGQ_ERR_FORMAT, "pos must be a U32 input");
+    Node nd{Op::LatentCacheWrite, "", nc.shape, nc.dtype, {down, weight, cache, pos}};
+    nd.f0 = eps; nd.f1 = rot_base;
+    nd.at = {(uint32_t)rank, rot_dim, (uint32_t)nc.shape[0]};
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_latent_attention(mgq_graph *g, int q, int cache, int uk, int uv, int pos, uint32_t heads, uint32_t dim, uint32_t rot_dim, uint32_t vdim,
+                               uint32_t window, float scale, float rot_base)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {q, cache, uk, uv, pos})) return -fail(MGQ_ERR_NAME, "latent_attention: node id out of range");
+    const Node &nq = g->nodes[q], &nc = g->nodes[cache];
+    if (heads == 0 || dim == 0 || vdim == 0 || rot_dim % 2 || nq.shape.size() != 2 || nq.dtype != MGQ_FMT_F32 || nq.shape[1] != (size_t)heads * (dim + rot_dim))
+        return -fail(MGQ_ERR_SHAPE, "latent_attention: q must be f32 rows of heads * (dim + rot_dim)");
+    if (nc.shape.size() != 2 || !operand_dtype(nc.dtype) || nc.shape[1] <= rot_dim) return -fail(MGQ_ERR_SHAPE, "latent_attention: the cache must be [slots, rank + rot_dim]");
+    const size_t rank = nc.shape[1] - rot_dim;
+    if (rank > 1024) return -fail(MGQ_ERR_SHAPE, "latent_attention: a latent of %zu elements (at most 1024)", rank);
+    if (!is_param(g, uk, MGQ_FMT_BF16, (size_t)heads * dim * rank) || !is_param(g, uv, MGQ_FMT_BF16, (size_t)heads * vdim * rank))
+        return -fail(MGQ_ERR_SHAPE, "latent_attention: W_uk and W_uv must be bf16 parameters [heads * dim, rank]");
+    if (window == 0 || window + nq.shape[0] - 1 > nc.shape[0]) return -fail(MGQ_ERR_SHAPE, "latent_attention: a window of %u and %zu rows need %zu cache rows, there are %zu", window, nq.shape[0], window + nq.shape[0] - 1, nc.shape[0]);
+    if (g->nodes[pos].dtype != kU32) return -fail(MGQ_ERR_FORMAT, "pos must be a U32 input");
+    Node nd{Op::LatentAttention, "", {nq.shape[0], (size_t)heads * vdim}, MGQ_FMT_F32, {q, cache, uk, uv, pos}};
+    nd.f0 = scale; nd.f1 = rot_base;
+    nd.at = {heads, dim, rot_dim, vdim, (uint32_t)rank, (uint32_t)nc.shape[0], window};
+    nd.rows = nq.rows;
     return push_node(g, std::move(nd));
 }
 
@@ -533,6 +824,89 @@ void merge_rope_cache(mgq_session *s)
     }
 }
 
+// Producer-consumer merges of the recurrent / latent operators.  A merged producer turns into Nop, or
+// stays "absorbed" when its consumer's dispatch still needs its buffer.
+void fuse_mixers(mgq_session *s)
+{
+    std::vector<Node> &nodes = s->nodes;
+    auto is_output = [&](int id) { for (int o : s->outputs) if (o == id) return true; return false; };
+    auto single = [&](int id) { return count_uses(nodes, id) == 1 && !is_output(id); };
+    auto linear = [&](int id) { return nodes[id].op == Op::MatMulBT && nodes[id].inputs.size() == 4; };
+    auto drop = [&](int id) { nodes[id].op = Op::Nop; nodes[id].inputs.clear(); };
+    for (size_t id = 0; id < nodes.size(); id++) {
+        Node &nd = nodes[id];
+        if (nd.op == Op::BiasAdd) {
+            const int mm = nd.inputs[0];
+            if (!linear(mm) || !single(mm) || nodes[mm].inputs[2] >= 0 || nodes[mm].inputs[3] >= 0) continue;
+            nd.op = Op::MatMulBT;
+            nd.inputs = {nodes[mm].inputs[0], nodes[mm].inputs[1], nd.inputs[1], -1};
+            drop(mm);
+        } else if (nd.op == Op::Add) {
+            int mm = -1, addend = -1;
+            for (int side = 0; side < 2 && mm < 0; side++)
+                if (linear(nd.inputs[side]) && single(nd.inputs[side]) && nodes[nd.inputs[side]].inputs[3] < 0) { mm = nd.inputs[side]; addend = nd.inputs[1 - side]; }
+            if (mm < 0 || mm == addend) continue;
+            nd.op = Op::MatMulBT;
+            nd.inputs = {nodes[mm].inputs[0], nodes[mm].inputs[1], nodes[mm].inputs[2], addend};
+            drop(mm);
+        } else if (nd.op == Op::ClampedGlu) {
+            const int ga = nd.inputs[0], up = nd.inputs[1];
+            if (ga == up || !linear(ga) || !linear(up) || !single(ga) || !single(up)) continue;
+            const std::vector<int> &a = nodes[ga].inputs, &b = nodes[up].inputs;
+            if (a[0] != b[0] || a[2] < 0 || b[2] < 0 || a[3] >= 0 || b[3] >= 0) continue;
+            nd.op = Op::LinearGlu;
+            nd.inputs = {a[0], a[1], a[2], b[1], b[2]};
+            drop(ga);
+            drop(up);
+        } else if (nd.op == Op::Norm) {
+            const int x = nd.inputs[0];
+            if (nodes[x].op != Op::PickRows || !single(x)) continue;
+            nd.inputs = {nodes[x].inputs[0], nd.inputs[1], nodes[x].inputs[1]};
+            drop(x);
+        } else if (nd.op == Op::TokenShift) {
+            const int h = nd.inputs[0];
+            if (nodes[h].op != Op::Norm || nodes[h].inputs[2] >= 0 || nodes[h].dtype != MGQ_FMT_F32 || !single(h)) continue;
+            nd.inputs[0] = nodes[h].inputs[0];
+            nd.inputs[2] = nodes[h].inputs[1];
+            nd.f0 = nodes[h].f0; nd.f1 = nodes[h].f1;
+            drop(h);
+        } else if (nd.op == Op::HeadGate) {
+            const int o = nd.inputs[0];
+            const Op producer = nodes[o].op;
+            if (!single(o) || nodes[o].rows != nd.rows) continue;
+            const bool recurrent = producer == Op::Wkv || producer == Op::Mlstm;
+            if (recurrent && nd.inputs[2] >= 0 && nodes[o].at[0] == nd.at[0]) nodes[o].absorbed = true;
+            if (producer == Op::Wkv && nodes[o].absorbed) {
+                const int w = nodes[o].inputs[3];
+                if (nodes[w].op == Op::Decay && single(w)) nodes[w].absorbed = true;
+                else nodes[o].absorbed = false;
+            }
+            if (producer == Op::LatentAttention && nd.inputs[2] < 0) nodes[o].absorbed = true;
+        }
+    }
+}
+
+// Consecutive independent bf16 linear layers of one K, row set and activation type form one dispatch.
+void group_linears(mgq_session *s)
+{
+    std::vector<Dispatch> &ds = s->dispatches;
+    for (size_t i = 0; i + 1 < ds.size(); ) {
+        Dispatch &a = ds[i];
+        const Dispatch &b = ds[i + 1];
+        bool merge = a.shader == MGQ_SHADER_LINEAR && b.shader == MGQ_SHADER_LINEAR && a.members.size() + b.members.size() <= mgq::kMaxSegments;
+        if (merge) {
+            const Node &na = s->nodes[a.members[0]], &nb = s->nodes[b.members[0]];
+            merge = s->nodes[na.inputs[1]].shape[1] == s->nodes[nb.inputs[1]].shape[1] && na.rows == nb.rows && na.shape[0] == nb.shape[0] &&
+                    s->nodes[na.inputs[0]].dtype == s->nodes[nb.inputs[0]].dtype;
+            for (int m : a.members) merge = merge && nb.inputs[0] != m && nb.inputs[3] != m;
+        }
+        if (!merge) { i++; continue; }
+        a.members.insert(a.members.end(), b.members.begin(), b.members.end());
+        a.out = b.out;
+        ds.erase(ds.begin() + i + 1);
+    }
+}
+
 void set_label(Dispatch &d, const char *fmt, ...)
 {
     char lab[128];
@@ -541,6 +915,31 @@ void set_label(Dispatch &d, const char *fmt, ...)
     std::vsnprintf(lab, sizeof lab, fmt, ap);
     va_end(ap);
     d.label = lab;
+}
+
+// freq_i = base^(-2i / dims), rounded once from f64; the buffer is the dispatch's workspace.
+int rotation_table(mgq_session *s, uint32_t dims, float base, Dispatch &d)
+{
+    if (dims == 0) return MGQ_OK;
+    std::vector<float> freq(dims / 2);
+    for (uint32_t i = 0; i < dims / 2; i++) freq[i] = (float)std::pow((double)base, -2.0 * i / dims);
+    if (int rc = mgq_buffer_create(freq.size() * 4, &d.workspace)) return rc;
+    s->workspaces.push_back(d.workspace);
+    return mgq_buffer_upload(d.workspace, freq.data(), freq.size() * 4, s->stream);
+}
+
+// Rotation table first (padded to 256 bytes), then the attention kernels' scratch.
+size_t rotation_bytes(uint32_t dims) { return ((size_t)dims * 2 + 255) & ~(size_t)255; }
+int latent_workspace(mgq_session *s, const Node &nd, Dispatch &d)
+{
+    const std::vector<uint32_t> &a = nd.at;
+    const size_t rot = rotation_bytes(a[2]);
+    const size_t bytes = mgq::latent_attention_workspace((uint32_t)nd.shape[0], a[0], a[1], a[2], a[3], a[4], a[5], a[6], s->nodes[nd.inputs[1]].dtype == MGQ_FMT_BF16);
+    if (int rc = mgq_buffer_create(rot + bytes, &d.workspace)) return rc;
+    s->workspaces.push_back(d.workspace);
+    std::vector<float> freq(a[2] / 2);
+    for (uint32_t i = 0; i < a[2] / 2; i++) freq[i] = (float)std::pow((double)nd.f1, -2.0 * i / a[2]);
+    return freq.empty() ? MGQ_OK : mgq_buffer_upload(d.workspace, freq.data(), freq.size() * 4, s->stream);
 }
 
 }  // namespace
@@ -557,6 +956,12 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
     s->outputs = g->outputs;
     for (size_t id = 0; id < s->nodes.size(); id++) s->order.push_back((int)id);
 
+    if (g_fuse_mixer) fuse_mixers(s);
+    for (const Node &nd : s->nodes)
+        if (nd.op == Op::Input && nd.rows) {
+            uint32_t &cap = s->row_cap[nd.rows];
+            cap = cap ? std::min(cap, (uint32_t)nd.shape[0]) : (uint32_t)nd.shape[0];
+        }
     fuse_matmul_add(s);
     fuse_horizontal(s, g_horizontal_fusion);
 
@@ -572,6 +977,16 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
         if (nd.op == Op::View) {
             s->node_buffer[id] = s->node_buffer[nd.inputs[0]];
             s->node_offset[id] = s->node_offset[nd.inputs[0]] + (size_t)nd.u0 * 4;
+            continue;
+        }
+        if (nd.op == Op::Slot) {
+            s->node_buffer[id] = s->node_buffer[nd.inputs[0]];
+            s->node_offset[id] = s->node_offset[nd.inputs[0]] + (size_t)nd.u0 * node_bytes(nd);
+            continue;
+        }
+        if (nd.op == Op::LatentCacheWrite) {
+            s->node_buffer[id] = s->node_buffer[nd.inputs[2]];
+            s->node_offset[id] = s->node_offset[nd.inputs[2]];
             continue;
         }
         if (nd.op == Op::CacheWrite) {
@@ -602,7 +1017,8 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
         for (size_t i = 0; i < nd.inputs.size() && i < 4; i++) d.in[i] = nd.inputs[i];
         d.out = id;
         d.weight_format = MGQ_FMT_F32;
-        d.workgroups[1] = d.workgroups[2] = 1;
+        d.workgroups[0] = d.workgroups[1] = d.workgroups[2] = 1;
+        if (nd.absorbed) continue;
         switch (nd.op) {
             case Op::MatMul:
             case Op::FusedMatMulAdd: {
@@ -633,6 +1049,12 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
             case Op::MatMulBT: {
                 const Node &na = s->nodes[nd.inputs[0]], &nb = s->nodes[nd.inputs[1]];
                 const uint32_t m = (uint32_t)na.shape[0], k = (uint32_t)na.shape[1], n = (uint32_t)nb.shape[0];
+                if (nb.dtype == MGQ_FMT_BF16) {
+                    d.shader = MGQ_SHADER_LINEAR;
+                    d.weight_format = MGQ_FMT_BF16;
+                    d.members = {id};
+                    break;                                   // labelled once the groups are known
+                }
                 if (m != 1 || k % 4 != 0) {          // the reference's tiled MatMulBT (m > 1) is outside this library
                     mgq_session_free(s);
                     return fail(MGQ_ERR_SHAPE, "matmul_bt: only the single-row form with K %% 4 == 0 is lowered (got %ux%ux%u)", m, n, k);
@@ -654,6 +1076,7 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
             case Op::Embedding: {
                 d.shader = MGQ_SHADER_EMBEDDING;
                 const uint32_t seq = (uint32_t)nd.shape[0], hidden = (uint32_t)nd.shape[1];
+                d.f0 = nd.f0;
                 d.workgroups[0] = (seq * hidden + 255) / 256;
                 d.params[0] = seq; d.params[1] = hidden; d.params[2] = (uint32_t)s->nodes[nd.inputs[1]].shape[0];
                 set_label(d, "Embedding[%ux%u]", seq, hidden);
@@ -745,11 +1168,97 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
                 }
                 break;
             }
-            default: continue;           // Input, Parameter, View, Nop: nothing to run
+            case Op::LinearGlu: {
+                d.shader = MGQ_SHADER_LINEAR_GLU;
+                d.weight_format = MGQ_FMT_BF16;
+                d.members = {id};
+                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = (uint32_t)s->nodes[nd.inputs[1]].shape[1]; d.params[2] = (uint32_t)nd.shape[1];
+                set_label(d, "LinearGLU[%ux%u]", d.params[2], d.params[1]);
+                break;
+            }
+            case Op::BiasAdd:
+            case Op::PickRows:
+            case Op::ClampedGlu: {
+                d.shader = nd.op == Op::BiasAdd ? MGQ_SHADER_BIAS_ADD : nd.op == Op::PickRows ? MGQ_SHADER_PICK_ROWS : MGQ_SHADER_CLAMPED_GLU;
+                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = (uint32_t)nd.shape[1];
+                set_label(d, "%s[%u]", shader_name(d.shader), d.params[1]);
+                break;
+            }
+            case Op::Norm: {
+                d.shader = MGQ_SHADER_NORM;
+                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = (uint32_t)nd.shape[1];
+                set_label(d, "Norm[%u]", d.params[1]);
+                break;
+            }
+            case Op::TokenShift: {
+                d.shader = MGQ_SHADER_TOKEN_SHIFT;
+                d.params[0] = (uint32_t)nd.shape[1]; d.params[1] = (uint32_t)nd.shape[2]; d.params[2] = (uint32_t)nd.shape[0];
+                set_label(d, "TokenShift[%ux%u]", d.params[2], d.params[1]);
+                s->states.push_back(nd.inputs[1]);
+                break;
+            }
+            case Op::Decay: {
+                d.shader = MGQ_SHADER_DECAY;
+                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = (uint32_t)nd.shape[1];
+                set_label(d, "Decay[%u]", d.params[1]);
+                break;
+            }
+            case Op::Wkv: {
+                d.shader = MGQ_SHADER_WKV;
+                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = nd.at[1];
+                set_label(d, "Wkv[%ux%u]", nd.at[0], nd.at[1]);
+                s->states.push_back(nd.inputs[5]);
+                break;
+            }
+            case Op::Mlstm: {
+                d.shader = MGQ_SHADER_MLSTM;
+                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = nd.at[1]; d.params[3] = nd.at[2];
+                set_label(d, "Mlstm[%ux%ux%u]", nd.at[0], nd.at[1], nd.at[2]);
+                s->states.push_back(nd.inputs[5]);
+                break;
+            }
+            case Op::HeadGate: {
+                const Node &o = s->nodes[nd.inputs[0]];
+                d.shader = o.absorbed && o.op == Op::Wkv ? MGQ_SHADER_WKV : o.absorbed && o.op == Op::Mlstm ? MGQ_SHADER_MLSTM
+                         : o.absorbed ? MGQ_SHADER_LATENT_ATTENTION : MGQ_SHADER_HEAD_GATE;
+                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = (uint32_t)(nd.shape[1] / nd.at[0]);
+                set_label(d, "%s%s[%ux%u]", o.absorbed ? shader_name(d.shader) : "", o.absorbed ? "+HeadGate" : "HeadGate", d.params[1], d.params[2]);
+                if (o.absorbed && o.op != Op::LatentAttention) s->states.push_back(o.inputs[5]);
+                if (!(o.absorbed && o.op == Op::LatentAttention)) break;
+                rc = latent_workspace(s, o, d);
+                if (rc) { mgq_session_free(s); return rc; }
+                break;
+            }
+            case Op::LatentCacheWrite: {
+                d.shader = MGQ_SHADER_LATENT_CACHE_WRITE;
+                d.params[0] = (uint32_t)s->nodes[nd.inputs[0]].shape[0]; d.params[1] = nd.at[0]; d.params[2] = nd.at[1]; d.params[3] = nd.at[2];
+                set_label(d, "LatentCacheWrite[%u+%u]", nd.at[0], nd.at[1]);
+                s->states.push_back(nd.inputs[2]);
+                rc = rotation_table(s, nd.at[1], nd.f1, d);
+                if (rc) { mgq_session_free(s); return rc; }
+                break;
+            }
+            case Op::LatentAttention: {
+                d.shader = MGQ_SHADER_LATENT_ATTENTION;
+                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = nd.at[4]; d.params[3] = nd.at[6];
+                set_label(d, "LatentAttention[%ux%u]", nd.at[0], nd.at[4]);
+                rc = latent_workspace(s, nd, d);
+                if (rc) { mgq_session_free(s); return rc; }
+                break;
+            }
+            default: continue;           // Input, Parameter, View, Slot, Nop: nothing to run
         }
         s->dispatches.push_back(d);
     }
     if (g_fuse_rope_cache) merge_rope_cache(s);
+    if (g_fuse_mixer) group_linears(s);
+    for (Dispatch &d : s->dispatches) {
+        if (d.shader != MGQ_SHADER_LINEAR) continue;
+        uint32_t n = 0;
+        for (int m : d.members) n += (uint32_t)s->nodes[m].shape[1];
+        d.params[0] = (uint32_t)s->nodes[d.out].shape[0]; d.params[1] = (uint32_t)s->nodes[s->nodes[d.out].inputs[1]].shape[1]; d.params[2] = n;
+        set_label(d, "Linear[%ux%u]%s", n, d.params[1], s->nodes[d.members[0]].inputs[3] >= 0 ? "+Add" : "");
+    }
     *out = s;
     return MGQ_OK;
 }
@@ -920,6 +1429,16 @@ int mgq_session_set_parameter(mgq_session *s, const char *name, const float *dat
         if (int rc = mgq_convert_f16(data, len, reinterpret_cast<uint16_t *>(s->staging.data()))) return rc;
         return mgq_buffer_upload(s->ptr(id), s->staging.data(), len * 2, s->stream);
     }
+    if (nd.dtype == MGQ_FMT_BF16) {
+        s->staging.resize(len * 2);
+        uint16_t *out = reinterpret_cast<uint16_t *>(s->staging.data());
+        for (size_t i = 0; i < len; i++) {               // round to nearest even; NaN stays NaN
+            uint32_t b;
+            std::memcpy(&b, data + i, 4);
+            out[i] = (b & 0x7FFFFFFFu) > 0x7F800000u ? (uint16_t)((b >> 16) | 0x40u) : (uint16_t)((b + 0x7FFFu + ((b >> 16) & 1u)) >> 16);
+        }
+        return mgq_buffer_upload(s->ptr(id), s->staging.data(), len * 2, s->stream);
+    }
     if (!mgq::is_quant(nd.dtype)) return mgq_buffer_upload(s->ptr(id), data, len * 4, s->stream);
     s->staging.resize(mgq_packed_bytes(nd.dtype, nd.shape[0], nd.shape[1]));
     const int rc = nd.dtype == MGQ_FMT_Q4 ? mgq_quantize_q4(data, nd.shape[0], nd.shape[1], s->staging.data())
@@ -955,8 +1474,154 @@ int mgq_session_set_input_u32(mgq_session *s, const char *name, const uint32_t *
     const int id = find_named(s, Op::Input, name);
     if (id < 0 || s->nodes[id].dtype != kU32) return fail(MGQ_ERR_NAME, "unknown u32 input: %s", name);
     const Node &nd = s->nodes[id];
-    if (len != nd.elements()) return fail(MGQ_ERR_SIZE, "input '%s' has %zu elements, got %zu", name, nd.elements(), len);
+    if (nd.rows ? len == 0 || len > nd.elements() : len != nd.elements()) return fail(MGQ_ERR_SIZE, "input '%s' has %zu elements, got %zu", name, nd.elements(), len);
     return mgq_buffer_upload(s->ptr(id), data, len * 4, s->stream);
+}
+
+int mgq_session_set_rows(mgq_session *s, int which, uint32_t count)
+{
+    if (!s) return fail(MGQ_ERR_NULL, "null session");
+    if ((which != MGQ_ROWS_TOKENS && which != MGQ_ROWS_PICKED) || s->row_cap[which] == 0) return fail(MGQ_ERR_NAME, "the graph has no row set %d", which);
+    if (count > s->row_cap[which] || (which == MGQ_ROWS_TOKENS && count == 0)) return fail(MGQ_ERR_SIZE, "row set %d holds up to %u rows, got %u", which, s->row_cap[which], count);
+    s->row_count[which] = count;
+    return MGQ_OK;
+}
+
+int mgq_session_reset_state(mgq_session *s)
+{
+    if (!s) return fail(MGQ_ERR_NULL, "null session");
+    for (int id : s->states) MGQ_CUDA(cudaMemsetAsync(s->ptr(id), 0, node_bytes(s->nodes[id]), s->stream));
+    return MGQ_OK;
+}
+
+static mgq::HeadGate head_gate_args(mgq_session *s, const Node &nd, int id)
+{
+    mgq::HeadGate hg{};
+    hg.gate = static_cast<const float *>(s->ptr(nd.inputs[1]));
+    hg.weight = nd.inputs[2] >= 0 ? static_cast<const float *>(s->ptr(nd.inputs[2])) : nullptr;
+    hg.out = s->ptr(id);
+    hg.out_bf16 = nd.dtype == MGQ_FMT_BF16;
+    hg.silu = nd.at[1] == MGQ_GATE_SILU;
+    hg.eps = nd.f0;
+    return hg;
+}
+
+static int run_linear(mgq_session *s, const Dispatch &d)
+{
+    mgq::LinearGroup g{};
+    g.count = (uint32_t)d.members.size();
+    g.glu = d.shader == MGQ_SHADER_LINEAR_GLU;
+    for (uint32_t i = 0; i < g.count; i++) {
+        const int id = d.members[i];
+        const Node &nd = s->nodes[id];
+        mgq::LinearSegment &sg = g.seg[i];
+        auto f = [&](int j) { return nd.inputs[j] >= 0 ? static_cast<const float *>(s->ptr(nd.inputs[j])) : nullptr; };
+        sg.a = s->ptr(nd.inputs[0]);
+        sg.w = s->ptr(nd.inputs[1]);
+        sg.bias = f(2);
+        if (g.glu) {
+            sg.w2 = s->ptr(nd.inputs[3]);
+            sg.bias2 = f(4);
+            g.limit = nd.f0; g.alpha = nd.f1;
+            g.out_bf16 = nd.dtype == MGQ_FMT_BF16;
+        } else {
+            sg.addend = f(3);
+        }
+        sg.out = s->ptr(id);
+        sg.n = (uint32_t)nd.shape[1];
+        g.m = s->rows_of(id);
+        g.k = (uint32_t)s->nodes[nd.inputs[1]].shape[1];
+        g.a_bf16 = s->bf16(nd.inputs[0]);
+    }
+    return mgq::launch_linear_group(g, s->stream);
+}
+
+// The recurrent, latent and row-dynamic operators.
+static int run_mixer(mgq_session *s, const Dispatch &d)
+{
+    const Node &nd = s->nodes[d.out];
+    const uint32_t rows = s->rows_of(d.out);
+    auto f = [&](int id) { return id >= 0 ? static_cast<float *>(s->ptr(id)) : nullptr; };
+    auto u = [&](int id) { return id >= 0 ? static_cast<uint32_t *>(s->ptr(id)) : nullptr; };
+    switch (nd.op) {
+        case Op::BiasAdd: return mgq::launch_bias_add(f(nd.inputs[0]), f(nd.inputs[1]), f(d.out), rows, d.params[1], s->stream);
+        case Op::PickRows: return mgq::launch_pick_rows(f(nd.inputs[0]), u(nd.inputs[1]), f(d.out), rows, s->rows_of(nd.inputs[0]), d.params[1], s->stream);
+        case Op::ClampedGlu: return mgq::launch_clamped_glu(f(nd.inputs[0]), f(nd.inputs[1]), s->ptr(d.out), s->bf16(d.out), (size_t)rows * d.params[1], nd.f0, nd.f1, s->stream);
+        case Op::Norm:
+            return mgq::launch_norm(f(nd.inputs[0]), f(nd.inputs[1]), u(nd.inputs[2]), s->ptr(d.out), s->bf16(d.out), rows, s->rows_of(nd.inputs[0]), d.params[1],
+                                    nd.f0, nd.f1, s->stream);
+        case Op::TokenShift: {
+            mgq::TokenShift a{};
+            a.x = f(nd.inputs[0]); a.state = f(nd.inputs[1]); a.norm_weight = f(nd.inputs[2]);
+            a.eps = nd.f0; a.offset = nd.f1;
+            a.slots = (uint32_t)nd.shape[0]; a.width = (uint32_t)nd.shape[2];
+            for (uint32_t i = 0; i < a.slots; i++) a.mu[i] = f(nd.inputs[3 + i]);
+            a.rows = s->rows_of(nd.inputs[0]);
+            a.out = s->ptr(d.out); a.out_bf16 = s->bf16(d.out); a.slot_stride = nd.shape[1] * nd.shape[2];
+            return mgq::launch_token_shift(a, s->stream);
+        }
+        case Op::LatentCacheWrite: {
+            mgq::LatentCache a{};
+            a.down = f(nd.inputs[0]); a.weight = f(nd.inputs[1]); a.cache = s->ptr(nd.inputs[2]); a.cache_bf16 = s->bf16(nd.inputs[2]);
+            a.pos = u(nd.inputs[3]); a.freq = static_cast<const float *>(d.workspace);
+            a.rows = s->rows_of(nd.inputs[0]); a.rank = nd.at[0]; a.rot_dim = nd.at[1]; a.slots = nd.at[2]; a.eps = nd.f0;
+            return mgq::launch_latent_cache_write(a, s->stream);
+        }
+        default: break;
+    }
+    // recurrences and latent attention, alone or with the head gate that consumes them
+    const bool gated = nd.op == Op::HeadGate;
+    const int oid = gated && s->nodes[nd.inputs[0]].absorbed ? nd.inputs[0] : d.out;
+    const Node &o = s->nodes[oid];
+    const bool fused = gated && oid != d.out;
+    mgq::HeadGate hg{};
+    if (gated) hg = head_gate_args(s, nd, d.out);
+    if (o.op == Op::Wkv || o.op == Op::Decay) {
+        mgq::Wkv a{};
+        const int did = o.op == Op::Decay ? oid : o.inputs[3];
+        const Node &dn = s->nodes[did];
+        a.rows = rows;
+        a.decay = f(did);
+        if (dn.op == Op::Decay) {
+            a.low = f(dn.inputs[0]); a.w2 = s->ptr(dn.inputs[1]); a.w0 = f(dn.inputs[2]);
+            a.rank = (uint32_t)s->nodes[dn.inputs[0]].shape[1];
+        }
+        if (o.op == Op::Decay) {
+            a.heads = 1; a.dim = (uint32_t)dn.shape[1];
+            return mgq::launch_decay(a, s->stream);
+        }
+        a.r = f(o.inputs[0]); a.k = f(o.inputs[1]); a.v = f(o.inputs[2]); a.u = f(o.inputs[4]);
+        a.state = f(o.inputs[5]); a.shift_state = f(o.inputs[6]); a.o = f(oid);
+        a.heads = o.at[0]; a.dim = o.at[1];
+        a.shift_width = o.inputs[6] >= 0 ? (uint32_t)(s->nodes[o.inputs[6]].elements() / 2) : 0;
+        if (!fused) return mgq::launch_wkv_scan(a, s->stream);
+        if (rows == 1) return mgq::launch_wkv_step(a, hg, s->stream);
+        if (int rc = mgq::launch_decay(a, s->stream)) return rc;
+        if (int rc = mgq::launch_wkv_scan(a, s->stream)) return rc;
+        return mgq::launch_head_gate(a.o, hg, rows, o.at[0], o.at[1], s->stream);
+    }
+    if (o.op == Op::Mlstm) {
+        mgq::Mlstm a{};
+        a.q = f(o.inputs[0]); a.k = f(o.inputs[1]); a.v = f(o.inputs[2]); a.gi = f(o.inputs[3]); a.gf = f(o.inputs[4]);
+        a.state = f(o.inputs[5]); a.o = f(oid);
+        a.rows = rows; a.heads = o.at[0]; a.dim = o.at[1]; a.vdim = o.at[2]; a.cap = o.f0;
+        if (!fused) return mgq::launch_mlstm_scan(a, s->stream);
+        if (rows == 1) return mgq::launch_mlstm_step(a, hg, s->stream);
+        if (int rc = mgq::launch_mlstm_scan(a, s->stream)) return rc;
+        return mgq::launch_head_gate(a.o, hg, rows, o.at[0], o.at[2], s->stream);
+    }
+    if (o.op == Op::LatentAttention) {
+        mgq::LatentAttention a{};
+        a.q = f(o.inputs[0]); a.cache = s->ptr(o.inputs[1]); a.cache_bf16 = s->bf16(o.inputs[1]);
+        a.uk = s->ptr(o.inputs[2]); a.uv = s->ptr(o.inputs[3]); a.pos = u(o.inputs[4]); a.o = f(oid);
+        a.rows = rows; a.heads = o.at[0]; a.dim = o.at[1]; a.rot_dim = o.at[2]; a.vdim = o.at[3]; a.rank = o.at[4]; a.slots = o.at[5]; a.window = o.at[6];
+        a.scale = o.f0;
+        a.freq = static_cast<const float *>(d.workspace);
+        a.workspace = static_cast<uint8_t *>(d.workspace) + rotation_bytes(a.rot_dim);
+        a.gate = fused ? &hg : nullptr;
+        return mgq::launch_latent_attention(a, s->stream);
+    }
+    return mgq::launch_head_gate(f(nd.inputs[0]), hg, rows, nd.at[0], (uint32_t)(nd.shape[1] / nd.at[0]), s->stream);
 }
 
 static int run_dispatch(mgq_session *s, const Dispatch &d)
@@ -964,12 +1629,27 @@ static int run_dispatch(mgq_session *s, const Dispatch &d)
     auto f = [&](int i) { return static_cast<const float *>(s->ptr(d.in[i])); };
     auto u = [&](int i) { return static_cast<const uint32_t *>(s->ptr(d.in[i])); };
     float *outp = static_cast<float *>(s->ptr(d.out));
+    if (s->nodes[d.out].rows && s->row_count[s->nodes[d.out].rows] == 0) return MGQ_OK;      // no row of this set is wanted
     switch (d.shader) {
+        case MGQ_SHADER_LINEAR:
+        case MGQ_SHADER_LINEAR_GLU: return run_linear(s, d);
+        case MGQ_SHADER_BIAS_ADD: case MGQ_SHADER_PICK_ROWS: case MGQ_SHADER_NORM: case MGQ_SHADER_TOKEN_SHIFT: case MGQ_SHADER_DECAY:
+        case MGQ_SHADER_WKV: case MGQ_SHADER_MLSTM: case MGQ_SHADER_HEAD_GATE: case MGQ_SHADER_LATENT_CACHE_WRITE:
+        case MGQ_SHADER_LATENT_ATTENTION: case MGQ_SHADER_CLAMPED_GLU: return run_mixer(s, d);
         case MGQ_SHADER_ADD:
+            if (s->nodes[d.out].rows) {
+                const uint32_t len = s->rows_of(d.out) * (uint32_t)s->nodes[d.out].shape[1];
+                add_kernel<<<(len + 255) / 256, 256, 0, s->stream>>>(f(0), f(1), outp, len);
+                MGQ_CUDA(cudaGetLastError());
+                return MGQ_OK;
+            }
             add_kernel<<<d.workgroups[0], 256, 0, s->stream>>>(f(0), f(1), outp, d.params[0]);
             MGQ_CUDA(cudaGetLastError());
             return MGQ_OK;
-        case MGQ_SHADER_EMBEDDING: return mgq_embedding(u(0), f(1), outp, d.params[0], d.params[1], d.params[2], s->stream);
+        case MGQ_SHADER_EMBEDDING:
+            if (s->nodes[d.out].u0)
+                return mgq::launch_embedding_scaled(u(0), s->ptr(d.in[1]), s->bf16(d.in[1]), outp, s->rows_of(d.out), d.params[1], d.params[2], d.f0, s->stream);
+            return mgq_embedding(u(0), f(1), outp, d.params[0], d.params[1], d.params[2], s->stream);
         case MGQ_SHADER_RMS_NORM: return mgq_rms_norm(f(0), f(1), outp, d.params[0], d.params[1], d.f0, s->stream);
         case MGQ_SHADER_ROPE_DYNAMIC: return mgq_rope_dynamic(f(0), outp, u(1), d.params[0], d.params[1], d.params[3], d.f0, s->stream);
         case MGQ_SHADER_CACHE_WRITE: return mgq_cache_write(f(0), outp, u(2), d.params[0], d.params[1], s->stream);
@@ -1021,16 +1701,25 @@ static int exchanges_bound(const mgq_session *s)
     return MGQ_OK;
 }
 
+// Greedy pick over the first row of the chosen output.  In a row-dynamic session it runs only when a row
+// was picked, and the position moves past all tokens of the step.
+static int greedy_pick(mgq_session *s)
+{
+    const Node &lo = s->nodes[s->greedy_output];
+    if (lo.rows && s->row_count[lo.rows] == 0) return MGQ_OK;
+    const Node &tok = s->nodes[s->greedy_token_input];
+    return mgq::launch_argmax(static_cast<const float *>(s->ptr(s->greedy_output)), lo.rows ? (uint32_t)lo.shape[1] : (uint32_t)lo.elements(), s->greedy_ws,
+                              s->greedy_token, static_cast<uint32_t *>(s->ptr(s->greedy_token_input)),
+                              static_cast<uint32_t *>(s->ptr(s->greedy_pos_input)), s->greedy_history, s->greedy_cap,
+                              tok.rows ? s->row_count[tok.rows] : 1u, s->stream);
+}
+
 static int enqueue_all(mgq_session *s)
 {
     for (const Dispatch &d : s->dispatches)
         if (int rc = run_dispatch(s, d)) return rc;
     if (s->greedy) {
-        const Node &lo = s->nodes[s->greedy_output];
-        const int rc = mgq_argmax(static_cast<const float *>(s->ptr(s->greedy_output)), (uint32_t)lo.elements(), s->greedy_ws,
-                                  s->greedy_token, static_cast<uint32_t *>(s->ptr(s->greedy_token_input)),
-                                  static_cast<uint32_t *>(s->ptr(s->greedy_pos_input)), s->greedy_history, s->greedy_cap, s->stream);
-        if (rc) return rc;
+        if (int rc = greedy_pick(s)) return rc;
     }
     return end_token(s);
 }
@@ -1054,11 +1743,7 @@ static int enqueue_profiled(mgq_session *s)
     }
     MGQ_CUDA(cudaEventRecord(s->events[n], s->stream));
     if (s->greedy) {
-        const Node &lo = s->nodes[s->greedy_output];
-        if (int rc = mgq_argmax(static_cast<const float *>(s->ptr(s->greedy_output)), (uint32_t)lo.elements(), s->greedy_ws,
-                                s->greedy_token, static_cast<uint32_t *>(s->ptr(s->greedy_token_input)),
-                                static_cast<uint32_t *>(s->ptr(s->greedy_pos_input)), s->greedy_history, s->greedy_cap, s->stream))
-            return rc;
+        if (int rc = greedy_pick(s)) return rc;
     }
     s->profiled = true;
     return end_token(s);
@@ -1073,7 +1758,7 @@ int mgq_session_step(mgq_session *s)
     int rc = MGQ_OK;
     if (s->profiling) {
         rc = enqueue_profiled(s);
-    } else if (s->graph_exec) {
+    } else if (s->graph_exec && !std::memcmp(s->graph_rows, s->row_count, sizeof s->graph_rows)) {
         rc = mgq::cuda_check((int)cudaGraphLaunch(s->graph_exec, s->stream), "cudaGraphLaunch", __FILE__, __LINE__);
     } else {
         rc = enqueue_all(s);
@@ -1188,6 +1873,8 @@ int mgq_session_num_groups(const mgq_session *s)
 {
     if (!s) return -fail(MGQ_ERR_NULL, "null session");
     const size_t n = s->dispatches.size();
+    for (const Dispatch &d : s->dispatches)
+        if (!d.members.empty() || d.shader > MGQ_SHADER_MATMUL_GEMV_BT) return (int)n;      // recurrent decoders run as one dependent chain
     std::vector<int32_t> ins(n * 4), outs(n * 4);
     auto buf = [&](int node) { return node < 0 ? -1 : s->node_buffer[node]; };
     for (size_t i = 0; i < n; i++) {
@@ -1215,6 +1902,7 @@ int mgq_session_capture(mgq_session *s)
     if (rc) { if (graph) cudaGraphDestroy(graph); return rc; }
     MGQ_CUDA(end);
     s->graph = graph;
+    std::memcpy(s->graph_rows, s->row_count, sizeof s->graph_rows);
     MGQ_CUDA(cudaGraphInstantiate(&s->graph_exec, s->graph, 0));
     return MGQ_OK;
 }
@@ -1226,7 +1914,7 @@ int mgq_session_enable_greedy(mgq_session *s, size_t output_index, const char *t
     if (output_index >= s->outputs.size()) return fail(MGQ_ERR_NAME, "output index %zu out of range", output_index);
     const int tok = find_named(s, Op::Input, token_input), pos = find_named(s, Op::Input, pos_input);
     if (tok < 0 || pos < 0 || s->nodes[tok].dtype != kU32 || s->nodes[pos].dtype != kU32) return fail(MGQ_ERR_NAME, "greedy feedback needs two u32 inputs");
-    if (s->nodes[tok].elements() != 1 || s->nodes[pos].elements() != 1) return fail(MGQ_ERR_SHAPE, "greedy feedback takes one token and one position");
+    if ((!s->nodes[tok].rows && s->nodes[tok].elements() != 1) || s->nodes[pos].elements() != 1) return fail(MGQ_ERR_SHAPE, "greedy feedback takes one token and one position");
     if (history_cap == 0) return fail(MGQ_ERR_SHAPE, "history capacity must be positive");
     void *p = nullptr;
     if (!s->greedy_ws) {

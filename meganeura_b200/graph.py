@@ -13,7 +13,7 @@ from enum import IntEnum
 
 import numpy as np
 
-from ._lib import check, last_error, lib, MgqError
+from ._lib import FMT_F32, GATE_SIGMOID, check, last_error, lib, MgqError
 
 
 class ShaderEntry(IntEnum):
@@ -32,6 +32,19 @@ class ShaderEntry(IntEnum):
     RoPECacheWrite = 12
     AllGather = 13
     MatMulGemvBT = 14
+    Linear = 15
+    LinearGLU = 16
+    BiasAdd = 17
+    PickRows = 18
+    Norm = 19
+    TokenShift = 20
+    Decay = 21
+    Wkv = 22
+    Mlstm = 23
+    HeadGate = 24
+    LatentCacheWrite = 25
+    LatentAttention = 26
+    ClampedGLU = 27
 
 
 class WeightFormat(IntEnum):
@@ -39,6 +52,7 @@ class WeightFormat(IntEnum):
     F16 = 1
     Q4 = 2
     Q8 = 3
+    BF16 = 4
 
 
 @dataclass
@@ -125,6 +139,57 @@ class Graph:
         """Graph::matmul_bt (src/graph.rs:809-817): a [M, K] @ b[N, K]^T, b an f32 parameter."""
         return _node(lib.mgq_graph_matmul_bt(self._h, a, b))
 
+    # ---- row-dynamic graphs and the operators of recurrent / latent-attention decoders (mgq.h)
+    def input_u32_rows(self, name: str, capacity: int, which: int) -> int:
+        """u32 input of up to `capacity` rows; Session.set_rows(which, n) sets the count of a step."""
+        return _node(lib.mgq_graph_input_u32_rows(self._h, name.encode(), capacity, which))
+
+    def parameter_bf16(self, name: str, shape) -> int:
+        return _node(lib.mgq_graph_parameter_bf16(self._h, name.encode(), *_shape(shape)))
+
+    def embedding_scaled(self, indices: int, table: int, scale: float) -> int:
+        return _node(lib.mgq_graph_embedding_scaled(self._h, indices, table, scale))
+
+    def pick_rows(self, x: int, index: int) -> int:
+        return _node(lib.mgq_graph_pick_rows(self._h, x, index))
+
+    def norm(self, x: int, weight: int, eps: float, weight_offset: float = 0.0, out_dtype: int = FMT_F32) -> int:
+        return _node(lib.mgq_graph_norm(self._h, x, weight, eps, weight_offset, out_dtype))
+
+    def bias_add(self, x: int, bias: int) -> int:
+        return _node(lib.mgq_graph_bias_add(self._h, x, bias))
+
+    def clamped_glu(self, gate: int, up: int, limit: float, alpha: float, out_dtype: int = FMT_F32) -> int:
+        return _node(lib.mgq_graph_clamped_glu(self._h, gate, up, limit, alpha, out_dtype))
+
+    def token_shift(self, h: int, mu, state: int, out_dtype: int = FMT_F32) -> int:
+        """[len(mu), rows, width] mixes of every token with the one before it; take one with slot()."""
+        arr = (ctypes.c_int * len(mu))(*mu)
+        return _node(lib.mgq_graph_token_shift(self._h, h, arr, len(mu), state, out_dtype))
+
+    def slot(self, x: int, index: int) -> int:
+        return _node(lib.mgq_graph_slot(self._h, x, index))
+
+    def lora_decay(self, low: int, w2: int, w0: int) -> int:
+        return _node(lib.mgq_graph_lora_decay(self._h, low, w2, w0))
+
+    def wkv(self, r: int, k: int, v: int, decay: int, u: int, state: int, heads: int, shift_state: int = -1) -> int:
+        return _node(lib.mgq_graph_wkv(self._h, r, k, v, decay, u, state, shift_state, heads))
+
+    def mlstm(self, q: int, k: int, v: int, gate_i: int, gate_f: int, state: int, heads: int, gate_cap: float) -> int:
+        return _node(lib.mgq_graph_mlstm(self._h, q, k, v, gate_i, gate_f, state, heads, gate_cap))
+
+    def head_gate(self, o: int, gate: int, heads: int, weight: int = -1, eps: float = 0.0, act: int = GATE_SIGMOID,
+                  out_dtype: int = FMT_F32) -> int:
+        return _node(lib.mgq_graph_head_gate(self._h, o, weight, gate, heads, eps, act, out_dtype))
+
+    def latent_cache_write(self, down: int, weight: int, cache: int, pos: int, rot_dim: int, rot_base: float, eps: float) -> int:
+        return _node(lib.mgq_graph_latent_cache_write(self._h, down, weight, cache, pos, rot_dim, rot_base, eps))
+
+    def latent_attention(self, q: int, cache: int, uk: int, uv: int, pos: int, heads: int, dim: int, rot_dim: int, vdim: int, window: int,
+                         scale: float, rot_base: float) -> int:
+        return _node(lib.mgq_graph_latent_attention(self._h, q, cache, uk, uv, pos, heads, dim, rot_dim, vdim, window, scale, rot_base))
+
     def all_gather(self, x: int, world: int) -> int:
         """This rank's [1, n] slice -> the whole [1, n * world] vector, rank-major (column-sharded
         models; no reference counterpart: the reference is single-device)."""
@@ -169,6 +234,14 @@ class Session:
     def set_input_u32(self, name: str, data) -> None:
         data = np.ascontiguousarray(data, dtype=np.uint32).reshape(-1)
         check(lib.mgq_session_set_input_u32(self._h, name.encode(), data.ctypes.data, data.size))
+
+    def set_rows(self, which: int, count: int) -> None:
+        """Row-dynamic sessions: rows of the following steps (ROWS_TOKENS or ROWS_PICKED)."""
+        check(lib.mgq_session_set_rows(self._h, which, count))
+
+    def reset_state(self) -> None:
+        """Clear every recurrent state and latent cache (the next step starts a new sequence)."""
+        check(lib.mgq_session_reset_state(self._h))
 
     def step(self) -> None:
         check(lib.mgq_session_step(self._h))
