@@ -567,6 +567,10 @@ def main():
                          "whichever of the two is faster in a short calibration, on several GPUs the persistent kernel")
     ap.add_argument("--exchange", choices=["peer", "nccl"], default="peer",
                     help="launches mode on several GPUs: slices pushed over NVLink by the GEMV kernels (default) or NCCL all-gather")
+    ap.add_argument("--design", choices=["petotar"], default=None,
+                    help="instead of the default workload: prefill and decode of this decoder design at layer sizes of real models, "
+                         "beside the closest existing decoder (one JSON line per size)")
+    ap.add_argument("--sizes", default="2048,4096", help="with --design: widths to measure")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-extras", action="store_true", help="skip the extra keys (gemm, gemv_cases, batch8, per_gemv_launches, decode)")
     ap.add_argument("--no-decode", action="store_true", help="skip the whole-model decode tokens/s measurement")
@@ -577,6 +581,17 @@ def main():
 
     if args.impl == "reference":
         run_reference(args, shape_t, fmt)
+        return
+
+    if args.design:
+        from meganeura_b200 import design_bench
+        hbm, tensor, source = measured_peaks()
+        for name in args.sizes.split(","):
+            sampler = ClockSampler(0)
+            sampler.start()
+            line = design_bench.measure(name, (hbm, tensor))
+            line.update(peaks=f"{hbm} GB/s, {tensor} TFLOP/s bf16 (of {source})", clocks=sampler.stop(), data="synthetic")
+            print(json.dumps(line), flush=True)
         return
 
     import torch

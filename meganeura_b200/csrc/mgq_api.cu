@@ -37,7 +37,9 @@ int mgq_buffer_create(size_t bytes, void **out_dev)
     if (bytes == 0) return fail(MGQ_ERR_SHAPE, "zero-sized buffer");
     void *p = nullptr;
     MGQ_CUDA(cudaMalloc(&p, bytes));
-    const int rc = cuda_check((int)cudaMemset(p, 0, bytes), "cudaMemset", __FILE__, __LINE__);
+    int rc = cuda_check((int)cudaMemset(p, 0, bytes), "cudaMemset", __FILE__, __LINE__);
+    // the fill is asynchronous and sessions use non-blocking streams: it must not land on top of a later upload
+    if (rc == MGQ_OK) rc = cuda_check((int)cudaStreamSynchronize(0), "cudaStreamSynchronize", __FILE__, __LINE__);
     if (rc != MGQ_OK) { cudaFree(p); return rc; }
     *out_dev = p;
     return MGQ_OK;

@@ -58,7 +58,8 @@ template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
-// 8 consecutive elements, 16-byte aligned source.
+// 8 consecutive elements, 16-byte aligned source.  Plain loads: activations are written by the kernel this one
+// overlaps with, and a read-only-path load might be moved across the wait for it.
 __device__ __forceinline__ void unpack8(const uint4 &q, float (&f)[8])
 {
     const uint32_t w[4] = {q.x, q.y, q.z, q.w};
@@ -68,10 +69,10 @@ __device__ __forceinline__ void unpack8(const uint4 &q, float (&f)[8])
         f[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
     }
 }
-__device__ __forceinline__ void load8(const __nv_bfloat16 *p, float (&f)[8]) { unpack8(__ldg(reinterpret_cast<const uint4 *>(p)), f); }
+__device__ __forceinline__ void load8(const __nv_bfloat16 *p, float (&f)[8]) { unpack8(*reinterpret_cast<const uint4 *>(p), f); }
 __device__ __forceinline__ void load8(const float *p, float (&f)[8])
 {
-    const float4 a = __ldg(reinterpret_cast<const float4 *>(p)), b = __ldg(reinterpret_cast<const float4 *>(p) + 1);
+    const float4 a = *reinterpret_cast<const float4 *>(p), b = *(reinterpret_cast<const float4 *>(p) + 1);
     f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
 }
 

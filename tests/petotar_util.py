@@ -36,7 +36,7 @@ CONFIGS = {
     "odd": (config(203, 90, [wkv(3, 22, ff=51, limit=0.9), latent(5, 18, 6, 13, 27, 9, base=500.0), mlstm(1, 35, 17, 3.5, ff=33),
                              latent(2, 10, 6, 20, 27, 30, base=500.0, kv_from=1, ff=70)], eps=1e-3, scale=1.0), 5),
     "wide": (config(512, 256, [mlstm(2, 128, 96, 10.0, ff=320), latent(12, 64, 32, 64, 256, 70, base=2e5, ff=256), wkv(2, 128, ff=256)], eps=1e-6,
-                    scale=12.0), 32),
+                    scale=1.5), 32),
 }
 
 

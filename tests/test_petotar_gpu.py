@@ -14,7 +14,7 @@ from petotar_util import CONFIGS, Tensors, row_errors, weights, write_folder
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-TOL = {"float32": 5e-5, "bfloat16": 4e-2}
+TOL = {"float32": 5e-5, "bfloat16": 8e-2}       # worst row; bf16 operands cost the median row about 1e-2
 _cache = {}
 
 
@@ -58,7 +58,9 @@ def test_logits_do_not_depend_on_the_cut(name, dtype):
     for label, sizes in (("whole", [150]), ("single", [1]), ("two", [2]), ("cuts", [37, 2, 3, 64, 1, 16, 9, 8]), ("mostly", [118] + [1] * 32)):
         got = feed_cut(e, tokens, sizes)
         e.end()
-        worst[label] = row_errors(got, want).max()
+        errors = row_errors(got, want)
+        worst[label] = errors.max()
+        assert np.median(errors) <= TOL[dtype] / 3
     assert max(worst.values()) <= TOL[dtype], worst
 
 
