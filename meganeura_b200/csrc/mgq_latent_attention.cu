@@ -1,11 +1,11 @@
 // Latent attention over a sliding window: the cache holds, per position, an RMS-normed latent of
 // `rank` elements and one rotated key part of `rot_dim` elements shared by all heads.
 //
-// Absorbed form (few rows, and every f32 session): the query is folded through W_uk once,
+// Absorbed form (few rows, and every f32 session; many rows: mgq_latent_prefill.cu): the query is folded through W_uk once,
 //   score = (W_uk^T q_nope) . c + q_rot . k_rot,   o' = softmax . c,   o = W_uv o',
 // so attention runs against the latents themselves and every head shares one key/value row.
 //   latent_absorb_kernel   q' = scale * [W_uk^T q_nope | rotate(q_rot)]
-//   latent_attend_kernel   CTA = 8 heads x one row x one slice of the window, 32 keys per tile,
+//   latent_attend_kernel   CTA = 8 heads (a warp each) x one row x one slice of the window, 32 keys per tile,
 //                          online softmax in f32; slices leave (max, sum, unnormalised o')
 //   latent_out_kernel      merges the slices, applies W_uv and the output gate
 // The ring cache is addressed by position % slots, so a sequence may be longer than the cache.
@@ -18,7 +18,7 @@ namespace {
 
 constexpr uint32_t kHeads = 8;             // heads per CTA in latent_attend_kernel
 constexpr uint32_t kTile = 32;             // keys per tile
-constexpr uint32_t kSliceKeys = 64;        // window positions per slice when the window is split
+constexpr uint32_t kSliceKeys = 32;        // window positions per slice when the window is split
 constexpr uint32_t kSplitRows = 16;        // at most this many rows split the window over CTAs
 
 __device__ __forceinline__ void rotate_pair(float u, float v, uint32_t pos, float freq, float &ru, float &rv)
@@ -126,32 +126,45 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constan
 }
 
 // ---------------------------------------------------------------- attention against the latents
-__device__ __forceinline__ void load4(const float *p, float (&f)[4])
+// Shared-memory row pitch in elements: 16-byte pieces of consecutive rows fall into different banks.
+template <typename CT> __host__ __device__ inline uint32_t key_pitch(uint32_t width)
+{
+    constexpr uint32_t per = 16 / sizeof(CT);
+    const uint32_t pieces = (width + per - 1) / per;
+    return (pieces | 1u) * per;
+}
+__host__ __device__ inline uint32_t query_pitch(uint32_t width) { return (width + 7u) & ~7u; }
+
+__device__ __forceinline__ void unpack_piece(const float *p, float (&f)[4])
 {
     const float4 v = *reinterpret_cast<const float4 *>(p);
     f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
 }
-__device__ __forceinline__ void load4(const __nv_bfloat16 *p, float (&f)[4])
+__device__ __forceinline__ void unpack_piece(const __nv_bfloat16 *p, float (&f)[8]) { unpack8(*reinterpret_cast<const uint4 *>(p), f); }
+
+__device__ __forceinline__ void cp_async16(void *smem, const void *gmem)
 {
-    const uint2 v = *reinterpret_cast<const uint2 *>(p);
-    f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xFFFF0000u);
-    f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xFFFF0000u);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((unsigned)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
 }
 
-__host__ __device__ inline uint32_t tile_pitch(uint32_t width) { return ((width + 3u) & ~3u) + 4u; }
-
-// DPT: rank elements per thread (128 threads).  Partials: po [row][split][heads][rank], ml [row][split][heads][2].
+// DPT: pairs of rank elements per thread (256 threads).  A warp scores one head against a tile of 32
+// keys (lane = key), then every thread adds its rank elements for all 8 heads.
+// Partials: po [row][split][heads][rank], ml [row][split][heads][2].
 template <typename CT, int DPT>
-__global__ void __launch_bounds__(128) latent_attend_kernel(const __grid_constant__ LatentAttention a, const float *qx, float *po, float *ml)
+__global__ void __launch_bounds__(256) latent_attend_kernel(const __grid_constant__ LatentAttention a, const float *qx, float *po, float *ml)
 {
+    constexpr uint32_t PER = 16 / sizeof(CT);
     extern __shared__ __align__(16) float smem[];
-    const uint32_t t = threadIdx.x, lane = t & 31u, warp = t >> 5, width = a.rank + a.rot_dim, pitch = tile_pitch(width);
-    float *s_k = smem, *s_q = s_k + kTile * pitch;                       // [32][pitch], [8][pitch]
+    const uint32_t t = threadIdx.x, lane = t & 31u, warp = t >> 5, width = a.rank + a.rot_dim, kp = key_pitch<CT>(width), qp = query_pitch(width);
+    float *s_q = smem;                                                   // [8][qp]
+    CT *s_k = reinterpret_cast<CT *>(smem + kHeads * qp);                // [32][kp]
     __shared__ __align__(16) float s_p[kHeads][kTile];
     __shared__ float s_corr[kHeads];
     const uint32_t h0 = blockIdx.x * kHeads, split = blockIdx.y, splits = gridDim.y, row = blockIdx.z;
     const uint32_t heads = min(kHeads, a.heads - h0);
     pdl_launch_dependents();
+    // the padding behind a row must stay finite
+    for (uint32_t i = t; i < kTile * (kp - width); i += 256) s_k[(i / (kp - width)) * kp + width + i % (kp - width)] = from_f32<CT>(0.f);
     pdl_wait();
     const uint32_t pos = a.pos[0] + row, lo = pos + 1 > a.window ? pos + 1 - a.window : 0u, total = pos + 1 - lo;
     const uint32_t per = ((total + splits - 1) / splits + kTile - 1) / kTile * kTile;
@@ -161,113 +174,127 @@ __global__ void __launch_bounds__(128) latent_attend_kernel(const __grid_constan
         if (t < heads) { ml[(part + t) * 2] = -INFINITY; ml[(part + t) * 2 + 1] = 0.f; }
         return;
     }
-    for (uint32_t i = t; i < kHeads * pitch; i += 128) {
-        const uint32_t h = i / pitch, j = i - h * pitch;
-        s_q[i] = h < heads && j < width ? qx[((size_t)row * a.heads + h0 + h) * width + j] : 0.f;
+    const CT *cache = static_cast<const CT *>(a.cache);
+    const bool vec = width % PER == 0;
+    auto stage = [&](uint32_t kt) {
+#pragma unroll
+        for (uint32_t r = warp; r < kTile; r += 8) {
+            if (kt + r < k1) {
+                const CT *src = cache + (size_t)((kt + r) % a.slots) * width;
+                CT *dst = s_k + r * kp;
+                if (vec) {
+                    for (uint32_t j = lane * PER; j < width; j += 32 * PER) cp_async16(dst + j, src + j);
+                } else {
+                    for (uint32_t j = lane; j < width; j += 32) dst[j] = src[j];
+                }
+            } else {
+                for (uint32_t j = lane; j < width; j += 32) s_k[r * kp + j] = from_f32<CT>(0.f);
+            }
+        }
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+    };
+    stage(k0);
+    const float *qsrc = qx + ((size_t)row * a.heads + h0) * width;
+    if (width % 4 == 0) {
+        for (uint32_t h = warp; h < kHeads; h += 8)
+            for (uint32_t j = lane * 4; j < qp; j += 128)
+                *reinterpret_cast<float4 *>(s_q + h * qp + j) = h < heads && j < width ? *reinterpret_cast<const float4 *>(qsrc + h * width + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+    } else {
+        for (uint32_t h = warp; h < kHeads; h += 8)
+            for (uint32_t j = lane; j < qp; j += 32) s_q[h * qp + j] = h < heads && j < width ? qsrc[h * width + j] : 0.f;
     }
-    for (uint32_t i = t; i < kTile * pitch; i += 128) s_k[i] = 0.f;      // the padding must stay finite
-    __syncthreads();
-    float acc[kHeads][DPT], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    float acc[kHeads][2 * DPT], m = -INFINITY, l = 0.f;
 #pragma unroll
     for (int h = 0; h < (int)kHeads; h++)
 #pragma unroll
-        for (int i = 0; i < DPT; i++) acc[h][i] = 0.f;
-    const CT *cache = static_cast<const CT *>(a.cache);
-    const bool vec = width % 4 == 0;
+        for (int i = 0; i < 2 * DPT; i++) acc[h][i] = 0.f;
     for (uint32_t kt = k0; kt < k1; kt += kTile) {
-        const uint32_t cnt = min(kTile, k1 - kt);
+        asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        __syncthreads();
+        float s4[4] = {0.f, 0.f, 0.f, 0.f};
+        const CT *kr = s_k + lane * kp;
+        const float *q = s_q + warp * qp;
 #pragma unroll 4
-        for (uint32_t r = warp; r < kTile; r += 4) {
-            if (r >= cnt) continue;
-            const CT *src = cache + (size_t)((kt + r) % a.slots) * width;
-            float *dst = s_k + r * pitch;
-            if (vec) {
-                for (uint32_t j = lane * 4; j < width; j += 128) {
-                    float f[4];
-                    load4(src + j, f);
-                    *reinterpret_cast<float4 *>(dst + j) = make_float4(f[0], f[1], f[2], f[3]);
-                }
-            } else {
-                for (uint32_t j = lane; j < width; j += 32) dst[j] = to_f32(src[j]);
+        for (uint32_t d = 0; d < width; d += PER) {                      // the query is zero beyond width
+            float kv[PER];
+            unpack_piece(kr + d, kv);
+#pragma unroll
+            for (int j = 0; j < (int)PER; j += 4) {
+                const float4 x = *reinterpret_cast<const float4 *>(q + d + j);
+                s4[0] = fmaf(kv[j], x.x, s4[0]); s4[1] = fmaf(kv[j + 1], x.y, s4[1]);
+                s4[2] = fmaf(kv[j + 2], x.z, s4[2]); s4[3] = fmaf(kv[j + 3], x.w, s4[3]);
             }
         }
-        __syncthreads();
-        // scores: lane = key, warp w = heads 2w and 2w + 1
-        float s0 = 0.f, s1 = 0.f;
-        const float *kr = s_k + lane * pitch, *q0 = s_q + (2 * warp) * pitch, *q1 = q0 + pitch;
-#pragma unroll 4
-        for (uint32_t d = 0; d < width; d += 4) {
-            const float4 kv = *reinterpret_cast<const float4 *>(kr + d), x = *reinterpret_cast<const float4 *>(q0 + d),
-                         y = *reinterpret_cast<const float4 *>(q1 + d);
-            s0 = fmaf(kv.x, x.x, s0); s0 = fmaf(kv.y, x.y, s0); s0 = fmaf(kv.z, x.z, s0); s0 = fmaf(kv.w, x.w, s0);
-            s1 = fmaf(kv.x, y.x, s1); s1 = fmaf(kv.y, y.y, s1); s1 = fmaf(kv.z, y.z, s1); s1 = fmaf(kv.w, y.w, s1);
-        }
-        float s[2] = {lane < cnt ? s0 : -INFINITY, lane < cnt ? s1 : -INFINITY};
-#pragma unroll
-        for (int i = 0; i < 2; i++) {
-            const float m_new = fmaxf(m[i], warp_max(s[i]));             // cnt >= 1: finite
-            const float corr = expf(m[i] - m_new), p = expf(s[i] - m_new);
-            l[i] = l[i] * corr + warp_sum(p);
-            m[i] = m_new;
-            s_p[2 * warp + i][lane] = p;
-            if (lane == 0) s_corr[2 * warp + i] = corr;
-        }
+        const float s = kt + lane < k1 ? (s4[0] + s4[1]) + (s4[2] + s4[3]) : -INFINITY;
+        const float m_new = fmaxf(m, warp_max(s));                       // at least one key: finite
+        const float corr = expf(m - m_new), p = expf(s - m_new);
+        l = l * corr + warp_sum(p);
+        m = m_new;
+        s_p[warp][lane] = p;
+        if (lane == 0) s_corr[warp] = corr;
         __syncthreads();
 #pragma unroll
         for (int h = 0; h < (int)kHeads; h++) {
-            const float corr = s_corr[h];
+            const float c = s_corr[h];
 #pragma unroll
-            for (int i = 0; i < DPT; i++) acc[h][i] *= corr;
+            for (int i = 0; i < 2 * DPT; i++) acc[h][i] *= c;
         }
-        for (uint32_t k = 0; k < cnt; k += 4) {                          // rows beyond cnt: p = 0 and finite contents
-            float kv[4][DPT];
+#pragma unroll 2
+        for (uint32_t k = 0; k < kTile; k += 4) {
+            float kv[4][2 * DPT];
 #pragma unroll
             for (int u = 0; u < 4; u++)
 #pragma unroll
                 for (int i = 0; i < DPT; i++) {
-                    const uint32_t d = t + 128u * i;
-                    kv[u][i] = d < a.rank ? s_k[(k + u) * pitch + d] : 0.f;
+                    const uint32_t d = 2 * (t + 256u * i);               // an odd rank reads one element of the rotated part, never stored
+                    kv[u][2 * i] = d < a.rank ? to_f32(s_k[(k + u) * kp + d]) : 0.f;
+                    kv[u][2 * i + 1] = d < a.rank ? to_f32(s_k[(k + u) * kp + d + 1]) : 0.f;
                 }
 #pragma unroll
             for (int h = 0; h < (int)kHeads; h++) {
-                const float4 p = *reinterpret_cast<const float4 *>(&s_p[h][k]);
+                const float4 p4 = *reinterpret_cast<const float4 *>(&s_p[h][k]);
 #pragma unroll
-                for (int i = 0; i < DPT; i++) {
-                    acc[h][i] = fmaf(p.x, kv[0][i], acc[h][i]);
-                    acc[h][i] = fmaf(p.y, kv[1][i], acc[h][i]);
-                    acc[h][i] = fmaf(p.z, kv[2][i], acc[h][i]);
-                    acc[h][i] = fmaf(p.w, kv[3][i], acc[h][i]);
+                for (int i = 0; i < 2 * DPT; i++) {
+                    acc[h][i] = fmaf(p4.x, kv[0][i], acc[h][i]);
+                    acc[h][i] = fmaf(p4.y, kv[1][i], acc[h][i]);
+                    acc[h][i] = fmaf(p4.z, kv[2][i], acc[h][i]);
+                    acc[h][i] = fmaf(p4.w, kv[3][i], acc[h][i]);
                 }
             }
         }
         __syncthreads();
+        if (kt + kTile < k1) stage(kt + kTile);
     }
 #pragma unroll
     for (int h = 0; h < (int)kHeads; h++) {
         if (h >= (int)heads) break;
 #pragma unroll
         for (int i = 0; i < DPT; i++) {
-            const uint32_t d = t + 128u * i;
-            if (d < a.rank) po[(part + h) * a.rank + d] = acc[h][i];
+            const uint32_t d = 2 * (t + 256u * i);
+            float *dst = po + (part + h) * a.rank + d;
+            if (d < a.rank) dst[0] = acc[h][2 * i];
+            if (d + 1 < a.rank) dst[1] = acc[h][2 * i + 1];
         }
     }
-    if (lane == 0) {
-#pragma unroll
-        for (int i = 0; i < 2; i++)
-            if (2 * warp + i < heads) { ml[(part + 2 * warp + i) * 2] = m[i]; ml[(part + 2 * warp + i) * 2 + 1] = l[i]; }
-    }
+    if (lane == 0 && warp < heads) { ml[(part + warp) * 2] = m; ml[(part + warp) * 2 + 1] = l; }
 }
 
-// ---------------------------------------------------------------- merge, W_uv, gate: CTA = row x head x 32 value dimensions
+// ---------------------------------------------------------------- merge, W_uv, gate: CTA = row x head x 64 value dimensions
+constexpr uint32_t kOutThreads = 512, kOutDims = 64;
+
 template <typename OT>
-__global__ void __launch_bounds__(256) latent_out_kernel(const __grid_constant__ LatentAttention a, const float *po, const float *ml, uint32_t splits,
-                                                         const __grid_constant__ HeadGate hg, OT *out)
+__global__ void __launch_bounds__(kOutThreads) latent_out_kernel(const __grid_constant__ LatentAttention a, const float *po, const float *ml, uint32_t splits,
+                                                                 const __grid_constant__ HeadGate hg, OT *out)
 {
     extern __shared__ __align__(16) float smem[];        // o' [rank], slice weights [splits]
     float *s_o = smem, *s_w = smem + ((a.rank + 3u) & ~3u);
-    const uint32_t t = threadIdx.x, lane = t & 31u, warp = t >> 5, head = blockIdx.x, row = blockIdx.y, v0 = blockIdx.z * 32;
+    const uint32_t t = threadIdx.x, lane = t & 31u, warp = t >> 5, head = blockIdx.x, row = blockIdx.y, v0 = blockIdx.z * kOutDims + warp * 4;
     const size_t part = (size_t)row * splits * a.heads + head;
+    const __nv_bfloat16 *uv = static_cast<const __nv_bfloat16 *>(a.uv) + (size_t)head * a.vdim * a.rank;
     pdl_launch_dependents();
+#pragma unroll
+    for (int i = 0; i < 4; i++)                          // weights are immutable: towards L2 before the wait
+        if (v0 + i < a.vdim && lane * 64u < a.rank) asm volatile("prefetch.global.L2 [%0];" ::"l"(uv + (size_t)(v0 + i) * a.rank + lane * 64u));
     pdl_wait();
     float m = -INFINITY, l = 0.f;
     for (uint32_t s = lane; s < splits; s += 32) m = fmaxf(m, ml[(part + (size_t)s * a.heads) * 2]);
@@ -280,21 +307,23 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const __grid_constant__
     }
     const float inv = 1.0f / warp_sum(l);
     __syncthreads();
-    for (uint32_t d = t; d < a.rank; d += 256) {
+    for (uint32_t d = t; d < a.rank; d += kOutThreads) {
+        const float *src = po + part * a.rank + d;
+        const size_t step = (size_t)a.heads * a.rank;
         float s = 0.f;
-#pragma unroll 4
+#pragma unroll 16
         for (uint32_t i = 0; i < splits; i++) {
             const float w = s_w[i];
-            if (w != 0.f) s = fmaf(po[(part + (size_t)i * a.heads) * a.rank + d], w, s);      // an empty slice has no partial
+            s = w != 0.f ? fmaf(src[i * step], w, s) : s;              // an empty slice has no partial
         }
         s_o[d] = s * inv;
     }
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < 4; i++) {
-        const uint32_t v = v0 + warp * 4 + i;
+        const uint32_t v = v0 + i;
         if (v >= a.vdim) break;
-        const __nv_bfloat16 *w = static_cast<const __nv_bfloat16 *>(a.uv) + ((size_t)head * a.vdim + v) * a.rank;
+        const __nv_bfloat16 *w = uv + (size_t)v * a.rank;
         float s = 0.f;
         if (a.rank % 8 == 0) {
             for (uint32_t c = lane * 8; c < a.rank; c += 256) {
@@ -324,18 +353,17 @@ uint32_t window_splits(uint32_t rows, uint32_t window) { return rows <= kSplitRo
 template <typename CT, int DPT>
 int launch_attend_dpt(const LatentAttention &a, const float *qx, float *po, float *ml, uint32_t splits, cudaStream_t st)
 {
-    const size_t smem = (size_t)(kTile + kHeads) * tile_pitch(a.rank + a.rot_dim) * sizeof(float);
+    const uint32_t width = a.rank + a.rot_dim;
+    const size_t smem = (size_t)kHeads * query_pitch(width) * sizeof(float) + (size_t)kTile * key_pitch<CT>(width) * sizeof(CT);
     if (int rc = allow_smem(latent_attend_kernel<CT, DPT>, smem)) return rc;
-    return launch(latent_attend_kernel<CT, DPT>, dim3((a.heads + kHeads - 1) / kHeads, splits, a.rows), dim3(128), smem, st, a, qx, po, ml);
+    return launch(latent_attend_kernel<CT, DPT>, dim3((a.heads + kHeads - 1) / kHeads, splits, a.rows), dim3(256), smem, st, a, qx, po, ml);
 }
 
 template <typename CT>
 int launch_attend(const LatentAttention &a, const float *qx, float *po, float *ml, uint32_t splits, cudaStream_t st)
 {
-    if (a.rank <= 128) return launch_attend_dpt<CT, 1>(a, qx, po, ml, splits, st);
-    if (a.rank <= 256) return launch_attend_dpt<CT, 2>(a, qx, po, ml, splits, st);
-    if (a.rank <= 512) return launch_attend_dpt<CT, 4>(a, qx, po, ml, splits, st);
-    return launch_attend_dpt<CT, 8>(a, qx, po, ml, splits, st);
+    if (a.rank <= 512) return launch_attend_dpt<CT, 1>(a, qx, po, ml, splits, st);
+    return launch_attend_dpt<CT, 2>(a, qx, po, ml, splits, st);
 }
 
 template <int AR>
@@ -350,7 +378,8 @@ template <typename OT>
 int launch_out(const LatentAttention &a, const float *po, const float *ml, uint32_t splits, const HeadGate &hg, void *out, cudaStream_t st)
 {
     const size_t smem = (size_t)(((a.rank + 3) & ~3u) + splits) * sizeof(float);
-    return launch(latent_out_kernel<OT>, dim3(a.heads, a.rows, (a.vdim + 31) / 32), dim3(256), smem, st, a, po, ml, splits, hg, static_cast<OT *>(out));
+    if (int rc = allow_smem(latent_out_kernel<OT>, smem)) return rc;
+    return launch(latent_out_kernel<OT>, dim3(a.heads, a.rows, (a.vdim + kOutDims - 1) / kOutDims), dim3(kOutThreads), smem, st, a, po, ml, splits, hg, static_cast<OT *>(out));
 }
 
 size_t align256(size_t n) { return (n + 255) & ~(size_t)255; }
@@ -374,8 +403,9 @@ int launch_latent_cache_write(const LatentCache &a, void *stream)
 size_t latent_attention_workspace(uint32_t max_rows, uint32_t heads, uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t rank, uint32_t slots,
                                   uint32_t window, bool cache_bf16)
 {
-    (void)dim; (void)vdim; (void)slots; (void)cache_bf16;
-    return absorbed_bytes(max_rows, heads, rot_dim, rank, window);
+    if (!latent_prefill_eligible(dim, rot_dim, vdim, rank, cache_bf16)) return absorbed_bytes(max_rows, heads, rot_dim, rank, window);
+    const size_t few = absorbed_bytes(std::min(max_rows, kPrefillRows - 1), heads, rot_dim, rank, window);
+    return max_rows < kPrefillRows ? few : std::max(few, latent_prefill_workspace(heads, dim, vdim, slots));
 }
 
 int launch_latent_attention(const LatentAttention &a, void *stream)
@@ -383,6 +413,7 @@ int launch_latent_attention(const LatentAttention &a, void *stream)
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     if (a.rank > 1024) return fail(MGQ_ERR_SHAPE, "latent attention: a latent of %u elements (at most 1024)", a.rank);
     if (a.rows > a.slots || a.window + a.rows - 1 > a.slots) return fail(MGQ_ERR_SHAPE, "latent attention: %u rows and a window of %u need more than %u cache rows", a.rows, a.window, a.slots);
+    if (a.rows >= kPrefillRows && latent_prefill_eligible(a.dim, a.rot_dim, a.vdim, a.rank, a.cache_bf16)) return launch_latent_prefill(a, stream);
     const uint32_t width = a.rank + a.rot_dim, splits = window_splits(a.rows, a.window);
     float *qx = static_cast<float *>(a.workspace);
     uint8_t *at = static_cast<uint8_t *>(a.workspace) + align256((size_t)a.rows * a.heads * width * 4);

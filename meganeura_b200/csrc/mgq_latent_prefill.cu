@@ -1,0 +1,274 @@
+// Latent attention for many rows (a prompt's portion), bf16 cache.
+//
+// The keys W_uk c and values W_uv c of all live cache rows are expanded once per step by the tcgen05
+// linear kernel (ring order, bf16); the attention kernel then works like a blockwise exact softmax:
+// CTA = one head x 64 query rows (4 warps x 16 rows), 64 keys per tile, double-buffered cp.async,
+// tensor-core products with f32 accumulation.  The shared rotated key part is read from the cache
+// itself, next to the head's expanded key.  Scores, maxima, sums and weights are f32; a weight enters the
+// product with the values as the sum of two bf16 (16 significant bits).  Only tiles that some row of the
+// CTA can see are visited; positions map to ring rows by position % slots.
+#include "mgq_linear.cuh"
+#include "mgq_mixer.cuh"
+
+namespace mgq {
+namespace {
+
+constexpr uint32_t BM = 64, BN = 64;
+
+__device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void cp_async16(uint32_t smem, const void *gmem)
+{
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void ldmatrix4(uint32_t addr, uint32_t (&r)[4])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldmatrix4_t(uint32_t addr, uint32_t (&r)[4])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
+{
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack2(float x, float y)
+{
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    return *reinterpret_cast<const uint32_t *>(&h);
+}
+
+struct Prefill {
+    const float *q, *freq;
+    const __nv_bfloat16 *keys, *values, *cache;     // keys [slots, heads * dim], values [slots, heads * vdim]
+    const uint32_t *pos;
+    const float *gate;
+    void *out;
+    uint32_t rows, heads, dim, rot, vdim, rank, slots, window;
+    float scale_log2;                               // scale * log2(e)
+    uint32_t out_bf16, silu;
+};
+
+// DK: dim + rot, DV: vdim, both rounded up to a multiple of 16.
+template <int DK, int DV>
+__global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_constant__ Prefill p)
+{
+    constexpr int PK = DK + 8, PV = DV + 8;          // row pitch in elements: an odd number of 16-byte pieces
+    extern __shared__ __align__(16) __nv_bfloat16 sm[];
+    __nv_bfloat16 *s_q = sm, *s_k = s_q + BM * PK, *s_v = s_k + 2 * BN * PK;
+    const uint32_t t = threadIdx.x, lane = t & 31u, warp = t >> 5, head = blockIdx.y;
+    const uint32_t row0 = (gridDim.x - 1 - blockIdx.x) * BM, dk = p.dim + p.rot, width = p.rank + p.rot;      // longest rows first
+    pdl_launch_dependents();
+    for (uint32_t i = t; i < (BM + 2 * BN) * PK + 2 * BN * PV; i += 128) sm[i] = __float2bfloat16_rn(0.f);    // padding columns stay zero
+    pdl_wait();
+    const uint32_t pos0 = p.pos[0], first = pos0 + row0, last = pos0 + min(row0 + BM, p.rows) - 1;
+    const uint32_t lo = first + 1 > p.window ? first + 1 - p.window : 0u, tiles = (last - lo) / BN + 1;
+    __syncthreads();
+
+    auto stage = [&](uint32_t tile, uint32_t buf) {
+        const uint32_t kt = lo + tile * BN;
+        const uint32_t kb = smem_addr(s_k + buf * BN * PK), vb = smem_addr(s_v + buf * BN * PV);
+        const uint32_t per_k = p.dim / 8, per_r = p.rot / 8, per_v = p.vdim / 8;
+        // two threads per key row
+        const uint32_t r = t >> 1, half = t & 1u;
+        const size_t slot = min(kt + r, last) % p.slots;                  // beyond the last key: a valid row, masked below
+        const __nv_bfloat16 *ksrc = p.keys + (slot * p.heads + head) * p.dim, *rsrc = p.cache + slot * width + p.rank,
+                            *vsrc = p.values + (slot * p.heads + head) * p.vdim;
+        for (uint32_t c = half; c < per_k; c += 2) cp_async16(kb + (r * PK + c * 8) * 2, ksrc + c * 8);
+        for (uint32_t c = half; c < per_r; c += 2) cp_async16(kb + (r * PK + p.dim + c * 8) * 2, rsrc + c * 8);
+        for (uint32_t c = half; c < per_v; c += 2) cp_async16(vb + (r * PV + c * 8) * 2, vsrc + c * 8);
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+    };
+    stage(0, 0);
+
+    // queries: unrotated part as it is, rotated part turned by its position
+    {
+        const uint32_t half = p.rot / 2;
+        const size_t pitch = (size_t)p.heads * dk;
+        for (uint32_t r = warp; r < BM; r += 4) {
+            if (row0 + r >= p.rows) break;
+            const float *src = p.q + (size_t)(row0 + r) * pitch + head * dk;
+            for (uint32_t j = lane; j < p.dim; j += 32) s_q[r * PK + j] = __float2bfloat16_rn(src[j]);
+            for (uint32_t i = lane; i < half; i += 32) {
+                float s, c;
+                sincosf((float)(pos0 + row0 + r) * p.freq[i], &s, &c);
+                const float u = src[p.dim + i], v = src[p.dim + half + i];
+                s_q[r * PK + p.dim + i] = __float2bfloat16_rn(u * c - v * s);
+                s_q[r * PK + p.dim + half + i] = __float2bfloat16_rn(v * c + u * s);
+            }
+        }
+    }
+    float o[DV / 8][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+#pragma unroll
+    for (int n = 0; n < DV / 8; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) o[n][e] = 0.f;
+    const uint32_t qrow = warp * 16 + lane / 4;                          // this thread's rows: qrow, qrow + 8
+    const uint32_t qp[2] = {first + qrow, first + qrow + 8};
+    const uint32_t a_addr = smem_addr(s_q + (warp * 16 + (lane & 7u) + ((lane >> 3) & 1u) * 8) * PK + (lane >> 4) * 8);
+    const uint32_t b_off = (((lane & 7u) + (lane >> 4) * 8) * PK + ((lane >> 3) & 1u) * 8) * 2;
+    const uint32_t v_off = (((lane & 7u) + ((lane >> 3) & 1u) * 8) * PV + (lane >> 4) * 8) * 2;
+
+    for (uint32_t tile = 0; tile < tiles; tile++) {
+        const uint32_t buf = tile & 1u, kt = lo + tile * BN;
+        if (tile + 1 < tiles) {
+            stage(tile + 1, buf ^ 1u);
+            asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        }
+        __syncthreads();
+        const uint32_t kb = smem_addr(s_k + buf * BN * PK) + b_off, vb = smem_addr(s_v + buf * BN * PV) + v_off;
+        float s[BN / 8][4];
+#pragma unroll
+        for (int n = 0; n < (int)BN / 8; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) s[n][e] = 0.f;
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; kk++) {
+            uint32_t a[4];
+            ldmatrix4(a_addr + kk * 32, a);
+#pragma unroll
+            for (int n = 0; n < (int)BN / 16; n++) {
+                uint32_t b[4];
+                ldmatrix4(kb + (n * 16 * PK + kk * 16) * 2, b);
+                mma16816(s[2 * n], a, b[0], b[1]);
+                mma16816(s[2 * n + 1], a, b[2], b[3]);
+            }
+        }
+        // mask only where the tile crosses the diagonal or a row's window edge
+        const bool edge = kt + BN - 1 > first + warp * 16 || kt + p.window <= first + warp * 16 + 15;
+#pragma unroll
+        for (int h = 0; h < 2; h++) {
+            float mx = -INFINITY;
+#pragma unroll
+            for (int n = 0; n < (int)BN / 8; n++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    float &x = s[n][2 * h + e];
+                    x *= p.scale_log2;
+                    const uint32_t key = kt + n * 8 + (lane & 3u) * 2 + e;
+                    if (edge && !(key <= qp[h] && key + p.window > qp[h])) x = -INFINITY;
+                    mx = fmaxf(mx, x);
+                }
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+            const float m_new = fmaxf(m[h], mx), base = m_new == -INFINITY ? 0.f : m_new;
+            const float corr = exp2f(m[h] - base);        // nothing seen yet: exp2(-inf) = 0
+            m[h] = m_new;
+            float sum = 0.f;
+#pragma unroll
+            for (int n = 0; n < (int)BN / 8; n++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    float &x = s[n][2 * h + e];
+                    x = exp2f(x - base);
+                    sum += x;
+                }
+            l[h] = l[h] * corr + sum;
+#pragma unroll
+            for (int n = 0; n < DV / 8; n++) { o[n][2 * h] *= corr; o[n][2 * h + 1] *= corr; }
+        }
+#pragma unroll
+        for (int kk = 0; kk < (int)BN / 16; kk++) {
+            uint32_t hi[4], lo2[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const float x = s[2 * kk + j / 2][(j & 1) * 2], y = s[2 * kk + j / 2][(j & 1) * 2 + 1];
+                hi[j] = pack2(x, y);
+                lo2[j] = pack2(x - __uint_as_float(hi[j] << 16), y - __uint_as_float(hi[j] & 0xFFFF0000u));
+            }
+#pragma unroll
+            for (int n = 0; n < DV / 16; n++) {
+                uint32_t b[4];
+                ldmatrix4_t(vb + (kk * 16 * PV + n * 16) * 2, b);
+                mma16816(o[2 * n], hi, b[0], b[1]);
+                mma16816(o[2 * n + 1], hi, b[2], b[3]);
+                mma16816(o[2 * n], lo2, b[0], b[1]);
+                mma16816(o[2 * n + 1], lo2, b[2], b[3]);
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
+        l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
+        const uint32_t row = row0 + qrow + h * 8;
+        if (row >= p.rows) continue;
+        const float inv = 1.0f / l[h];
+        const size_t base = ((size_t)row * p.heads + head) * p.vdim;
+#pragma unroll
+        for (int n = 0; n < DV / 8; n++) {
+            const uint32_t v = n * 8 + (lane & 3u) * 2;
+            if (v >= p.vdim) break;
+            float x = o[n][2 * h] * inv, y = o[n][2 * h + 1] * inv;
+            if (p.gate) {
+                const float2 g = *reinterpret_cast<const float2 *>(p.gate + base + v);
+                x *= sigmoid_f(g.x) * (p.silu ? g.x : 1.f);
+                y *= sigmoid_f(g.y) * (p.silu ? g.y : 1.f);
+            }
+            if (p.out_bf16) *reinterpret_cast<uint32_t *>(static_cast<__nv_bfloat16 *>(p.out) + base + v) = pack2(x, y);
+            else            *reinterpret_cast<float2 *>(static_cast<float *>(p.out) + base + v) = make_float2(x, y);
+        }
+    }
+}
+
+template <int DK, int DV>
+int launch_prefill(const Prefill &p, cudaStream_t st)
+{
+    const size_t smem = ((size_t)(BM + 2 * BN) * (DK + 8) + (size_t)2 * BN * (DV + 8)) * 2;
+    if (int rc = allow_smem(latent_prefill_kernel<DK, DV>, smem)) return rc;
+    return launch(latent_prefill_kernel<DK, DV>, dim3((p.rows + BM - 1) / BM, p.heads), dim3(128), smem, st, p);
+}
+
+template <int DK>
+int launch_prefill_v(const Prefill &p, cudaStream_t st)
+{
+    if (p.vdim <= 64) return launch_prefill<DK, 64>(p, st);
+    return launch_prefill<DK, 128>(p, st);
+}
+
+size_t align256(size_t n) { return (n + 255) & ~(size_t)255; }
+
+}  // namespace
+
+bool latent_prefill_eligible(uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t rank, bool cache_bf16)
+{
+    return cache_bf16 && dim % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 && rank % 8 == 0 && dim + rot_dim <= 256 && vdim <= 128;
+}
+
+size_t latent_prefill_workspace(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t slots)
+{
+    return align256((size_t)slots * heads * dim * 2) + align256((size_t)slots * heads * vdim * 2);
+}
+
+int launch_latent_prefill(const LatentAttention &a, void *stream)
+{
+    __nv_bfloat16 *keys = static_cast<__nv_bfloat16 *>(a.workspace);
+    __nv_bfloat16 *values = reinterpret_cast<__nv_bfloat16 *>(static_cast<uint8_t *>(a.workspace) + align256((size_t)a.slots * a.heads * a.dim * 2));
+    LinearGroup g{};
+    g.count = 2; g.m = a.slots; g.k = a.rank; g.lda = a.rank + a.rot_dim;
+    g.a_bf16 = 1; g.out_bf16 = 1; g.live = a.pos; g.live_add = a.rows;
+    g.seg[0].a = g.seg[1].a = a.cache;
+    g.seg[0].w = a.uk; g.seg[0].out = keys; g.seg[0].n = a.heads * a.dim;
+    g.seg[1].w = a.uv; g.seg[1].out = values; g.seg[1].n = a.heads * a.vdim;
+    if (int rc = launch_linear_tc(g, stream)) return rc;
+    Prefill p{};
+    p.q = a.q; p.freq = a.freq; p.keys = keys; p.values = values; p.cache = static_cast<const __nv_bfloat16 *>(a.cache); p.pos = a.pos;
+    p.gate = a.gate ? a.gate->gate : nullptr;
+    p.out = a.gate ? a.gate->out : a.o;
+    p.rows = a.rows; p.heads = a.heads; p.dim = a.dim; p.rot = a.rot_dim; p.vdim = a.vdim; p.rank = a.rank; p.slots = a.slots; p.window = a.window;
+    p.scale_log2 = a.scale * 1.4426950408889634f;
+    p.out_bf16 = a.gate && a.gate->out_bf16; p.silu = a.gate && a.gate->silu;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const uint32_t dk = a.dim + a.rot_dim;
+    if (dk <= 64) return launch_prefill_v<64>(p, st);
+    if (dk <= 96) return launch_prefill_v<96>(p, st);
+    if (dk <= 128) return launch_prefill_v<128>(p, st);
+    if (dk <= 192) return launch_prefill_v<192>(p, st);
+    return launch_prefill_v<256>(p, st);
+}
+
+}  // namespace mgq

@@ -11,14 +11,18 @@ struct LinearSegment {
     const void *w, *w2;           // [n, k] bf16; w2: the up projection of a GLU pair (w is the gate)
     const float *bias, *bias2;    // [n] or null
     const float *addend;          // [m, n] f32 or null
-    void *out;                    // [m, n] f32 (GLU: f32 or bf16)
+    void *out;                    // [m, n] f32, or bf16 when the group says so
     uint32_t n;
 };
 
 struct LinearGroup {
     LinearSegment seg[kMaxSegments];
     uint32_t count, m, k;
-    uint32_t a_bf16, glu, out_bf16;
+    uint32_t a_bf16, glu;
+    uint32_t out_bf16;            // GLU, and the tcgen05 path without an addend
+    uint32_t lda;                 // elements between rows of a; 0: k (tcgen05 path only)
+    const uint32_t *live;         // tcgen05 path: only rows below *live + live_add are wanted; null: all
+    uint32_t live_add;
     float limit, alpha;           // clamped GLU
 };
 

@@ -43,9 +43,8 @@ struct Tile {
 
 // Tile index -> layer, row block, column block (COLS output columns per tile).
 template <uint32_t COLS>
-__device__ __forceinline__ Tile find_tile(const LinearGroup &g, uint32_t tile)
+__device__ __forceinline__ Tile find_tile(const LinearGroup &g, uint32_t tile, uint32_t mt)
 {
-    const uint32_t mt = (g.m + TM - 1) / TM;
     uint32_t nt = tile / mt, si = 0;
     const uint32_t m0 = (tile - nt * mt) * TM;
     while (si + 1 < g.count) {
@@ -88,6 +87,12 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
     const uint32_t tmem = sh.tmem_base;
     pdl_launch_dependents();
     pdl_wait();
+    uint32_t mt = (g.m + TM - 1) / TM;
+    if (g.live) {                                        // fewer row blocks, so fewer tiles
+        const uint32_t all = mt;
+        mt = min(mt, (g.live[0] + g.live_add + TM - 1) / TM);
+        tiles = tiles / all * mt;
+    }
 
     if (warp == 0) {
         if (lane == 0) {
@@ -95,7 +100,7 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
             int armed = -1;
             bool ok = true;
             for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
-                const Tile tl = find_tile<COLS>(g, tile);
+                const Tile tl = find_tile<COLS>(g, tile, mt);
                 for (uint32_t kc = 0; kc < nk; kc++, it++) {
                     const uint32_t s = it % S, ph = (it / S) & 1u;
                     ok = mbar_wait(&sh.empty[s], ph ^ 1u, &sh.failed, &g_linear_tc_error);
@@ -146,7 +151,7 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             tc_fence_after();
-            const Tile tl = find_tile<COLS>(g, tile);
+            const Tile tl = find_tile<COLS>(g, tile, mt);
             const LinearSegment &sg = g.seg[tl.si];
             const uint32_t row = tl.m0 + quad * 32 + lane, n = sg.n;
             const bool live = row < g.m;
@@ -169,7 +174,7 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
                         else if (sg.bias) y[e] += __ldg(sg.bias + col + e);
                     }
                 }
-                if (GLU && g.out_bf16) {
+                if (g.out_bf16) {
                     __nv_bfloat16 *out = static_cast<__nv_bfloat16 *>(sg.out) + o;
                     if (n % 8 == 0 && col + 16 <= n) {
                         uint32_t q[8];
@@ -218,10 +223,10 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
     }
 }
 
-int encode_rows(EncodeTiledFn encode, CUtensorMap &map, const void *base, uint32_t k, uint32_t rows, uint32_t box_rows)
+int encode_rows(EncodeTiledFn encode, CUtensorMap &map, const void *base, uint32_t k, uint32_t ld, uint32_t rows, uint32_t box_rows)
 {
     const cuuint64_t dims[2] = {k, rows};
-    const cuuint64_t strides[1] = {(cuuint64_t)k * 2};
+    const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
     const cuuint32_t box[2] = {TK, box_rows};
     const cuuint32_t elem[2] = {1, 1};
     const CUresult cr = encode(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, elem,
@@ -240,10 +245,10 @@ int launch_tc(const LinearGroup &g, cudaStream_t stream)
     uint32_t tiles = 0;
     for (uint32_t i = 0; i < g.count; i++) {
         const LinearSegment &s = g.seg[i];
-        if (int rc = encode_rows(encode, maps.a[i], s.a, g.k, g.m, TM)) return rc;
-        if (int rc = encode_rows(encode, maps.w[i], s.w, g.k, s.n, COLS)) return rc;
+        if (int rc = encode_rows(encode, maps.a[i], s.a, g.k, g.lda ? g.lda : g.k, g.m, TM)) return rc;
+        if (int rc = encode_rows(encode, maps.w[i], s.w, g.k, g.k, s.n, COLS)) return rc;
         if (GLU)
-            if (int rc = encode_rows(encode, maps.w2[i], s.w2, g.k, s.n, COLS)) return rc;
+            if (int rc = encode_rows(encode, maps.w2[i], s.w2, g.k, g.k, s.n, COLS)) return rc;
         tiles += (s.n + COLS - 1) / COLS;
     }
     tiles *= (g.m + TM - 1) / TM;

@@ -25,6 +25,14 @@ __device__ __forceinline__ float block_sum(float v, float *s_part)
     return total;
 }
 
+template <typename OT> __device__ __forceinline__ void store4(OT *p, float a, float b, float c, float d);
+template <> __device__ __forceinline__ void store4<float>(float *p, float a, float b, float c, float d) { *reinterpret_cast<float4 *>(p) = make_float4(a, b, c, d); }
+template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16 *p, float a, float b, float c, float d)
+{
+    const __nv_bfloat162 x = __floats2bfloat162_rn(a, b), y = __floats2bfloat162_rn(c, d);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&x), *reinterpret_cast<const uint32_t *>(&y));
+}
+
 // ---------------------------------------------------------------- embedding, rows, element-wise
 template <typename T>
 __global__ void embedding_scaled_kernel(const uint32_t *ids, const T *table, float *out, uint32_t rows, uint32_t width, uint32_t vocab, float scale)
@@ -72,6 +80,29 @@ __global__ void __launch_bounds__(256) norm_kernel(const float *x, const float *
     constexpr int HOLD = 16;                     // values a thread keeps between the two passes
     __shared__ float s_part[8];
     const uint32_t t = threadIdx.x;
+    if (cols % 4 == 0 && cols <= 4096) {         // float4 form
+        const uint32_t n4 = cols / 4;
+        float4 w[4], v[4];
+        pdl_launch_dependents();
+#pragma unroll
+        for (int i = 0; i < 4; i++) w[i] = t + 256u * i < n4 ? __ldg(reinterpret_cast<const float4 *>(weight) + t + 256u * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        pdl_wait();
+        const float4 *src = reinterpret_cast<const float4 *>(x + (size_t)(index ? min(index[blockIdx.x], src_rows - 1u) : blockIdx.x) * cols);
+        OT *dst = out + (size_t)blockIdx.x * cols;
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            v[i] = t + 256u * i < n4 ? src[t + 256u * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+            ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+        }
+        const float r = 1.0f / sqrtf(block_sum(ss, s_part) / (float)cols + eps);
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+            if (t + 256u * i < n4)
+                store4<OT>(dst + 4 * (t + 256u * i), v[i].x * r * (offset + w[i].x), v[i].y * r * (offset + w[i].y), v[i].z * r * (offset + w[i].z),
+                           v[i].w * r * (offset + w[i].w));
+        return;
+    }
     float w[HOLD], v[HOLD];
     pdl_launch_dependents();
 #pragma unroll
@@ -121,6 +152,68 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const __grid_constant_
         const float hp = row && a.norm_weight ? before[j] * r_before * g : before[j];        // the state already holds a normed h
         for (uint32_t s = 0; s < a.slots; s++) out[s * a.slot_stride + j] = from_f32<OT>(fmaf(hp - h, a.mu[s][j], h));
         if (last) a.state[width + j] = h;
+    }
+}
+
+// Vector form: NV float4 of a row per thread, RB consecutive rows per CTA (the previous row stays in
+// registers).  A single row is spread over gridDim.y CTAs, each of which sums the whole row and writes
+// one group of 1024 channels.
+template <typename OT, int NV>
+__global__ void __launch_bounds__(256) token_shift_vec_kernel(const __grid_constant__ TokenShift a, uint32_t rows_per_cta)
+{
+    __shared__ float s_part[8];
+    const uint32_t t = threadIdx.x, width = a.width, n4 = width / 4, row0 = blockIdx.x * rows_per_cta, row1 = min(row0 + rows_per_cta, a.rows);
+    const bool sliced = gridDim.y > 1;
+    float4 g[NV];
+    pdl_launch_dependents();
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const uint32_t j = t + 256u * i;
+        g[i] = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (a.norm_weight && j < n4) {
+            const float4 w = __ldg(reinterpret_cast<const float4 *>(a.norm_weight) + j);
+            g[i] = make_float4(a.offset + w.x, a.offset + w.y, a.offset + w.z, a.offset + w.w);
+        }
+        if (sliced && (uint32_t)i == blockIdx.y && j < n4)
+            for (uint32_t s = 0; s < a.slots; s++) asm volatile("prefetch.global.L1 [%0];" ::"l"(a.mu[s] + 4 * j));
+    }
+    pdl_wait();
+    auto load_h = [&](uint32_t row, float4 (&h)[NV]) {
+        const float4 *src = reinterpret_cast<const float4 *>(a.x + (size_t)row * width);
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; i++) {
+            h[i] = t + 256u * i < n4 ? src[t + 256u * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+            ss += h[i].x * h[i].x + h[i].y * h[i].y + h[i].z * h[i].z + h[i].w * h[i].w;
+        }
+        if (!a.norm_weight) return;
+        const float r = 1.0f / sqrtf(block_sum(ss, s_part) / (float)width + a.eps);
+#pragma unroll
+        for (int i = 0; i < NV; i++) { h[i].x *= r * g[i].x; h[i].y *= r * g[i].y; h[i].z *= r * g[i].z; h[i].w *= r * g[i].w; }
+    };
+    float4 prev[NV], h[NV];
+    if (row0) {
+        load_h(row0 - 1, prev);
+    } else {
+#pragma unroll
+        for (int i = 0; i < NV; i++) prev[i] = t + 256u * i < n4 ? reinterpret_cast<const float4 *>(a.state)[t + 256u * i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    for (uint32_t row = row0; row < row1; row++) {
+        load_h(row, h);
+        OT *out = static_cast<OT *>(a.out) + (size_t)row * width;
+#pragma unroll
+        for (int i = 0; i < NV; i++) {
+            const uint32_t j = t + 256u * i;
+            if (j >= n4 || (sliced && (uint32_t)i != blockIdx.y)) continue;
+            const float4 d = make_float4(prev[i].x - h[i].x, prev[i].y - h[i].y, prev[i].z - h[i].z, prev[i].w - h[i].w);
+            for (uint32_t s = 0; s < a.slots; s++) {
+                const float4 m = *(reinterpret_cast<const float4 *>(a.mu[s]) + j);
+                store4<OT>(out + s * a.slot_stride + 4 * j, fmaf(d.x, m.x, h[i].x), fmaf(d.y, m.y, h[i].y), fmaf(d.z, m.z, h[i].z), fmaf(d.w, m.w, h[i].w));
+            }
+            if (row + 1 == a.rows) reinterpret_cast<float4 *>(a.state + width)[j] = h[i];
+        }
+#pragma unroll
+        for (int i = 0; i < NV; i++) prev[i] = h[i];
     }
 }
 
@@ -208,9 +301,9 @@ template <int RPT> __host__ __device__ constexpr int chunk_tokens() { return RPT
 
 __device__ __forceinline__ float log_sigmoid(float z) { return z < 0.f ? z - log1pf(expf(z)) : -log1pf(expf(-z)); }
 
-// One token of one value column for the RPT keys this thread owns; returns the partial dot products.
+// One token of one value column for the RPT keys this thread owns; returns its share of the dot products.
 template <int MODE, int RPT>
-__device__ __forceinline__ void token_step(const float *q, const float *k, const float *w, const float (&u)[RPT], float v, float a, float b,
+__device__ __forceinline__ void token_update(const float *q, const float *k, const float *w, const float (&u)[RPT], float v, float a, float b,
                                            float (&S)[RPT], float (&n)[RPT], float &out, float &den)
 {
     float o[2] = {0.f, 0.f}, d[2] = {0.f, 0.f};
@@ -240,11 +333,38 @@ __device__ __forceinline__ void token_step(const float *q, const float *k, const
     }
     out = o[0] + o[1];
     den = d[0] + d[1];
+}
+
+// The same with the sums over the column's 8 threads.
+template <int MODE, int RPT>
+__device__ __forceinline__ void token_step(const float *q, const float *k, const float *w, const float (&u)[RPT], float v, float a, float b,
+                                           float (&S)[RPT], float (&n)[RPT], float &out, float &den)
+{
+    token_update<MODE, RPT>(q, k, w, u, v, a, b, S, n, out, den);
 #pragma unroll
     for (int off = 4; off > 0; off >>= 1) {
         out += __shfl_xor_sync(0xffffffffu, out, off);
         if (MODE == kMlstm) den += __shfl_xor_sync(0xffffffffu, den, off);
     }
+}
+
+// Sums x[t] over the 8 threads of a column for 8 tokens at once: every exchange halves the tokens a
+// thread is responsible for; thread ks ends up with the total of token ks.
+__device__ __forceinline__ float reduce8(const float (&x)[8], uint32_t ks)
+{
+    float y[4], z[2];
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const bool up = ks & 4u;
+        y[i] = (up ? x[i + 4] : x[i]) + __shfl_xor_sync(0xffffffffu, up ? x[i] : x[i + 4], 4);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+        const bool up = ks & 2u;
+        z[i] = (up ? y[i + 2] : y[i]) + __shfl_xor_sync(0xffffffffu, up ? y[i] : y[i + 2], 2);
+    }
+    const bool up = ks & 1u;
+    return (up ? z[1] : z[0]) + __shfl_xor_sync(0xffffffffu, up ? z[0] : z[1], 1);
 }
 
 __device__ __forceinline__ float mlstm_out(float out, float den, float qscale, float floor_)
@@ -285,7 +405,7 @@ __device__ __forceinline__ float *normalizer(const Scan &p, uint32_t head, uint3
 }
 
 template <int MODE, int RPT>
-__global__ void __launch_bounds__(kScanThreads) scan_kernel(const __grid_constant__ Scan p)
+__global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_constant__ Scan p)
 {
     constexpr int TC = chunk_tokens<RPT>(), KS = RPT * 8, NA = MODE == kWkv ? 3 : 2;
     extern __shared__ __align__(16) float smem[];
@@ -376,8 +496,20 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const __grid_constan
         const float *sv = base + NA * TC * KS + t / 8;
         const uint32_t r0 = c * TC, cnt = min((uint32_t)TC, p.rows - r0);
         float *dst = p.o + (size_t)r0 * vpitch + head * vdim + col;
-#pragma unroll 2
-        for (uint32_t r = 0; r < cnt; r++) {
+        uint32_t r = 0;
+        for (; r + 8 <= cnt; r += 8) {                       // 8 tokens at a time: one shared reduction, loads run ahead
+            float out[8], den[8];
+#pragma unroll
+            for (int i = 0; i < 8; i++) {
+                float a = 0.f, b = 0.f;
+                if (MODE == kMlstm) { a = s_gate[buf][0][r + i]; b = s_gate[buf][1][r + i]; }
+                token_update<MODE, RPT>(sq + (r + i) * KS, sk + (r + i) * KS, sw + (r + i) * KS, u, sv[(r + i) * kScanCols], a, b, S, n, out[i], den[i]);
+            }
+            float y = reduce8(out, ks);
+            if (MODE == kMlstm) y = mlstm_out(y, reduce8(den, ks), p.qscale, s_gate[buf][2][r + ks]);
+            if (live) dst[(size_t)(r + ks) * vpitch] = y;
+        }
+        for (; r < cnt; r++) {
             float out, den, a = 0.f, b = 0.f;
             if (MODE == kMlstm) { a = s_gate[buf][0][r]; b = s_gate[buf][1][r]; }
             token_step<MODE, RPT>(sq + r * KS, sk + r * KS, sw + r * KS, u, sv[r * kScanCols], a, b, S, n, out, den);
@@ -582,10 +714,23 @@ int launch_clamped_glu(const float *gate, const float *up, void *out, bool out_b
     return launch(clamped_glu_kernel<float>, dim3(blocks_for(len)), dim3(256), 0, st, gate, up, static_cast<float *>(out), len, limit, alpha);
 }
 
+template <typename OT>
+static int launch_token_shift_vec(const TokenShift &a, cudaStream_t st)
+{
+    const uint32_t nv = (a.width + 1023) / 1024, per = a.rows >= 592 ? 4 : 1;
+    const dim3 grid((a.rows + per - 1) / per, a.rows == 1 ? nv : 1);
+    if (nv <= 1) return launch(token_shift_vec_kernel<OT, 1>, grid, dim3(256), 0, st, a, per);
+    if (nv <= 2) return launch(token_shift_vec_kernel<OT, 2>, grid, dim3(256), 0, st, a, per);
+    if (nv <= 4) return launch(token_shift_vec_kernel<OT, 4>, grid, dim3(256), 0, st, a, per);
+    return launch(token_shift_vec_kernel<OT, 8>, grid, dim3(256), 0, st, a, per);
+}
+
 int launch_token_shift(const TokenShift &a, void *stream)
 {
     if (a.slots == 0 || a.slots > kMaxShifts) return fail(MGQ_ERR_SHAPE, "token_shift: %u mixes (1..%d)", a.slots, kMaxShifts);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (a.width % 4 == 0 && a.width <= 8192 && reinterpret_cast<uintptr_t>(a.x) % 16 == 0)
+        return a.out_bf16 ? launch_token_shift_vec<__nv_bfloat16>(a, st) : launch_token_shift_vec<float>(a, st);
     if (a.out_bf16) return launch(token_shift_kernel<__nv_bfloat16>, dim3(a.rows), dim3(256), 0, st, a);
     return launch(token_shift_kernel<float>, dim3(a.rows), dim3(256), 0, st, a);
 }

@@ -297,13 +297,13 @@ def test_latent_attention_portions_and_ring(fuse, heads, dim, rot, vdim, rank, w
         at += n
 
 
-@pytest.mark.parametrize("rows", [1, 2, 40])
+@pytest.mark.parametrize("rows", [1, 2, 40, 64, 150])
 @pytest.mark.parametrize("cache_bf16", [False, True])
-@pytest.mark.parametrize("window", [7, 32, 64, 65])
+@pytest.mark.parametrize("window", [7, 32, 64, 65, 130])
 def test_window_edge_is_exact(rows, cache_bf16, window):
     """One key stands out by a score of about 50: while it is visible it takes the whole softmax."""
     heads, dim, rot, vdim, rank = 2, 16, 8, 16, 32
-    feed, oracle, s, tables = latent_case(heads, dim, rot, vdim, rank, window, 40, cache_bf16=cache_bf16, q_gain=0.05, base=1e9)
+    feed, oracle, s, tables = latent_case(heads, dim, rot, vdim, rank, window, 150, cache_bf16=cache_bf16, q_gain=0.05, base=1e9)
     r = rng_of(77)
     down = (r.standard_normal((64, rank + rot)) * 0.5).astype(np.float32)
     q = (r.standard_normal((64, heads, dim + rot)) * 0.05).astype(np.float32)
@@ -324,6 +324,19 @@ def test_window_edge_is_exact(rows, cache_bf16, window):
     while at < len(tokens):
         n = min(rows, len(tokens) - at)
         close(feed(tokens[at:at + n], at)[0], want[at:at + n], 2e-2 if cache_bf16 else 1e-4)
+        at += n
+
+
+@pytest.mark.parametrize("heads,dim,rot,vdim,rank,window", [(2, 16, 8, 24, 32, 10), (3, 32, 16, 40, 64, 300), (9, 64, 32, 64, 136, 100), (2, 72, 24, 128, 256, 77),
+                                                            (1, 128, 64, 128, 512, 128), (4, 184, 8, 8, 40, 64)])
+def test_latent_attention_many_rows(heads, dim, rot, vdim, rank, window):
+    """Portions of 64 and more rows (expanded keys and values), with fewer rows in between, several rings long."""
+    feed, oracle, _, _ = latent_case(heads, dim, rot, vdim, rank, window, 200, cache_bf16=True, q_gain=2.0)
+    sizes = [200, 64, 1, 100, 63, 65, 2, 199, 128]
+    tokens = rng_of(5, window).integers(0, 64, sum(sizes))
+    want, at = oracle(tokens, window), 0
+    for n in sizes:
+        close(feed(tokens[at:at + n], at)[0], want[at:at + n], 3e-2)
         at += n
 
 
