@@ -7,6 +7,8 @@
 //   latent_absorb_kernel   q' = scale * [W_uk^T q_nope | rotate(q_rot)]
 //   latent_attend_kernel   CTA = 8 heads (a warp each) x one row x one slice of the window, 32 keys per tile,
 //                          online softmax in f32; slices leave (max, sum, unnormalised o')
+//   latent_attend_mma_kernel   the same for bf16 caches: 16 heads x 64 keys on the tensor cores; the f32
+//                          query and the f32 weights enter as sums of two bf16
 //   latent_out_kernel      merges the slices, applies W_uv and the output gate
 // The ring cache is addressed by position % slots, so a sequence may be longer than the cache.
 #include <algorithm>
@@ -18,7 +20,7 @@ namespace {
 
 constexpr uint32_t kHeads = 8;             // heads per CTA in latent_attend_kernel
 constexpr uint32_t kTile = 32;             // keys per tile
-constexpr uint32_t kSliceKeys = 32;        // window positions per slice when the window is split
+constexpr uint32_t kSliceKeys = 64;        // window positions per slice when the window is split
 constexpr uint32_t kSplitRows = 16;        // at most this many rows split the window over CTAs
 
 __device__ __forceinline__ void rotate_pair(float u, float v, uint32_t pos, float freq, float &ru, float &rv)
@@ -65,6 +67,8 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constan
     const uint32_t qpitch = a.heads * (dim + rot), width = a.rank + rot, rows = min((uint32_t)AR, a.rows - row0);
     float *s_q = smem, *s_p = smem + AR * dim;
     pdl_launch_dependents();
+    for (uint32_t d = t; d < dim; d += 256)              // weights are immutable: towards L2 before the wait
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(static_cast<const __nv_bfloat16 *>(a.uk) + ((size_t)head * dim + d) * a.rank + c0));
     pdl_wait();
     for (uint32_t i = t; i < AR * dim; i += 256) {
         const uint32_t r = i / dim;
@@ -79,7 +83,7 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constan
         const bool two = c + 1 < a.rank;
         const bool wide = two && a.rank % 2 == 0;
         const __nv_bfloat16 *w = static_cast<const __nv_bfloat16 *>(a.uk) + (size_t)head * dim * a.rank + c;
-#pragma unroll 8
+#pragma unroll(AR == 1 ? 16 : 8)
         for (uint32_t d = slice; d < dim; d += 8) {
             float w0, w1;
             if (wide) {
@@ -279,6 +283,153 @@ __global__ void __launch_bounds__(256) latent_attend_kernel(const __grid_constan
     if (lane == 0 && warp < heads) { ml[(part + warp) * 2] = m; ml[(part + warp) * 2 + 1] = l; }
 }
 
+// ---------------------------------------------------------------- the same on the tensor cores (bf16 cache, sizes in multiples of 8)
+__device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldmatrix4(uint32_t addr, uint32_t (&r)[4])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldmatrix2(uint32_t addr, uint32_t (&r)[2])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldmatrix4_t(uint32_t addr, uint32_t (&r)[4])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
+{
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+constexpr uint32_t kMmaHeads = 16, kMmaTile = 64;
+__host__ __device__ inline uint32_t mma_pitch(uint32_t width) { return (width + 15u) / 16u * 16u + 8u; }      // an odd number of 16-byte pieces
+inline size_t mma_smem(uint32_t width) { return ((size_t)kMmaTile + 2 * kMmaHeads) * mma_pitch(width) * 2; }
+
+// NT: 16-column groups of the latent per warp (8 warps): rank <= 128 * NT.
+template <int NT>
+__global__ void __launch_bounds__(256) latent_attend_mma_kernel(const __grid_constant__ LatentAttention a, const float *qx, float *po, float *ml)
+{
+    extern __shared__ __align__(16) __nv_bfloat16 sm[];
+    __shared__ float s_s[kMmaHeads][kMmaTile + 1], s_corr[kMmaHeads];
+    __shared__ __align__(16) __nv_bfloat16 s_p[2][kMmaHeads][kMmaTile + 8];
+    const uint32_t t = threadIdx.x, lane = t & 31u, warp = t >> 5, width = a.rank + a.rot_dim, pitch = mma_pitch(width), k16 = (width + 15u) / 16u;
+    __nv_bfloat16 *s_k = sm, *s_hi = s_k + kMmaTile * pitch, *s_lo = s_hi + kMmaHeads * pitch;
+    const uint32_t h0 = blockIdx.x * kMmaHeads, split = blockIdx.y, splits = gridDim.y, row = blockIdx.z;
+    const uint32_t heads = min(kMmaHeads, a.heads - h0);
+    pdl_launch_dependents();
+    const uint32_t pad = k16 * 16 - width;               // zero columns behind the rows, so that garbage never meets a zero
+    for (uint32_t i = t; i < kMmaTile * pad; i += 256) s_k[(i / pad) * pitch + width + i % pad] = __float2bfloat16_rn(0.f);
+    pdl_wait();
+    const uint32_t pos = a.pos[0] + row, lo = pos + 1 > a.window ? pos + 1 - a.window : 0u, total = pos + 1 - lo;
+    const uint32_t per = ((total + splits - 1) / splits + kMmaTile - 1) / kMmaTile * kMmaTile;
+    const uint32_t k0 = min(lo + split * per, pos + 1), k1 = min(k0 + per, pos + 1);
+    const size_t part = ((size_t)row * splits + split) * a.heads + h0;
+    if (k0 >= k1) {
+        if (t < heads) { ml[(part + t) * 2] = -INFINITY; ml[(part + t) * 2 + 1] = 0.f; }
+        return;
+    }
+    const __nv_bfloat16 *cache = static_cast<const __nv_bfloat16 *>(a.cache);
+    auto stage = [&](uint32_t kt) {
+#pragma unroll
+        for (uint32_t r = warp; r < kMmaTile; r += 8) {                   // beyond the last key: a valid row, masked below
+            const __nv_bfloat16 *src = cache + (size_t)(min(kt + r, k1 - 1u) % a.slots) * width;
+            for (uint32_t j = lane * 8; j < width; j += 256) cp_async16(s_k + r * pitch + j, src + j);
+        }
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+    };
+    stage(k0);
+    const float *qsrc = qx + ((size_t)row * a.heads + h0) * width;
+    for (uint32_t h = warp; h < kMmaHeads; h += 8)
+#pragma unroll 4
+        for (uint32_t j = lane * 2; j < k16 * 16; j += 64) {
+            const float2 q = h < heads && j < width ? *reinterpret_cast<const float2 *>(qsrc + h * width + j) : make_float2(0.f, 0.f);
+            const __nv_bfloat162 hi = __floats2bfloat162_rn(q.x, q.y);
+            const float2 f = __bfloat1622float2(hi);
+            *reinterpret_cast<__nv_bfloat162 *>(s_hi + h * pitch + j) = hi;
+            *reinterpret_cast<__nv_bfloat162 *>(s_lo + h * pitch + j) = __floats2bfloat162_rn(q.x - f.x, q.y - f.y);
+        }
+    float o[2 * NT][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};      // m, l: heads 2 * warp, 2 * warp + 1
+#pragma unroll
+    for (int n = 0; n < 2 * NT; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) o[n][e] = 0.f;
+    const uint32_t a_off = (((lane & 7u) + ((lane >> 3) & 1u) * 8) * pitch + (lane >> 4) * 8) * 2;
+    const uint32_t hi_addr = smem_addr(s_hi) + a_off, lo_addr = smem_addr(s_lo) + a_off;
+    const uint32_t b_addr = smem_addr(s_k + (warp * 8 + (lane & 7u)) * pitch + ((lane >> 3) & 1u) * 8);
+    const uint32_t v_addr = smem_addr(s_k) + (((lane & 7u) + ((lane >> 3) & 1u) * 8) * pitch + (lane >> 4) * 8) * 2;
+    const uint32_t p_off = (((lane & 7u) + ((lane >> 3) & 1u) * 8) * (kMmaTile + 8) + (lane >> 4) * 8) * 2;
+    for (uint32_t kt = k0; kt < k1; kt += kMmaTile) {
+        asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        __syncthreads();
+        float s_hi_acc[4] = {0.f, 0.f, 0.f, 0.f}, s_lo_acc[4] = {0.f, 0.f, 0.f, 0.f};       // warp w: keys 8w .. 8w + 7
+#pragma unroll 4
+        for (uint32_t kk = 0; kk < k16; kk++) {
+            uint32_t ah[4], al[4], b[2];
+            ldmatrix4(hi_addr + kk * 32, ah);
+            ldmatrix4(lo_addr + kk * 32, al);
+            ldmatrix2(b_addr + kk * 32, b);
+            mma16816(s_hi_acc, ah, b[0], b[1]);
+            mma16816(s_lo_acc, al, b[0], b[1]);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; e++) s_s[lane / 4 + (e >> 1) * 8][warp * 8 + (lane & 3u) * 2 + (e & 1)] = s_hi_acc[e] + s_lo_acc[e];
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const uint32_t h = warp * 2 + i;
+            const float x = kt + lane < k1 ? s_s[h][lane] : -INFINITY, y = kt + lane + 32 < k1 ? s_s[h][lane + 32] : -INFINITY;
+            const float m_new = fmaxf(m[i], warp_max(fmaxf(x, y)));      // at least one key: finite
+            const float corr = expf(m[i] - m_new), px = expf(x - m_new), py = expf(y - m_new);
+            l[i] = l[i] * corr + warp_sum(px + py);
+            m[i] = m_new;
+            const __nv_bfloat16 hx = __float2bfloat16_rn(px), hy = __float2bfloat16_rn(py);
+            s_p[0][h][lane] = hx;
+            s_p[0][h][lane + 32] = hy;
+            s_p[1][h][lane] = __float2bfloat16_rn(px - __bfloat162float(hx));
+            s_p[1][h][lane + 32] = __float2bfloat16_rn(py - __bfloat162float(hy));
+            if (lane == 0) s_corr[h] = corr;
+        }
+        __syncthreads();
+        const float c0 = s_corr[lane / 4], c1 = s_corr[lane / 4 + 8];
+#pragma unroll
+        for (int n = 0; n < 2 * NT; n++) { o[n][0] *= c0; o[n][1] *= c0; o[n][2] *= c1; o[n][3] *= c1; }
+#pragma unroll
+        for (int kk = 0; kk < (int)kMmaTile / 16; kk++) {
+            uint32_t ph[4], pl[4];
+            ldmatrix4(smem_addr(s_p[0]) + p_off + kk * 32, ph);
+            ldmatrix4(smem_addr(s_p[1]) + p_off + kk * 32, pl);
+#pragma unroll
+            for (int n = 0; n < NT; n++) {
+                const uint32_t col = (warp * NT + n) * 16;
+                if (col >= a.rank) break;
+                uint32_t b[4];
+                ldmatrix4_t(v_addr + (kk * 16 * pitch + col) * 2, b);
+                mma16816(o[2 * n], ph, b[0], b[1]);
+                mma16816(o[2 * n + 1], ph, b[2], b[3]);
+                mma16816(o[2 * n], pl, b[0], b[1]);
+                mma16816(o[2 * n + 1], pl, b[2], b[3]);
+            }
+        }
+        __syncthreads();
+        if (kt + kMmaTile < k1) stage(kt + kMmaTile);
+    }
+#pragma unroll
+    for (int n = 0; n < 2 * NT; n++) {
+        const uint32_t col = (warp * NT + n / 2) * 16 + (n & 1) * 8 + (lane & 3u) * 2;
+        if (col >= a.rank) break;                        // rank % 8 == 0: pairs never straddle it
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const uint32_t h = lane / 4 + 8 * i;
+            if (h < heads) *reinterpret_cast<float2 *>(po + (part + h) * a.rank + col) = make_float2(o[n][2 * i], o[n][2 * i + 1]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 2; i++)
+        if (lane == 0 && warp * 2 + i < heads) { ml[(part + warp * 2 + i) * 2] = m[i]; ml[(part + warp * 2 + i) * 2 + 1] = l[i]; }
+}
+
 // ---------------------------------------------------------------- merge, W_uv, gate: CTA = row x head x 64 value dimensions
 constexpr uint32_t kOutThreads = 512, kOutDims = 64;
 
@@ -366,6 +517,22 @@ int launch_attend(const LatentAttention &a, const float *qx, float *po, float *m
     return launch_attend_dpt<CT, 2>(a, qx, po, ml, splits, st);
 }
 
+template <int NT>
+int launch_mma_nt(const LatentAttention &a, const float *qx, float *po, float *ml, uint32_t splits, cudaStream_t st)
+{
+    const size_t smem = mma_smem(a.rank + a.rot_dim);
+    if (int rc = allow_smem(latent_attend_mma_kernel<NT>, smem)) return rc;
+    return launch(latent_attend_mma_kernel<NT>, dim3((a.heads + kMmaHeads - 1) / kMmaHeads, splits, a.rows), dim3(256), smem, st, a, qx, po, ml);
+}
+
+int launch_mma(const LatentAttention &a, const float *qx, float *po, float *ml, uint32_t splits, cudaStream_t st)
+{
+    if (a.rank <= 128) return launch_mma_nt<1>(a, qx, po, ml, splits, st);
+    if (a.rank <= 256) return launch_mma_nt<2>(a, qx, po, ml, splits, st);
+    if (a.rank <= 512) return launch_mma_nt<4>(a, qx, po, ml, splits, st);
+    return launch_mma_nt<8>(a, qx, po, ml, splits, st);
+}
+
 template <int AR>
 int launch_absorb(const LatentAttention &a, float *qx, cudaStream_t st)
 {
@@ -405,7 +572,7 @@ size_t latent_attention_workspace(uint32_t max_rows, uint32_t heads, uint32_t di
 {
     if (!latent_prefill_eligible(dim, rot_dim, vdim, rank, cache_bf16)) return absorbed_bytes(max_rows, heads, rot_dim, rank, window);
     const size_t few = absorbed_bytes(std::min(max_rows, kPrefillRows - 1), heads, rot_dim, rank, window);
-    return max_rows < kPrefillRows ? few : std::max(few, latent_prefill_workspace(heads, dim, vdim, slots));
+    return max_rows < kPrefillRows ? few : std::max(few, latent_prefill_workspace(heads, dim, rot_dim, vdim, slots));
 }
 
 int launch_latent_attention(const LatentAttention &a, void *stream)
@@ -420,7 +587,8 @@ int launch_latent_attention(const LatentAttention &a, void *stream)
     float *po = reinterpret_cast<float *>(at);
     float *ml = reinterpret_cast<float *>(at + align256((size_t)a.rows * splits * a.heads * a.rank * 4));
     if (int rc = a.rows == 1 ? launch_absorb<1>(a, qx, st) : launch_absorb<8>(a, qx, st)) return rc;
-    if (int rc = a.cache_bf16 ? launch_attend<__nv_bfloat16>(a, qx, po, ml, splits, st) : launch_attend<float>(a, qx, po, ml, splits, st)) return rc;
+    const bool mma = a.cache_bf16 && a.rank % 8 == 0 && a.rot_dim % 8 == 0 && mma_smem(width) <= 210 * 1024;
+    if (int rc = mma ? launch_mma(a, qx, po, ml, splits, st) : a.cache_bf16 ? launch_attend<__nv_bfloat16>(a, qx, po, ml, splits, st) : launch_attend<float>(a, qx, po, ml, splits, st)) return rc;
     const HeadGate none{};
     const HeadGate &hg = a.gate ? *a.gate : none;
     void *out = a.gate ? a.gate->out : a.o;

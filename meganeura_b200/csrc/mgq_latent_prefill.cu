@@ -1,12 +1,15 @@
 // Latent attention for many rows (a prompt's portion), bf16 cache.
 //
 // The keys W_uk c and values W_uv c of all live cache rows are expanded once per step by the tcgen05
-// linear kernel (ring order, bf16); the attention kernel then works like a blockwise exact softmax:
+// linear kernel (ring order, f16); the attention kernel then works like a blockwise exact softmax:
 // CTA = one head x 64 query rows (4 warps x 16 rows), 64 keys per tile, double-buffered cp.async,
-// tensor-core products with f32 accumulation.  The shared rotated key part is read from the cache
-// itself, next to the head's expanded key.  Scores, maxima, sums and weights are f32; a weight enters the
-// product with the values as the sum of two bf16 (16 significant bits).  Only tiles that some row of the
+// tensor-core products with f32 accumulation.  The rotated key part, shared by the heads, is kept once.
+// Scores, maxima, sums and weights are f32.  The operands of the products are f16, not bf16: all are of
+// moderate size (a clamp guards the range), and with 11 significant bits the result stays close to the
+// absorbed form, which keeps the query in f32, so it hardly matters how a prompt is cut.  Only tiles that some row of the
 // CTA can see are visited; positions map to ring rows by position % slots.
+#include <cuda_fp16.h>
+
 #include "mgq_linear.cuh"
 #include "mgq_mixer.cuh"
 
@@ -30,18 +33,30 @@ __device__ __forceinline__ void ldmatrix4_t(uint32_t addr, uint32_t (&r)[4])
 }
 __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
 {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ uint32_t pack2(float x, float y)
 {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    const __half2 h = __floats2half2_rn(x, y);
     return *reinterpret_cast<const uint32_t *>(&h);
+}
+__device__ __forceinline__ __half to_half(float x) { return __float2half_rn(fminf(fmaxf(x, -65504.f), 65504.f)); }
+
+// The shared rotated key parts of the live cache rows as f16.
+__global__ void rotated_half_kernel(const __nv_bfloat16 *cache, const uint32_t *pos, __half *out, uint32_t rows, uint32_t slots, uint32_t rank, uint32_t rot)
+{
+    const uint32_t i = blockIdx.x * 256u + threadIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (i >= min(slots, pos[0] + rows) * rot) return;
+    const uint32_t slot = i / rot;
+    out[i] = to_half(__bfloat162float(cache[(size_t)slot * (rank + rot) + rank + i - slot * rot]));
 }
 
 struct Prefill {
     const float *q, *freq;
-    const __nv_bfloat16 *keys, *values, *cache;     // keys [slots, heads * dim], values [slots, heads * vdim]
+    const __half *keys, *values, *rotated;          // [slots, heads * dim], [slots, heads * vdim], [slots, rot]
     const uint32_t *pos;
     const float *gate;
     void *out;
@@ -55,12 +70,12 @@ template <int DK, int DV>
 __global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_constant__ Prefill p)
 {
     constexpr int PK = DK + 8, PV = DV + 8;          // row pitch in elements: an odd number of 16-byte pieces
-    extern __shared__ __align__(16) __nv_bfloat16 sm[];
-    __nv_bfloat16 *s_q = sm, *s_k = s_q + BM * PK, *s_v = s_k + 2 * BN * PK;
+    extern __shared__ __align__(16) __half sm[];
+    __half *s_q = sm, *s_k = s_q + BM * PK, *s_v = s_k + 2 * BN * PK;
     const uint32_t t = threadIdx.x, lane = t & 31u, warp = t >> 5, head = blockIdx.y;
-    const uint32_t row0 = (gridDim.x - 1 - blockIdx.x) * BM, dk = p.dim + p.rot, width = p.rank + p.rot;      // longest rows first
+    const uint32_t row0 = (gridDim.x - 1 - blockIdx.x) * BM, dk = p.dim + p.rot;      // longest rows first
     pdl_launch_dependents();
-    for (uint32_t i = t; i < (BM + 2 * BN) * PK + 2 * BN * PV; i += 128) sm[i] = __float2bfloat16_rn(0.f);    // padding columns stay zero
+    for (uint32_t i = t; i < (BM + 2 * BN) * PK + 2 * BN * PV; i += 128) sm[i] = __float2half_rn(0.f);    // padding columns stay zero
     pdl_wait();
     const uint32_t pos0 = p.pos[0], first = pos0 + row0, last = pos0 + min(row0 + BM, p.rows) - 1;
     const uint32_t lo = first + 1 > p.window ? first + 1 - p.window : 0u, tiles = (last - lo) / BN + 1;
@@ -73,7 +88,7 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_consta
         // two threads per key row
         const uint32_t r = t >> 1, half = t & 1u;
         const size_t slot = min(kt + r, last) % p.slots;                  // beyond the last key: a valid row, masked below
-        const __nv_bfloat16 *ksrc = p.keys + (slot * p.heads + head) * p.dim, *rsrc = p.cache + slot * width + p.rank,
+        const __half *ksrc = p.keys + (slot * p.heads + head) * p.dim, *rsrc = p.rotated + slot * p.rot,
                             *vsrc = p.values + (slot * p.heads + head) * p.vdim;
         for (uint32_t c = half; c < per_k; c += 2) cp_async16(kb + (r * PK + c * 8) * 2, ksrc + c * 8);
         for (uint32_t c = half; c < per_r; c += 2) cp_async16(kb + (r * PK + p.dim + c * 8) * 2, rsrc + c * 8);
@@ -89,13 +104,13 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_consta
         for (uint32_t r = warp; r < BM; r += 4) {
             if (row0 + r >= p.rows) break;
             const float *src = p.q + (size_t)(row0 + r) * pitch + head * dk;
-            for (uint32_t j = lane; j < p.dim; j += 32) s_q[r * PK + j] = __float2bfloat16_rn(src[j]);
+            for (uint32_t j = lane; j < p.dim; j += 32) s_q[r * PK + j] = to_half(src[j]);
             for (uint32_t i = lane; i < half; i += 32) {
                 float s, c;
                 sincosf((float)(pos0 + row0 + r) * p.freq[i], &s, &c);
                 const float u = src[p.dim + i], v = src[p.dim + half + i];
-                s_q[r * PK + p.dim + i] = __float2bfloat16_rn(u * c - v * s);
-                s_q[r * PK + p.dim + half + i] = __float2bfloat16_rn(v * c + u * s);
+                s_q[r * PK + p.dim + i] = to_half(u * c - v * s);
+                s_q[r * PK + p.dim + half + i] = to_half(v * c + u * s);
             }
         }
     }
@@ -172,21 +187,15 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_consta
         }
 #pragma unroll
         for (int kk = 0; kk < (int)BN / 16; kk++) {
-            uint32_t hi[4], lo2[4];
+            uint32_t w[4];
 #pragma unroll
-            for (int j = 0; j < 4; j++) {
-                const float x = s[2 * kk + j / 2][(j & 1) * 2], y = s[2 * kk + j / 2][(j & 1) * 2 + 1];
-                hi[j] = pack2(x, y);
-                lo2[j] = pack2(x - __uint_as_float(hi[j] << 16), y - __uint_as_float(hi[j] & 0xFFFF0000u));
-            }
+            for (int j = 0; j < 4; j++) w[j] = pack2(s[2 * kk + j / 2][(j & 1) * 2], s[2 * kk + j / 2][(j & 1) * 2 + 1]);
 #pragma unroll
             for (int n = 0; n < DV / 16; n++) {
                 uint32_t b[4];
                 ldmatrix4_t(vb + (kk * 16 * PV + n * 16) * 2, b);
-                mma16816(o[2 * n], hi, b[0], b[1]);
-                mma16816(o[2 * n + 1], hi, b[2], b[3]);
-                mma16816(o[2 * n], lo2, b[0], b[1]);
-                mma16816(o[2 * n + 1], lo2, b[2], b[3]);
+                mma16816(o[2 * n], w, b[0], b[1]);
+                mma16816(o[2 * n + 1], w, b[2], b[3]);
             }
         }
         __syncthreads();
@@ -209,7 +218,7 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_consta
                 x *= sigmoid_f(g.x) * (p.silu ? g.x : 1.f);
                 y *= sigmoid_f(g.y) * (p.silu ? g.y : 1.f);
             }
-            if (p.out_bf16) *reinterpret_cast<uint32_t *>(static_cast<__nv_bfloat16 *>(p.out) + base + v) = pack2(x, y);
+            if (p.out_bf16) *reinterpret_cast<__nv_bfloat162 *>(static_cast<__nv_bfloat16 *>(p.out) + base + v) = __floats2bfloat162_rn(x, y);
             else            *reinterpret_cast<float2 *>(static_cast<float *>(p.out) + base + v) = make_float2(x, y);
         }
     }
@@ -239,30 +248,37 @@ bool latent_prefill_eligible(uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint
     return cache_bf16 && dim % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 && rank % 8 == 0 && dim + rot_dim <= 256 && vdim <= 128;
 }
 
-size_t latent_prefill_workspace(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t slots)
+size_t latent_prefill_workspace(uint32_t heads, uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t slots)
 {
-    return align256((size_t)slots * heads * dim * 2) + align256((size_t)slots * heads * vdim * 2);
+    return align256((size_t)slots * heads * dim * 2) + align256((size_t)slots * heads * vdim * 2) + align256((size_t)slots * rot_dim * 2);
 }
 
 int launch_latent_prefill(const LatentAttention &a, void *stream)
 {
-    __nv_bfloat16 *keys = static_cast<__nv_bfloat16 *>(a.workspace);
-    __nv_bfloat16 *values = reinterpret_cast<__nv_bfloat16 *>(static_cast<uint8_t *>(a.workspace) + align256((size_t)a.slots * a.heads * a.dim * 2));
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    uint8_t *ws = static_cast<uint8_t *>(a.workspace);
+    __half *keys = reinterpret_cast<__half *>(ws);
+    ws += align256((size_t)a.slots * a.heads * a.dim * 2);
+    __half *values = reinterpret_cast<__half *>(ws);
+    ws += align256((size_t)a.slots * a.heads * a.vdim * 2);
+    __half *rotated = reinterpret_cast<__half *>(ws);
+    const __nv_bfloat16 *cache = static_cast<const __nv_bfloat16 *>(a.cache);
+    if (a.rot_dim)
+        if (int rc = launch(rotated_half_kernel, dim3((uint32_t)(((size_t)a.slots * a.rot_dim + 255) / 256)), dim3(256), 0, st, cache, a.pos, rotated, a.rows, a.slots, a.rank, a.rot_dim)) return rc;
     LinearGroup g{};
     g.count = 2; g.m = a.slots; g.k = a.rank; g.lda = a.rank + a.rot_dim;
-    g.a_bf16 = 1; g.out_bf16 = 1; g.live = a.pos; g.live_add = a.rows;
+    g.a_bf16 = 1; g.out_f16 = 1; g.live = a.pos; g.live_add = a.rows;
     g.seg[0].a = g.seg[1].a = a.cache;
     g.seg[0].w = a.uk; g.seg[0].out = keys; g.seg[0].n = a.heads * a.dim;
     g.seg[1].w = a.uv; g.seg[1].out = values; g.seg[1].n = a.heads * a.vdim;
     if (int rc = launch_linear_tc(g, stream)) return rc;
     Prefill p{};
-    p.q = a.q; p.freq = a.freq; p.keys = keys; p.values = values; p.cache = static_cast<const __nv_bfloat16 *>(a.cache); p.pos = a.pos;
+    p.q = a.q; p.freq = a.freq; p.keys = keys; p.values = values; p.rotated = rotated; p.pos = a.pos;
     p.gate = a.gate ? a.gate->gate : nullptr;
     p.out = a.gate ? a.gate->out : a.o;
     p.rows = a.rows; p.heads = a.heads; p.dim = a.dim; p.rot = a.rot_dim; p.vdim = a.vdim; p.rank = a.rank; p.slots = a.slots; p.window = a.window;
     p.scale_log2 = a.scale * 1.4426950408889634f;
     p.out_bf16 = a.gate && a.gate->out_bf16; p.silu = a.gate && a.gate->silu;
-    cudaStream_t st = static_cast<cudaStream_t>(stream);
     const uint32_t dk = a.dim + a.rot_dim;
     if (dk <= 64) return launch_prefill_v<64>(p, st);
     if (dk <= 96) return launch_prefill_v<96>(p, st);

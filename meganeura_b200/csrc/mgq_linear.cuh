@@ -19,7 +19,8 @@ struct LinearGroup {
     LinearSegment seg[kMaxSegments];
     uint32_t count, m, k;
     uint32_t a_bf16, glu;
-    uint32_t out_bf16;            // GLU, and the tcgen05 path without an addend
+    uint32_t out_bf16;            // GLU only
+    uint32_t out_f16;             // tcgen05 path without an addend: f16, clamped to its range
     uint32_t lda;                 // elements between rows of a; 0: k (tcgen05 path only)
     const uint32_t *live;         // tcgen05 path: only rows below *live + live_add are wanted; null: all
     uint32_t live_add;

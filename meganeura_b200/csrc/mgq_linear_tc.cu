@@ -11,6 +11,8 @@
 //               to empty[s] and the tile to acc_full[b].
 //   warps 2-5   epilogue of one accumulator while the other is being filled (2 x TN TMEM columns).
 // Every wait is bounded like in mgq_gemm_tc.cu.
+#include <cuda_fp16.h>
+
 #include "mgq_linear.cuh"
 #include "mgq_tcgen05.cuh"
 
@@ -174,7 +176,25 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
                         else if (sg.bias) y[e] += __ldg(sg.bias + col + e);
                     }
                 }
-                if (g.out_bf16) {
+                if (!GLU && g.out_f16) {
+                    __half *out = static_cast<__half *>(sg.out) + o;
+#pragma unroll
+                    for (int e = 0; e < 16; e++) y[e] = fminf(fmaxf(y[e], -65504.f), 65504.f);
+                    if (n % 8 == 0 && col + 16 <= n) {
+                        uint32_t q[8];
+#pragma unroll
+                        for (int e = 0; e < 8; e++) {
+                            const __half2 h = __floats2half2_rn(y[2 * e], y[2 * e + 1]);
+                            q[e] = *reinterpret_cast<const uint32_t *>(&h);
+                        }
+                        reinterpret_cast<uint4 *>(out)[0] = make_uint4(q[0], q[1], q[2], q[3]);
+                        reinterpret_cast<uint4 *>(out)[1] = make_uint4(q[4], q[5], q[6], q[7]);
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 16; e++)
+                            if (col + e < n) out[e] = __float2half_rn(y[e]);
+                    }
+                } else if (GLU && g.out_bf16) {
                     __nv_bfloat16 *out = static_cast<__nv_bfloat16 *>(sg.out) + o;
                     if (n % 8 == 0 && col + 16 <= n) {
                         uint32_t q[8];

@@ -99,7 +99,7 @@ int launch_latent_attention(const LatentAttention &a, void *stream);
 // from the latents once per step and the softmax runs tile by tile on the tensor cores.
 constexpr uint32_t kPrefillRows = 64;      // fewer rows take the absorbed form
 bool latent_prefill_eligible(uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t rank, bool cache_bf16);
-size_t latent_prefill_workspace(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t slots);
+size_t latent_prefill_workspace(uint32_t heads, uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t slots);
 int launch_latent_prefill(const LatentAttention &a, void *stream);
 
 }  // namespace mgq

@@ -45,6 +45,22 @@ __global__ void embedding_scaled_kernel(const uint32_t *ids, const T *table, flo
     out[i] = to_f32(table[(size_t)min(ids[row], vocab - 1u) * width + col]) * scale;
 }
 
+// 8 elements per thread (width % 8 == 0)
+template <typename T>
+__global__ void embedding_vec_kernel(const uint32_t *ids, const T *table, float *out, uint32_t rows, uint32_t width, uint32_t vocab, float scale)
+{
+    const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (i >= (size_t)rows * width) return;
+    const uint32_t row = (uint32_t)(i / width), col = (uint32_t)(i - (size_t)row * width);
+    float f[8];
+    load8(table + (size_t)min(ids[row], vocab - 1u) * width + col, f);
+    float4 *dst = reinterpret_cast<float4 *>(out + i);
+    dst[0] = make_float4(f[0] * scale, f[1] * scale, f[2] * scale, f[3] * scale);
+    dst[1] = make_float4(f[4] * scale, f[5] * scale, f[6] * scale, f[7] * scale);
+}
+
 __global__ void pick_rows_kernel(const float *x, const uint32_t *index, float *out, uint32_t rows, uint32_t src_rows, uint32_t cols)
 {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -247,30 +263,91 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const float *o, const __
     for (uint32_t j = lane + 32u * HOLD; j < dim; j += 32) put(j, o[base + j]);
 }
 
-// ---------------------------------------------------------------- decay: exp(-exp(tanh(low) . w2^T + w0)), 8 rows per CTA
-constexpr uint32_t kDecayRows = 8;
-__global__ void __launch_bounds__(128) decay_kernel(const __grid_constant__ Wkv a)
+// G lanes per (row, head), KV float4 per lane: dim <= 4 * G * KV, dim % 4 == 0.
+template <typename OT, int G, int KV>
+__global__ void __launch_bounds__(256) head_gate_vec_kernel(const float *o, const __grid_constant__ HeadGate hg, uint32_t total, uint32_t heads, uint32_t dim)
 {
-    extern __shared__ float s_low[];                     // [8][rank]
-    const uint32_t ch = blockIdx.x * 128u + threadIdx.x, row0 = blockIdx.y * kDecayRows, channels = a.heads * a.dim;
-    const uint32_t rows = min(kDecayRows, a.rows - row0);
+    const uint32_t unit = (blockIdx.x * 256u + threadIdx.x) / G, lane = threadIdx.x % G, n4 = dim / 4;
     pdl_launch_dependents();
     pdl_wait();
-    for (uint32_t i = threadIdx.x; i < kDecayRows * a.rank; i += 128)
-        s_low[i] = i < rows * a.rank ? tanhf(a.low[(size_t)row0 * a.rank + i]) : 0.f;
-    __syncthreads();
-    if (ch >= channels) return;
-    const __nv_bfloat16 *w = static_cast<const __nv_bfloat16 *>(a.w2) + (size_t)ch * a.rank;
-    const float w0 = a.w0[ch];
-    float acc[kDecayRows];
+    const bool live = unit < total;                      // no early return: the lanes of a warp reduce together
+    const size_t base = (size_t)(live ? unit : 0) * dim;
+    const uint32_t wbase = (live ? unit % heads : 0) * dim;
+    float4 v[KV], g[KV];
+    float ss = 0.f;
 #pragma unroll
-    for (int r = 0; r < (int)kDecayRows; r++) acc[r] = 0.f;
-    for (uint32_t j = 0; j < a.rank; j++) {
-        const float wv = __bfloat162float(w[j]);
-#pragma unroll
-        for (int r = 0; r < (int)kDecayRows; r++) acc[r] = fmaf(s_low[r * a.rank + j], wv, acc[r]);
+    for (int i = 0; i < KV; i++) {
+        const uint32_t j = lane + G * i;
+        v[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < n4) {
+            v[i] = *(reinterpret_cast<const float4 *>(o + base) + j);
+            g[i] = *(reinterpret_cast<const float4 *>(hg.gate + base) + j);
+        }
+        ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
     }
-    for (uint32_t r = 0; r < rows; r++) a.decay[(size_t)(row0 + r) * channels + ch] = expf(-expf(acc[r] + w0));
+    float r = 1.f;
+    if (hg.weight) {
+#pragma unroll
+        for (int off = G / 2; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+        r = 1.0f / sqrtf(ss / (float)dim + hg.eps);
+    }
+    if (!live) return;
+    OT *out = static_cast<OT *>(hg.out) + base;
+#pragma unroll
+    for (int i = 0; i < KV; i++) {
+        const uint32_t j = lane + G * i;
+        if (j >= n4) break;
+        float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (hg.weight) w = *(reinterpret_cast<const float4 *>(hg.weight + wbase) + j);
+        auto act = [&](float x) { const float sg = sigmoid_f(x); return hg.silu ? x * sg : sg; };
+        store4<OT>(out + 4 * j, v[i].x * r * w.x * act(g[i].x), v[i].y * r * w.y * act(g[i].y), v[i].z * r * w.z * act(g[i].z), v[i].w * r * w.w * act(g[i].w));
+    }
+}
+
+// ---------------------------------------------------------------- decay: exp(-exp(tanh(low) . w2^T + w0)), 64 rows x 64 channels per CTA
+constexpr uint32_t kDecayTile = 64, kDecayK = 16;
+__global__ void __launch_bounds__(256) decay_kernel(const __grid_constant__ Wkv a)
+{
+    __shared__ float s_low[kDecayK][kDecayTile + 4], s_w[kDecayK][kDecayTile + 4];
+    const uint32_t t = threadIdx.x, tx = t & 15u, ty = t >> 4, ch0 = blockIdx.x * kDecayTile, row0 = blockIdx.y * kDecayTile, channels = a.heads * a.dim;
+    const __nv_bfloat16 *w = static_cast<const __nv_bfloat16 *>(a.w2);
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) acc[i][j] = 0.f;
+    pdl_launch_dependents();
+    pdl_wait();
+    for (uint32_t k0 = 0; k0 < a.rank; k0 += kDecayK) {
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const uint32_t e = t + 256u * i, r = e / kDecayK, k = e % kDecayK;
+            const bool in = k0 + k < a.rank;
+            s_low[k][r] = in && row0 + r < a.rows ? tanhf(a.low[(size_t)(row0 + r) * a.rank + k0 + k]) : 0.f;
+            s_w[k][r] = in && ch0 + r < channels ? __bfloat162float(w[(size_t)(ch0 + r) * a.rank + k0 + k]) : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < (int)kDecayK; k++) {
+            const float4 x = *reinterpret_cast<const float4 *>(&s_low[k][ty * 4]), y = *reinterpret_cast<const float4 *>(&s_w[k][tx * 4]);
+            const float xr[4] = {x.x, x.y, x.z, x.w}, yr[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) acc[i][j] = fmaf(xr[i], yr[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const uint32_t row = row0 + ty * 4 + i;
+        if (row >= a.rows) break;
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const uint32_t ch = ch0 + tx * 4 + j;
+            if (ch < channels) a.decay[(size_t)row * channels + ch] = expf(-expf(acc[i][j] + a.w0[ch]));
+        }
+    }
 }
 
 // ---------------------------------------------------------------- recurrences
@@ -684,6 +761,11 @@ int launch_embedding_scaled(const uint32_t *ids, const void *table, bool table_b
 {
     const dim3 grid(blocks_for((size_t)rows * width));
     cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (width % 8 == 0) {
+        const dim3 grid8(blocks_for((size_t)rows * width / 8));
+        if (table_bf16) return launch(embedding_vec_kernel<__nv_bfloat16>, grid8, dim3(256), 0, st, ids, static_cast<const __nv_bfloat16 *>(table), out, rows, width, vocab, scale);
+        return launch(embedding_vec_kernel<float>, grid8, dim3(256), 0, st, ids, static_cast<const float *>(table), out, rows, width, vocab, scale);
+    }
     if (table_bf16) return launch(embedding_scaled_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, ids, static_cast<const __nv_bfloat16 *>(table), out, rows, width, vocab, scale);
     return launch(embedding_scaled_kernel<float>, grid, dim3(256), 0, st, ids, static_cast<const float *>(table), out, rows, width, vocab, scale);
 }
@@ -739,6 +821,16 @@ int launch_head_gate(const float *o, const HeadGate &hg, uint32_t rows, uint32_t
 {
     const uint32_t total = rows * heads;
     cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (dim % 4 == 0 && dim <= 512) {
+        auto go = [&](auto kernel_f32, auto kernel_bf16, uint32_t lanes) {
+            const dim3 grid((uint32_t)(((size_t)total * lanes + 255) / 256));
+            return hg.out_bf16 ? launch(kernel_bf16, grid, dim3(256), 0, st, o, hg, total, heads, dim) : launch(kernel_f32, grid, dim3(256), 0, st, o, hg, total, heads, dim);
+        };
+        if (dim <= 32) return go(head_gate_vec_kernel<float, 8, 1>, head_gate_vec_kernel<__nv_bfloat16, 8, 1>, 8);
+        if (dim <= 64) return go(head_gate_vec_kernel<float, 16, 1>, head_gate_vec_kernel<__nv_bfloat16, 16, 1>, 16);
+        if (dim <= 128) return go(head_gate_vec_kernel<float, 32, 1>, head_gate_vec_kernel<__nv_bfloat16, 32, 1>, 32);
+        return go(head_gate_vec_kernel<float, 32, 4>, head_gate_vec_kernel<__nv_bfloat16, 32, 4>, 32);
+    }
     if (hg.out_bf16) return launch(head_gate_kernel<__nv_bfloat16>, dim3((total + 7) / 8), dim3(256), 0, st, o, hg, total, heads, dim);
     return launch(head_gate_kernel<float>, dim3((total + 7) / 8), dim3(256), 0, st, o, hg, total, heads, dim);
 }
@@ -751,9 +843,7 @@ size_t mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim)
 
 int launch_decay(const Wkv &a, void *stream)
 {
-    const size_t smem = (size_t)kDecayRows * a.rank * sizeof(float);
-    if (int rc = allow_smem(decay_kernel, smem)) return rc;
-    return launch(decay_kernel, dim3((a.heads * a.dim + 127) / 128, (a.rows + kDecayRows - 1) / kDecayRows), dim3(128), smem,
+    return launch(decay_kernel, dim3((a.heads * a.dim + kDecayTile - 1) / kDecayTile, (a.rows + kDecayTile - 1) / kDecayTile), dim3(256), 0,
                   static_cast<cudaStream_t>(stream), a);
 }
 
