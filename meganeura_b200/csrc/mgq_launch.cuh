@@ -30,11 +30,11 @@ int launch(void (*kernel)(Params...), dim3 grid, dim3 block, size_t smem, cudaSt
     return MGQ_OK;
 }
 
-// Opts a kernel into more than 48 KB of dynamic shared memory (a no-op for the driver when repeated).
+// Opts a kernel into more than 48 KB of shared memory, static part included (a no-op for the driver when repeated).
 template <typename K>
 int allow_smem(K *kernel, size_t bytes)
 {
-    if (bytes <= 48 * 1024) return MGQ_OK;
+    if (bytes <= 32 * 1024) return MGQ_OK;
     MGQ_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes));
     return MGQ_OK;
 }

@@ -51,6 +51,7 @@ struct Wkv {
     const void *w2;
     float *decay, *o, *state, *shift_state;
     uint32_t rows, heads, dim, rank, shift_width;
+    void *workspace;                       // scan_workspace bytes, or null (long portions then run in one piece)
 };
 size_t wkv_state_elements(uint32_t heads, uint32_t dim);
 int launch_decay(const Wkv &a, void *stream);
@@ -58,13 +59,15 @@ int launch_wkv_scan(const Wkv &a, void *stream);
 int launch_wkv_step(const Wkv &a, const HeadGate &hg, void *stream);      // rows == 1: decay, recurrence, head gate in one launch
 
 // mLSTM recurrence.  q, k [rows, heads * dim], v, o [rows, heads * vdim], gate pre-activations
-// gi, gf [rows, heads].  State: per head [vdim][pad4(dim)], then n [heads][pad4(dim)], then m [heads].
+// gi, gf [rows, heads].  State: per head [vdim][pad4(dim)], then n and m per head and block of columns.
 struct Mlstm {
     const float *q, *k, *v, *gi, *gf;
     float *o, *state;
     uint32_t rows, heads, dim, vdim;
     float cap;
+    void *workspace;                       // as in Wkv
 };
+size_t scan_workspace(uint32_t max_rows, uint32_t heads, uint32_t dim, uint32_t vdim);
 size_t mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim);
 int launch_mlstm_scan(const Mlstm &a, void *stream);
 int launch_mlstm_step(const Mlstm &a, const HeadGate &hg, void *stream);

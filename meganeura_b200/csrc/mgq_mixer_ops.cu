@@ -3,12 +3,14 @@
 // operands of the next projection may be stored as bf16.
 //
 // The two recurrences share one schedule.  A head's state is kept value-major, [value][key], and a
-// thread owns RPT keys of one value column (8 threads per column), so a token step is register
-// arithmetic plus a 3-step shuffle; keys beyond `dim` are zero.
-//   scan_kernel  several tokens: CTA = head x 16 value columns, state in registers over the whole
-//                portion, the tokens' vectors staged through a double-buffered cp.async ring.
+// thread owns RPT keys of a few value columns (8 threads per group of columns), so a token step is
+// register arithmetic plus a short shuffle reduction; keys beyond `dim` are zero.
+//   scan_kernel  several tokens: CTA = head x a block of value columns (x a segment of a long portion),
+//                state in registers, the tokens' vectors staged through a double-buffered cp.async ring.
 //   step_kernel  one token: CTA = head; the decay projection (or the gates), the recurrence, the
 //                per-head norm and the output gate in one launch, state streamed once.
+#include <algorithm>
+
 #include "mgq_mixer.cuh"
 
 namespace mgq {
@@ -369,60 +371,75 @@ struct Scan {
     const float *u;                      // wkv bonus [heads, dim]
     const float *gi, *gf;                // mlstm gate pre-activations [rows, heads]
     float *o, *state, *shift_state;
+    float *segments;                     // scratch: end states of the segments (several segments only)
     uint32_t rows, heads, dim, vdim, shift_width;
+    uint32_t seg_len, seg_count, phase;  // see scan_kernel
     float cap, qscale;
 };
 
 __host__ __device__ inline uint32_t pad4(uint32_t d) { return (d + 3u) & ~3u; }
 template <int RPT> __host__ __device__ constexpr int chunk_tokens() { return RPT <= 8 ? 32 : RPT == 16 ? 16 : 8; }
+// Value columns per thread and per CTA (128 threads, 8 per group of columns): as many as registers hold, since every
+// column reuses the key vectors read from shared memory.
+template <int RPT> __host__ __device__ constexpr int thread_cols() { return RPT <= 16 ? 4 : 2; }
+__host__ __device__ inline uint32_t block_cols(uint32_t dim) { return dim <= 128 ? 64u : 32u; }
 
 __device__ __forceinline__ float log_sigmoid(float z) { return z < 0.f ? z - log1pf(expf(z)) : -log1pf(expf(-z)); }
 
-// One token of one value column for the RPT keys this thread owns; returns its share of the dot products.
-template <int MODE, int RPT>
-__device__ __forceinline__ void token_update(const float *q, const float *k, const float *w, const float (&u)[RPT], float v, float a, float b,
-                                           float (&S)[RPT], float (&n)[RPT], float &out, float &den)
+// One token of C value columns for the RPT keys this thread owns; OUT: out / den receive its share of the
+// dot products.  n: mlstm normalizer; without OUT a wkv thread multiplies its decays into it instead.
+template <int MODE, int RPT, int C, bool OUT>
+__device__ __forceinline__ void token_update(const float *q, const float *k, const float *w, const float (&u)[RPT], const float (&v_in)[C], float a, float b,
+                                             float (&S)[C][RPT], float (&n)[RPT], float (&out)[C], float &den)
 {
-    float o[2] = {0.f, 0.f}, d[2] = {0.f, 0.f};
-    if (MODE == kMlstm) v *= b;
+    float v[C], d = 0.f;
+#pragma unroll
+    for (int c = 0; c < C; c++) {
+        v[c] = MODE == kMlstm ? v_in[c] * b : v_in[c];
+        out[c] = 0.f;
+    }
 #pragma unroll
     for (int i = 0; i < RPT; i += 4) {
-        const float4 q4 = *reinterpret_cast<const float4 *>(q + i * 8), k4 = *reinterpret_cast<const float4 *>(k + i * 8);
-        const float qv[4] = {q4.x, q4.y, q4.z, q4.w}, kv[4] = {k4.x, k4.y, k4.z, k4.w};
+        const float4 k4 = *reinterpret_cast<const float4 *>(k + i * 8);
+        const float kv[4] = {k4.x, k4.y, k4.z, k4.w};
+        float qv[4] = {0.f, 0.f, 0.f, 0.f}, wv[4] = {0.f, 0.f, 0.f, 0.f};
+        if (OUT) {
+            const float4 q4 = *reinterpret_cast<const float4 *>(q + i * 8);
+            qv[0] = q4.x; qv[1] = q4.y; qv[2] = q4.z; qv[3] = q4.w;
+        }
         if (MODE == kWkv) {
             const float4 w4 = *reinterpret_cast<const float4 *>(w + i * 8);
-            const float wv[4] = {w4.x, w4.y, w4.z, w4.w};
+            wv[0] = w4.x; wv[1] = w4.y; wv[2] = w4.z; wv[3] = w4.w;
+        }
 #pragma unroll
-            for (int j = 0; j < 4; j++) {
-                const float x = kv[j] * v;
-                o[j & 1] = fmaf(qv[j], fmaf(u[i + j], x, S[i + j]), o[j & 1]);
-                S[i + j] = fmaf(wv[j], S[i + j], x);
-            }
-        } else {
+        for (int j = 0; j < 4; j++) {
+            if (MODE == kWkv) {
+                if (!OUT) n[i + j] *= wv[j];
 #pragma unroll
-            for (int j = 0; j < 4; j++) {
-                S[i + j] = fmaf(kv[j], v, a * S[i + j]);
+                for (int c = 0; c < C; c++) {
+                    const float x = kv[j] * v[c];
+                    if (OUT) out[c] = fmaf(qv[j], fmaf(u[i + j], x, S[c][i + j]), out[c]);
+                    S[c][i + j] = fmaf(wv[j], S[c][i + j], x);
+                }
+            } else {
                 n[i + j] = fmaf(kv[j], b, a * n[i + j]);
-                o[j & 1] = fmaf(qv[j], S[i + j], o[j & 1]);
-                d[j & 1] = fmaf(qv[j], n[i + j], d[j & 1]);
+                if (OUT) d = fmaf(qv[j], n[i + j], d);
+#pragma unroll
+                for (int c = 0; c < C; c++) {
+                    S[c][i + j] = fmaf(kv[j], v[c], a * S[c][i + j]);
+                    if (OUT) out[c] = fmaf(qv[j], S[c][i + j], out[c]);
+                }
             }
         }
     }
-    out = o[0] + o[1];
-    den = d[0] + d[1];
+    den = d;
 }
 
-// The same with the sums over the column's 8 threads.
-template <int MODE, int RPT>
-__device__ __forceinline__ void token_step(const float *q, const float *k, const float *w, const float (&u)[RPT], float v, float a, float b,
-                                           float (&S)[RPT], float (&n)[RPT], float &out, float &den)
+__device__ __forceinline__ float sum8(float x)
 {
-    token_update<MODE, RPT>(q, k, w, u, v, a, b, S, n, out, den);
 #pragma unroll
-    for (int off = 4; off > 0; off >>= 1) {
-        out += __shfl_xor_sync(0xffffffffu, out, off);
-        if (MODE == kMlstm) den += __shfl_xor_sync(0xffffffffu, den, off);
-    }
+    for (int off = 4; off > 0; off >>= 1) x += __shfl_xor_sync(0xffffffffu, x, off);
+    return x;
 }
 
 // Sums x[t] over the 8 threads of a column for 8 tokens at once: every exchange halves the tokens a
@@ -470,83 +487,142 @@ __device__ __forceinline__ void store_keys(float *row, uint32_t ks, uint32_t kp,
     }
 }
 
-constexpr uint32_t kScanThreads = 128, kScanCols = 16;
+constexpr uint32_t kScanThreads = 128;
 
-// mLSTM: n [pad4(dim)] and m of a head, one copy per block of 16 value columns (every CTA of a head
-// advances its own, so no CTA reads what another one writes).
-__host__ __device__ inline uint32_t value_blocks(uint32_t vdim) { return (vdim + kScanCols - 1) / kScanCols; }
-__device__ __forceinline__ float *normalizer(const Scan &p, uint32_t head, uint32_t block)
+// A state block: [heads][vdim][pad4(dim)], then per head and block of value columns [pad4(dim)] plus 4
+// scalars.  In an mlstm state those hold n and m, one copy per block (every CTA of a head advances its own,
+// so no CTA reads what another one writes); in a segment's end state also the decay product (wkv: per key in
+// place of n) or the sum of log forget gates (mlstm: scalar 1).
+__host__ __device__ inline uint32_t value_blocks(uint32_t dim, uint32_t vdim) { return (vdim + block_cols(dim) - 1) / block_cols(dim); }
+__host__ __device__ inline size_t block_elements(uint32_t heads, uint32_t dim, uint32_t vdim)
+{
+    return (size_t)heads * vdim * pad4(dim) + (size_t)heads * value_blocks(dim, vdim) * (pad4(dim) + 4u);
+}
+__device__ __forceinline__ float *normalizer(const Scan &p, float *base, uint32_t head, uint32_t block)
 {
     const uint32_t kp = pad4(p.dim);
-    return p.state + (size_t)p.heads * p.vdim * kp + (size_t)(head * value_blocks(p.vdim) + block) * (kp + 4u);
+    return base + (size_t)p.heads * p.vdim * kp + (size_t)(head * value_blocks(p.dim, p.vdim) + block) * (kp + 4u);
 }
 
+// One launch (phase 0) runs all tokens from the state.  A long portion is cut into segments of seg_len
+// tokens and takes two launches of seg_count - 1 segments each: phase 1 runs segment 0 from the state,
+// with outputs, and the middle segments from nothing, for their end states only; phase 2 starts segments
+// 1.. from the end states before them, put together in order.  Decays are only ever multiplied, and
+// mlstm end states carry their own maximum, so nothing can overflow.
 template <int MODE, int RPT>
 __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_constant__ Scan p)
 {
-    constexpr int TC = chunk_tokens<RPT>(), KS = RPT * 8, NA = MODE == kWkv ? 3 : 2;
+    constexpr int TC = chunk_tokens<RPT>(), KS = RPT * 8, NA = MODE == kWkv ? 3 : 2, C = thread_cols<RPT>(), COLS = 16 * C;
     extern __shared__ __align__(16) float smem[];
-    // per buffer: NA x [TC][KS] key vectors, [TC][16] values
-    constexpr int kBuf = NA * TC * KS + TC * (int)kScanCols;
+    // per buffer: NA x [TC][KS] key vectors, [TC][COLS] values
+    constexpr int kBuf = NA * TC * KS + TC * COLS;
     __shared__ float s_gate[2][3][32];                   // mlstm: keep, write, exp(-m) per token of a chunk
-    const uint32_t t = threadIdx.x, head = blockIdx.x, col0 = blockIdx.y * kScanCols, col = col0 + t / 8, ks = t & 7u;
+    __shared__ float s_end[2];                           // mlstm: m and the sum of log forget gates at the end
+    const uint32_t t = threadIdx.x, head = blockIdx.x, block = blockIdx.y, ks = t & 7u, vc = t / 8 * C, col = block * COLS + vc;
     const uint32_t dim = p.dim, vdim = p.vdim, kp = pad4(dim), kpitch = p.heads * dim, vpitch = p.heads * vdim;
-    const bool live = col < vdim;
-    const uint32_t chunks = (p.rows + TC - 1) / TC;
+    const uint32_t seg = p.phase == 2 ? blockIdx.z + 1 : blockIdx.z, row0 = seg * p.seg_len, rows = min(p.seg_len, p.rows - row0);
+    const bool outputs = p.phase != 1 || seg == 0, from_state = seg == 0;
+    const uint32_t chunks = (rows + TC - 1) / TC;
     for (uint32_t i = t; i < 2u * kBuf; i += kScanThreads) smem[i] = 0.f;          // keys beyond dim stay zero
-    float S[RPT], n[RPT], u[RPT];
+    float S[C][RPT], n[RPT], u[RPT], m = 0.f;
 #pragma unroll
-    for (int i = 0; i < RPT; i++) { S[i] = 0.f; n[i] = 0.f; u[i] = 0.f; }
-    if (MODE == kWkv) {
+    for (int i = 0; i < RPT; i++) {
+        const uint32_t key = (i / 4 * 8 + ks) * 4 + i % 4;
+        u[i] = MODE == kWkv && key < dim ? __ldg(p.u + head * dim + key) : 0.f;
+        n[i] = MODE == kWkv ? 1.f : 0.f;
 #pragma unroll
-        for (int i = 0; i < RPT; i++) {
-            const uint32_t key = (i / 4 * 8 + ks) * 4 + i % 4;
-            if (key < dim) u[i] = __ldg(p.u + head * dim + key);
-        }
+        for (int c = 0; c < C; c++) S[c][i] = 0.f;
     }
     pdl_launch_dependents();
     pdl_wait();
     __syncthreads();
-    float *srow = p.state + ((size_t)head * vdim + col) * kp;
-    float *nrow = normalizer(p, head, blockIdx.y), *mrow = nrow + kp;
-    if (live) load_keys<RPT>(srow, ks, kp, S);
-    if (MODE == kMlstm) load_keys<RPT>(nrow, ks, kp, n);
     const bool vec = dim % 4 == 0 && (reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.w)) % 16 == 0;
+    const bool vec_v = vdim % 4 == 0 && COLS % 4 == 0 && (reinterpret_cast<uintptr_t>(p.v) | reinterpret_cast<uintptr_t>(p.o)) % 16 == 0;
 
     auto stage = [&](uint32_t c, uint32_t buf) {
         float *base = smem + buf * kBuf;
-        const uint32_t r0 = c * TC, cnt = min((uint32_t)TC, p.rows - r0);
+        const uint32_t r0 = row0 + c * TC, cnt = min((uint32_t)TC, rows - c * TC);
 #pragma unroll
         for (int arr = 0; arr < NA; arr++) {
+            if (arr == 0 && !outputs) continue;
             const float *src = (arr == 0 ? p.q : arr == 1 ? p.k : p.w) + (size_t)r0 * kpitch + head * dim;
             float *dst = base + arr * TC * KS;
             if (vec) {
-                const uint32_t per = dim / 4;
-                for (uint32_t i = t; i < cnt * per; i += kScanThreads) {
-                    const uint32_t r = i / per, j = (i - r * per) * 4;
-                    cp_async16(dst + r * KS + j, src + (size_t)r * kpitch + j);
-                }
+                for (uint32_t j = (t & 7u) * 4; j < dim; j += 32)
+                    for (uint32_t r = t / 8; r < cnt; r += kScanThreads / 8) cp_async16(dst + r * KS + j, src + (size_t)r * kpitch + j);
             } else {
-                for (uint32_t i = t; i < cnt * dim; i += kScanThreads) {
-                    const uint32_t r = i / dim, j = i - r * dim;
-                    cp_async4(dst + r * KS + j, src + (size_t)r * kpitch + j);
-                }
+                for (uint32_t j = t & 7u; j < dim; j += 8)
+                    for (uint32_t r = t / 8; r < cnt; r += kScanThreads / 8) cp_async4(dst + r * KS + j, src + (size_t)r * kpitch + j);
             }
         }
         float *dv = base + NA * TC * KS;
-        const float *sv = p.v + (size_t)r0 * vpitch + head * vdim + col0;
-        for (uint32_t i = t; i < cnt * kScanCols; i += kScanThreads) {
-            const uint32_t r = i / kScanCols, j = i % kScanCols;
-            if (col0 + j < vdim) cp_async4(dv + i, sv + (size_t)r * vpitch + j);
+        const float *sv = p.v + (size_t)r0 * vpitch + head * vdim + block * COLS;
+        const uint32_t cols = min((uint32_t)COLS, vdim - block * COLS);
+        if (vec_v) {
+            for (uint32_t j = (t & 7u) * 4; j < cols; j += 32)
+                for (uint32_t r = t / 8; r < cnt; r += kScanThreads / 8) cp_async16(dv + r * COLS + j, sv + (size_t)r * vpitch + j);
+        } else {
+            for (uint32_t j = t & 7u; j < cols; j += 8)
+                for (uint32_t r = t / 8; r < cnt; r += kScanThreads / 8) cp_async4(dv + r * COLS + j, sv + (size_t)r * vpitch + j);
         }
         cp_commit();
     };
+    stage(0, 0);
+
+    // the state in front of the segment
+    auto load_state = [&](float *base, float (&X)[C][RPT]) {
+#pragma unroll
+        for (int c = 0; c < C; c++)
+            if (col + c < vdim) load_keys<RPT>(base + ((size_t)head * vdim + col + c) * kp, ks, kp, X[c]);
+    };
+    const size_t stride = block_elements(p.heads, dim, vdim);
+    if (from_state) {
+        load_state(p.state, S);
+        if (MODE == kMlstm) {
+            const float *nb = normalizer(p, p.state, head, block);
+            load_keys<RPT>(nb, ks, kp, n);
+            m = nb[kp];
+        }
+    } else if (outputs) {
+        load_state(p.segments, S);
+        if (MODE == kMlstm) {
+            const float *nb = normalizer(p, p.segments, head, block);
+            load_keys<RPT>(nb, ks, kp, n);
+            m = nb[kp];
+        }
+        for (uint32_t g = 1; g < seg; g++) {
+            float *base = p.segments + g * stride;
+            const float *nb = normalizer(p, base, head, block);
+            float f[RPT];
+            load_keys<RPT>(nb, ks, kp, f);
+            float keep = 1.f, add = 1.f;
+            if (MODE == kMlstm) {
+                const float m_new = fmaxf(nb[kp + 1] + m, nb[kp]);
+                keep = expf(nb[kp + 1] + m - m_new);
+                add = expf(nb[kp] - m_new);
+                m = m_new;
+#pragma unroll
+                for (int i = 0; i < RPT; i++) n[i] = fmaf(add, f[i], keep * n[i]);
+            }
+#pragma unroll
+            for (int c = 0; c < C; c++) {
+                if (col + c >= vdim) continue;
+                float x[RPT];
+                load_keys<RPT>(base + ((size_t)head * vdim + col + c) * kp, ks, kp, x);
+#pragma unroll
+                for (int i = 0; i < RPT; i++) S[c][i] = MODE == kWkv ? fmaf(f[i], S[c][i], x[i]) : fmaf(add, x[i], keep * S[c][i]);
+            }
+        }
+    } else if (MODE == kMlstm) {
+        m = -INFINITY;
+    }
     // mlstm gates of a chunk by one warp: m_t = max(f_t + m_{t-1}, i_t) is a scan of (sum f, max) pairs
-    float m_carry = 0.f;
+    float f_sum = 0.f;
     auto gates = [&](uint32_t c, uint32_t buf) {
-        const uint32_t lane = t, row = c * TC + lane;
-        const bool in = lane < (uint32_t)TC && row < p.rows;
-        const float xi = in ? p.gi[(size_t)row * p.heads + head] : 0.f, xf = in ? p.gf[(size_t)row * p.heads + head] : 0.f;
+        const uint32_t lane = t, row = c * TC + lane, cnt = min((uint32_t)TC, rows - c * TC);
+        const bool in = lane < cnt;
+        const size_t at = (size_t)(row0 + row) * p.heads + head;
+        const float xi = in ? p.gi[at] : 0.f, xf = in ? p.gf[at] : 0.f;
         const float li = p.cap * tanhf(xi / p.cap), lf = in ? log_sigmoid(p.cap * tanhf(xf / p.cap)) : 0.f;
         float F = lf, M = in ? li : -INFINITY;
 #pragma unroll
@@ -554,53 +630,100 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_cons
             const float Fp = __shfl_up_sync(0xffffffffu, F, off), Mp = __shfl_up_sync(0xffffffffu, M, off);
             if (lane >= (uint32_t)off) { M = fmaxf(M, F + Mp); F += Fp; }
         }
-        const float m = fmaxf(F + m_carry, M);
-        float prev = __shfl_up_sync(0xffffffffu, m, 1);
-        if (lane == 0) prev = m_carry;
-        s_gate[buf][0][lane] = expf(lf + prev - m);
-        s_gate[buf][1][lane] = in ? expf(li - m) : 0.f;
-        s_gate[buf][2][lane] = expf(-m);
-        const uint32_t cnt = min((uint32_t)TC, p.rows - c * TC);
-        m_carry = __shfl_sync(0xffffffffu, m, cnt - 1);
+        const float mt = fmaxf(F + m, M);
+        float prev = __shfl_up_sync(0xffffffffu, mt, 1);
+        if (lane == 0) prev = m;
+        s_gate[buf][0][lane] = expf(lf + prev - mt);         // a segment that starts from nothing: exp(-inf) = 0
+        s_gate[buf][1][lane] = in ? expf(li - mt) : 0.f;
+        s_gate[buf][2][lane] = expf(-mt);
+        m = __shfl_sync(0xffffffffu, mt, cnt - 1);
+        f_sum += __shfl_sync(0xffffffffu, F, cnt - 1);
     };
-    if (MODE == kMlstm && t < 32) { m_carry = *mrow; gates(0, 0); }
-    stage(0, 0);
+    if (MODE == kMlstm && t < 32) gates(0, 0);
     for (uint32_t c = 0; c < chunks; c++) {
         const uint32_t buf = c & 1u;
         if (c + 1 < chunks) { stage(c + 1, buf ^ 1u); cp_wait<1>(); } else { cp_wait<0>(); }
         __syncthreads();
         const float *base = smem + buf * kBuf, *sq = base + ks * 4, *sk = sq + TC * KS, *sw = sk + (NA == 3 ? TC * KS : 0);
-        const float *sv = base + NA * TC * KS + t / 8;
-        const uint32_t r0 = c * TC, cnt = min((uint32_t)TC, p.rows - r0);
+        const float *sv = base + NA * TC * KS + vc;
+        const uint32_t r0 = row0 + c * TC, cnt = min((uint32_t)TC, rows - c * TC);
         float *dst = p.o + (size_t)r0 * vpitch + head * vdim + col;
+        auto values = [&](uint32_t r, float (&v)[C]) {
+#pragma unroll
+            for (int i = 0; i < C; i += 2) {
+                const float2 x = *reinterpret_cast<const float2 *>(sv + r * COLS + i);
+                v[i] = x.x; v[i + 1] = x.y;
+            }
+        };
         uint32_t r = 0;
+        if (!outputs) {
+            for (; r < cnt; r++) {
+                float v[C], out[C], den;
+                values(r, v);
+                token_update<MODE, RPT, C, false>(sq, sk + r * KS, sw + r * KS, u, v, MODE == kMlstm ? s_gate[buf][0][r] : 0.f,
+                                                  MODE == kMlstm ? s_gate[buf][1][r] : 0.f, S, n, out, den);
+            }
+        }
         for (; r + 8 <= cnt; r += 8) {                       // 8 tokens at a time: one shared reduction, loads run ahead
-            float out[8], den[8];
+            float out[C][8], den[8];
 #pragma unroll
             for (int i = 0; i < 8; i++) {
-                float a = 0.f, b = 0.f;
-                if (MODE == kMlstm) { a = s_gate[buf][0][r + i]; b = s_gate[buf][1][r + i]; }
-                token_update<MODE, RPT>(sq + (r + i) * KS, sk + (r + i) * KS, sw + (r + i) * KS, u, sv[(r + i) * kScanCols], a, b, S, n, out[i], den[i]);
+                float v[C], o1[C];
+                values(r + i, v);
+                token_update<MODE, RPT, C, true>(sq + (r + i) * KS, sk + (r + i) * KS, sw + (r + i) * KS, u, v, MODE == kMlstm ? s_gate[buf][0][r + i] : 0.f,
+                                                 MODE == kMlstm ? s_gate[buf][1][r + i] : 0.f, S, n, o1, den[i]);
+#pragma unroll
+                for (int j = 0; j < C; j++) out[j][i] = o1[j];
             }
-            float y = reduce8(out, ks);
-            if (MODE == kMlstm) y = mlstm_out(y, reduce8(den, ks), p.qscale, s_gate[buf][2][r + ks]);
-            if (live) dst[(size_t)(r + ks) * vpitch] = y;
+            const float d = MODE == kMlstm ? reduce8(den, ks) : 0.f;
+            float y[C];
+#pragma unroll
+            for (int j = 0; j < C; j++) {
+                y[j] = reduce8(out[j], ks);
+                if (MODE == kMlstm) y[j] = mlstm_out(y[j], d, p.qscale, s_gate[buf][2][r + ks]);
+            }
+            float *at = dst + (size_t)(r + ks) * vpitch;
+            if (C == 4 && vec_v) {
+                if (col < vdim) *reinterpret_cast<float4 *>(at) = make_float4(y[0], y[1], y[C - 2], y[C - 1]);
+            } else {
+#pragma unroll
+                for (int j = 0; j < C; j++)
+                    if (col + j < vdim) at[j] = y[j];
+            }
         }
         for (; r < cnt; r++) {
-            float out, den, a = 0.f, b = 0.f;
-            if (MODE == kMlstm) { a = s_gate[buf][0][r]; b = s_gate[buf][1][r]; }
-            token_step<MODE, RPT>(sq + r * KS, sk + r * KS, sw + r * KS, u, sv[r * kScanCols], a, b, S, n, out, den);
-            if (ks == 0 && live) dst[(size_t)r * vpitch] = MODE == kMlstm ? mlstm_out(out, den, p.qscale, s_gate[buf][2][r]) : out;
+            float v[C], out[C], den;
+            values(r, v);
+            token_update<MODE, RPT, C, true>(sq + r * KS, sk + r * KS, sw + r * KS, u, v, MODE == kMlstm ? s_gate[buf][0][r] : 0.f,
+                                             MODE == kMlstm ? s_gate[buf][1][r] : 0.f, S, n, out, den);
+            den = sum8(den);
+#pragma unroll
+            for (int j = 0; j < C; j++) {
+                const float y = sum8(out[j]);
+                if (ks == 0 && col + j < vdim) dst[(size_t)r * vpitch + j] = MODE == kMlstm ? mlstm_out(y, den, p.qscale, s_gate[buf][2][r]) : y;
+            }
         }
         if (MODE == kMlstm && t < 32 && c + 1 < chunks) gates(c + 1, buf ^ 1u);
         __syncthreads();
     }
-    if (live) store_keys<RPT>(srow, ks, kp, S);
     if (MODE == kMlstm) {
-        if (t < 8) store_keys<RPT>(nrow, ks, kp, n);
-        if (t == 0) *mrow = m_carry;
+        if (t == 0) { s_end[0] = m; s_end[1] = f_sum; }
+        __syncthreads();
     }
-    if (MODE == kWkv && p.shift_state && blockIdx.y == 0) {
+    const bool last = row0 + rows == p.rows;
+    float *end = last ? p.state : p.segments + seg * stride;
+#pragma unroll
+    for (int c = 0; c < C; c++)
+        if (col + c < vdim) store_keys<RPT>(end + ((size_t)head * vdim + col + c) * kp, ks, kp, S[c]);
+    if (MODE == kMlstm || !last) {
+        float *nb = normalizer(p, end, head, block);
+        if (t < 8) store_keys<RPT>(nb, ks, kp, n);
+        if (MODE == kMlstm && t == 0) {
+            nb[kp] = s_end[0];
+            if (!last) nb[kp + 1] = s_end[1];
+        }
+    }
+    if (MODE == kWkv && p.shift_state && p.phase != 1 && block == 0 && blockIdx.z == 0) {
         for (uint32_t j = head * kScanThreads + t; j < p.shift_width; j += p.heads * kScanThreads) p.shift_state[j] = p.shift_state[p.shift_width + j];
     }
 }
@@ -631,7 +754,7 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
         sk[i] = i < dim ? p.k[head * dim + i] : 0.f;
         sw[i] = 0.f;
     }
-    float *nrow = normalizer(p, head, 0);
+    float *nrow = normalizer(p, p.state, head, 0);
     if (MODE == kWkv) {
         for (uint32_t i = t; i < rank; i += kStepThreads) s_low[i] = tanhf(low[i]);
         __syncthreads();
@@ -661,19 +784,20 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
     for (uint32_t col = t / 8; col < (vdim + kStepCols - 1) / kStepCols * kStepCols; col += kStepCols) {
         const bool live = col < vdim;
         float *srow = p.state + ((size_t)head * vdim + (live ? col : 0)) * kp;
-        float S[RPT], nn[RPT], out, den;
-        load_keys<RPT>(srow, ks, kp, S);
+        float S[1][RPT], nn[RPT], out1[1], den;
+        load_keys<RPT>(srow, ks, kp, S[0]);
 #pragma unroll
         for (int i = 0; i < RPT; i++) nn[i] = n[i];
-        const float v = live ? p.v[head * vdim + col] : 0.f;
-        token_step<MODE, RPT>(sq + ks * 4, sk + ks * 4, sw + ks * 4, u, v, a, b, S, nn, out, den);
+        const float v[1] = {live ? p.v[head * vdim + col] : 0.f};
+        token_update<MODE, RPT, 1, true>(sq + ks * 4, sk + ks * 4, sw + ks * 4, u, v, a, b, S, nn, out1, den);
+        float out = sum8(out1[0]);
         if (MODE == kMlstm) {
-            out = mlstm_out(out, den, p.qscale, expf(-m_new));
+            out = mlstm_out(out, sum8(den), p.qscale, expf(-m_new));
 #pragma unroll
             for (int i = 0; i < RPT; i++) n_out[i] = nn[i];
         }
         if (live) {
-            store_keys<RPT>(srow, ks, kp, S);
+            store_keys<RPT>(srow, ks, kp, S[0]);
             if (ks == 0) { so[col] = out; ss = fmaf(out, out, ss); }
         }
     }
@@ -684,31 +808,60 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
         dst[j] = from_f32<OT>(so[j] * r * hg.weight[head * vdim + j] * (hg.silu ? g * s : s));
     }
     if (MODE == kMlstm) {
-        for (uint32_t blk = t / 8; blk < value_blocks(vdim); blk += kStepCols) {
-            store_keys<RPT>(normalizer(p, head, blk), ks, kp, n_out);
-            if (ks == 0) normalizer(p, head, blk)[kp] = m_new;
+        for (uint32_t blk = t / 8; blk < value_blocks(dim, vdim); blk += kStepCols) {
+            float *nb = normalizer(p, p.state, head, blk);
+            store_keys<RPT>(nb, ks, kp, n_out);
+            if (ks == 0) nb[kp] = m_new;
         }
     } else if (p.shift_state) {
         for (uint32_t j = head * kStepThreads + t; j < p.shift_width; j += p.heads * kStepThreads) p.shift_state[j] = p.shift_state[p.shift_width + j];
     }
 }
 
-template <int MODE, int RPT>
-int launch_scan_rpt(const Scan &p, cudaStream_t stream)
+// Tokens per segment; rows: no cut.  Segments pay only when two launches of all but one of them are
+// shorter than one pass, i.e. from three segments on.
+uint32_t segment_length(uint32_t rows, uint32_t heads, uint32_t dim, uint32_t vdim)
 {
-    constexpr int NA = MODE == kWkv ? 3 : 2, TC = chunk_tokens<RPT>();
-    const size_t smem = (size_t)2 * (NA * TC * RPT * 8 + TC * kScanCols) * sizeof(float);
+    const uint32_t ctas = heads * value_blocks(dim, vdim);
+    const uint32_t want = std::min(8u, (148u * 3u + ctas - 1) / ctas) + 1;
+    if (want < 3 || rows < 256) return rows;
+    const uint32_t len = std::max(64u, ((rows + want - 1) / want + 31u) & ~31u);
+    return (rows + len - 1) / len < 3 ? rows : len;
+}
+
+// Launched without programmatic overlap: few long-running CTAs that would otherwise be packed onto the
+// SMs that the preceding kernel happens to leave first.
+template <int MODE, int RPT>
+int launch_scan_rpt(Scan p, void *workspace, cudaStream_t stream)
+{
+    constexpr int NA = MODE == kWkv ? 3 : 2, TC = chunk_tokens<RPT>(), COLS = 16 * thread_cols<RPT>();
+    const size_t smem = (size_t)2 * (NA * TC * RPT * 8 + TC * COLS) * sizeof(float);
     if (int rc = allow_smem(scan_kernel<MODE, RPT>, smem)) return rc;
-    return launch(scan_kernel<MODE, RPT>, dim3(p.heads, value_blocks(p.vdim)), dim3(kScanThreads), smem, stream, p);
+    p.segments = static_cast<float *>(workspace);
+    p.seg_len = p.segments ? segment_length(p.rows, p.heads, p.dim, p.vdim) : p.rows;
+    p.seg_count = (p.rows + p.seg_len - 1) / p.seg_len;
+    dim3 grid(p.heads, value_blocks(p.dim, p.vdim));
+    if (p.seg_count == 1) {
+        scan_kernel<MODE, RPT><<<grid, kScanThreads, smem, stream>>>(p);
+    } else {
+        grid.z = p.seg_count - 1;
+        p.phase = 1;
+        scan_kernel<MODE, RPT><<<grid, kScanThreads, smem, stream>>>(p);
+        MGQ_CUDA(cudaGetLastError());
+        p.phase = 2;
+        scan_kernel<MODE, RPT><<<grid, kScanThreads, smem, stream>>>(p);
+    }
+    MGQ_CUDA(cudaGetLastError());
+    return MGQ_OK;
 }
 
 template <int MODE>
-int launch_scan(const Scan &p, cudaStream_t stream)
+int launch_scan(const Scan &p, void *workspace, cudaStream_t stream)
 {
-    if (p.dim <= 32) return launch_scan_rpt<MODE, 4>(p, stream);
-    if (p.dim <= 64) return launch_scan_rpt<MODE, 8>(p, stream);
-    if (p.dim <= 128) return launch_scan_rpt<MODE, 16>(p, stream);
-    if (p.dim <= kMaxStateDim) return launch_scan_rpt<MODE, 32>(p, stream);
+    if (p.dim <= 32) return launch_scan_rpt<MODE, 4>(p, workspace, stream);
+    if (p.dim <= 64) return launch_scan_rpt<MODE, 8>(p, workspace, stream);
+    if (p.dim <= 128) return launch_scan_rpt<MODE, 16>(p, workspace, stream);
+    if (p.dim <= kMaxStateDim) return launch_scan_rpt<MODE, 32>(p, workspace, stream);
     return fail(MGQ_ERR_SHAPE, "recurrent heads of %u key dimensions (at most %u)", p.dim, kMaxStateDim);
 }
 
@@ -836,9 +989,10 @@ int launch_head_gate(const float *o, const HeadGate &hg, uint32_t rows, uint32_t
 }
 
 size_t wkv_state_elements(uint32_t heads, uint32_t dim) { return (size_t)heads * dim * pad4(dim); }
-size_t mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim)
+size_t mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim) { return block_elements(heads, dim, vdim); }
+size_t scan_workspace(uint32_t max_rows, uint32_t heads, uint32_t dim, uint32_t vdim)
 {
-    return (size_t)heads * vdim * pad4(dim) + (size_t)heads * value_blocks(vdim) * (pad4(dim) + 4u);
+    return max_rows < 256 ? 0 : 8 * block_elements(heads, dim, vdim) * sizeof(float);       // at most 9 segments, the last one ends in the state
 }
 
 int launch_decay(const Wkv &a, void *stream)
@@ -847,8 +1001,8 @@ int launch_decay(const Wkv &a, void *stream)
                   static_cast<cudaStream_t>(stream), a);
 }
 
-int launch_wkv_scan(const Wkv &a, void *stream) { return launch_scan<kWkv>(wkv_args(a), static_cast<cudaStream_t>(stream)); }
-int launch_mlstm_scan(const Mlstm &a, void *stream) { return launch_scan<kMlstm>(mlstm_args(a), static_cast<cudaStream_t>(stream)); }
+int launch_wkv_scan(const Wkv &a, void *stream) { return launch_scan<kWkv>(wkv_args(a), a.workspace, static_cast<cudaStream_t>(stream)); }
+int launch_mlstm_scan(const Mlstm &a, void *stream) { return launch_scan<kMlstm>(mlstm_args(a), a.workspace, static_cast<cudaStream_t>(stream)); }
 int launch_wkv_step(const Wkv &a, const HeadGate &hg, void *stream)
 {
     return launch_step<kWkv>(wkv_args(a), hg, a.low, a.w2, a.w0, a.rank, static_cast<cudaStream_t>(stream));

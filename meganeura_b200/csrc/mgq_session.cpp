@@ -61,7 +61,7 @@ struct Node {
     float f0 = 0.f;               // eps (RmsNorm), theta (RoPE)
     float f1 = 0.f, f2 = 0.f;
     int rows = 0;                 // leading dimension: 0 fixed, MGQ_ROWS_TOKENS / MGQ_ROWS_PICKED: set per step
-    std::vector<uint32_t> at;     // integer attributes of the recurrent and latent operators
+    std::vector<uint32_t> at = {};     // integer attributes of the recurrent and latent operators
     bool absorbed = false;        // runs inside the dispatch of its consumer (keeps its buffer)
     uint32_t u0 = 0, u1 = 0, u2 = 0;   // head_dim (RoPE); num_heads, num_kv_heads, head_dim (CachedAttention); column offset (View)
     size_t elements() const { size_t e = 1; for (size_t s : shape) e *= s; return e; }
@@ -928,6 +928,15 @@ int rotation_table(mgq_session *s, uint32_t dims, float base, Dispatch &d)
     return mgq_buffer_upload(d.workspace, freq.data(), freq.size() * 4, s->stream);
 }
 
+int recurrence_workspace(mgq_session *s, const Node &nd, Dispatch &d)
+{
+    const size_t bytes = mgq::scan_workspace((uint32_t)nd.shape[0], nd.at[0], nd.at[1], nd.at.back());
+    if (bytes == 0) return MGQ_OK;
+    if (int rc = mgq_buffer_create(bytes, &d.workspace)) return rc;
+    s->workspaces.push_back(d.workspace);
+    return MGQ_OK;
+}
+
 // Rotation table first (padded to 256 bytes), then the attention kernels' scratch.
 size_t rotation_bytes(uint32_t dims) { return ((size_t)dims * 2 + 255) & ~(size_t)255; }
 int latent_workspace(mgq_session *s, const Node &nd, Dispatch &d)
@@ -1208,6 +1217,8 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
                 d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = nd.at[1];
                 set_label(d, "Wkv[%ux%u]", nd.at[0], nd.at[1]);
                 s->states.push_back(nd.inputs[5]);
+                rc = recurrence_workspace(s, nd, d);
+                if (rc) { mgq_session_free(s); return rc; }
                 break;
             }
             case Op::Mlstm: {
@@ -1215,6 +1226,8 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
                 d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = nd.at[1]; d.params[3] = nd.at[2];
                 set_label(d, "Mlstm[%ux%ux%u]", nd.at[0], nd.at[1], nd.at[2]);
                 s->states.push_back(nd.inputs[5]);
+                rc = recurrence_workspace(s, nd, d);
+                if (rc) { mgq_session_free(s); return rc; }
                 break;
             }
             case Op::HeadGate: {
@@ -1223,9 +1236,9 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
                          : o.absorbed ? MGQ_SHADER_LATENT_ATTENTION : MGQ_SHADER_HEAD_GATE;
                 d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = (uint32_t)(nd.shape[1] / nd.at[0]);
                 set_label(d, "%s%s[%ux%u]", o.absorbed ? shader_name(d.shader) : "", o.absorbed ? "+HeadGate" : "HeadGate", d.params[1], d.params[2]);
-                if (o.absorbed && o.op != Op::LatentAttention) s->states.push_back(o.inputs[5]);
-                if (!(o.absorbed && o.op == Op::LatentAttention)) break;
-                rc = latent_workspace(s, o, d);
+                if (!o.absorbed) break;
+                if (o.op != Op::LatentAttention) s->states.push_back(o.inputs[5]);
+                rc = o.op == Op::LatentAttention ? latent_workspace(s, o, d) : recurrence_workspace(s, o, d);
                 if (rc) { mgq_session_free(s); return rc; }
                 break;
             }
@@ -1581,6 +1594,7 @@ static int run_mixer(mgq_session *s, const Dispatch &d)
         const int did = o.op == Op::Decay ? oid : o.inputs[3];
         const Node &dn = s->nodes[did];
         a.rows = rows;
+        a.workspace = d.workspace;
         a.decay = f(did);
         if (dn.op == Op::Decay) {
             a.low = f(dn.inputs[0]); a.w2 = s->ptr(dn.inputs[1]); a.w0 = f(dn.inputs[2]);
@@ -1605,6 +1619,7 @@ static int run_mixer(mgq_session *s, const Dispatch &d)
         a.q = f(o.inputs[0]); a.k = f(o.inputs[1]); a.v = f(o.inputs[2]); a.gi = f(o.inputs[3]); a.gf = f(o.inputs[4]);
         a.state = f(o.inputs[5]); a.o = f(oid);
         a.rows = rows; a.heads = o.at[0]; a.dim = o.at[1]; a.vdim = o.at[2]; a.cap = o.f0;
+        a.workspace = d.workspace;
         if (!fused) return mgq::launch_mlstm_scan(a, s->stream);
         if (rows == 1) return mgq::launch_mlstm_step(a, hg, s->stream);
         if (int rc = mgq::launch_mlstm_scan(a, s->stream)) return rc;

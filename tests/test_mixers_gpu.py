@@ -135,11 +135,12 @@ def test_embedding_scaled():
 # ---------------------------------------------------------------- token shift and RWKV-style mixing
 @pytest.mark.parametrize("heads,dim,rank,width", [(2, 32, 8, 64), (3, 22, 5, 50), (1, 64, 16, 300), (2, 128, 4, 40), (1, 200, 3, 33), (7, 6, 9, 20)])
 def test_wkv_portions_carry_state_and_previous_token(fuse, heads, dim, rank, width):
-    """Portions of 1, 40, 2, 1 and 33 tokens of one sequence, then a second sequence from cleared state."""
+    """Portions of 1, 600 (cut into segments), 2, 1, 33 and 300 tokens of one sequence, then a second sequence from
+    cleared state."""
     import meganeura_b200 as mg
     from meganeura_b200._lib import GATE_SILU, ROWS_TOKENS, lib
     r = rng_of(heads, dim, rank)
-    n, cap = heads * dim, 40
+    n, cap = heads * dim, 600
     table = r.standard_normal((90, width)).astype(np.float32)
     nw = r.standard_normal(width).astype(np.float32) * 0.2
     mus = r.uniform(0, 1, (5, width)).astype(np.float32)
@@ -164,7 +165,7 @@ def test_wkv_portions_carry_state_and_previous_token(fuse, heads, dim, rank, wid
         prev, S = np.zeros(width), np.zeros((heads, dim, dim))
         s.reset_state()
         at = 0
-        for cnt in (1, 40, 2, 1, 33) if seq == 0 else (3, 1):
+        for cnt in (1, 600, 2, 1, 33, 300) if seq == 0 else (3, 1):
             toks = (np.arange(at, at + cnt) * 7 + seq * 13) % 90
             at += cnt
             s.set_rows(ROWS_TOKENS, cnt)
@@ -185,7 +186,7 @@ def test_mlstm_portions(fuse, heads, dim, vdim, cap):
     import meganeura_b200 as mg
     from meganeura_b200._lib import GATE_SIGMOID, ROWS_TOKENS, lib
     r = rng_of(heads, dim, vdim)
-    n, nv, rows = heads * dim, heads * vdim, 70
+    n, nv, rows = heads * dim, heads * vdim, 700
     tabs = {"q": r.standard_normal((90, n)), "k": r.standard_normal((90, n)), "v": r.standard_normal((90, nv)), "g": r.standard_normal((90, nv)),
             "i": r.standard_normal((90, heads)) * 6 - 2, "f": r.standard_normal((90, heads)) * 6 + 3}
     tabs = {c: a.astype(np.float32) for c, a in tabs.items()}
@@ -201,7 +202,7 @@ def test_mlstm_portions(fuse, heads, dim, vdim, cap):
         S, nn, m = np.zeros((heads, dim, vdim)), np.zeros((heads, dim)), np.zeros(heads)
         s.reset_state()
         at = 0
-        for cnt in (2, 70, 1, 1, 33, 5) if seq == 0 else (1, 4):
+        for cnt in (2, 700, 1, 1, 33, 5, 257) if seq == 0 else (1, 4):
             toks = (np.arange(at, at + cnt) * 11 + seq * 5) % 90
             at += cnt
             s.set_rows(ROWS_TOKENS, cnt)
