@@ -2,7 +2,7 @@
 //
 // The keys W_uk c and values W_uv c of all live cache rows are expanded once per step by the tcgen05
 // linear kernel (ring order, f16); the attention kernel then works like a blockwise exact softmax:
-// CTA = one head x 64 query rows (4 warps x 16 rows), 64 keys per tile, double-buffered cp.async,
+// CTA = one head x 128 query rows (8 warps x 16 rows), 64 keys per tile, three cp.async stages,
 // tensor-core products with f32 accumulation.  The rotated key part, shared by the heads, is kept once.
 // Scores, maxima, sums and weights are f32.  The operands of the products are f16, not bf16: all are of
 // moderate size (a clamp guards the range), and with 11 significant bits the result stays close to the
@@ -16,7 +16,7 @@
 namespace mgq {
 namespace {
 
-constexpr uint32_t BM = 64, BN = 64;
+constexpr uint32_t BM = 128, BN = 64, kStages = 3, kThreads = 256;
 
 __device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void cp_async16(uint32_t smem, const void *gmem)
@@ -67,15 +67,22 @@ struct Prefill {
 
 // DK: dim + rot, DV: vdim, both rounded up to a multiple of 16.
 template <int DK, int DV>
-__global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_constant__ Prefill p)
+__global__ void __launch_bounds__(kThreads, 1) latent_prefill_kernel(const __grid_constant__ Prefill p)
 {
     constexpr int PK = DK + 8, PV = DV + 8;          // row pitch in elements: an odd number of 16-byte pieces
     extern __shared__ __align__(16) __half sm[];
-    __half *s_q = sm, *s_k = s_q + BM * PK, *s_v = s_k + 2 * BN * PK;
-    const uint32_t t = threadIdx.x, lane = t & 31u, warp = t >> 5, head = blockIdx.y;
-    const uint32_t row0 = (gridDim.x - 1 - blockIdx.x) * BM, dk = p.dim + p.rot;      // longest rows first
+    __half *s_q = sm, *s_k = s_q + BM * PK, *s_v = s_k + kStages * BN * PK;
+    const uint32_t t = threadIdx.x, lane = t & 31u, warp = t >> 5, head = blockIdx.x;
+    const uint32_t row0 = (gridDim.y - 1 - blockIdx.y) * BM, dk = p.dim + p.rot;      // longest rows first
     pdl_launch_dependents();
-    for (uint32_t i = t; i < (BM + 2 * BN) * PK + 2 * BN * PV; i += 128) sm[i] = __float2half_rn(0.f);    // padding columns stay zero
+    // zero padding columns (they meet in products), and query rows that do not exist
+    const __half zero = __float2half_rn(0.f);
+    if (dk < DK)
+        for (uint32_t i = t; i < (BM + kStages * BN) * (DK - dk); i += kThreads) s_q[i / (DK - dk) * PK + dk + i % (DK - dk)] = zero;
+    if (p.vdim < DV)
+        for (uint32_t i = t; i < kStages * BN * (DV - p.vdim); i += kThreads) s_v[i / (DV - p.vdim) * PV + p.vdim + i % (DV - p.vdim)] = zero;
+    for (uint32_t r = p.rows - row0; r < BM; r++)
+        for (uint32_t j = t; j < dk; j += kThreads) s_q[r * PK + j] = zero;
     pdl_wait();
     const uint32_t pos0 = p.pos[0], first = pos0 + row0, last = pos0 + min(row0 + BM, p.rows) - 1;
     const uint32_t lo = first + 1 > p.window ? first + 1 - p.window : 0u, tiles = (last - lo) / BN + 1;
@@ -85,33 +92,42 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_consta
         const uint32_t kt = lo + tile * BN;
         const uint32_t kb = smem_addr(s_k + buf * BN * PK), vb = smem_addr(s_v + buf * BN * PV);
         const uint32_t per_k = p.dim / 8, per_r = p.rot / 8, per_v = p.vdim / 8;
-        // two threads per key row
-        const uint32_t r = t >> 1, half = t & 1u;
+        const uint32_t r = t >> 2, part = t & 3u;                         // four threads per key row
         const size_t slot = min(kt + r, last) % p.slots;                  // beyond the last key: a valid row, masked below
         const __half *ksrc = p.keys + (slot * p.heads + head) * p.dim, *rsrc = p.rotated + slot * p.rot,
                             *vsrc = p.values + (slot * p.heads + head) * p.vdim;
-        for (uint32_t c = half; c < per_k; c += 2) cp_async16(kb + (r * PK + c * 8) * 2, ksrc + c * 8);
-        for (uint32_t c = half; c < per_r; c += 2) cp_async16(kb + (r * PK + p.dim + c * 8) * 2, rsrc + c * 8);
-        for (uint32_t c = half; c < per_v; c += 2) cp_async16(vb + (r * PV + c * 8) * 2, vsrc + c * 8);
+        for (uint32_t c = part; c < per_k; c += 4) cp_async16(kb + (r * PK + c * 8) * 2, ksrc + c * 8);
+        for (uint32_t c = part; c < per_r; c += 4) cp_async16(kb + (r * PK + p.dim + c * 8) * 2, rsrc + c * 8);
+        for (uint32_t c = part; c < per_v; c += 4) cp_async16(vb + (r * PV + c * 8) * 2, vsrc + c * 8);
         asm volatile("cp.async.commit_group;\n" ::: "memory");
     };
     stage(0, 0);
+    if (tiles > 1) stage(1, 1);
+    else asm volatile("cp.async.commit_group;\n" ::: "memory");
 
     // queries: unrotated part as it is, rotated part turned by its position
     {
         const uint32_t half = p.rot / 2;
         const size_t pitch = (size_t)p.heads * dk;
-        for (uint32_t r = warp; r < BM; r += 4) {
-            if (row0 + r >= p.rows) break;
-            const float *src = p.q + (size_t)(row0 + r) * pitch + head * dk;
-            for (uint32_t j = lane; j < p.dim; j += 32) s_q[r * PK + j] = to_half(src[j]);
-            for (uint32_t i = lane; i < half; i += 32) {
-                float s, c;
-                sincosf((float)(pos0 + row0 + r) * p.freq[i], &s, &c);
-                const float u = src[p.dim + i], v = src[p.dim + half + i];
-                s_q[r * PK + p.dim + i] = to_half(u * c - v * s);
-                s_q[r * PK + p.dim + half + i] = to_half(v * c + u * s);
-            }
+        const uint32_t n = min(BM, p.rows - row0), d4 = p.dim / 4;
+        const float *base = p.q + (size_t)row0 * pitch + head * dk;
+#pragma unroll 8
+        for (uint32_t i = t; i < n * d4; i += kThreads) {
+            const uint32_t r = i / d4, j = (i - r * d4) * 4;
+            const float4 v = *reinterpret_cast<const float4 *>(base + r * pitch + j);
+            __half2 *dst = reinterpret_cast<__half2 *>(s_q + r * PK + j);
+            dst[0] = __halves2half2(to_half(v.x), to_half(v.y));
+            dst[1] = __halves2half2(to_half(v.z), to_half(v.w));
+        }
+#pragma unroll 4
+        for (uint32_t i = t; i < n * half; i += kThreads) {
+            const uint32_t r = i / half, j = i - r * half;
+            const float *src = base + r * pitch + p.dim;
+            const float u = src[j], v = src[half + j];
+            float sn, cs;
+            sincosf((float)(first + r) * p.freq[j], &sn, &cs);
+            s_q[r * PK + p.dim + j] = to_half(u * cs - v * sn);
+            s_q[r * PK + p.dim + half + j] = to_half(v * cs + u * sn);
         }
     }
     float o[DV / 8][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
@@ -126,14 +142,13 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_consta
     const uint32_t v_off = (((lane & 7u) + ((lane >> 3) & 1u) * 8) * PV + (lane >> 4) * 8) * 2;
 
     for (uint32_t tile = 0; tile < tiles; tile++) {
-        const uint32_t buf = tile & 1u, kt = lo + tile * BN;
-        if (tile + 1 < tiles) {
-            stage(tile + 1, buf ^ 1u);
-            asm volatile("cp.async.wait_group 1;\n" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;\n" ::: "memory");
-        }
-        __syncthreads();
+        const uint32_t buf = tile % kStages, kt = lo + tile * BN;
+        asm volatile("cp.async.wait_group 1;\n" ::: "memory");           // one group per tile, the next one may be in flight
+        __syncthreads();                                                 // and every warp has left the buffer that is filled now
+        if (tile + 2 < tiles) stage(tile + 2, (tile + 2) % kStages);
+        else asm volatile("cp.async.commit_group;\n" ::: "memory");
+        const uint32_t w_first = first + warp * 16, w_last = w_first + 15;
+        if (kt > w_last || kt + BN - 1 + p.window <= w_first) continue;  // no row of this warp sees the tile
         const uint32_t kb = smem_addr(s_k + buf * BN * PK) + b_off, vb = smem_addr(s_v + buf * BN * PV) + v_off;
         float s[BN / 8][4];
 #pragma unroll
@@ -153,7 +168,7 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_consta
             }
         }
         // mask only where the tile crosses the diagonal or a row's window edge
-        const bool edge = kt + BN - 1 > first + warp * 16 || kt + p.window <= first + warp * 16 + 15;
+        const bool edge = kt + BN - 1 > w_first || kt + p.window <= w_last;
 #pragma unroll
         for (int h = 0; h < 2; h++) {
             float mx = -INFINITY;
@@ -198,7 +213,6 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_consta
                 mma16816(o[2 * n + 1], w, b[2], b[3]);
             }
         }
-        __syncthreads();
     }
 #pragma unroll
     for (int h = 0; h < 2; h++) {
@@ -227,9 +241,9 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const __grid_consta
 template <int DK, int DV>
 int launch_prefill(const Prefill &p, cudaStream_t st)
 {
-    const size_t smem = ((size_t)(BM + 2 * BN) * (DK + 8) + (size_t)2 * BN * (DV + 8)) * 2;
+    const size_t smem = ((size_t)(BM + kStages * BN) * (DK + 8) + (size_t)kStages * BN * (DV + 8)) * 2;
     if (int rc = allow_smem(latent_prefill_kernel<DK, DV>, smem)) return rc;
-    return launch(latent_prefill_kernel<DK, DV>, dim3((p.rows + BM - 1) / BM, p.heads), dim3(128), smem, st, p);
+    return launch(latent_prefill_kernel<DK, DV>, dim3(p.heads, (p.rows + BM - 1) / BM), dim3(kThreads), smem, st, p);
 }
 
 template <int DK>
