@@ -14,7 +14,10 @@ from petotar_util import CONFIGS, Tensors, row_errors, weights, write_folder
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-TOL = {"float32": 5e-5, "bfloat16": 8e-2}       # worst row; bf16 operands cost the median row about 1e-2
+# Worst row and median row.  Rounding the operands of the linear layers alone, in the plain restatement, costs
+# these models 0.04-0.07 in the worst and 0.013 in the median row.
+TOL = {"float32": 5e-5, "bfloat16": 0.1}
+MEDIAN = {"float32": 1e-5, "bfloat16": 2.5e-2}
 _cache = {}
 
 
@@ -60,7 +63,7 @@ def test_logits_do_not_depend_on_the_cut(name, dtype):
         e.end()
         errors = row_errors(got, want)
         worst[label] = errors.max()
-        assert np.median(errors) <= TOL[dtype] / 3
+        assert np.median(errors) <= MEDIAN[dtype]
     assert max(worst.values()) <= TOL[dtype], worst
 
 
