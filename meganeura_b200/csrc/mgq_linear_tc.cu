@@ -39,6 +39,19 @@ struct __align__(8) LinearShared {
     volatile int failed;
 };
 
+constexpr uint32_t kStgBytes = 32 * 36 * 4;              // epilogue staging of one warp: 32 rows x 32 columns, padded rows
+
+// Two values of a 2-byte output: bf16 for a GLU, f16 otherwise.
+template <bool BF16> __device__ __forceinline__ uint32_t pack_pair(float x, float y)
+{
+    if (BF16) {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+        return *reinterpret_cast<const uint32_t *>(&h);
+    }
+    const __half2 h = __floats2half2_rn(x, y);
+    return *reinterpret_cast<const uint32_t *>(&h);
+}
+
 struct Tile {
     uint32_t si, m0, n0;
 };
@@ -146,6 +159,7 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
         }
     } else {
         const uint32_t quad = warp & 3u;                 // TMEM lanes this warp may read
+        float *stg = reinterpret_cast<float *>(ring + S * kStage) + quad * (kStgBytes / 4);
         uint32_t at = 0;
         for (uint32_t tile = blockIdx.x; tile < tiles; tile += gridDim.x, at++) {
             const uint32_t b = at & 1u;
@@ -155,78 +169,93 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
             tc_fence_after();
             const Tile tl = find_tile<COLS>(g, tile, mt);
             const LinearSegment &sg = g.seg[tl.si];
-            const uint32_t row = tl.m0 + quad * 32 + lane, n = sg.n;
-            const bool live = row < g.m;
+            const uint32_t rbase = tl.m0 + quad * 32, n = sg.n;
             const uint32_t acc = tmem + ((quad * 32u) << 16) + b * TN;
+            const bool narrow = (GLU && g.out_bf16) || (!GLU && g.out_f16);       // 2-byte outputs
 #pragma unroll 1
-            for (uint32_t c0 = 0; c0 < COLS; c0 += 16) {
-                if (tl.n0 + c0 >= n) break;              // uniform over the warp
-                uint32_t r[16], r2[16];
-                tmem_ld16(acc + c0, r);
-                if (GLU) tmem_ld16(acc + COLS + c0, r2);
-                if (!live) continue;
+            for (uint32_t c0 = 0; c0 < COLS; c0 += 32) {
                 const uint32_t col = tl.n0 + c0;
-                const size_t o = (size_t)row * n + col;
-                float y[16];
+                if (col >= n) break;                     // uniform over the warp
+                const bool whole = col + 32 <= n && n % (narrow ? 8 : 4) == 0;
+                // lane = row of the accumulator: bias and GLU here
+                float y[32];
+                tmem_ld32(acc + c0, y);
+                if (GLU) {
+                    float up[32];
+                    tmem_ld32(acc + COLS + c0, up);
+                    if (whole) {
 #pragma unroll
-                for (int e = 0; e < 16; e++) {
-                    y[e] = __uint_as_float(r[e]);
-                    if (col + e < n) {
-                        if (GLU) y[e] = clamped_glu_f(y[e] + __ldg(sg.bias + col + e), __uint_as_float(r2[e]) + __ldg(sg.bias2 + col + e), g.limit, g.alpha);
-                        else if (sg.bias) y[e] += __ldg(sg.bias + col + e);
+                        for (int e = 0; e < 32; e += 4) {
+                            const float4 bg = __ldg(reinterpret_cast<const float4 *>(sg.bias + col + e)), bu = __ldg(reinterpret_cast<const float4 *>(sg.bias2 + col + e));
+                            y[e] = clamped_glu_f(y[e] + bg.x, up[e] + bu.x, g.limit, g.alpha);
+                            y[e + 1] = clamped_glu_f(y[e + 1] + bg.y, up[e + 1] + bu.y, g.limit, g.alpha);
+                            y[e + 2] = clamped_glu_f(y[e + 2] + bg.z, up[e + 2] + bu.z, g.limit, g.alpha);
+                            y[e + 3] = clamped_glu_f(y[e + 3] + bg.w, up[e + 3] + bu.w, g.limit, g.alpha);
+                        }
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 32; e++)
+                            if (col + e < n) y[e] = clamped_glu_f(y[e] + __ldg(sg.bias + col + e), up[e] + __ldg(sg.bias2 + col + e), g.limit, g.alpha);
+                    }
+                } else if (sg.bias) {
+                    if (whole) {
+#pragma unroll
+                        for (int e = 0; e < 32; e += 4) {
+                            const float4 v = __ldg(reinterpret_cast<const float4 *>(sg.bias + col + e));
+                            y[e] += v.x; y[e + 1] += v.y; y[e + 2] += v.z; y[e + 3] += v.w;
+                        }
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 32; e++)
+                            if (col + e < n) y[e] += __ldg(sg.bias + col + e);
                     }
                 }
                 if (!GLU && g.out_f16) {
-                    __half *out = static_cast<__half *>(sg.out) + o;
 #pragma unroll
-                    for (int e = 0; e < 16; e++) y[e] = fminf(fmaxf(y[e], -65504.f), 65504.f);
-                    if (n % 8 == 0 && col + 16 <= n) {
-                        uint32_t q[8];
+                    for (int e = 0; e < 32; e++) y[e] = fminf(fmaxf(y[e], -65504.f), 65504.f);
+                }
+                // through shared memory, so that a store instruction covers whole pieces of few rows
+                if (whole && narrow) {
+                    uint32_t *mine = reinterpret_cast<uint32_t *>(stg) + lane * 20;
 #pragma unroll
-                        for (int e = 0; e < 8; e++) {
-                            const __half2 h = __floats2half2_rn(y[2 * e], y[2 * e + 1]);
-                            q[e] = *reinterpret_cast<const uint32_t *>(&h);
-                        }
-                        reinterpret_cast<uint4 *>(out)[0] = make_uint4(q[0], q[1], q[2], q[3]);
-                        reinterpret_cast<uint4 *>(out)[1] = make_uint4(q[4], q[5], q[6], q[7]);
-                    } else {
+                    for (int e = 0; e < 16; e += 4)
+                        *reinterpret_cast<uint4 *>(mine + e) = make_uint4(pack_pair<GLU>(y[2 * e], y[2 * e + 1]), pack_pair<GLU>(y[2 * e + 2], y[2 * e + 3]),
+                                                                          pack_pair<GLU>(y[2 * e + 4], y[2 * e + 5]), pack_pair<GLU>(y[2 * e + 6], y[2 * e + 7]));
+                    __syncwarp();
 #pragma unroll
-                        for (int e = 0; e < 16; e++)
-                            if (col + e < n) out[e] = __float2half_rn(y[e]);
+                    for (int i = 0; i < 4; i++) {
+                        const uint32_t r = i * 8 + lane / 4, piece = lane & 3u;
+                        const uint4 v = *reinterpret_cast<const uint4 *>(reinterpret_cast<const uint32_t *>(stg) + r * 20 + piece * 4);
+                        if (rbase + r < g.m) *reinterpret_cast<uint4 *>(static_cast<uint16_t *>(sg.out) + (size_t)(rbase + r) * n + col + piece * 8) = v;
                     }
-                } else if (GLU && g.out_bf16) {
-                    __nv_bfloat16 *out = static_cast<__nv_bfloat16 *>(sg.out) + o;
-                    if (n % 8 == 0 && col + 16 <= n) {
-                        uint32_t q[8];
+                    __syncwarp();
+                } else if (whole) {
+                    float *mine = stg + lane * 36;
+                    float4 add[8];
 #pragma unroll
-                        for (int e = 0; e < 8; e++) {
-                            const __nv_bfloat162 h = __floats2bfloat162_rn(y[2 * e], y[2 * e + 1]);
-                            q[e] = *reinterpret_cast<const uint32_t *>(&h);
-                        }
-                        reinterpret_cast<uint4 *>(out)[0] = make_uint4(q[0], q[1], q[2], q[3]);
-                        reinterpret_cast<uint4 *>(out)[1] = make_uint4(q[4], q[5], q[6], q[7]);
-                    } else {
-#pragma unroll
-                        for (int e = 0; e < 16; e++)
-                            if (col + e < n) out[e] = __float2bfloat16_rn(y[e]);
+                    for (int i = 0; i < 8; i++) {        // all addends requested before the first one is needed
+                        const uint32_t r = i * 4 + lane / 8;
+                        add[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                        if (!GLU && sg.addend && rbase + r < g.m) add[i] = *reinterpret_cast<const float4 *>(sg.addend + (size_t)(rbase + r) * n + col + (lane & 7u) * 4);
                     }
-                } else {
-                    float *out = static_cast<float *>(sg.out) + o;
-                    const float *add = GLU ? nullptr : sg.addend;
-                    if (n % 4 == 0 && col + 16 <= n) {
 #pragma unroll
-                        for (int e = 0; e < 16; e += 4) {
-                            float4 v = make_float4(y[e], y[e + 1], y[e + 2], y[e + 3]);
-                            if (add) {
-                                const float4 d = *reinterpret_cast<const float4 *>(add + o + e);
-                                v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
-                            }
-                            *reinterpret_cast<float4 *>(out + e) = v;
-                        }
-                    } else {
+                    for (int e = 0; e < 32; e += 4) *reinterpret_cast<float4 *>(mine + e) = make_float4(y[e], y[e + 1], y[e + 2], y[e + 3]);
+                    __syncwarp();
 #pragma unroll
-                        for (int e = 0; e < 16; e++)
-                            if (col + e < n) out[e] = add ? y[e] + add[o + e] : y[e];
+                    for (int i = 0; i < 8; i++) {
+                        const uint32_t r = i * 4 + lane / 8;
+                        float4 v = *reinterpret_cast<const float4 *>(stg + r * 36 + (lane & 7u) * 4);
+                        v.x += add[i].x; v.y += add[i].y; v.z += add[i].z; v.w += add[i].w;
+                        if (rbase + r < g.m) *reinterpret_cast<float4 *>(static_cast<float *>(sg.out) + (size_t)(rbase + r) * n + col + (lane & 7u) * 4) = v;
+                    }
+                    __syncwarp();
+                } else if (rbase + lane < g.m) {         // ragged columns
+                    const size_t o = (size_t)(rbase + lane) * n + col;
+#pragma unroll
+                    for (int e = 0; e < 32; e++) {
+                        if (col + e >= n) continue;
+                        if (narrow) static_cast<uint16_t *>(sg.out)[o + e] = (uint16_t)pack_pair<GLU>(y[e], 0.f);
+                        else        static_cast<float *>(sg.out)[o + e] = !GLU && sg.addend ? y[e] + sg.addend[o + e] : y[e];
                     }
                 }
             }
@@ -272,7 +301,7 @@ int launch_tc(const LinearGroup &g, cudaStream_t stream)
         tiles += (s.n + COLS - 1) / COLS;
     }
     tiles *= (g.m + TM - 1) / TM;
-    const size_t smem = (size_t)stages<TN>() * stage_bytes<TN>() + 1024;
+    const size_t smem = (size_t)stages<TN>() * stage_bytes<TN>() + 4 * kStgBytes + 1024;
     if (int rc = allow_smem(linear_tc_kernel<TN, GLU>, smem)) return rc;
     return launch(linear_tc_kernel<TN, GLU>, dim3(min(tiles, 148u)), dim3(kThreads), smem, stream, maps, g, tiles);
 }
