@@ -378,6 +378,14 @@ typedef struct mgq_session mgq_session;
 #define MGQ_SHADER_LATENT_CACHE_WRITE 25
 #define MGQ_SHADER_LATENT_ATTENTION  26   /* alone, or with the output gate behind it */
 #define MGQ_SHADER_CLAMPED_GLU       27
+#define MGQ_SHADER_CAST              28
+#define MGQ_SHADER_SCALED_SUM        29
+#define MGQ_SHADER_RESIDUAL_NORM     30
+#define MGQ_SHADER_GLA               31
+#define MGQ_SHADER_QUERY_TEMPERATURE 32
+#define MGQ_SHADER_CACHE_APPEND      33
+#define MGQ_SHADER_ATTENTION         34
+#define MGQ_SHADER_ATTENTION_INPUTS  35
 
 mgq_graph *mgq_graph_new(void);
 void mgq_graph_free(mgq_graph *g);
@@ -416,7 +424,7 @@ int mgq_graph_all_gather(mgq_graph *g, int x, uint32_t world);
  * a whole vector that belongs to this rank, e.g. the residual a sharded projection adds to. */
 int mgq_graph_slice_columns(mgq_graph *g, int x, uint32_t first, uint32_t count);
 
-/* ---- row-dynamic graphs and the operators of decoders with recurrent and latent-attention mixers
+/* ---- row-dynamic graphs and the operators of decoders with recurrent, softmax- and latent-attention mixers
  * (no reference counterpart).
  *
  * mgq_graph_input_u32_rows declares a u32 input of up to `capacity` rows whose count is set per step
@@ -429,20 +437,33 @@ int mgq_graph_slice_columns(mgq_graph *g, int x, uint32_t first, uint32_t count)
  * matmul_bt with a parameter_bf16 [N, K]  linear layer, any number of rows, f32 accumulation and output
  * bias_add            x[r, c] + bias[c]
  * embedding_scaled    table[id] * scale, table f32 or bf16
+ * embedding_positions the same plus a sinusoidal vector of the token's position p = pos + row: column 2i is
+ *                     sin(p * base^(-2i / width)), column 2i + 1 its cosine
+ * cast                a bf16 copy of an f32 node, as operand of linear layers
+ * scaled_sum          sa * a + sb * b
  * pick_rows           x[index[r], :]
  * norm                x / sqrt(mean(x^2) + eps) * (weight_offset + weight)
  * clamped_glu         g = min(gate, limit), u = clamp(up, +-limit): g sigmoid(alpha g) (u + 1)
+ * silu_glu            silu(gate) * up
  * token_shift         `count` mixes h_t + (h_(t-1) - h_t) * mu_i as a [count, rows, width] node (take one
  *                     with slot); state: zero-filled f32 parameter [2, width], row 0 the previous
  *                     portion's last h, row 1 the pending one that wkv commits
  * lora_decay          exp(-exp(tanh(low) . w2^T + w0)), low [rows, rank], w2 bf16 [channels, rank]
+ * lora_sigmoid_decay  sigmoid(low . w2^T + bias)^(1 / tau)
  * wkv                 per head: o_t = (S + diag(u) k_t v_t^T)^T r_t, then S = diag(w_t) S + k_t v_t^T;
  *                     state: f32 parameter of mgq_wkv_state_elements
  * mlstm               matrix memory with running maximum m (zero at the start), capped log gates
  *                     i = cap tanh(gate_i / cap), f = logsigmoid(cap tanh(gate_f / cap)), q scaled by
  *                     dim^-1/2, o = S^T q / (max(|n . q|, exp(-m)) + 1e-6); state: f32 parameter of
  *                     mgq_mlstm_state_elements
- * head_gate           per head o / rms(o) * weight * act(gate); weight -1: o * act(gate) without the norm
+ * gla                 gated linear attention, per head: S = diag(decay_t) S + k_t v_t^T, then o = S^T q dim^-1/2;
+ *                     state: f32 parameter of mgq_gla_state_elements
+ * head_gate           per head o / rms(o) * weight * act(gate), the weight for all heads side by side or one of a
+ *                     head's size shared by them; weight -1: o * act(gate) without the norm
+ * query_temperature   x * (1 + coef * ln(floor((p + 1) / every) + 1)) at position p = pos + row
+ * cache_append        row pos + r of an f32 or f16 cache parameter [slots, cols] = x[r]
+ * attention           causal softmax of (q . k) * scale over positions 0 .. p, query head h on key / value head
+ *                     h / (heads / kv_heads); caches [slots, kv_heads * dim] and [slots, kv_heads * vdim]
  * latent_cache_write  ring cache row pos % slots = [norm(down[:rank]) * weight | rotated down[rank:]]
  * latent_attention    softmax over the last `window` positions of
  *                     (q_nope . W_uk c + rotate(q_rot) . k_rot) * scale, values W_uv c; q is laid out head
@@ -455,21 +476,32 @@ int mgq_graph_slice_columns(mgq_graph *g, int x, uint32_t first, uint32_t count)
 int mgq_graph_input_u32_rows(mgq_graph *g, const char *name, size_t capacity, int which);
 int mgq_graph_parameter_bf16(mgq_graph *g, const char *name, const size_t *shape, size_t rank);
 int mgq_graph_embedding_scaled(mgq_graph *g, int indices, int table, float scale);
+int mgq_graph_embedding_positions(mgq_graph *g, int indices, int table, int pos, float scale, float base);
+int mgq_graph_cast(mgq_graph *g, int x, int out_dtype);
+int mgq_graph_scaled_sum(mgq_graph *g, int a, int b, float sa, float sb);
 int mgq_graph_pick_rows(mgq_graph *g, int x, int index);
 int mgq_graph_norm(mgq_graph *g, int x, int weight, float eps, float weight_offset, int out_dtype);
 int mgq_graph_bias_add(mgq_graph *g, int x, int bias);
 int mgq_graph_clamped_glu(mgq_graph *g, int gate, int up, float limit, float alpha, int out_dtype);
+int mgq_graph_silu_glu(mgq_graph *g, int gate, int up, int out_dtype);
 int mgq_graph_token_shift(mgq_graph *g, int h, const int *mu, size_t count, int state, int out_dtype);
 int mgq_graph_slot(mgq_graph *g, int x, uint32_t index);
 size_t mgq_wkv_state_elements(uint32_t heads, uint32_t dim);
 size_t mgq_mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim);
+size_t mgq_gla_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim);
 int mgq_graph_lora_decay(mgq_graph *g, int low, int w2, int w0);
+int mgq_graph_lora_sigmoid_decay(mgq_graph *g, int low, int w2, int bias, float tau);
+int mgq_graph_gla(mgq_graph *g, int q, int k, int v, int decay, int state, uint32_t heads);
 int mgq_graph_wkv(mgq_graph *g, int r, int k, int v, int decay, int u, int state, int shift_state, uint32_t heads);
 int mgq_graph_mlstm(mgq_graph *g, int q, int k, int v, int gate_i, int gate_f, int state, uint32_t heads, float gate_cap);
 int mgq_graph_head_gate(mgq_graph *g, int o, int weight, int gate, uint32_t heads, float eps, int act, int out_dtype);
 int mgq_graph_latent_cache_write(mgq_graph *g, int down, int weight, int cache, int pos, uint32_t rot_dim, float rot_base, float eps);
 int mgq_graph_latent_attention(mgq_graph *g, int q, int cache, int uk, int uv, int pos, uint32_t heads, uint32_t dim, uint32_t rot_dim,
                                uint32_t vdim, uint32_t window, float scale, float rot_base);
+int mgq_graph_query_temperature(mgq_graph *g, int x, int pos, float coef, float every);
+int mgq_graph_cache_append(mgq_graph *g, int x, int cache, int pos);
+int mgq_graph_attention(mgq_graph *g, int q, int k_cache, int v_cache, int pos, uint32_t heads, uint32_t kv_heads, uint32_t dim, uint32_t vdim,
+                        float scale);
 int mgq_graph_set_outputs(mgq_graph *g, const int *ids, size_t count);
 
 /* build_inference_session (src/train.rs:380-389): fuse, lower, allocate zero-filled buffers. */

@@ -112,6 +112,16 @@ SIGNATURES = {
     "mgq_graph_input_u32_rows": (_int, [_vp, ctypes.c_char_p, _sz, _int]),
     "mgq_graph_parameter_bf16": (_int, [_vp, ctypes.c_char_p, _szp, _sz]),
     "mgq_graph_embedding_scaled": (_int, [_vp, _int, _int, ctypes.c_float]),
+    "mgq_graph_embedding_positions": (_int, [_vp, _int, _int, _int, ctypes.c_float, ctypes.c_float]),
+    "mgq_graph_cast": (_int, [_vp, _int, _int]),
+    "mgq_graph_scaled_sum": (_int, [_vp, _int, _int, ctypes.c_float, ctypes.c_float]),
+    "mgq_graph_silu_glu": (_int, [_vp, _int, _int, _int]),
+    "mgq_graph_lora_sigmoid_decay": (_int, [_vp, _int, _int, _int, ctypes.c_float]),
+    "mgq_gla_state_elements": (_sz, [_u32, _u32, _u32]),
+    "mgq_graph_gla": (_int, [_vp, _int, _int, _int, _int, _int, _u32]),
+    "mgq_graph_query_temperature": (_int, [_vp, _int, _int, ctypes.c_float, ctypes.c_float]),
+    "mgq_graph_cache_append": (_int, [_vp, _int, _int, _int]),
+    "mgq_graph_attention": (_int, [_vp, _int, _int, _int, _int, _u32, _u32, _u32, _u32, ctypes.c_float]),
     "mgq_graph_pick_rows": (_int, [_vp, _int, _int]),
     "mgq_graph_norm": (_int, [_vp, _int, _int, ctypes.c_float, ctypes.c_float, _int]),
     "mgq_graph_bias_add": (_int, [_vp, _int, _int]),

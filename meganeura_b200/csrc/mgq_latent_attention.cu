@@ -1,7 +1,7 @@
 // Latent attention over a sliding window: the cache holds, per position, an RMS-normed latent of
 // `rank` elements and one rotated key part of `rot_dim` elements shared by all heads.
 //
-// Absorbed form (few rows, and every f32 session; many rows: mgq_latent_prefill.cu): the query is folded through W_uk once,
+// Absorbed form (few rows, and every f32 session; many rows: mgq_prefill_attention.cu): the query is folded through W_uk once,
 //   score = (W_uk^T q_nope) . c + q_rot . k_rot,   o' = softmax . c,   o = W_uv o',
 // so attention runs against the latents themselves and every head shares one key/value row.
 //   latent_absorb_kernel   q' = scale * [W_uk^T q_nope | rotate(q_rot)]

@@ -2,6 +2,7 @@
 // reductions, f32 <-> bf16 element access.
 #pragma once
 #include <cuda_bf16.h>
+#include <cuda_fp16.h>
 #include <cuda_runtime.h>
 
 #include <cstdint>
@@ -54,9 +55,11 @@ __device__ __forceinline__ float warp_max(float v)
 
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float to_f32(__half v) { return __half2float(v); }
 template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+template <> __device__ __forceinline__ __half from_f32<__half>(float v) { return __float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f)); }       // clamped to the range
 
 // 8 consecutive elements, 16-byte aligned source.  Plain loads: activations are written by the kernel this one
 // overlaps with, and a read-only-path load might be moved across the wait for it.
@@ -78,11 +81,15 @@ __device__ __forceinline__ void load8(const float *p, float (&f)[8])
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 
-// g = min(gate, limit), u = clamp(up, +-limit):  g sigmoid(alpha g) (u + 1)
-__device__ __forceinline__ float clamped_glu_f(float gate, float up, float limit, float alpha)
+// g = min(gate, limit), u = clamp(up, +-limit):  g sigmoid(alpha g) (u + offset).
+// limit = infinity, alpha = 1, offset = 0 is the plain silu(gate) * up.
+struct Glu {
+    float limit, alpha, offset;
+};
+__device__ __forceinline__ float glu_f(float gate, float up, const Glu &p)
 {
-    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
-    return g * sigmoid_f(alpha * g) * (u + 1.0f);
+    const float g = fminf(gate, p.limit), u = fminf(fmaxf(up, -p.limit), p.limit);
+    return g * sigmoid_f(p.alpha * g) * (u + p.offset);
 }
 
 }  // namespace mgq

@@ -1,9 +1,9 @@
 // Linear layers over bf16 weights stored [N, K]:  y[m, n] = sum_k x[m, k] W[n, k] (+ bias[n]) (+ addend[m, n]).
 //
-// One launch takes a GROUP of up to kMaxSegments independent layers that share M and K (the
-// projections of one mixer: same or different inputs, different widths), so a decode step pays one
-// kernel boundary for all of them.  A gated feed-forward's pair of projections runs as one segment
-// with two weights whose epilogue applies the clamped GLU.
+// One launch takes a GROUP of up to kMaxSegments independent layers that share M (the projections of
+// one mixer: same or different inputs, different widths), so a decode step pays one kernel boundary
+// for all of them.  A gated feed-forward's pair of projections runs as one segment with two weights
+// whose epilogue applies the GLU.
 //
 //   linear_gemv_kernel   M <= 8: HBM-bound, a warp streams R weight rows with 16-byte loads for all M
 //                        activation rows at once (every weight byte is read once per 8 rows).
@@ -32,7 +32,7 @@ __global__ void __launch_bounds__(128) linear_gemv_kernel(const __grid_constant_
     }
     if (si >= g.count) return;
     const LinearSegment &s = g.seg[si];
-    const uint32_t n0 = unit * COLS, k = g.k;
+    const uint32_t n0 = unit * COLS, k = s.k;
     const __nv_bfloat16 *w[R];
 #pragma unroll
     for (int r = 0; r < R; r++) {
@@ -99,7 +99,7 @@ __global__ void __launch_bounds__(128) linear_gemv_kernel(const __grid_constant_
             if (lane != (uint32_t)(i * COLS + c) % 32u || n >= s.n) continue;
             const size_t o = (size_t)(row0 + i) * s.n + n;
             if (GLU) {
-                const float y = clamped_glu_f(acc[i][2 * c] + s.bias[n], acc[i][2 * c + 1] + s.bias2[n], g.limit, g.alpha);
+                const float y = glu_f(acc[i][2 * c] + (s.bias ? s.bias[n] : 0.f), acc[i][2 * c + 1] + (s.bias ? s.bias2[n] : 0.f), g.act);
                 if (g.out_bf16) static_cast<__nv_bfloat16 *>(s.out)[o] = __float2bfloat16_rn(y);
                 else            static_cast<float *>(s.out)[o] = y;
             } else {
@@ -170,7 +170,7 @@ __global__ void __launch_bounds__(256) linear_tiled_kernel(const __grid_constant
     }
     if (si >= g.count) return;
     const LinearSegment &s = g.seg[si];
-    const uint32_t n0 = tile * BN, m0 = blockIdx.y * BM, k = g.k, t = threadIdx.x;
+    const uint32_t n0 = tile * BN, m0 = blockIdx.y * BM, k = s.k, t = threadIdx.x;
     const uint32_t tx = t & 15u, ty = t >> 4;
     const XT *a = static_cast<const XT *>(s.a);
     const __nv_bfloat16 *w = static_cast<const __nv_bfloat16 *>(s.w), *w2 = static_cast<const __nv_bfloat16 *>(s.w2);
@@ -220,7 +220,7 @@ __global__ void __launch_bounds__(256) linear_tiled_kernel(const __grid_constant
             const size_t o = (size_t)row * s.n + n;
             float y = acc[0][i][j];
             if (GLU) {
-                y = clamped_glu_f(y + s.bias[n], acc[GLU ? 1 : 0][i][j] + s.bias2[n], g.limit, g.alpha);
+                y = glu_f(y + (s.bias ? s.bias[n] : 0.f), acc[GLU ? 1 : 0][i][j] + (s.bias ? s.bias2[n] : 0.f), g.act);
                 if (g.out_bf16) static_cast<__nv_bfloat16 *>(s.out)[o] = __float2bfloat16_rn(y);
                 else            static_cast<float *>(s.out)[o] = y;
                 continue;
@@ -259,12 +259,13 @@ int launch_linear_group(const LinearGroup &g, void *stream_v)
 {
     cudaStream_t stream = static_cast<cudaStream_t>(stream_v);
     if (g.m == 0) return MGQ_OK;
-    if (g.count == 0 || g.count > kMaxSegments || g.k == 0) return fail(MGQ_ERR_SHAPE, "linear: %u layers, K %u", g.count, g.k);
-    bool vec = g.k % 8 == 0;
+    if (g.count == 0 || g.count > kMaxSegments || (g.glu && g.count != 1)) return fail(MGQ_ERR_SHAPE, "linear: %u layers", g.count);
+    bool vec = true;
     for (uint32_t i = 0; i < g.count; i++) {
         const LinearSegment &s = g.seg[i];
-        if (!s.a || !s.w || !s.out || (g.glu && (!s.w2 || !s.bias || !s.bias2))) return fail(MGQ_ERR_NULL, "linear: null operand");
-        vec = vec && reinterpret_cast<uintptr_t>(s.a) % 16 == 0 && reinterpret_cast<uintptr_t>(s.w) % 16 == 0 &&
+        if (!s.a || !s.w || !s.out || (g.glu && (!s.w2 || !s.bias != !s.bias2))) return fail(MGQ_ERR_NULL, "linear: null operand");
+        if (s.k == 0) return fail(MGQ_ERR_SHAPE, "linear: K is 0");
+        vec = vec && s.k % 8 == 0 && reinterpret_cast<uintptr_t>(s.a) % 16 == 0 && reinterpret_cast<uintptr_t>(s.w) % 16 == 0 &&
               reinterpret_cast<uintptr_t>(s.w2) % 16 == 0;
     }
     if (g.m <= 8) return g.a_bf16 ? launch_gemv_typed<__nv_bfloat16>(g, vec, stream) : launch_gemv_typed<float>(g, vec, stream);

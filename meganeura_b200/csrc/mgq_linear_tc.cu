@@ -1,7 +1,7 @@
 // Linear layers over bf16 weights on the sm_100a tensor cores (M > 8 rows, bf16 activations):
 //     y[m, n] = sum_k x[m, k] W[n, k] (+ bias) (+ addend), f32 accumulation in TMEM;
 // a GLU pair keeps gate and up columns of a tile side by side in one accumulator and applies the
-// clamped GLU in the epilogue, so neither projection is written to memory.
+// GLU in the epilogue, so neither projection is written to memory.
 //
 // Persistent: one CTA per SM walks the output tiles (128 rows x TN columns) of all layers of the
 // group, rows fastest, so that consecutive CTAs share a weight tile in L2.
@@ -26,7 +26,7 @@ constexpr int kThreads = 192;
 __device__ unsigned int g_linear_tc_error = 0;
 
 struct LinearMaps {
-    CUtensorMap a[kMaxSegments], w[kMaxSegments], w2[kMaxSegments];
+    CUtensorMap a[kMaxSegments], w[kMaxSegments];        // a GLU group has one layer: w[1] is its second weight
 };
 
 template <int TN> __host__ __device__ constexpr uint32_t stage_bytes() { return kBytesA + TN * TK * 2; }
@@ -81,7 +81,6 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
     __shared__ LinearShared<S> sh;
     uint8_t *ring = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
-    const uint32_t nk = (g.k + TK - 1) / TK;
 
     if (tid == 0) {
         for (int s = 0; s < S; s++) {
@@ -116,6 +115,7 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
             bool ok = true;
             for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
                 const Tile tl = find_tile<COLS>(g, tile, mt);
+                const uint32_t nk = (g.seg[tl.si].k + TK - 1) / TK;
                 for (uint32_t kc = 0; kc < nk; kc++, it++) {
                     const uint32_t s = it % S, ph = (it / S) & 1u;
                     ok = mbar_wait(&sh.empty[s], ph ^ 1u, &sh.failed, &g_linear_tc_error);
@@ -124,7 +124,7 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
                     mbar_arrive_expect_tx(&sh.full[s], kStage);
                     tma_load_2d(st, &maps.a[tl.si], (int)(kc * TK), (int)tl.m0, &sh.full[s]);
                     tma_load_2d(st + kBytesA, &maps.w[tl.si], (int)(kc * TK), (int)tl.n0, &sh.full[s]);
-                    if (GLU) tma_load_2d(st + kBytesA + COLS * TK * 2, &maps.w2[tl.si], (int)(kc * TK), (int)tl.n0, &sh.full[s]);
+                    if (GLU) tma_load_2d(st + kBytesA + COLS * TK * 2, &maps.w[1], (int)(kc * TK), (int)tl.n0, &sh.full[s]);
                     armed = (int)it;
                 }
             }
@@ -142,6 +142,7 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
                 ok = mbar_wait(&sh.acc_empty[b], ((at >> 1) & 1u) ^ 1u, &sh.failed, &g_linear_tc_error);
                 if (!ok) break;
                 tc_fence_after();
+                const uint32_t nk = (g.seg[find_tile<COLS>(g, tile, mt).si].k + TK - 1) / TK;
                 for (uint32_t kc = 0; kc < nk; kc++, it++) {
                     const uint32_t s = it % S, ph = (it / S) & 1u;
                     ok = mbar_wait(&sh.full[s], ph, &sh.failed, &g_linear_tc_error);
@@ -183,20 +184,20 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
                 if (GLU) {
                     float up[32];
                     tmem_ld32(acc + COLS + c0, up);
-                    if (whole) {
+                    if (whole && sg.bias) {
 #pragma unroll
                         for (int e = 0; e < 32; e += 4) {
                             const float4 bg = __ldg(reinterpret_cast<const float4 *>(sg.bias + col + e)), bu = __ldg(reinterpret_cast<const float4 *>(sg.bias2 + col + e));
-                            y[e] = clamped_glu_f(y[e] + bg.x, up[e] + bu.x, g.limit, g.alpha);
-                            y[e + 1] = clamped_glu_f(y[e + 1] + bg.y, up[e + 1] + bu.y, g.limit, g.alpha);
-                            y[e + 2] = clamped_glu_f(y[e + 2] + bg.z, up[e + 2] + bu.z, g.limit, g.alpha);
-                            y[e + 3] = clamped_glu_f(y[e + 3] + bg.w, up[e + 3] + bu.w, g.limit, g.alpha);
+                            y[e] += bg.x; y[e + 1] += bg.y; y[e + 2] += bg.z; y[e + 3] += bg.w;
+                            up[e] += bu.x; up[e + 1] += bu.y; up[e + 2] += bu.z; up[e + 3] += bu.w;
                         }
-                    } else {
+                    } else if (sg.bias) {
 #pragma unroll
                         for (int e = 0; e < 32; e++)
-                            if (col + e < n) y[e] = clamped_glu_f(y[e] + __ldg(sg.bias + col + e), up[e] + __ldg(sg.bias2 + col + e), g.limit, g.alpha);
+                            if (col + e < n) { y[e] += __ldg(sg.bias + col + e); up[e] += __ldg(sg.bias2 + col + e); }
                     }
+#pragma unroll
+                    for (int e = 0; e < 32; e++) y[e] = glu_f(y[e], up[e], g.act);
                 } else if (sg.bias) {
                     if (whole) {
 #pragma unroll
@@ -294,10 +295,10 @@ int launch_tc(const LinearGroup &g, cudaStream_t stream)
     uint32_t tiles = 0;
     for (uint32_t i = 0; i < g.count; i++) {
         const LinearSegment &s = g.seg[i];
-        if (int rc = encode_rows(encode, maps.a[i], s.a, g.k, g.lda ? g.lda : g.k, g.m, TM)) return rc;
-        if (int rc = encode_rows(encode, maps.w[i], s.w, g.k, g.k, s.n, COLS)) return rc;
+        if (int rc = encode_rows(encode, maps.a[i], s.a, s.k, g.lda ? g.lda : s.k, g.m, TM)) return rc;
+        if (int rc = encode_rows(encode, maps.w[i], s.w, s.k, s.k, s.n, COLS)) return rc;
         if (GLU)
-            if (int rc = encode_rows(encode, maps.w2[i], s.w2, g.k, g.k, s.n, COLS)) return rc;
+            if (int rc = encode_rows(encode, maps.w[1], s.w2, s.k, s.k, s.n, COLS)) return rc;
         tiles += (s.n + COLS - 1) / COLS;
     }
     tiles *= (g.m + TM - 1) / TM;

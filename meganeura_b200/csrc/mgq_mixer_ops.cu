@@ -1,8 +1,8 @@
-// Norms, token shift, recurrences (RWKV-style time mixing, mLSTM matrix memory), per-head output
-// gates and the clamped GLU.  All statistics, gates, decays and recurrent state are f32; only the
+// Embedding, norms, token shift, recurrences (RWKV-style time mixing, gated linear attention, mLSTM
+// matrix memory), per-head output gates and the GLU.  All statistics, gates, decays and recurrent state are f32; only the
 // operands of the next projection may be stored as bf16.
 //
-// The two recurrences share one schedule.  A head's state is kept value-major, [value][key], and a
+// The recurrences share one schedule.  A head's state is kept value-major, [value][key], and a
 // thread owns RPT keys of a few value columns (8 threads per group of columns), so a token step is
 // register arithmetic plus a short shuffle reduction; keys beyond `dim` are zero.
 //   scan_kernel  several tokens: CTA = head x a block of value columns (x a segment of a long portion),
@@ -36,31 +36,63 @@ template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16 
 }
 
 // ---------------------------------------------------------------- embedding, rows, element-wise
+// Sine and cosine of p * f for f = f.x + f.y: the product's rounding error and the low part of f enter to first order.
+__device__ __forceinline__ void sincos_product(float p, float2 f, float &s, float &c)
+{
+    const float hi = p * f.x, lo = fmaf(p, f.y, fmaf(p, f.x, -hi));
+    float s0, c0;
+    sincosf(hi, &s0, &c0);
+    s = fmaf(lo, c0, s0);
+    c = fmaf(-lo, s0, c0);
+}
+
 template <typename T>
-__global__ void embedding_scaled_kernel(const uint32_t *ids, const T *table, float *out, uint32_t rows, uint32_t width, uint32_t vocab, float scale)
+__global__ void embedding_scaled_kernel(const __grid_constant__ Embedding a)
 {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     pdl_launch_dependents();
     pdl_wait();
-    if (i >= (size_t)rows * width) return;
-    const uint32_t row = (uint32_t)(i / width), col = (uint32_t)(i - (size_t)row * width);
-    out[i] = to_f32(table[(size_t)min(ids[row], vocab - 1u) * width + col]) * scale;
+    if (i >= (size_t)a.rows * a.width) return;
+    const uint32_t row = (uint32_t)(i / a.width), col = (uint32_t)(i - (size_t)row * a.width);
+    float x = to_f32(static_cast<const T *>(a.table)[(size_t)min(a.ids[row], a.vocab - 1u) * a.width + col]) * a.scale;
+    if (a.sinusoid) {
+        float s, c;
+        sincos_product((float)(a.pos[0] + row), a.sinusoid[col / 2], s, c);
+        x += col & 1u ? c : s;
+    }
+    a.out[i] = x;
+    if (a.copy) a.copy[i] = __float2bfloat16_rn(x);
 }
 
 // 8 elements per thread (width % 8 == 0)
 template <typename T>
-__global__ void embedding_vec_kernel(const uint32_t *ids, const T *table, float *out, uint32_t rows, uint32_t width, uint32_t vocab, float scale)
+__global__ void embedding_vec_kernel(const __grid_constant__ Embedding a)
 {
     const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 8;
     pdl_launch_dependents();
     pdl_wait();
-    if (i >= (size_t)rows * width) return;
-    const uint32_t row = (uint32_t)(i / width), col = (uint32_t)(i - (size_t)row * width);
+    if (i >= (size_t)a.rows * a.width) return;
+    const uint32_t row = (uint32_t)(i / a.width), col = (uint32_t)(i - (size_t)row * a.width);
     float f[8];
-    load8(table + (size_t)min(ids[row], vocab - 1u) * width + col, f);
-    float4 *dst = reinterpret_cast<float4 *>(out + i);
-    dst[0] = make_float4(f[0] * scale, f[1] * scale, f[2] * scale, f[3] * scale);
-    dst[1] = make_float4(f[4] * scale, f[5] * scale, f[6] * scale, f[7] * scale);
+    load8(static_cast<const T *>(a.table) + (size_t)min(a.ids[row], a.vocab - 1u) * a.width + col, f);
+#pragma unroll
+    for (int j = 0; j < 8; j++) f[j] *= a.scale;
+    if (a.sinusoid) {
+        const float p = (float)(a.pos[0] + row);
+#pragma unroll
+        for (int j = 0; j < 8; j += 2) {
+            float s, c;
+            sincos_product(p, a.sinusoid[(col + j) / 2], s, c);
+            f[j] += s;
+            f[j + 1] += c;
+        }
+    }
+    store4<float>(a.out + i, f[0], f[1], f[2], f[3]);
+    store4<float>(a.out + i + 4, f[4], f[5], f[6], f[7]);
+    if (a.copy) {
+        store4<__nv_bfloat16>(a.copy + i, f[0], f[1], f[2], f[3]);
+        store4<__nv_bfloat16>(a.copy + i + 4, f[4], f[5], f[6], f[7]);
+    }
 }
 
 __global__ void pick_rows_kernel(const float *x, const uint32_t *index, float *out, uint32_t rows, uint32_t src_rows, uint32_t cols)
@@ -82,12 +114,28 @@ __global__ void bias_add_kernel(const float *x, const float *bias, float *out, s
 }
 
 template <typename OT>
-__global__ void clamped_glu_kernel(const float *gate, const float *up, OT *out, size_t len, float limit, float alpha)
+__global__ void glu_kernel(const float *gate, const float *up, OT *out, size_t len, Glu act)
 {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     pdl_launch_dependents();
     pdl_wait();
-    if (i < len) out[i] = from_f32<OT>(clamped_glu_f(gate[i], up[i], limit, alpha));
+    if (i < len) out[i] = from_f32<OT>(glu_f(gate[i], up[i], act));
+}
+
+__global__ void cast_kernel(const float *x, __nv_bfloat16 *out, size_t len)
+{
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (i < len) out[i] = __float2bfloat16_rn(x[i]);
+}
+
+__global__ void scaled_sum_kernel(const float *a, const float *b, float *out, size_t len, float sa, float sb)
+{
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (i < len) out[i] = fmaf(sa, a[i], sb * b[i]);
 }
 
 // ---------------------------------------------------------------- RMS norm with a weight offset, optional row index
@@ -141,6 +189,82 @@ __global__ void __launch_bounds__(256) norm_kernel(const float *x, const float *
     for (int i = 0; i < HOLD; i++)
         if (t + 256u * i < cols) dst[t + 256u * i] = from_f32<OT>(v[i] * r * w[i]);
     for (uint32_t j = t + 256u * HOLD; j < cols; j += 256) dst[j] = from_f32<OT>(src[j] * r * (offset + weight[j]));
+}
+
+// ---------------------------------------------------------------- norm behind a sublayer, added to the residual
+// V elements per access.  NV accesses of a row per thread stay in registers; a wider row is summed and read again.
+template <int V, int NV>
+__global__ void __launch_bounds__(256) residual_norm_kernel(const __grid_constant__ ResidualNorm p)
+{
+    __shared__ float s_part[8];
+    const uint32_t t = threadIdx.x, n = p.cols / V;
+    const size_t base = (size_t)blockIdx.x * p.cols;
+    auto load = [&](const float *src, uint32_t j, float (&x)[V]) {
+        if (V == 4) {
+            const float4 f = *reinterpret_cast<const float4 *>(src + 4 * j);
+            x[0] = f.x; x[V / 4] = f.y; x[V / 2] = f.z; x[V - 1] = f.w;
+        } else {
+            x[0] = src[j];
+        }
+    };
+    auto value = [&](uint32_t j, float (&y)[V]) {
+        load(p.a + base, j, y);
+#pragma unroll
+        for (int e = 0; e < V; e++) y[e] *= p.sa;
+        if (!p.b) return;
+        float z[V];
+        load(p.b + base, j, z);
+#pragma unroll
+        for (int e = 0; e < V; e++) y[e] = fmaf(p.sb, z[e], y[e]);
+    };
+    float w[NV][V], y[NV][V], x[NV][V];
+    pdl_launch_dependents();
+#pragma unroll
+    for (int i = 0; i < NV; i++)
+        if (t + 256u * i < n) load(p.weight, t + 256u * i, w[i]);
+    pdl_wait();
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        if (t + 256u * i >= n) break;
+        value(t + 256u * i, y[i]);
+        load(p.addend + base, t + 256u * i, x[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        if (t + 256u * i >= n) break;
+#pragma unroll
+        for (int e = 0; e < V; e++) ss = fmaf(y[i][e], y[i][e], ss);
+    }
+    for (uint32_t j = t + 256u * NV; j < n; j += 256) {
+        float z[V];
+        value(j, z);
+#pragma unroll
+        for (int e = 0; e < V; e++) ss = fmaf(z[e], z[e], ss);
+    }
+    const float r = 1.0f / sqrtf(block_sum(ss, s_part) / (float)p.cols + p.eps);
+    auto put = [&](uint32_t j, const float (&yy)[V], const float (&ww)[V], const float (&xx)[V]) {
+        float o[V];
+#pragma unroll
+        for (int e = 0; e < V; e++) o[e] = fmaf(yy[e] * r, p.offset + ww[e], xx[e]);
+        if (V == 4) {
+            store4<float>(p.out + base + 4 * j, o[0], o[V / 4], o[V / 2], o[V - 1]);
+            if (p.copy) store4<__nv_bfloat16>(p.copy + base + 4 * j, o[0], o[V / 4], o[V / 2], o[V - 1]);
+        } else {
+            p.out[base + j] = o[0];
+            if (p.copy) p.copy[base + j] = __float2bfloat16_rn(o[0]);
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < NV; i++)
+        if (t + 256u * i < n) put(t + 256u * i, y[i], w[i], x[i]);
+    for (uint32_t j = t + 256u * NV; j < n; j += 256) {
+        float yy[V], ww[V], xx[V];
+        value(j, yy);
+        load(p.weight, j, ww);
+        load(p.addend + base, j, xx);
+        put(j, yy, ww, xx);
+    }
 }
 
 // ---------------------------------------------------------------- token shift (with the norm in front of it)
@@ -245,7 +369,7 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const float *o, const __
     pdl_wait();
     if (unit >= total) return;
     const size_t base = (size_t)unit * dim;
-    const uint32_t wbase = (unit % heads) * dim;
+    const uint32_t wbase = hg.shared ? 0 : (unit % heads) * dim;
     float v[HOLD], ss = 0.f, r = 1.f;
 #pragma unroll
     for (int i = 0; i < HOLD; i++) {
@@ -274,7 +398,7 @@ __global__ void __launch_bounds__(256) head_gate_vec_kernel(const float *o, cons
     pdl_wait();
     const bool live = unit < total;                      // no early return: the lanes of a warp reduce together
     const size_t base = (size_t)(live ? unit : 0) * dim;
-    const uint32_t wbase = (live ? unit % heads : 0) * dim;
+    const uint32_t wbase = hg.shared || !live ? 0 : unit % heads * dim;
     float4 v[KV], g[KV];
     float ss = 0.f;
 #pragma unroll
@@ -306,12 +430,16 @@ __global__ void __launch_bounds__(256) head_gate_vec_kernel(const float *o, cons
     }
 }
 
-// ---------------------------------------------------------------- decay: exp(-exp(tanh(low) . w2^T + w0)), 64 rows x 64 channels per CTA
+// ---------------------------------------------------------------- decays, 64 rows x 64 channels per CTA
+__device__ __forceinline__ float log_sigmoid(float z) { return z < 0.f ? z - log1pf(expf(z)) : -log1pf(expf(-z)); }
+__device__ __forceinline__ float decay_input(float low, float inv_tau) { return inv_tau == 0.f ? tanhf(low) : low; }
+__device__ __forceinline__ float decay_value(float z, float inv_tau) { return inv_tau == 0.f ? expf(-expf(z)) : expf(log_sigmoid(z) * inv_tau); }
+
 constexpr uint32_t kDecayTile = 64, kDecayK = 16;
-__global__ void __launch_bounds__(256) decay_kernel(const __grid_constant__ Wkv a)
+__global__ void __launch_bounds__(256) decay_kernel(const __grid_constant__ Decay a)
 {
     __shared__ float s_low[kDecayK][kDecayTile + 4], s_w[kDecayK][kDecayTile + 4];
-    const uint32_t t = threadIdx.x, tx = t & 15u, ty = t >> 4, ch0 = blockIdx.x * kDecayTile, row0 = blockIdx.y * kDecayTile, channels = a.heads * a.dim;
+    const uint32_t t = threadIdx.x, tx = t & 15u, ty = t >> 4, ch0 = blockIdx.x * kDecayTile, row0 = blockIdx.y * kDecayTile, channels = a.channels;
     const __nv_bfloat16 *w = static_cast<const __nv_bfloat16 *>(a.w2);
     float acc[4][4];
 #pragma unroll
@@ -325,7 +453,7 @@ __global__ void __launch_bounds__(256) decay_kernel(const __grid_constant__ Wkv 
         for (int i = 0; i < 4; i++) {
             const uint32_t e = t + 256u * i, r = e / kDecayK, k = e % kDecayK;
             const bool in = k0 + k < a.rank;
-            s_low[k][r] = in && row0 + r < a.rows ? tanhf(a.low[(size_t)(row0 + r) * a.rank + k0 + k]) : 0.f;
+            s_low[k][r] = in && row0 + r < a.rows ? decay_input(a.low[(size_t)(row0 + r) * a.rank + k0 + k], a.inv_tau) : 0.f;
             s_w[k][r] = in && ch0 + r < channels ? __bfloat162float(w[(size_t)(ch0 + r) * a.rank + k0 + k]) : 0.f;
         }
         __syncthreads();
@@ -347,7 +475,7 @@ __global__ void __launch_bounds__(256) decay_kernel(const __grid_constant__ Wkv 
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const uint32_t ch = ch0 + tx * 4 + j;
-            if (ch < channels) a.decay[(size_t)row * channels + ch] = expf(-expf(acc[i][j] + a.w0[ch]));
+            if (ch < channels) a.out[(size_t)row * channels + ch] = decay_value(acc[i][j] + a.w0[ch], a.inv_tau);
         }
     }
 }
@@ -364,10 +492,10 @@ __device__ __forceinline__ void cp_async16(void *smem, const void *gmem)
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
 
-enum { kWkv = 0, kMlstm = 1 };
+enum { kWkv = 0, kMlstm = 1, kGla = 2 };
 
 struct Scan {
-    const float *q, *k, *v, *w;          // wkv: r, k, v, decay;  mlstm: q, k, v, -
+    const float *q, *k, *v, *w;          // wkv, gla: with a decay per key channel;  mlstm: w unused
     const float *u;                      // wkv bonus [heads, dim]
     const float *gi, *gf;                // mlstm gate pre-activations [rows, heads]
     float *o, *state, *shift_state;
@@ -384,10 +512,8 @@ template <int RPT> __host__ __device__ constexpr int chunk_tokens() { return RPT
 template <int RPT> __host__ __device__ constexpr int thread_cols() { return RPT <= 16 ? 4 : 2; }
 __host__ __device__ inline uint32_t block_cols(uint32_t dim) { return dim <= 128 ? 64u : 32u; }
 
-__device__ __forceinline__ float log_sigmoid(float z) { return z < 0.f ? z - log1pf(expf(z)) : -log1pf(expf(-z)); }
-
 // One token of C value columns for the RPT keys this thread owns; OUT: out / den receive its share of the
-// dot products.  n: mlstm normalizer; without OUT a wkv thread multiplies its decays into it instead.
+// dot products.  n: mlstm normalizer; without OUT a thread with channel decays multiplies them into it instead.
 template <int MODE, int RPT, int C, bool OUT>
 __device__ __forceinline__ void token_update(const float *q, const float *k, const float *w, const float (&u)[RPT], const float (&v_in)[C], float a, float b,
                                              float (&S)[C][RPT], float (&n)[RPT], float (&out)[C], float &den)
@@ -407,19 +533,20 @@ __device__ __forceinline__ void token_update(const float *q, const float *k, con
             const float4 q4 = *reinterpret_cast<const float4 *>(q + i * 8);
             qv[0] = q4.x; qv[1] = q4.y; qv[2] = q4.z; qv[3] = q4.w;
         }
-        if (MODE == kWkv) {
+        if (MODE != kMlstm) {
             const float4 w4 = *reinterpret_cast<const float4 *>(w + i * 8);
             wv[0] = w4.x; wv[1] = w4.y; wv[2] = w4.z; wv[3] = w4.w;
         }
 #pragma unroll
         for (int j = 0; j < 4; j++) {
-            if (MODE == kWkv) {
+            if (MODE != kMlstm) {
                 if (!OUT) n[i + j] *= wv[j];
 #pragma unroll
                 for (int c = 0; c < C; c++) {
                     const float x = kv[j] * v[c];
-                    if (OUT) out[c] = fmaf(qv[j], fmaf(u[i + j], x, S[c][i + j]), out[c]);
+                    if (OUT && MODE == kWkv) out[c] = fmaf(qv[j], fmaf(u[i + j], x, S[c][i + j]), out[c]);
                     S[c][i + j] = fmaf(wv[j], S[c][i + j], x);
+                    if (OUT && MODE == kGla) out[c] = fmaf(qv[j], S[c][i + j], out[c]);
                 }
             } else {
                 n[i + j] = fmaf(kv[j], b, a * n[i + j]);
@@ -491,8 +618,8 @@ constexpr uint32_t kScanThreads = 128;
 
 // A state block: [heads][vdim][pad4(dim)], then per head and block of value columns [pad4(dim)] plus 4
 // scalars.  In an mlstm state those hold n and m, one copy per block (every CTA of a head advances its own,
-// so no CTA reads what another one writes); in a segment's end state also the decay product (wkv: per key in
-// place of n) or the sum of log forget gates (mlstm: scalar 1).
+// so no CTA reads what another one writes); in a segment's end state also the decay product (per key in
+// place of n: channel decays) or the sum of log forget gates (mlstm: scalar 1).
 __host__ __device__ inline uint32_t value_blocks(uint32_t dim, uint32_t vdim) { return (vdim + block_cols(dim) - 1) / block_cols(dim); }
 __host__ __device__ inline size_t block_elements(uint32_t heads, uint32_t dim, uint32_t vdim)
 {
@@ -512,7 +639,7 @@ __device__ __forceinline__ float *normalizer(const Scan &p, float *base, uint32_
 template <int MODE, int RPT>
 __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_constant__ Scan p)
 {
-    constexpr int TC = chunk_tokens<RPT>(), KS = RPT * 8, NA = MODE == kWkv ? 3 : 2, C = thread_cols<RPT>(), COLS = 16 * C;
+    constexpr int TC = chunk_tokens<RPT>(), KS = RPT * 8, NA = MODE != kMlstm ? 3 : 2, C = thread_cols<RPT>(), COLS = 16 * C;
     extern __shared__ __align__(16) float smem[];
     // per buffer: NA x [TC][KS] key vectors, [TC][COLS] values
     constexpr int kBuf = NA * TC * KS + TC * COLS;
@@ -529,7 +656,7 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_cons
     for (int i = 0; i < RPT; i++) {
         const uint32_t key = (i / 4 * 8 + ks) * 4 + i % 4;
         u[i] = MODE == kWkv && key < dim ? __ldg(p.u + head * dim + key) : 0.f;
-        n[i] = MODE == kWkv ? 1.f : 0.f;
+        n[i] = MODE != kMlstm ? 1.f : 0.f;
 #pragma unroll
         for (int c = 0; c < C; c++) S[c][i] = 0.f;
     }
@@ -610,7 +737,7 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_cons
                 float x[RPT];
                 load_keys<RPT>(base + ((size_t)head * vdim + col + c) * kp, ks, kp, x);
 #pragma unroll
-                for (int i = 0; i < RPT; i++) S[c][i] = MODE == kWkv ? fmaf(f[i], S[c][i], x[i]) : fmaf(add, x[i], keep * S[c][i]);
+                for (int i = 0; i < RPT; i++) S[c][i] = MODE != kMlstm ? fmaf(f[i], S[c][i], x[i]) : fmaf(add, x[i], keep * S[c][i]);
             }
         }
     } else if (MODE == kMlstm) {
@@ -681,6 +808,7 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_cons
             for (int j = 0; j < C; j++) {
                 y[j] = reduce8(out[j], ks);
                 if (MODE == kMlstm) y[j] = mlstm_out(y[j], d, p.qscale, s_gate[buf][2][r + ks]);
+                if (MODE == kGla) y[j] *= p.qscale;
             }
             float *at = dst + (size_t)(r + ks) * vpitch;
             if (C == 4 && vec_v) {
@@ -699,7 +827,7 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_cons
             den = sum8(den);
 #pragma unroll
             for (int j = 0; j < C; j++) {
-                const float y = sum8(out[j]);
+                const float y = sum8(out[j]) * (MODE == kGla ? p.qscale : 1.f);
                 if (ks == 0 && col + j < vdim) dst[(size_t)r * vpitch + j] = MODE == kMlstm ? mlstm_out(y, den, p.qscale, s_gate[buf][2][r]) : y;
             }
         }
@@ -732,11 +860,11 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_cons
 constexpr uint32_t kStepThreads = 512, kStepCols = kStepThreads / 8;
 
 template <int MODE, int RPT, typename OT>
-__global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constant__ Scan p, const __grid_constant__ HeadGate hg, const float *low,
-                                                            const __nv_bfloat16 *w2, const float *w0, uint32_t rank)
+__global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constant__ Scan p, const __grid_constant__ HeadGate hg,
+                                                            const __grid_constant__ Decay d)
 {
     constexpr int KS = RPT * 8;
-    extern __shared__ __align__(16) float smem[];        // q, k, w [KS] each; o [vdim]; tanh(low) [rank]
+    extern __shared__ __align__(16) float smem[];        // q, k, w [KS] each; o [vdim]; the decay's low-rank input [rank]
     __shared__ float s_part[kStepThreads / 32], s_gate[3];
     const uint32_t t = threadIdx.x, head = blockIdx.x, ks = t & 7u, dim = p.dim, vdim = p.vdim, kp = pad4(dim);
     float *sq = smem, *sk = sq + KS, *sw = sk + KS, *so = sw + KS, *s_low = so + vdim;
@@ -755,8 +883,10 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
         sw[i] = 0.f;
     }
     float *nrow = normalizer(p, p.state, head, 0);
-    if (MODE == kWkv) {
-        for (uint32_t i = t; i < rank; i += kStepThreads) s_low[i] = tanhf(low[i]);
+    if (MODE != kMlstm) {
+        const __nv_bfloat16 *w2 = static_cast<const __nv_bfloat16 *>(d.w2);
+        const uint32_t rank = d.rank;
+        for (uint32_t i = t; i < rank; i += kStepThreads) s_low[i] = decay_input(d.low[i], d.inv_tau);
         __syncthreads();
         for (uint32_t ch = t / 8; ch < ((dim + 3u) & ~3u); ch += kStepCols) {       // a warp covers 4 channels: uniform trip count
             float acc = 0.f;
@@ -764,7 +894,7 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
                 for (uint32_t j = ks; j < rank; j += 8) acc = fmaf(s_low[j], __bfloat162float(w2[(size_t)(head * dim + ch) * rank + j]), acc);
 #pragma unroll
             for (int off = 4; off > 0; off >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
-            if (ks == 0 && ch < dim) sw[ch] = expf(-expf(acc + w0[head * dim + ch]));
+            if (ks == 0 && ch < dim) sw[ch] = decay_value(acc + d.w0[head * dim + ch], d.inv_tau);
         }
     } else {
         load_keys<RPT>(nrow, ks, kp, n);
@@ -791,6 +921,7 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
         const float v[1] = {live ? p.v[head * vdim + col] : 0.f};
         token_update<MODE, RPT, 1, true>(sq + ks * 4, sk + ks * 4, sw + ks * 4, u, v, a, b, S, nn, out1, den);
         float out = sum8(out1[0]);
+        if (MODE == kGla) out *= p.qscale;
         if (MODE == kMlstm) {
             out = mlstm_out(out, sum8(den), p.qscale, expf(-m_new));
 #pragma unroll
@@ -805,7 +936,7 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
     OT *dst = static_cast<OT *>(hg.out) + head * vdim;
     for (uint32_t j = t; j < vdim; j += kStepThreads) {
         const float g = hg.gate[head * vdim + j], s = sigmoid_f(g);
-        dst[j] = from_f32<OT>(so[j] * r * hg.weight[head * vdim + j] * (hg.silu ? g * s : s));
+        dst[j] = from_f32<OT>(so[j] * r * hg.weight[hg.shared ? j : head * vdim + j] * (hg.silu ? g * s : s));
     }
     if (MODE == kMlstm) {
         for (uint32_t blk = t / 8; blk < value_blocks(dim, vdim); blk += kStepCols) {
@@ -834,7 +965,7 @@ uint32_t segment_length(uint32_t rows, uint32_t heads, uint32_t dim, uint32_t vd
 template <int MODE, int RPT>
 int launch_scan_rpt(Scan p, void *workspace, cudaStream_t stream)
 {
-    constexpr int NA = MODE == kWkv ? 3 : 2, TC = chunk_tokens<RPT>(), COLS = 16 * thread_cols<RPT>();
+    constexpr int NA = MODE != kMlstm ? 3 : 2, TC = chunk_tokens<RPT>(), COLS = 16 * thread_cols<RPT>();
     const size_t smem = (size_t)2 * (NA * TC * RPT * 8 + TC * COLS) * sizeof(float);
     if (int rc = allow_smem(scan_kernel<MODE, RPT>, smem)) return rc;
     p.segments = static_cast<float *>(workspace);
@@ -866,34 +997,33 @@ int launch_scan(const Scan &p, void *workspace, cudaStream_t stream)
 }
 
 template <int MODE, int RPT>
-int launch_step_rpt(const Scan &p, const HeadGate &hg, const float *low, const void *w2, const float *w0, uint32_t rank, cudaStream_t stream)
+int launch_step_rpt(const Scan &p, const HeadGate &hg, const Decay &d, cudaStream_t stream)
 {
-    const size_t smem = (size_t)(3 * RPT * 8 + p.vdim + rank) * sizeof(float);
-    const __nv_bfloat16 *w2b = static_cast<const __nv_bfloat16 *>(w2);
+    const size_t smem = (size_t)(3 * RPT * 8 + p.vdim + d.rank) * sizeof(float);
     if (hg.out_bf16) {
         if (int rc = allow_smem(step_kernel<MODE, RPT, __nv_bfloat16>, smem)) return rc;
-        return launch(step_kernel<MODE, RPT, __nv_bfloat16>, dim3(p.heads), dim3(kStepThreads), smem, stream, p, hg, low, w2b, w0, rank);
+        return launch(step_kernel<MODE, RPT, __nv_bfloat16>, dim3(p.heads), dim3(kStepThreads), smem, stream, p, hg, d);
     }
     if (int rc = allow_smem(step_kernel<MODE, RPT, float>, smem)) return rc;
-    return launch(step_kernel<MODE, RPT, float>, dim3(p.heads), dim3(kStepThreads), smem, stream, p, hg, low, w2b, w0, rank);
+    return launch(step_kernel<MODE, RPT, float>, dim3(p.heads), dim3(kStepThreads), smem, stream, p, hg, d);
 }
 
 template <int MODE>
-int launch_step(const Scan &p, const HeadGate &hg, const float *low, const void *w2, const float *w0, uint32_t rank, cudaStream_t stream)
+int launch_step(const Scan &p, const HeadGate &hg, const Decay &d, cudaStream_t stream)
 {
-    if (p.dim <= 32) return launch_step_rpt<MODE, 4>(p, hg, low, w2, w0, rank, stream);
-    if (p.dim <= 64) return launch_step_rpt<MODE, 8>(p, hg, low, w2, w0, rank, stream);
-    if (p.dim <= 128) return launch_step_rpt<MODE, 16>(p, hg, low, w2, w0, rank, stream);
-    if (p.dim <= kMaxStateDim) return launch_step_rpt<MODE, 32>(p, hg, low, w2, w0, rank, stream);
+    if (p.dim <= 32) return launch_step_rpt<MODE, 4>(p, hg, d, stream);
+    if (p.dim <= 64) return launch_step_rpt<MODE, 8>(p, hg, d, stream);
+    if (p.dim <= 128) return launch_step_rpt<MODE, 16>(p, hg, d, stream);
+    if (p.dim <= kMaxStateDim) return launch_step_rpt<MODE, 32>(p, hg, d, stream);
     return fail(MGQ_ERR_SHAPE, "recurrent heads of %u key dimensions (at most %u)", p.dim, kMaxStateDim);
 }
 
-Scan wkv_args(const Wkv &a)
+Scan channel_decay_args(const ChannelDecay &a)
 {
     Scan p{};
-    p.q = a.r; p.k = a.k; p.v = a.v; p.w = a.decay; p.u = a.u; p.o = a.o; p.state = a.state; p.shift_state = a.shift_state;
-    p.rows = a.rows; p.heads = a.heads; p.dim = a.dim; p.vdim = a.dim; p.shift_width = a.shift_width;
-    p.cap = 1.f; p.qscale = 1.f;
+    p.q = a.q; p.k = a.k; p.v = a.v; p.w = a.d.out; p.u = a.u; p.o = a.o; p.state = a.state; p.shift_state = a.shift_state;
+    p.rows = a.rows; p.heads = a.heads; p.dim = a.dim; p.vdim = a.vdim; p.shift_width = a.shift_width;
+    p.cap = 1.f; p.qscale = a.u ? 1.f : (float)(1.0 / sqrt((double)a.dim));
     return p;
 }
 Scan mlstm_args(const Mlstm &a)
@@ -909,18 +1039,15 @@ inline uint32_t blocks_for(size_t n) { return (uint32_t)((n + 255) / 256); }
 
 }  // namespace
 
-int launch_embedding_scaled(const uint32_t *ids, const void *table, bool table_bf16, float *out, uint32_t rows, uint32_t width, uint32_t vocab,
-                            float scale, void *stream)
+int launch_embedding_scaled(const Embedding &a, void *stream)
 {
-    const dim3 grid(blocks_for((size_t)rows * width));
     cudaStream_t st = static_cast<cudaStream_t>(stream);
-    if (width % 8 == 0) {
-        const dim3 grid8(blocks_for((size_t)rows * width / 8));
-        if (table_bf16) return launch(embedding_vec_kernel<__nv_bfloat16>, grid8, dim3(256), 0, st, ids, static_cast<const __nv_bfloat16 *>(table), out, rows, width, vocab, scale);
-        return launch(embedding_vec_kernel<float>, grid8, dim3(256), 0, st, ids, static_cast<const float *>(table), out, rows, width, vocab, scale);
+    if (a.width % 8 == 0) {
+        const dim3 grid(blocks_for((size_t)a.rows * a.width / 8));
+        return a.table_bf16 ? launch(embedding_vec_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, a) : launch(embedding_vec_kernel<float>, grid, dim3(256), 0, st, a);
     }
-    if (table_bf16) return launch(embedding_scaled_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, ids, static_cast<const __nv_bfloat16 *>(table), out, rows, width, vocab, scale);
-    return launch(embedding_scaled_kernel<float>, grid, dim3(256), 0, st, ids, static_cast<const float *>(table), out, rows, width, vocab, scale);
+    const dim3 grid(blocks_for((size_t)a.rows * a.width));
+    return a.table_bf16 ? launch(embedding_scaled_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, a) : launch(embedding_scaled_kernel<float>, grid, dim3(256), 0, st, a);
 }
 
 int launch_norm(const float *x, const float *weight, const uint32_t *index, void *out, bool out_bf16, uint32_t rows, uint32_t src_rows,
@@ -942,11 +1069,30 @@ int launch_bias_add(const float *x, const float *bias, float *out, uint32_t rows
     return launch(bias_add_kernel, dim3(blocks_for(len)), dim3(256), 0, static_cast<cudaStream_t>(stream), x, bias, out, len, cols);
 }
 
-int launch_clamped_glu(const float *gate, const float *up, void *out, bool out_bf16, size_t len, float limit, float alpha, void *stream)
+int launch_glu(const float *gate, const float *up, void *out, bool out_bf16, size_t len, const Glu &act, void *stream)
 {
     cudaStream_t st = static_cast<cudaStream_t>(stream);
-    if (out_bf16) return launch(clamped_glu_kernel<__nv_bfloat16>, dim3(blocks_for(len)), dim3(256), 0, st, gate, up, static_cast<__nv_bfloat16 *>(out), len, limit, alpha);
-    return launch(clamped_glu_kernel<float>, dim3(blocks_for(len)), dim3(256), 0, st, gate, up, static_cast<float *>(out), len, limit, alpha);
+    if (out_bf16) return launch(glu_kernel<__nv_bfloat16>, dim3(blocks_for(len)), dim3(256), 0, st, gate, up, static_cast<__nv_bfloat16 *>(out), len, act);
+    return launch(glu_kernel<float>, dim3(blocks_for(len)), dim3(256), 0, st, gate, up, static_cast<float *>(out), len, act);
+}
+
+int launch_cast(const float *x, __nv_bfloat16 *out, size_t len, void *stream)
+{
+    return launch(cast_kernel, dim3(blocks_for(len)), dim3(256), 0, static_cast<cudaStream_t>(stream), x, out, len);
+}
+
+int launch_scaled_sum(const float *a, const float *b, float *out, size_t len, float sa, float sb, void *stream)
+{
+    return launch(scaled_sum_kernel, dim3(blocks_for(len)), dim3(256), 0, static_cast<cudaStream_t>(stream), a, b, out, len, sa, sb);
+}
+
+int launch_residual_norm(const ResidualNorm &a, void *stream)
+{
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (a.cols % 4) return launch(residual_norm_kernel<1, 4>, dim3(a.rows), dim3(256), 0, st, a);
+    if (a.cols <= 1024) return launch(residual_norm_kernel<4, 1>, dim3(a.rows), dim3(256), 0, st, a);
+    if (a.cols <= 2048) return launch(residual_norm_kernel<4, 2>, dim3(a.rows), dim3(256), 0, st, a);
+    return launch(residual_norm_kernel<4, 4>, dim3(a.rows), dim3(256), 0, st, a);
 }
 
 template <typename OT>
@@ -988,28 +1134,35 @@ int launch_head_gate(const float *o, const HeadGate &hg, uint32_t rows, uint32_t
     return launch(head_gate_kernel<float>, dim3((total + 7) / 8), dim3(256), 0, st, o, hg, total, heads, dim);
 }
 
-size_t wkv_state_elements(uint32_t heads, uint32_t dim) { return (size_t)heads * dim * pad4(dim); }
+size_t channel_decay_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim) { return (size_t)heads * vdim * pad4(dim); }
 size_t mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim) { return block_elements(heads, dim, vdim); }
 size_t scan_workspace(uint32_t max_rows, uint32_t heads, uint32_t dim, uint32_t vdim)
 {
     return max_rows < 256 ? 0 : 8 * block_elements(heads, dim, vdim) * sizeof(float);       // at most 9 segments, the last one ends in the state
 }
 
-int launch_decay(const Wkv &a, void *stream)
+int launch_decay(const Decay &a, void *stream)
 {
-    return launch(decay_kernel, dim3((a.heads * a.dim + kDecayTile - 1) / kDecayTile, (a.rows + kDecayTile - 1) / kDecayTile), dim3(256), 0,
+    return launch(decay_kernel, dim3((a.channels + kDecayTile - 1) / kDecayTile, (a.rows + kDecayTile - 1) / kDecayTile), dim3(256), 0,
                   static_cast<cudaStream_t>(stream), a);
 }
 
-int launch_wkv_scan(const Wkv &a, void *stream) { return launch_scan<kWkv>(wkv_args(a), a.workspace, static_cast<cudaStream_t>(stream)); }
-int launch_mlstm_scan(const Mlstm &a, void *stream) { return launch_scan<kMlstm>(mlstm_args(a), a.workspace, static_cast<cudaStream_t>(stream)); }
-int launch_wkv_step(const Wkv &a, const HeadGate &hg, void *stream)
+int launch_channel_decay_scan(const ChannelDecay &a, void *stream)
 {
-    return launch_step<kWkv>(wkv_args(a), hg, a.low, a.w2, a.w0, a.rank, static_cast<cudaStream_t>(stream));
+    const Scan p = channel_decay_args(a);
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    return a.u ? launch_scan<kWkv>(p, a.workspace, st) : launch_scan<kGla>(p, a.workspace, st);
+}
+int launch_mlstm_scan(const Mlstm &a, void *stream) { return launch_scan<kMlstm>(mlstm_args(a), a.workspace, static_cast<cudaStream_t>(stream)); }
+int launch_channel_decay_step(const ChannelDecay &a, const HeadGate &hg, void *stream)
+{
+    const Scan p = channel_decay_args(a);
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    return a.u ? launch_step<kWkv>(p, hg, a.d, st) : launch_step<kGla>(p, hg, a.d, st);
 }
 int launch_mlstm_step(const Mlstm &a, const HeadGate &hg, void *stream)
 {
-    return launch_step<kMlstm>(mlstm_args(a), hg, nullptr, nullptr, nullptr, 0, static_cast<cudaStream_t>(stream));
+    return launch_step<kMlstm>(mlstm_args(a), hg, Decay{}, static_cast<cudaStream_t>(stream));
 }
 
 }  // namespace mgq

@@ -1,15 +1,13 @@
-// Latent attention for many rows (a prompt's portion), bf16 cache.
+// Softmax attention for many rows (a prompt's portion) over f16 keys and values: a blockwise exact softmax,
+// CTA = one head x 128 query rows (8 warps x 16 rows) x up to 128 value columns, 64 keys per tile, three
+// cp.async stages, tensor-core products with f32 accumulation.  Query heads may share key / value heads.
 //
-// The keys W_uk c and values W_uv c of all live cache rows are expanded once per step by the tcgen05
-// linear kernel (ring order, f16); the attention kernel then works like a blockwise exact softmax:
-// CTA = one head x 128 query rows (8 warps x 16 rows), 64 keys per tile, three cp.async stages,
-// tensor-core products with f32 accumulation.  The rotated key part, shared by the heads, is kept once.
+// Latent attention, bf16 cache: the keys W_uk c and values W_uv c of all live cache rows are expanded once
+// per step by the tcgen05 linear kernel (ring order, f16).  The rotated key part, shared by the heads, is kept once.
 // Scores, maxima, sums and weights are f32.  The operands of the products are f16, not bf16: all are of
 // moderate size (a clamp guards the range), and with 11 significant bits the result stays close to the
 // absorbed form, which keeps the query in f32, so it hardly matters how a prompt is cut.  Only tiles that some row of the
 // CTA can see are visited; positions map to ring rows by position % slots.
-#include <cuda_fp16.h>
-
 #include "mgq_linear.cuh"
 #include "mgq_mixer.cuh"
 
@@ -41,7 +39,7 @@ __device__ __forceinline__ uint32_t pack2(float x, float y)
     const __half2 h = __floats2half2_rn(x, y);
     return *reinterpret_cast<const uint32_t *>(&h);
 }
-__device__ __forceinline__ __half to_half(float x) { return __float2half_rn(fminf(fmaxf(x, -65504.f), 65504.f)); }
+__device__ __forceinline__ __half to_half(float x) { return from_f32<__half>(x); }
 
 // The shared rotated key parts of the live cache rows as f16.
 __global__ void rotated_half_kernel(const __nv_bfloat16 *cache, const uint32_t *pos, __half *out, uint32_t rows, uint32_t slots, uint32_t rank, uint32_t rot)
@@ -56,31 +54,32 @@ __global__ void rotated_half_kernel(const __nv_bfloat16 *cache, const uint32_t *
 
 struct Prefill {
     const float *q, *freq;
-    const __half *keys, *values, *rotated;          // [slots, heads * dim], [slots, heads * vdim], [slots, rot]
+    const __half *keys, *values, *rotated;          // [slots, kv_heads * dim], [slots, kv_heads * vdim], [slots, rot]
     const uint32_t *pos;
     const float *gate;
     void *out;
-    uint32_t rows, heads, dim, rot, vdim, rank, slots, window;
+    uint32_t rows, heads, kv_heads, dim, rot, vdim, slots, window;
     float scale_log2;                               // scale * log2(e)
     uint32_t out_bf16, silu;
 };
 
-// DK: dim + rot, DV: vdim, both rounded up to a multiple of 16.
+// DK: dim + rot, DV: value columns of the CTA (blockIdx.z: which), both rounded up to a multiple of 16.
 template <int DK, int DV>
-__global__ void __launch_bounds__(kThreads, 1) latent_prefill_kernel(const __grid_constant__ Prefill p)
+__global__ void __launch_bounds__(kThreads, 1) prefill_attention_kernel(const __grid_constant__ Prefill p)
 {
     constexpr int PK = DK + 8, PV = DV + 8;          // row pitch in elements: an odd number of 16-byte pieces
     extern __shared__ __align__(16) __half sm[];
     __half *s_q = sm, *s_k = s_q + BM * PK, *s_v = s_k + kStages * BN * PK;
     const uint32_t t = threadIdx.x, lane = t & 31u, warp = t >> 5, head = blockIdx.x;
+    const uint32_t kv_head = head / (p.heads / p.kv_heads), v0 = blockIdx.z * DV, vcols = min(p.vdim - v0, (uint32_t)DV);
     const uint32_t row0 = (gridDim.y - 1 - blockIdx.y) * BM, dk = p.dim + p.rot;      // longest rows first
     pdl_launch_dependents();
     // zero padding columns (they meet in products), and query rows that do not exist
     const __half zero = __float2half_rn(0.f);
     if (dk < DK)
         for (uint32_t i = t; i < (BM + kStages * BN) * (DK - dk); i += kThreads) s_q[i / (DK - dk) * PK + dk + i % (DK - dk)] = zero;
-    if (p.vdim < DV)
-        for (uint32_t i = t; i < kStages * BN * (DV - p.vdim); i += kThreads) s_v[i / (DV - p.vdim) * PV + p.vdim + i % (DV - p.vdim)] = zero;
+    if (vcols < DV)
+        for (uint32_t i = t; i < kStages * BN * (DV - vcols); i += kThreads) s_v[i / (DV - vcols) * PV + vcols + i % (DV - vcols)] = zero;
     for (uint32_t r = p.rows - row0; r < BM; r++)
         for (uint32_t j = t; j < dk; j += kThreads) s_q[r * PK + j] = zero;
     pdl_wait();
@@ -91,11 +90,11 @@ __global__ void __launch_bounds__(kThreads, 1) latent_prefill_kernel(const __gri
     auto stage = [&](uint32_t tile, uint32_t buf) {
         const uint32_t kt = lo + tile * BN;
         const uint32_t kb = smem_addr(s_k + buf * BN * PK), vb = smem_addr(s_v + buf * BN * PV);
-        const uint32_t per_k = p.dim / 8, per_r = p.rot / 8, per_v = p.vdim / 8;
+        const uint32_t per_k = p.dim / 8, per_r = p.rot / 8, per_v = vcols / 8;
         const uint32_t r = t >> 2, part = t & 3u;                         // four threads per key row
         const size_t slot = min(kt + r, last) % p.slots;                  // beyond the last key: a valid row, masked below
-        const __half *ksrc = p.keys + (slot * p.heads + head) * p.dim, *rsrc = p.rotated + slot * p.rot,
-                            *vsrc = p.values + (slot * p.heads + head) * p.vdim;
+        const __half *ksrc = p.keys + (slot * p.kv_heads + kv_head) * p.dim, *rsrc = p.rotated + slot * p.rot,
+                            *vsrc = p.values + (slot * p.kv_heads + kv_head) * p.vdim + v0;
         for (uint32_t c = part; c < per_k; c += 4) cp_async16(kb + (r * PK + c * 8) * 2, ksrc + c * 8);
         for (uint32_t c = part; c < per_r; c += 4) cp_async16(kb + (r * PK + p.dim + c * 8) * 2, rsrc + c * 8);
         for (uint32_t c = part; c < per_v; c += 4) cp_async16(vb + (r * PV + c * 8) * 2, vsrc + c * 8);
@@ -221,11 +220,11 @@ __global__ void __launch_bounds__(kThreads, 1) latent_prefill_kernel(const __gri
         const uint32_t row = row0 + qrow + h * 8;
         if (row >= p.rows) continue;
         const float inv = 1.0f / l[h];
-        const size_t base = ((size_t)row * p.heads + head) * p.vdim;
+        const size_t base = ((size_t)row * p.heads + head) * p.vdim + v0;
 #pragma unroll
         for (int n = 0; n < DV / 8; n++) {
             const uint32_t v = n * 8 + (lane & 3u) * 2;
-            if (v >= p.vdim) break;
+            if (v >= vcols) break;
             float x = o[n][2 * h] * inv, y = o[n][2 * h + 1] * inv;
             if (p.gate) {
                 const float2 g = *reinterpret_cast<const float2 *>(p.gate + base + v);
@@ -242,8 +241,8 @@ template <int DK, int DV>
 int launch_prefill(const Prefill &p, cudaStream_t st)
 {
     const size_t smem = ((size_t)(BM + kStages * BN) * (DK + 8) + (size_t)kStages * BN * (DV + 8)) * 2;
-    if (int rc = allow_smem(latent_prefill_kernel<DK, DV>, smem)) return rc;
-    return launch(latent_prefill_kernel<DK, DV>, dim3(p.heads, (p.rows + BM - 1) / BM), dim3(kThreads), smem, st, p);
+    if (int rc = allow_smem(prefill_attention_kernel<DK, DV>, smem)) return rc;
+    return launch(prefill_attention_kernel<DK, DV>, dim3(p.heads, (p.rows + BM - 1) / BM, (p.vdim + DV - 1) / DV), dim3(kThreads), smem, st, p);
 }
 
 template <int DK>
@@ -253,13 +252,31 @@ int launch_prefill_v(const Prefill &p, cudaStream_t st)
     return launch_prefill<DK, 128>(p, st);
 }
 
+int launch_prefill_sized(const Prefill &p, cudaStream_t st)
+{
+    const uint32_t dk = p.dim + p.rot;
+    if (dk <= 64) return launch_prefill_v<64>(p, st);
+    if (dk <= 96) return launch_prefill_v<96>(p, st);
+    if (dk <= 128) return launch_prefill_v<128>(p, st);
+    if (dk <= 192) return launch_prefill_v<192>(p, st);
+    return launch_prefill_v<256>(p, st);
+}
+
+void set_output(Prefill &p, const HeadGate *gate, float *o)
+{
+    p.gate = gate ? gate->gate : nullptr;
+    p.out = gate ? gate->out : o;
+    p.out_bf16 = gate && gate->out_bf16;
+    p.silu = gate && gate->silu;
+}
+
 size_t align256(size_t n) { return (n + 255) & ~(size_t)255; }
 
 }  // namespace
 
 bool latent_prefill_eligible(uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t rank, bool cache_bf16)
 {
-    return cache_bf16 && dim % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 && rank % 8 == 0 && dim + rot_dim <= 256 && vdim <= 128;
+    return cache_bf16 && dim % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 && rank % 8 == 0 && dim + rot_dim <= 256;
 }
 
 size_t latent_prefill_workspace(uint32_t heads, uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t slots)
@@ -280,25 +297,32 @@ int launch_latent_prefill(const LatentAttention &a, void *stream)
     if (a.rot_dim)
         if (int rc = launch(rotated_half_kernel, dim3((uint32_t)(((size_t)a.slots * a.rot_dim + 255) / 256)), dim3(256), 0, st, cache, a.pos, rotated, a.rows, a.slots, a.rank, a.rot_dim)) return rc;
     LinearGroup g{};
-    g.count = 2; g.m = a.slots; g.k = a.rank; g.lda = a.rank + a.rot_dim;
+    g.count = 2; g.m = a.slots; g.lda = a.rank + a.rot_dim;
     g.a_bf16 = 1; g.out_f16 = 1; g.live = a.pos; g.live_add = a.rows;
     g.seg[0].a = g.seg[1].a = a.cache;
+    g.seg[0].k = g.seg[1].k = a.rank;
     g.seg[0].w = a.uk; g.seg[0].out = keys; g.seg[0].n = a.heads * a.dim;
     g.seg[1].w = a.uv; g.seg[1].out = values; g.seg[1].n = a.heads * a.vdim;
     if (int rc = launch_linear_tc(g, stream)) return rc;
     Prefill p{};
     p.q = a.q; p.freq = a.freq; p.keys = keys; p.values = values; p.rotated = rotated; p.pos = a.pos;
-    p.gate = a.gate ? a.gate->gate : nullptr;
-    p.out = a.gate ? a.gate->out : a.o;
-    p.rows = a.rows; p.heads = a.heads; p.dim = a.dim; p.rot = a.rot_dim; p.vdim = a.vdim; p.rank = a.rank; p.slots = a.slots; p.window = a.window;
+    set_output(p, a.gate, a.o);
+    p.rows = a.rows; p.heads = p.kv_heads = a.heads; p.dim = a.dim; p.rot = a.rot_dim; p.vdim = a.vdim; p.slots = a.slots; p.window = a.window;
     p.scale_log2 = a.scale * 1.4426950408889634f;
-    p.out_bf16 = a.gate && a.gate->out_bf16; p.silu = a.gate && a.gate->silu;
-    const uint32_t dk = a.dim + a.rot_dim;
-    if (dk <= 64) return launch_prefill_v<64>(p, st);
-    if (dk <= 96) return launch_prefill_v<96>(p, st);
-    if (dk <= 128) return launch_prefill_v<128>(p, st);
-    if (dk <= 192) return launch_prefill_v<192>(p, st);
-    return launch_prefill_v<256>(p, st);
+    return launch_prefill_sized(p, st);
+}
+
+bool attention_prefill_eligible(const Attention &a) { return a.half && a.rows >= kPrefillRows && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.dim <= 256; }
+
+int launch_attention_prefill(const Attention &a, void *stream)
+{
+    Prefill p{};
+    p.q = a.q; p.keys = static_cast<const __half *>(a.keys); p.values = static_cast<const __half *>(a.values); p.pos = a.pos;
+    set_output(p, a.gate, a.o);
+    p.rows = a.rows; p.heads = a.heads; p.kv_heads = a.kv_heads; p.dim = a.dim; p.vdim = a.vdim; p.slots = a.slots;
+    p.window = 1u << 30;                                 // no position is that far away
+    p.scale_log2 = a.scale * 1.4426950408889634f;
+    return launch_prefill_sized(p, static_cast<cudaStream_t>(stream));
 }
 
 }  // namespace mgq

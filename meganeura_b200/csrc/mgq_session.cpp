@@ -25,9 +25,9 @@
 // no host round trip.  (4) Row-dynamic graphs: activations whose leading dimension is a capacity
 // (input_u32_rows) run with the row count set by mgq_session_set_rows, so one session serves both a
 // prompt's portions and single-token steps; a captured CUDA graph is replayed for the row counts it
-// was captured with.  (5) Recurrent mixers (token shift, RWKV-style time mixing, mLSTM), latent
-// attention over a ring cache, clamped GLUs and bf16 linear layers, with their state in zero-filled
-// parameters that mgq_session_reset_state clears.
+// was captured with.  (5) Recurrent mixers (token shift, RWKV-style time mixing, mLSTM, gated linear
+// attention), latent attention over a ring cache, softmax attention over grouped key / value heads, GLUs
+// and bf16 linear layers, with recurrent state in zero-filled parameters that mgq_session_reset_state clears.
 #include <cuda_runtime.h>
 #include <nvtx3/nvToolsExt.h>
 
@@ -49,7 +49,8 @@ constexpr int kU32 = 100;         // node dtype of input_u32 (not a weight forma
 enum class Op {
     Input, Parameter, MatMul, Add, FusedMatMulAdd, Embedding, RmsNorm, RoPE, CacheWrite, CachedAttention,
     SwiGLU, SwiGLUConcat, AllGather, MatMulBT, View, Nop,
-    BiasAdd, PickRows, Norm, TokenShift, Slot, Decay, Wkv, Mlstm, HeadGate, LatentCacheWrite, LatentAttention, ClampedGlu, LinearGlu
+    BiasAdd, PickRows, Norm, TokenShift, Slot, Decay, Wkv, Mlstm, HeadGate, LatentCacheWrite, LatentAttention, Glu, LinearGlu,
+    Cast, ScaledSum, ResidualNorm, Gla, QueryTemperature, CacheAppend, Attention
 };
 
 struct Node {
@@ -59,10 +60,11 @@ struct Node {
     int dtype;                    // MGQ_FMT_F32 / Q4 / Q8, or kU32
     std::vector<int> inputs;
     float f0 = 0.f;               // eps (RmsNorm), theta (RoPE)
-    float f1 = 0.f, f2 = 0.f;
+    float f1 = 0.f, f2 = 0.f, f3 = 0.f;
     int rows = 0;                 // leading dimension: 0 fixed, MGQ_ROWS_TOKENS / MGQ_ROWS_PICKED: set per step
     std::vector<uint32_t> at = {};     // integer attributes of the recurrent and latent operators
     bool absorbed = false;        // runs inside the dispatch of its consumer (keeps its buffer)
+    int copy = -1;                // Embedding, ResidualNorm: the Cast node whose bf16 copy this dispatch writes too
     uint32_t u0 = 0, u1 = 0, u2 = 0;   // head_dim (RoPE); num_heads, num_kv_heads, head_dim (CachedAttention); column offset (View)
     size_t elements() const { size_t e = 1; for (size_t s : shape) e *= s; return e; }
 };
@@ -132,6 +134,14 @@ const char *shader_name(int s)
         case MGQ_SHADER_LATENT_CACHE_WRITE: return "LatentCacheWrite";
         case MGQ_SHADER_LATENT_ATTENTION: return "LatentAttention";
         case MGQ_SHADER_CLAMPED_GLU: return "ClampedGLU";
+        case MGQ_SHADER_CAST: return "Cast";
+        case MGQ_SHADER_SCALED_SUM: return "ScaledSum";
+        case MGQ_SHADER_RESIDUAL_NORM: return "ResidualNorm";
+        case MGQ_SHADER_GLA: return "Gla";
+        case MGQ_SHADER_QUERY_TEMPERATURE: return "QueryTemperature";
+        case MGQ_SHADER_CACHE_APPEND: return "CacheAppend";
+        case MGQ_SHADER_ATTENTION: return "Attention";
+        case MGQ_SHADER_ATTENTION_INPUTS: return "AttentionInputs";
     }
     return "?";
 }
@@ -445,7 +455,7 @@ int mgq_graph_all_gather(mgq_graph *g, int x, uint32_t world)
 
 }  // extern "C"
 
-// ---- operators of decoders with recurrent and latent-attention mixers
+// ---- operators of decoders with recurrent, softmax- and latent-attention mixers
 namespace {
 
 bool is_param(const mgq_graph *g, int id, int dtype, size_t elements)
@@ -482,6 +492,40 @@ int mgq_graph_embedding_scaled(mgq_graph *g, int indices, int table, float scale
     nd.u0 = 1;                            // scaled form
     nd.rows = ni.rows;
     return push_node(g, std::move(nd));
+}
+
+int mgq_graph_embedding_positions(mgq_graph *g, int indices, int table, int pos, float scale, float base)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!valid(g, pos)) return -fail(MGQ_ERR_NAME, "embedding: node id out of range");
+    if (g->nodes[pos].dtype != kU32) return -fail(MGQ_ERR_FORMAT, "pos must be a U32 input");
+    if (!(base > 0.f)) return -fail(MGQ_ERR_SHAPE, "embedding: the base of the positions must be positive");
+    const int id = mgq_graph_embedding_scaled(g, indices, table, scale);
+    if (id < 0) return id;
+    g->nodes[id].inputs.push_back(pos);
+    g->nodes[id].f1 = base;
+    return id;
+}
+
+int mgq_graph_cast(mgq_graph *g, int x, int out_dtype)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!valid(g, x)) return -fail(MGQ_ERR_NAME, "cast: node id out of range");
+    const Node &nx = g->nodes[x];
+    if (nx.shape.size() != 2 || nx.dtype != MGQ_FMT_F32 || out_dtype != MGQ_FMT_BF16) return -fail(MGQ_ERR_FORMAT, "cast turns a 2D f32 tensor into bf16");
+    Node nd{Op::Cast, "", nx.shape, MGQ_FMT_BF16, {x}};
+    nd.rows = nx.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_scaled_sum(mgq_graph *g, int a, int b, float sa, float sb)
+{
+    const int id = mgq_graph_add(g, a, b);
+    if (id < 0) return id;
+    if (g->nodes[id].shape.size() != 2) return -fail(MGQ_ERR_SHAPE, "scaled_sum takes 2D tensors");
+    g->nodes[id].op = Op::ScaledSum;
+    g->nodes[id].f0 = sa; g->nodes[id].f1 = sb;
+    return id;
 }
 
 int mgq_graph_pick_rows(mgq_graph *g, int x, int index)
@@ -522,18 +566,20 @@ int mgq_graph_bias_add(mgq_graph *g, int x, int bias)
     return push_node(g, std::move(nd));
 }
 
-int mgq_graph_clamped_glu(mgq_graph *g, int gate, int up, float limit, float alpha, int out_dtype)
+static int glu_node(mgq_graph *g, int gate, int up, const mgq::Glu &act, int out_dtype)
 {
     if (!g) return -fail(MGQ_ERR_NULL, "null graph");
-    if (!all_valid(g, {gate, up})) return -fail(MGQ_ERR_NAME, "clamped_glu: node id out of range");
+    if (!all_valid(g, {gate, up})) return -fail(MGQ_ERR_NAME, "glu: node id out of range");
     const Node &ng = g->nodes[gate], &nu = g->nodes[up];
-    if (ng.shape.size() != 2 || ng.shape != nu.shape || ng.rows != nu.rows) return -fail(MGQ_ERR_SHAPE, "clamped_glu: shapes differ");
-    if (ng.dtype != MGQ_FMT_F32 || nu.dtype != MGQ_FMT_F32 || !operand_dtype(out_dtype)) return -fail(MGQ_ERR_FORMAT, "clamped_glu: f32 operands, f32 or bf16 output");
-    Node nd{Op::ClampedGlu, "", ng.shape, out_dtype, {gate, up}};
-    nd.f0 = limit; nd.f1 = alpha;
+    if (ng.shape.size() != 2 || ng.shape != nu.shape || ng.rows != nu.rows) return -fail(MGQ_ERR_SHAPE, "glu: shapes differ");
+    if (ng.dtype != MGQ_FMT_F32 || nu.dtype != MGQ_FMT_F32 || !operand_dtype(out_dtype)) return -fail(MGQ_ERR_FORMAT, "glu: f32 operands, f32 or bf16 output");
+    Node nd{Op::Glu, "", ng.shape, out_dtype, {gate, up}};
+    nd.f0 = act.limit; nd.f1 = act.alpha; nd.f2 = act.offset;
     nd.rows = ng.rows;
     return push_node(g, std::move(nd));
 }
+int mgq_graph_clamped_glu(mgq_graph *g, int gate, int up, float limit, float alpha, int out_dtype) { return glu_node(g, gate, up, {limit, alpha, 1.f}, out_dtype); }
+int mgq_graph_silu_glu(mgq_graph *g, int gate, int up, int out_dtype) { return glu_node(g, gate, up, {INFINITY, 1.f, 0.f}, out_dtype); }
 
 int mgq_graph_token_shift(mgq_graph *g, int h, const int *mu, size_t count, int state, int out_dtype)
 {
@@ -565,7 +611,8 @@ int mgq_graph_slot(mgq_graph *g, int x, uint32_t index)
     return push_node(g, std::move(nd));
 }
 
-size_t mgq_wkv_state_elements(uint32_t heads, uint32_t dim) { return mgq::wkv_state_elements(heads, dim); }
+size_t mgq_wkv_state_elements(uint32_t heads, uint32_t dim) { return mgq::channel_decay_state_elements(heads, dim, dim); }
+size_t mgq_gla_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim) { return mgq::channel_decay_state_elements(heads, dim, vdim); }
 size_t mgq_mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim) { return mgq::mlstm_state_elements(heads, dim, vdim); }
 
 int mgq_graph_lora_decay(mgq_graph *g, int low, int w2, int w0)
@@ -581,6 +628,32 @@ int mgq_graph_lora_decay(mgq_graph *g, int low, int w2, int w0)
     return push_node(g, std::move(nd));
 }
 
+int mgq_graph_lora_sigmoid_decay(mgq_graph *g, int low, int w2, int bias, float tau)
+{
+    if (!(tau > 0.f)) return -fail(MGQ_ERR_SHAPE, "lora_sigmoid_decay: tau must be positive");
+    const int id = mgq_graph_lora_decay(g, low, w2, bias);
+    if (id >= 0) g->nodes[id].f0 = (float)(1.0 / (double)tau);
+    return id;
+}
+
+int mgq_graph_gla(mgq_graph *g, int q, int k, int v, int decay, int state, uint32_t heads)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {q, k, v, decay, state})) return -fail(MGQ_ERR_NAME, "gla: node id out of range");
+    const Node &nq = g->nodes[q], &nv = g->nodes[v];
+    if (nq.shape.size() != 2 || nv.shape.size() != 2 || heads == 0 || nq.shape[1] % heads || nv.shape[1] % heads) return -fail(MGQ_ERR_SHAPE, "gla: widths do not divide over %u heads", heads);
+    const uint32_t dim = (uint32_t)(nq.shape[1] / heads), vdim = (uint32_t)(nv.shape[1] / heads);
+    if (dim > mgq::kMaxStateDim) return -fail(MGQ_ERR_SHAPE, "gla: heads of %u key dimensions (at most %u)", dim, mgq::kMaxStateDim);
+    for (int id : {q, k, decay})
+        if (!is_act(g, id, nq.shape[0], nq.shape[1], nq.rows)) return -fail(MGQ_ERR_SHAPE, "gla: q, k and the decay must be f32 of one shape");
+    if (!is_act(g, v, nq.shape[0], nv.shape[1], nq.rows)) return -fail(MGQ_ERR_SHAPE, "gla: v must be f32 rows like q");
+    if (!is_param(g, state, MGQ_FMT_F32, mgq_gla_state_elements(heads, dim, vdim))) return -fail(MGQ_ERR_SHAPE, "gla: state must be an f32 parameter of %zu elements", mgq_gla_state_elements(heads, dim, vdim));
+    Node nd{Op::Gla, "", nv.shape, MGQ_FMT_F32, {q, k, v, decay, -1, state, -1}};         // laid out like Wkv
+    nd.at = {heads, dim, vdim};
+    nd.rows = nq.rows;
+    return push_node(g, std::move(nd));
+}
+
 int mgq_graph_wkv(mgq_graph *g, int r, int k, int v, int decay, int u, int state, int shift_state, uint32_t heads)
 {
     if (!g) return -fail(MGQ_ERR_NULL, "null graph");
@@ -592,10 +665,10 @@ int mgq_graph_wkv(mgq_graph *g, int r, int k, int v, int decay, int u, int state
     for (int id : {r, k, v, decay})
         if (!is_act(g, id, nr.shape[0], nr.shape[1], nr.rows)) return -fail(MGQ_ERR_SHAPE, "wkv: r, k, v and the decay must be f32 of one shape");
     if (!is_param(g, u, MGQ_FMT_F32, nr.shape[1])) return -fail(MGQ_ERR_SHAPE, "wkv: u must be an f32 parameter of %zu elements", nr.shape[1]);
-    if (!is_param(g, state, MGQ_FMT_F32, mgq::wkv_state_elements(heads, dim))) return -fail(MGQ_ERR_SHAPE, "wkv: state must be an f32 parameter of %zu elements", mgq::wkv_state_elements(heads, dim));
+    if (!is_param(g, state, MGQ_FMT_F32, mgq_wkv_state_elements(heads, dim))) return -fail(MGQ_ERR_SHAPE, "wkv: state must be an f32 parameter of %zu elements", mgq_wkv_state_elements(heads, dim));
     if (shift_state >= 0 && !is_param(g, shift_state, MGQ_FMT_F32, 0)) return -fail(MGQ_ERR_SHAPE, "wkv: the shift state must be an f32 parameter");
     Node nd{Op::Wkv, "", nr.shape, MGQ_FMT_F32, {r, k, v, decay, u, state, shift_state}};
-    nd.at = {heads, dim};
+    nd.at = {heads, dim, dim};
     nd.rows = nr.rows;
     return push_node(g, std::move(nd));
 }
@@ -627,7 +700,8 @@ int mgq_graph_head_gate(mgq_graph *g, int o, int weight, int gate, uint32_t head
     const Node &no = g->nodes[o];
     if (no.shape.size() != 2 || heads == 0 || no.shape[1] % heads) return -fail(MGQ_ERR_SHAPE, "head_gate: width does not divide over %u heads", heads);
     if (!is_act(g, o, no.shape[0], no.shape[1], no.rows) || !is_act(g, gate, no.shape[0], no.shape[1], no.rows)) return -fail(MGQ_ERR_SHAPE, "head_gate: the gate must have the shape of its input");
-    if (weight >= 0 && !is_param(g, weight, MGQ_FMT_F32, no.shape[1])) return -fail(MGQ_ERR_SHAPE, "head_gate: weight must be an f32 parameter of %zu elements", no.shape[1]);
+    if (weight >= 0 && !is_param(g, weight, MGQ_FMT_F32, no.shape[1]) && !is_param(g, weight, MGQ_FMT_F32, no.shape[1] / heads))
+        return -fail(MGQ_ERR_SHAPE, "head_gate: weight must be an f32 parameter of %zu or %zu elements", no.shape[1], no.shape[1] / heads);
     if (act != MGQ_GATE_SIGMOID && act != MGQ_GATE_SILU) return -fail(MGQ_ERR_FORMAT, "head_gate: unknown activation %d", act);
     if (!operand_dtype(out_dtype)) return -fail(MGQ_ERR_FORMAT, "head_gate: output must be f32 or bf16");
     Node nd{Op::HeadGate, "", no.shape, out_dtype, {o, gate, weight}};
@@ -672,6 +746,51 @@ int mgq_graph_latent_attention(mgq_graph *g, int q, int cache, int uk, int uv, i
     Node nd{Op::LatentAttention, "", {nq.shape[0], (size_t)heads * vdim}, MGQ_FMT_F32, {q, cache, uk, uv, pos}};
     nd.f0 = scale; nd.f1 = rot_base;
     nd.at = {heads, dim, rot_dim, vdim, (uint32_t)rank, (uint32_t)nc.shape[0], window};
+    nd.rows = nq.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_query_temperature(mgq_graph *g, int x, int pos, float coef, float every)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {x, pos})) return -fail(MGQ_ERR_NAME, "query_temperature: node id out of range");
+    const Node &nx = g->nodes[x];
+    if (nx.shape.size() != 2 || nx.dtype != MGQ_FMT_F32) return -fail(MGQ_ERR_SHAPE, "query_temperature takes a 2D f32 tensor");
+    if (g->nodes[pos].dtype != kU32) return -fail(MGQ_ERR_FORMAT, "pos must be a U32 input");
+    if (!(every > 0.f)) return -fail(MGQ_ERR_SHAPE, "query_temperature: the step must be positive");
+    Node nd{Op::QueryTemperature, "", nx.shape, MGQ_FMT_F32, {x, pos}};
+    nd.f0 = coef; nd.f1 = every;
+    nd.rows = nx.rows;
+    return push_node(g, std::move(nd));
+}
+
+int mgq_graph_cache_append(mgq_graph *g, int x, int cache, int pos)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {x, cache, pos})) return -fail(MGQ_ERR_NAME, "cache_append: node id out of range");
+    const Node &nx = g->nodes[x], &nc = g->nodes[cache];
+    if (nx.shape.size() != 2 || nx.dtype != MGQ_FMT_F32) return -fail(MGQ_ERR_SHAPE, "cache_append takes a 2D f32 tensor");
+    if (nc.op != Op::Parameter || (nc.dtype != MGQ_FMT_F32 && nc.dtype != MGQ_FMT_F16) || nc.shape.size() != 2 || nc.shape[1] != nx.shape[1])
+        return -fail(MGQ_ERR_SHAPE, "cache_append: the cache must be an f32 or f16 parameter [slots, %zu]", nx.shape[1]);
+    if (g->nodes[pos].dtype != kU32) return -fail(MGQ_ERR_FORMAT, "pos must be a U32 input");
+    return push_node(g, Node{Op::CacheAppend, "", nc.shape, nc.dtype, {x, cache, pos}});
+}
+
+int mgq_graph_attention(mgq_graph *g, int q, int k_cache, int v_cache, int pos, uint32_t heads, uint32_t kv_heads, uint32_t dim, uint32_t vdim, float scale)
+{
+    if (!g) return -fail(MGQ_ERR_NULL, "null graph");
+    if (!all_valid(g, {q, k_cache, v_cache, pos})) return -fail(MGQ_ERR_NAME, "attention: node id out of range");
+    const Node &nq = g->nodes[q], &nk = g->nodes[k_cache], &nv = g->nodes[v_cache];
+    if (kv_heads == 0 || heads == 0 || heads % kv_heads || dim == 0 || vdim == 0) return -fail(MGQ_ERR_SHAPE, "attention: %u heads do not divide over %u key / value heads", heads, kv_heads);
+    if (nq.shape.size() != 2 || nq.dtype != MGQ_FMT_F32 || nq.shape[1] != (size_t)heads * dim) return -fail(MGQ_ERR_SHAPE, "attention: q must be f32 rows of heads * dim");
+    if ((nk.dtype != MGQ_FMT_F32 && nk.dtype != MGQ_FMT_F16) || nv.dtype != nk.dtype || nk.shape.size() != 2 || nv.shape.size() != 2 || nk.shape[0] != nv.shape[0] ||
+        nk.shape[1] != (size_t)kv_heads * dim || nv.shape[1] != (size_t)kv_heads * vdim)
+        return -fail(MGQ_ERR_SHAPE, "attention: the caches must be [slots, kv_heads * dim] and [slots, kv_heads * vdim], f32 or f16");
+    if (nk.shape[0] < nq.shape[0]) return -fail(MGQ_ERR_SHAPE, "attention: %zu cache rows for %zu tokens", nk.shape[0], nq.shape[0]);
+    if (g->nodes[pos].dtype != kU32) return -fail(MGQ_ERR_FORMAT, "pos must be a U32 input");
+    Node nd{Op::Attention, "", {nq.shape[0], (size_t)heads * vdim}, MGQ_FMT_F32, {q, k_cache, v_cache, pos}};
+    nd.f0 = scale;
+    nd.at = {heads, kv_heads, dim, vdim, (uint32_t)nk.shape[0]};
     nd.rows = nq.rows;
     return push_node(g, std::move(nd));
 }
@@ -824,7 +943,43 @@ void merge_rope_cache(mgq_session *s)
     }
 }
 
-// Producer-consumer merges of the recurrent / latent operators.  A merged producer turns into Nop, or
+// Norm(q), Norm(k), QueryTemperature, CacheAppend(k), CacheAppend(v) in a row, as an attention layer builds
+// them, become one dispatch; the normed q and k have no other reader.
+void merge_attention_inputs(mgq_session *s)
+{
+    std::vector<Dispatch> &ds = s->dispatches;
+    auto plain_norm = [&](const Dispatch &d) {
+        if (d.shader != MGQ_SHADER_NORM) return false;
+        const Node &nd = s->nodes[d.out];
+        return nd.dtype == MGQ_FMT_F32 && nd.inputs[2] < 0;
+    };
+    auto uses = [&](int id) {
+        int n = 0;
+        for (const Node &nd : s->nodes)
+            for (int in : nd.inputs) n += in == id;
+        for (int o : s->outputs) n += o == id;
+        return n;
+    };
+    for (size_t i = 0; i + 4 < ds.size(); i++) {
+        const Dispatch &qn = ds[i], &kn = ds[i + 1], &qt = ds[i + 2], &kc = ds[i + 3], &vc = ds[i + 4];
+        if (!plain_norm(qn) || !plain_norm(kn) || qt.shader != MGQ_SHADER_QUERY_TEMPERATURE || kc.shader != MGQ_SHADER_CACHE_APPEND ||
+            vc.shader != MGQ_SHADER_CACHE_APPEND) continue;
+        if (qt.in[0] != qn.out || kc.in[0] != kn.out || qt.in[1] != kc.in[2] || qt.in[1] != vc.in[2]) continue;
+        if (uses(qn.out) != 1 || uses(kn.out) != 1) continue;
+        const Node &cache_k = s->nodes[kc.in[1]], &cache_v = s->nodes[vc.in[1]];
+        if (cache_k.dtype != cache_v.dtype || cache_k.shape[0] != cache_v.shape[0]) continue;
+        Dispatch m = qt;
+        m.shader = MGQ_SHADER_ATTENTION_INPUTS;
+        m.members = {qn.out, kn.out, kc.out, vc.out};
+        char lab[96];
+        std::snprintf(lab, sizeof lab, "AttentionInputs[q%zu k%zu v%zu]", s->nodes[qn.out].shape[1], cache_k.shape[1], cache_v.shape[1]);
+        m.label = lab;
+        ds[i] = m;
+        ds.erase(ds.begin() + i + 1, ds.begin() + i + 5);
+    }
+}
+
+// Producer-consumer merges of the recurrent / attention operators.  A merged producer turns into Nop, or
 // stays "absorbed" when its consumer's dispatch still needs its buffer.
 void fuse_mixers(mgq_session *s)
 {
@@ -845,15 +1000,41 @@ void fuse_mixers(mgq_session *s)
             int mm = -1, addend = -1;
             for (int side = 0; side < 2 && mm < 0; side++)
                 if (linear(nd.inputs[side]) && single(nd.inputs[side]) && nodes[nd.inputs[side]].inputs[3] < 0) { mm = nd.inputs[side]; addend = nd.inputs[1 - side]; }
-            if (mm < 0 || mm == addend) continue;
-            nd.op = Op::MatMulBT;
-            nd.inputs = {nodes[mm].inputs[0], nodes[mm].inputs[1], nodes[mm].inputs[2], addend};
-            drop(mm);
-        } else if (nd.op == Op::ClampedGlu) {
+            if (mm >= 0) {
+                if (mm == addend) continue;
+                nd.op = Op::MatMulBT;
+                nd.inputs = {nodes[mm].inputs[0], nodes[mm].inputs[1], nodes[mm].inputs[2], addend};
+                drop(mm);
+                continue;
+            }
+            for (int side = 0; side < 2; side++) {           // a sublayer's norm and the residual, with the sum in front of the norm
+                const int nm = nd.inputs[side];
+                if (nodes[nm].op != Op::Norm || nodes[nm].dtype != MGQ_FMT_F32 || nodes[nm].inputs[2] >= 0 || nodes[nm].shape.size() != 2 || !single(nm)) continue;
+                int a = nodes[nm].inputs[0], b = -1;
+                float sa = 1.f, sb = 0.f;
+                if (nodes[a].op == Op::ScaledSum && single(a)) {
+                    const int sum = a;
+                    a = nodes[sum].inputs[0]; b = nodes[sum].inputs[1]; sa = nodes[sum].f0; sb = nodes[sum].f1;
+                    drop(sum);
+                }
+                const int residual = nd.inputs[1 - side];
+                nd.op = Op::ResidualNorm;
+                nd.inputs = {a, b, nodes[nm].inputs[1], residual};
+                nd.f0 = nodes[nm].f0; nd.f1 = nodes[nm].f1; nd.f2 = sa; nd.f3 = sb;
+                drop(nm);
+                break;
+            }
+        } else if (nd.op == Op::Cast) {
+            Node &x = nodes[nd.inputs[0]];
+            if ((x.op == Op::ResidualNorm || (x.op == Op::Embedding && x.u0)) && x.copy < 0) {
+                x.copy = (int)id;
+                nd.absorbed = true;
+            }
+        } else if (nd.op == Op::Glu) {
             const int ga = nd.inputs[0], up = nd.inputs[1];
             if (ga == up || !linear(ga) || !linear(up) || !single(ga) || !single(up)) continue;
             const std::vector<int> &a = nodes[ga].inputs, &b = nodes[up].inputs;
-            if (a[0] != b[0] || a[2] < 0 || b[2] < 0 || a[3] >= 0 || b[3] >= 0) continue;
+            if (a[0] != b[0] || (a[2] < 0) != (b[2] < 0) || a[3] >= 0 || b[3] >= 0) continue;
             nd.op = Op::LinearGlu;
             nd.inputs = {a[0], a[1], a[2], b[1], b[2]};
             drop(ga);
@@ -874,19 +1055,19 @@ void fuse_mixers(mgq_session *s)
             const int o = nd.inputs[0];
             const Op producer = nodes[o].op;
             if (!single(o) || nodes[o].rows != nd.rows) continue;
-            const bool recurrent = producer == Op::Wkv || producer == Op::Mlstm;
+            const bool recurrent = producer == Op::Wkv || producer == Op::Gla || producer == Op::Mlstm;
             if (recurrent && nd.inputs[2] >= 0 && nodes[o].at[0] == nd.at[0]) nodes[o].absorbed = true;
-            if (producer == Op::Wkv && nodes[o].absorbed) {
+            if ((producer == Op::Wkv || producer == Op::Gla) && nodes[o].absorbed) {
                 const int w = nodes[o].inputs[3];
                 if (nodes[w].op == Op::Decay && single(w)) nodes[w].absorbed = true;
                 else nodes[o].absorbed = false;
             }
-            if (producer == Op::LatentAttention && nd.inputs[2] < 0) nodes[o].absorbed = true;
+            if ((producer == Op::LatentAttention || producer == Op::Attention) && nd.inputs[2] < 0) nodes[o].absorbed = true;
         }
     }
 }
 
-// Consecutive independent bf16 linear layers of one K, row set and activation type form one dispatch.
+// Consecutive independent bf16 linear layers of one row set and activation type form one dispatch.
 void group_linears(mgq_session *s)
 {
     std::vector<Dispatch> &ds = s->dispatches;
@@ -896,8 +1077,7 @@ void group_linears(mgq_session *s)
         bool merge = a.shader == MGQ_SHADER_LINEAR && b.shader == MGQ_SHADER_LINEAR && a.members.size() + b.members.size() <= mgq::kMaxSegments;
         if (merge) {
             const Node &na = s->nodes[a.members[0]], &nb = s->nodes[b.members[0]];
-            merge = s->nodes[na.inputs[1]].shape[1] == s->nodes[nb.inputs[1]].shape[1] && na.rows == nb.rows && na.shape[0] == nb.shape[0] &&
-                    s->nodes[na.inputs[0]].dtype == s->nodes[nb.inputs[0]].dtype;
+            merge = na.rows == nb.rows && na.shape[0] == nb.shape[0] && s->nodes[na.inputs[0]].dtype == s->nodes[nb.inputs[0]].dtype;
             for (int m : a.members) merge = merge && nb.inputs[0] != m && nb.inputs[3] != m;
         }
         if (!merge) { i++; continue; }
@@ -926,6 +1106,29 @@ int rotation_table(mgq_session *s, uint32_t dims, float base, Dispatch &d)
     if (int rc = mgq_buffer_create(freq.size() * 4, &d.workspace)) return rc;
     s->workspaces.push_back(d.workspace);
     return mgq_buffer_upload(d.workspace, freq.data(), freq.size() * 4, s->stream);
+}
+
+// The same frequencies as sums of two f32 (embedding positions; an odd width ends with a sine).
+int sinusoid_table(mgq_session *s, uint32_t width, float base, Dispatch &d)
+{
+    std::vector<float> freq;
+    for (uint32_t i = 0; i < (width + 1) / 2; i++) {
+        const double f = std::pow((double)base, -2.0 * i / width);
+        freq.push_back((float)f);
+        freq.push_back((float)(f - (double)(float)f));
+    }
+    if (int rc = mgq_buffer_create(freq.size() * 4, &d.workspace)) return rc;
+    s->workspaces.push_back(d.workspace);
+    return mgq_buffer_upload(d.workspace, freq.data(), freq.size() * 4, s->stream);
+}
+
+int attention_scratch(mgq_session *s, const Node &nd, Dispatch &d)
+{
+    const std::vector<uint32_t> &a = nd.at;
+    const size_t bytes = mgq::attention_workspace((uint32_t)nd.shape[0], a[0], a[1], a[2], a[3], a[4], s->nodes[nd.inputs[1]].dtype == MGQ_FMT_F16);
+    if (int rc = mgq_buffer_create(bytes, &d.workspace)) return rc;
+    s->workspaces.push_back(d.workspace);
+    return MGQ_OK;
 }
 
 int recurrence_workspace(mgq_session *s, const Node &nd, Dispatch &d)
@@ -998,7 +1201,7 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
             s->node_offset[id] = s->node_offset[nd.inputs[2]];
             continue;
         }
-        if (nd.op == Op::CacheWrite) {
+        if (nd.op == Op::CacheWrite || nd.op == Op::CacheAppend) {
             s->node_buffer[id] = s->node_buffer[nd.inputs[1]];
             s->node_offset[id] = s->node_offset[nd.inputs[1]];
             continue;
@@ -1089,6 +1292,10 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
                 d.workgroups[0] = (seq * hidden + 255) / 256;
                 d.params[0] = seq; d.params[1] = hidden; d.params[2] = (uint32_t)s->nodes[nd.inputs[1]].shape[0];
                 set_label(d, "Embedding[%ux%u]", seq, hidden);
+                if (nd.u0 && nd.inputs.size() > 2) {
+                    rc = sinusoid_table(s, hidden, nd.f1, d);
+                    if (rc) { mgq_session_free(s); return rc; }
+                }
                 break;
             }
             case Op::RmsNorm: {
@@ -1187,8 +1394,14 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
             }
             case Op::BiasAdd:
             case Op::PickRows:
-            case Op::ClampedGlu: {
-                d.shader = nd.op == Op::BiasAdd ? MGQ_SHADER_BIAS_ADD : nd.op == Op::PickRows ? MGQ_SHADER_PICK_ROWS : MGQ_SHADER_CLAMPED_GLU;
+            case Op::Glu:
+            case Op::Cast:
+            case Op::ScaledSum:
+            case Op::ResidualNorm:
+            case Op::QueryTemperature: {
+                d.shader = nd.op == Op::BiasAdd ? MGQ_SHADER_BIAS_ADD : nd.op == Op::PickRows ? MGQ_SHADER_PICK_ROWS : nd.op == Op::Glu ? MGQ_SHADER_CLAMPED_GLU
+                         : nd.op == Op::Cast ? MGQ_SHADER_CAST : nd.op == Op::ScaledSum ? MGQ_SHADER_SCALED_SUM
+                         : nd.op == Op::ResidualNorm ? MGQ_SHADER_RESIDUAL_NORM : MGQ_SHADER_QUERY_TEMPERATURE;
                 d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = (uint32_t)nd.shape[1];
                 set_label(d, "%s[%u]", shader_name(d.shader), d.params[1]);
                 break;
@@ -1212,10 +1425,25 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
                 set_label(d, "Decay[%u]", d.params[1]);
                 break;
             }
-            case Op::Wkv: {
-                d.shader = MGQ_SHADER_WKV;
-                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = nd.at[1];
-                set_label(d, "Wkv[%ux%u]", nd.at[0], nd.at[1]);
+            case Op::CacheAppend: {
+                d.shader = MGQ_SHADER_CACHE_APPEND;
+                d.params[0] = (uint32_t)s->nodes[nd.inputs[0]].shape[0]; d.params[1] = (uint32_t)nd.shape[1]; d.params[2] = (uint32_t)nd.shape[0];
+                set_label(d, "CacheAppend[%u]", d.params[1]);
+                break;
+            }
+            case Op::Attention: {
+                d.shader = MGQ_SHADER_ATTENTION;
+                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = nd.at[2]; d.params[3] = nd.at[3];
+                set_label(d, "Attention[%u/%ux%u+%u]", nd.at[0], nd.at[1], nd.at[2], nd.at[3]);
+                rc = attention_scratch(s, nd, d);
+                if (rc) { mgq_session_free(s); return rc; }
+                break;
+            }
+            case Op::Wkv:
+            case Op::Gla: {
+                d.shader = nd.op == Op::Wkv ? MGQ_SHADER_WKV : MGQ_SHADER_GLA;
+                d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = nd.at[1]; d.params[3] = nd.at[2];
+                set_label(d, nd.op == Op::Wkv ? "Wkv[%ux%u]" : "Gla[%ux%ux%u]", nd.at[0], nd.at[1], nd.at[2]);
                 s->states.push_back(nd.inputs[5]);
                 rc = recurrence_workspace(s, nd, d);
                 if (rc) { mgq_session_free(s); return rc; }
@@ -1232,13 +1460,14 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
             }
             case Op::HeadGate: {
                 const Node &o = s->nodes[nd.inputs[0]];
-                d.shader = o.absorbed && o.op == Op::Wkv ? MGQ_SHADER_WKV : o.absorbed && o.op == Op::Mlstm ? MGQ_SHADER_MLSTM
-                         : o.absorbed ? MGQ_SHADER_LATENT_ATTENTION : MGQ_SHADER_HEAD_GATE;
+                d.shader = !o.absorbed ? MGQ_SHADER_HEAD_GATE : o.op == Op::Wkv ? MGQ_SHADER_WKV : o.op == Op::Gla ? MGQ_SHADER_GLA
+                         : o.op == Op::Mlstm ? MGQ_SHADER_MLSTM : o.op == Op::Attention ? MGQ_SHADER_ATTENTION : MGQ_SHADER_LATENT_ATTENTION;
                 d.params[0] = (uint32_t)nd.shape[0]; d.params[1] = nd.at[0]; d.params[2] = (uint32_t)(nd.shape[1] / nd.at[0]);
+                if (o.absorbed && (o.op == Op::Gla || o.op == Op::Attention)) d.params[3] = o.at[o.op == Op::Gla ? 1 : 2];      // key dimensions
                 set_label(d, "%s%s[%ux%u]", o.absorbed ? shader_name(d.shader) : "", o.absorbed ? "+HeadGate" : "HeadGate", d.params[1], d.params[2]);
                 if (!o.absorbed) break;
-                if (o.op != Op::LatentAttention) s->states.push_back(o.inputs[5]);
-                rc = o.op == Op::LatentAttention ? latent_workspace(s, o, d) : recurrence_workspace(s, o, d);
+                if (o.op != Op::LatentAttention && o.op != Op::Attention) s->states.push_back(o.inputs[5]);
+                rc = o.op == Op::LatentAttention ? latent_workspace(s, o, d) : o.op == Op::Attention ? attention_scratch(s, o, d) : recurrence_workspace(s, o, d);
                 if (rc) { mgq_session_free(s); return rc; }
                 break;
             }
@@ -1264,11 +1493,17 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
         s->dispatches.push_back(d);
     }
     if (g_fuse_rope_cache) merge_rope_cache(s);
+    if (g_fuse_mixer) merge_attention_inputs(s);
     if (g_fuse_mixer) group_linears(s);
     for (Dispatch &d : s->dispatches) {
         if (d.shader != MGQ_SHADER_LINEAR) continue;
         uint32_t n = 0;
-        for (int m : d.members) n += (uint32_t)s->nodes[m].shape[1];
+        size_t weights = 0;
+        for (int m : d.members) {
+            n += (uint32_t)s->nodes[m].shape[1];
+            weights += s->nodes[s->nodes[m].inputs[1]].elements();
+        }
+        d.params[3] = (uint32_t)std::min<size_t>(weights, 0xFFFFFFFFu);
         d.params[0] = (uint32_t)s->nodes[d.out].shape[0]; d.params[1] = (uint32_t)s->nodes[s->nodes[d.out].inputs[1]].shape[1]; d.params[2] = n;
         set_label(d, "Linear[%ux%u]%s", n, d.params[1], s->nodes[d.members[0]].inputs[3] >= 0 ? "+Add" : "");
     }
@@ -1515,6 +1750,7 @@ static mgq::HeadGate head_gate_args(mgq_session *s, const Node &nd, int id)
     hg.out = s->ptr(id);
     hg.out_bf16 = nd.dtype == MGQ_FMT_BF16;
     hg.silu = nd.at[1] == MGQ_GATE_SILU;
+    hg.shared = nd.inputs[2] >= 0 && s->nodes[nd.inputs[2]].elements() != nd.shape[1];
     hg.eps = nd.f0;
     return hg;
 }
@@ -1535,7 +1771,7 @@ static int run_linear(mgq_session *s, const Dispatch &d)
         if (g.glu) {
             sg.w2 = s->ptr(nd.inputs[3]);
             sg.bias2 = f(4);
-            g.limit = nd.f0; g.alpha = nd.f1;
+            g.act = mgq::Glu{nd.f0, nd.f1, nd.f2};
             g.out_bf16 = nd.dtype == MGQ_FMT_BF16;
         } else {
             sg.addend = f(3);
@@ -1543,7 +1779,7 @@ static int run_linear(mgq_session *s, const Dispatch &d)
         sg.out = s->ptr(id);
         sg.n = (uint32_t)nd.shape[1];
         g.m = s->rows_of(id);
-        g.k = (uint32_t)s->nodes[nd.inputs[1]].shape[1];
+        sg.k = (uint32_t)s->nodes[nd.inputs[1]].shape[1];
         g.a_bf16 = s->bf16(nd.inputs[0]);
     }
     return mgq::launch_linear_group(g, s->stream);
@@ -1559,7 +1795,30 @@ static int run_mixer(mgq_session *s, const Dispatch &d)
     switch (nd.op) {
         case Op::BiasAdd: return mgq::launch_bias_add(f(nd.inputs[0]), f(nd.inputs[1]), f(d.out), rows, d.params[1], s->stream);
         case Op::PickRows: return mgq::launch_pick_rows(f(nd.inputs[0]), u(nd.inputs[1]), f(d.out), rows, s->rows_of(nd.inputs[0]), d.params[1], s->stream);
-        case Op::ClampedGlu: return mgq::launch_clamped_glu(f(nd.inputs[0]), f(nd.inputs[1]), s->ptr(d.out), s->bf16(d.out), (size_t)rows * d.params[1], nd.f0, nd.f1, s->stream);
+        case Op::Glu:
+            return mgq::launch_glu(f(nd.inputs[0]), f(nd.inputs[1]), s->ptr(d.out), s->bf16(d.out), (size_t)rows * d.params[1], {nd.f0, nd.f1, nd.f2}, s->stream);
+        case Op::Cast: return mgq::launch_cast(f(nd.inputs[0]), static_cast<__nv_bfloat16 *>(s->ptr(d.out)), (size_t)rows * d.params[1], s->stream);
+        case Op::ScaledSum: return mgq::launch_scaled_sum(f(nd.inputs[0]), f(nd.inputs[1]), f(d.out), (size_t)rows * d.params[1], nd.f0, nd.f1, s->stream);
+        case Op::ResidualNorm: {
+            mgq::ResidualNorm a{};
+            a.a = f(nd.inputs[0]); a.b = f(nd.inputs[1]); a.weight = f(nd.inputs[2]); a.addend = f(nd.inputs[3]);
+            a.out = f(d.out); a.copy = nd.copy >= 0 ? static_cast<__nv_bfloat16 *>(s->ptr(nd.copy)) : nullptr;
+            a.rows = rows; a.cols = d.params[1]; a.eps = nd.f0; a.offset = nd.f1; a.sa = nd.f2; a.sb = nd.f3;
+            return mgq::launch_residual_norm(a, s->stream);
+        }
+        case Op::QueryTemperature: {
+            if (d.shader == MGQ_SHADER_QUERY_TEMPERATURE) return mgq::launch_query_temperature(f(nd.inputs[0]), u(nd.inputs[1]), f(d.out), rows, d.params[1], nd.f0, nd.f1, s->stream);
+            const Node &qn = s->nodes[d.members[0]], &kn = s->nodes[d.members[1]], &kc = s->nodes[d.members[2]], &vc = s->nodes[d.members[3]];
+            mgq::AttentionInputs a{};
+            a.q = f(qn.inputs[0]); a.k = f(kn.inputs[0]); a.v = f(vc.inputs[0]); a.q_weight = f(qn.inputs[1]); a.k_weight = f(kn.inputs[1]);
+            a.pos = u(nd.inputs[1]); a.q_out = f(d.out); a.keys = s->ptr(kc.inputs[1]); a.values = s->ptr(vc.inputs[1]); a.half = kc.dtype == MGQ_FMT_F16;
+            a.rows = rows; a.q_cols = (uint32_t)qn.shape[1]; a.k_cols = (uint32_t)kc.shape[1]; a.v_cols = (uint32_t)vc.shape[1]; a.slots = (uint32_t)kc.shape[0];
+            a.q_eps = qn.f0; a.k_eps = kn.f0; a.q_offset = qn.f1; a.k_offset = kn.f1; a.coef = nd.f0; a.every = nd.f1;
+            return mgq::launch_attention_inputs(a, s->stream);
+        }
+        case Op::CacheAppend:
+            return mgq::launch_cache_append(f(nd.inputs[0]), s->ptr(nd.inputs[1]), nd.dtype == MGQ_FMT_F16, u(nd.inputs[2]), s->rows_of(nd.inputs[0]), d.params[1],
+                                            (uint32_t)nd.shape[0], s->stream);
         case Op::Norm:
             return mgq::launch_norm(f(nd.inputs[0]), f(nd.inputs[1]), u(nd.inputs[2]), s->ptr(d.out), s->bf16(d.out), rows, s->rows_of(nd.inputs[0]), d.params[1],
                                     nd.f0, nd.f1, s->stream);
@@ -1589,30 +1848,39 @@ static int run_mixer(mgq_session *s, const Dispatch &d)
     const bool fused = gated && oid != d.out;
     mgq::HeadGate hg{};
     if (gated) hg = head_gate_args(s, nd, d.out);
-    if (o.op == Op::Wkv || o.op == Op::Decay) {
-        mgq::Wkv a{};
+    if (o.op == Op::Wkv || o.op == Op::Gla || o.op == Op::Decay) {
+        mgq::ChannelDecay a{};
         const int did = o.op == Op::Decay ? oid : o.inputs[3];
         const Node &dn = s->nodes[did];
-        a.rows = rows;
+        a.rows = a.d.rows = rows;
         a.workspace = d.workspace;
-        a.decay = f(did);
+        a.d.out = f(did);
         if (dn.op == Op::Decay) {
-            a.low = f(dn.inputs[0]); a.w2 = s->ptr(dn.inputs[1]); a.w0 = f(dn.inputs[2]);
-            a.rank = (uint32_t)s->nodes[dn.inputs[0]].shape[1];
+            a.d.low = f(dn.inputs[0]); a.d.w2 = s->ptr(dn.inputs[1]); a.d.w0 = f(dn.inputs[2]);
+            a.d.rank = (uint32_t)s->nodes[dn.inputs[0]].shape[1];
+            a.d.channels = (uint32_t)dn.shape[1];
+            a.d.inv_tau = dn.f0;
         }
-        if (o.op == Op::Decay) {
-            a.heads = 1; a.dim = (uint32_t)dn.shape[1];
-            return mgq::launch_decay(a, s->stream);
-        }
-        a.r = f(o.inputs[0]); a.k = f(o.inputs[1]); a.v = f(o.inputs[2]); a.u = f(o.inputs[4]);
+        if (o.op == Op::Decay) return mgq::launch_decay(a.d, s->stream);
+        a.q = f(o.inputs[0]); a.k = f(o.inputs[1]); a.v = f(o.inputs[2]); a.u = f(o.inputs[4]);
         a.state = f(o.inputs[5]); a.shift_state = f(o.inputs[6]); a.o = f(oid);
-        a.heads = o.at[0]; a.dim = o.at[1];
+        a.heads = o.at[0]; a.dim = o.at[1]; a.vdim = o.at[2];
         a.shift_width = o.inputs[6] >= 0 ? (uint32_t)(s->nodes[o.inputs[6]].elements() / 2) : 0;
-        if (!fused) return mgq::launch_wkv_scan(a, s->stream);
-        if (rows == 1) return mgq::launch_wkv_step(a, hg, s->stream);
-        if (int rc = mgq::launch_decay(a, s->stream)) return rc;
-        if (int rc = mgq::launch_wkv_scan(a, s->stream)) return rc;
-        return mgq::launch_head_gate(a.o, hg, rows, o.at[0], o.at[1], s->stream);
+        if (!fused) return mgq::launch_channel_decay_scan(a, s->stream);
+        if (rows == 1) return mgq::launch_channel_decay_step(a, hg, s->stream);
+        if (int rc = mgq::launch_decay(a.d, s->stream)) return rc;
+        if (int rc = mgq::launch_channel_decay_scan(a, s->stream)) return rc;
+        return mgq::launch_head_gate(a.o, hg, rows, o.at[0], o.at[2], s->stream);
+    }
+    if (o.op == Op::Attention) {
+        mgq::Attention a{};
+        a.q = f(o.inputs[0]); a.keys = s->ptr(o.inputs[1]); a.values = s->ptr(o.inputs[2]); a.pos = u(o.inputs[3]); a.o = f(oid);
+        a.half = s->nodes[o.inputs[1]].dtype == MGQ_FMT_F16;
+        a.rows = rows; a.heads = o.at[0]; a.kv_heads = o.at[1]; a.dim = o.at[2]; a.vdim = o.at[3]; a.slots = o.at[4];
+        a.scale = o.f0;
+        a.workspace = d.workspace;
+        a.gate = fused ? &hg : nullptr;
+        return mgq::launch_attention(a, s->stream);
     }
     if (o.op == Op::Mlstm) {
         mgq::Mlstm a{};
@@ -1650,7 +1918,9 @@ static int run_dispatch(mgq_session *s, const Dispatch &d)
         case MGQ_SHADER_LINEAR_GLU: return run_linear(s, d);
         case MGQ_SHADER_BIAS_ADD: case MGQ_SHADER_PICK_ROWS: case MGQ_SHADER_NORM: case MGQ_SHADER_TOKEN_SHIFT: case MGQ_SHADER_DECAY:
         case MGQ_SHADER_WKV: case MGQ_SHADER_MLSTM: case MGQ_SHADER_HEAD_GATE: case MGQ_SHADER_LATENT_CACHE_WRITE:
-        case MGQ_SHADER_LATENT_ATTENTION: case MGQ_SHADER_CLAMPED_GLU: return run_mixer(s, d);
+        case MGQ_SHADER_LATENT_ATTENTION: case MGQ_SHADER_CLAMPED_GLU: case MGQ_SHADER_CAST: case MGQ_SHADER_SCALED_SUM: case MGQ_SHADER_RESIDUAL_NORM:
+        case MGQ_SHADER_GLA: case MGQ_SHADER_QUERY_TEMPERATURE: case MGQ_SHADER_CACHE_APPEND: case MGQ_SHADER_ATTENTION: case MGQ_SHADER_ATTENTION_INPUTS:
+            return run_mixer(s, d);
         case MGQ_SHADER_ADD:
             if (s->nodes[d.out].rows) {
                 const uint32_t len = s->rows_of(d.out) * (uint32_t)s->nodes[d.out].shape[1];
@@ -1662,8 +1932,15 @@ static int run_dispatch(mgq_session *s, const Dispatch &d)
             MGQ_CUDA(cudaGetLastError());
             return MGQ_OK;
         case MGQ_SHADER_EMBEDDING:
-            if (s->nodes[d.out].u0)
-                return mgq::launch_embedding_scaled(u(0), s->ptr(d.in[1]), s->bf16(d.in[1]), outp, s->rows_of(d.out), d.params[1], d.params[2], d.f0, s->stream);
+            if (s->nodes[d.out].u0) {
+                const Node &nd = s->nodes[d.out];
+                mgq::Embedding a{};
+                a.ids = u(0); a.table = s->ptr(d.in[1]); a.table_bf16 = s->bf16(d.in[1]); a.out = outp; a.scale = d.f0;
+                a.rows = s->rows_of(d.out); a.width = d.params[1]; a.vocab = d.params[2];
+                if (nd.inputs.size() > 2) { a.pos = u(2); a.sinusoid = static_cast<const float2 *>(d.workspace); }
+                if (nd.copy >= 0) a.copy = static_cast<__nv_bfloat16 *>(s->ptr(nd.copy));
+                return mgq::launch_embedding_scaled(a, s->stream);
+            }
             return mgq_embedding(u(0), f(1), outp, d.params[0], d.params[1], d.params[2], s->stream);
         case MGQ_SHADER_RMS_NORM: return mgq_rms_norm(f(0), f(1), outp, d.params[0], d.params[1], d.f0, s->stream);
         case MGQ_SHADER_ROPE_DYNAMIC: return mgq_rope_dynamic(f(0), outp, u(1), d.params[0], d.params[1], d.params[3], d.f0, s->stream);

@@ -45,6 +45,14 @@ class ShaderEntry(IntEnum):
     LatentCacheWrite = 25
     LatentAttention = 26
     ClampedGLU = 27
+    Cast = 28
+    ScaledSum = 29
+    ResidualNorm = 30
+    Gla = 31
+    QueryTemperature = 32
+    CacheAppend = 33
+    Attention = 34
+    AttentionInputs = 35
 
 
 class WeightFormat(IntEnum):
@@ -139,7 +147,7 @@ class Graph:
         """Graph::matmul_bt (src/graph.rs:809-817): a [M, K] @ b[N, K]^T, b an f32 parameter."""
         return _node(lib.mgq_graph_matmul_bt(self._h, a, b))
 
-    # ---- row-dynamic graphs and the operators of recurrent / latent-attention decoders (mgq.h)
+    # ---- row-dynamic graphs and the operators of recurrent / attention decoders (mgq.h)
     def input_u32_rows(self, name: str, capacity: int, which: int) -> int:
         """u32 input of up to `capacity` rows; Session.set_rows(which, n) sets the count of a step."""
         return _node(lib.mgq_graph_input_u32_rows(self._h, name.encode(), capacity, which))
@@ -149,6 +157,16 @@ class Graph:
 
     def embedding_scaled(self, indices: int, table: int, scale: float) -> int:
         return _node(lib.mgq_graph_embedding_scaled(self._h, indices, table, scale))
+
+    def embedding_positions(self, indices: int, table: int, pos: int, scale: float = 1.0, base: float = 10000.0) -> int:
+        """embedding_scaled plus the sinusoidal vector of every token's position (pos: position of row 0)."""
+        return _node(lib.mgq_graph_embedding_positions(self._h, indices, table, pos, scale, base))
+
+    def cast(self, x: int, out_dtype: int) -> int:
+        return _node(lib.mgq_graph_cast(self._h, x, out_dtype))
+
+    def scaled_sum(self, a: int, b: int, sa: float, sb: float) -> int:
+        return _node(lib.mgq_graph_scaled_sum(self._h, a, b, sa, sb))
 
     def pick_rows(self, x: int, index: int) -> int:
         return _node(lib.mgq_graph_pick_rows(self._h, x, index))
@@ -162,6 +180,9 @@ class Graph:
     def clamped_glu(self, gate: int, up: int, limit: float, alpha: float, out_dtype: int = FMT_F32) -> int:
         return _node(lib.mgq_graph_clamped_glu(self._h, gate, up, limit, alpha, out_dtype))
 
+    def silu_glu(self, gate: int, up: int, out_dtype: int = FMT_F32) -> int:
+        return _node(lib.mgq_graph_silu_glu(self._h, gate, up, out_dtype))
+
     def token_shift(self, h: int, mu, state: int, out_dtype: int = FMT_F32) -> int:
         """[len(mu), rows, width] mixes of every token with the one before it; take one with slot()."""
         arr = (ctypes.c_int * len(mu))(*mu)
@@ -172,6 +193,21 @@ class Graph:
 
     def lora_decay(self, low: int, w2: int, w0: int) -> int:
         return _node(lib.mgq_graph_lora_decay(self._h, low, w2, w0))
+
+    def lora_sigmoid_decay(self, low: int, w2: int, bias: int, tau: float) -> int:
+        return _node(lib.mgq_graph_lora_sigmoid_decay(self._h, low, w2, bias, tau))
+
+    def gla(self, q: int, k: int, v: int, decay: int, state: int, heads: int) -> int:
+        return _node(lib.mgq_graph_gla(self._h, q, k, v, decay, state, heads))
+
+    def query_temperature(self, x: int, pos: int, coef: float, every: float) -> int:
+        return _node(lib.mgq_graph_query_temperature(self._h, x, pos, coef, every))
+
+    def cache_append(self, x: int, cache: int, pos: int) -> int:
+        return _node(lib.mgq_graph_cache_append(self._h, x, cache, pos))
+
+    def attention(self, q: int, k_cache: int, v_cache: int, pos: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float) -> int:
+        return _node(lib.mgq_graph_attention(self._h, q, k_cache, v_cache, pos, heads, kv_heads, dim, vdim, scale))
 
     def wkv(self, r: int, k: int, v: int, decay: int, u: int, state: int, heads: int, shift_state: int = -1) -> int:
         return _node(lib.mgq_graph_wkv(self._h, r, k, v, decay, u, state, shift_state, heads))

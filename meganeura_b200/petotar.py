@@ -13,10 +13,9 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Optional
 
-import numpy as np
-
-from ._lib import FMT_BF16, FMT_F32, GATE_SIGMOID, GATE_SILU, ROWS_PICKED, ROWS_TOKENS, lib
-from .graph import Graph, Session, build_inference_session
+from ._lib import FMT_BF16, GATE_SIGMOID, GATE_SILU, lib
+from .graph import Graph
+from .row_model import RowModel
 
 GLU_ALPHA = 1.702            # fixed by the design
 SHIFTS = "rkvgw"             # token-shift mixes of a wkv layer, in slot order
@@ -81,47 +80,15 @@ class PetotarConfig:
         return PetotarConfig(int(cfg["vocab"]), int(cfg["width"]), float(cfg["norm"]["eps"]), float(cfg["embedding"]["scale"]), tuple(layers))
 
 
-class Petotar:
-    """One sequence's session.  max_rows: tokens of the largest step; max_tokens: positions a sequence
-    may reach (bounds the latent caches together with the windows)."""
-
-    def __init__(self, cfg: PetotarConfig, dtype: str = "bfloat16", max_rows: int = 512, max_picked: int = 256, max_tokens: int = 4096,
-                 lora_rank=None, tap_layers: bool = False):
-        """lora_rank: {wkv layer: rows of its w1}.  tap_layers: the residual stream after every layer
-        becomes an output too (indices 1.. of read_output_by_index)."""
-        if dtype not in ("bfloat16", "float32"):
-            raise ValueError(f"dtype must be bfloat16 or float32, not {dtype}")
-        self.cfg, self.dtype = cfg, dtype
-        self.max_rows, self.max_picked, self.max_tokens = max_rows, min(max_picked, max_rows), max_tokens
-        self.lora_rank = lora_rank or {}
-        self._params = []                                      # (name, shape, bf16?)
-        self._operand = FMT_BF16 if dtype == "bfloat16" else FMT_F32
-        self.graph = Graph()
-        self._taps = []
-        logits = self._build(self.graph)
-        self.graph.set_outputs([logits] + (self._taps if tap_layers else []))
-        self.session: Session = build_inference_session(self.graph)
+class Petotar(RowModel):
+    """max_tokens bounds the latent caches together with the windows."""
 
     # ---- graph
-    def _vec(self, name, n):
-        self._params.append((name, (n,), False))
-        return self.graph.parameter(name, [n])
-
-    def _mat(self, name, n, k):
-        self._params.append((name, (n, k), True))
-        return self.graph.parameter_bf16(name, [n, k])
-
-    def _linear(self, x, name, n, k):
-        return self.graph.matmul_bt(x, self._mat(name, n, k))
-
     def _window(self, layer):
         return min(layer.window, self.max_tokens)
 
     def _build(self, g: Graph) -> int:
         cfg, op = self.cfg, self._operand
-        self.token_ids = g.input_u32_rows("token_ids", self.max_rows, ROWS_TOKENS)
-        self.picked = g.input_u32_rows("picked_rows", self.max_picked, ROWS_PICKED)
-        self.pos = g.input_u32("kv_pos", [1])
         embed = self._mat("embed", cfg.vocab, cfg.width)
         x = g.embedding_scaled(self.token_ids, embed, cfg.embedding_scale)
         caches = {}
@@ -186,22 +153,6 @@ class Petotar:
                                layer.rot_base)
         o = g.head_gate(o, gate, layer.heads, act=GATE_SIGMOID, out_dtype=self._operand)
         return self._linear(o, f"{p}.o", cfg.width, layer.heads * layer.vdim)
-
-    # ---- weights
-    def parameters(self):
-        """(name, shape, stored as bf16 on the device) of every weight."""
-        return list(self._params)
-
-    def load(self, tensors) -> None:
-        """tensors: a weights.SafeTensors, or anything with shape / dtype / raw / f32 of the names."""
-        for name, shape, bf16 in self._params:
-            have = tuple(tensors.shape(name))
-            if int(np.prod(have)) != int(np.prod(shape)) or (bf16 and have != tuple(shape)):
-                raise ValueError(f"tensor '{name}' has the shape {list(have)}, the configuration needs {list(shape)}")
-            if bf16 and tensors.dtype(name) == "BF16":
-                self.session.upload_param(name, tensors.raw(name))
-            else:
-                self.session.set_parameter(name, tensors.f32(name))
 
     @staticmethod
     def from_tensors(config: dict, tensors, **kw) -> "Petotar":

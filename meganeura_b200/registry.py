@@ -9,9 +9,10 @@ import os
 
 from . import decode_model
 from .petotar import Petotar
+from .tobovik import Tobovik
 from .weights import SafeTensors, read_config
 
-ARCHITECTURES = {"Petotar": Petotar}
+ARCHITECTURES = {"Petotar": Petotar, "Tobovik": Tobovik}
 DECODERS = {c.name: c for c in (decode_model.SMOLLM2_135M, decode_model.QWEN3_8B)}
 
 
