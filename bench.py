@@ -567,7 +567,7 @@ def main():
                          "whichever of the two is faster in a short calibration, on several GPUs the persistent kernel")
     ap.add_argument("--exchange", choices=["peer", "nccl"], default="peer",
                     help="launches mode on several GPUs: slices pushed over NVLink by the GEMV kernels (default) or NCCL all-gather")
-    ap.add_argument("--design", choices=["petotar"], default=None,
+    ap.add_argument("--design", choices=["petotar", "tobovik"], default=None,
                     help="instead of the default workload: prefill and decode of this decoder design at layer sizes of real models, "
                          "beside the closest existing decoder (one JSON line per size)")
     ap.add_argument("--sizes", default="2048,4096", help="with --design: widths to measure")
@@ -589,7 +589,7 @@ def main():
         for name in args.sizes.split(","):
             sampler = ClockSampler(0)
             sampler.start()
-            line = design_bench.measure(name, (hbm, tensor))
+            line = design_bench.measure(args.design, name, (hbm, tensor))
             line.update(peaks=f"{hbm} GB/s, {tensor} TFLOP/s bf16 (of {source})", clocks=sampler.stop(), data="synthetic")
             print(json.dumps(line), flush=True)
         return

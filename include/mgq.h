@@ -457,7 +457,8 @@ int mgq_graph_slice_columns(mgq_graph *g, int x, uint32_t first, uint32_t count)
  *                     dim^-1/2, o = S^T q / (max(|n . q|, exp(-m)) + 1e-6); state: f32 parameter of
  *                     mgq_mlstm_state_elements
  * gla                 gated linear attention, per head: S = diag(decay_t) S + k_t v_t^T, then o = S^T q dim^-1/2;
- *                     state: f32 parameter of mgq_gla_state_elements
+ *                     state: f32 parameter of mgq_gla_state_elements; product_dtype MGQ_FMT_F32: f32 arithmetic,
+ *                     MGQ_FMT_BF16: long portions multiply sums of two bf16 on the tensor cores
  * head_gate           per head o / rms(o) * weight * act(gate), the weight for all heads side by side or one of a
  *                     head's size shared by them; weight -1: o * act(gate) without the norm
  * query_temperature   x * (1 + coef * ln(floor((p + 1) / every) + 1)) at position p = pos + row
@@ -491,7 +492,7 @@ size_t mgq_mlstm_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim);
 size_t mgq_gla_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim);
 int mgq_graph_lora_decay(mgq_graph *g, int low, int w2, int w0);
 int mgq_graph_lora_sigmoid_decay(mgq_graph *g, int low, int w2, int bias, float tau);
-int mgq_graph_gla(mgq_graph *g, int q, int k, int v, int decay, int state, uint32_t heads);
+int mgq_graph_gla(mgq_graph *g, int q, int k, int v, int decay, int state, uint32_t heads, int product_dtype);
 int mgq_graph_wkv(mgq_graph *g, int r, int k, int v, int decay, int u, int state, int shift_state, uint32_t heads);
 int mgq_graph_mlstm(mgq_graph *g, int q, int k, int v, int gate_i, int gate_f, int state, uint32_t heads, float gate_cap);
 int mgq_graph_head_gate(mgq_graph *g, int o, int weight, int gate, uint32_t heads, float eps, int act, int out_dtype);

@@ -118,7 +118,7 @@ SIGNATURES = {
     "mgq_graph_silu_glu": (_int, [_vp, _int, _int, _int]),
     "mgq_graph_lora_sigmoid_decay": (_int, [_vp, _int, _int, _int, ctypes.c_float]),
     "mgq_gla_state_elements": (_sz, [_u32, _u32, _u32]),
-    "mgq_graph_gla": (_int, [_vp, _int, _int, _int, _int, _int, _u32]),
+    "mgq_graph_gla": (_int, [_vp, _int, _int, _int, _int, _int, _u32, _int]),
     "mgq_graph_query_temperature": (_int, [_vp, _int, _int, ctypes.c_float, ctypes.c_float]),
     "mgq_graph_cache_append": (_int, [_vp, _int, _int, _int]),
     "mgq_graph_attention": (_int, [_vp, _int, _int, _int, _int, _u32, _u32, _u32, _u32, ctypes.c_float]),

@@ -1,0 +1,377 @@
+// Gated linear attention over many tokens in chunks of 16 on the tensor cores.
+//
+// Inside a chunk, with a_t the decays per key channel, L_t = a_1 .. a_t, G_s = a_(s+1) .. a_16 and the
+// state S in front of the chunk:
+//     o_t = S^T (L_t q_t) + sum_(s <= t) A_ts v_s,      A_ts = sum_d q_t k_s a_(s+1) .. a_t
+//     S'  = diag(L_16) S + sum_s (G_s k_s) v_s^T
+// Only products of decays appear, never a quotient, so nothing overflows however strong the decay is.
+//   gla_prepare_kernel  CTA = chunk x head: A, L q, G k and L_16 into a record that the next kernel copies as it is
+//   gla_chunks_kernel   a warp keeps S^T for 16 value columns and all keys in registers, as f32 accumulators of
+//                       mma.sync whose layout is also that of the products' left operand, and walks the chunks;
+//                       the records come through a ring of cp.async copies
+// State and sums are f32.  The products' operands (state, decayed queries and keys, A, values) enter as sums of two
+// bf16, three products each: 16 to 17 significant bits with the range of f32.  A long portion is cut into segments
+// that run in two launches, like in the token-by-token scan (mgq_mixer_ops.cu).
+#include <algorithm>
+
+#include "mgq_mixer.cuh"
+
+namespace mgq {
+namespace {
+
+constexpr uint32_t kChunk = 16, kStages = 3, kMaxWarps = 8, kMaxSegs = 16;
+
+// Record of a chunk of a head: G k (high, low parts), L_16, L q (high, low), A (high, low); rows padded for ldmatrix.
+template <int D> struct Record {
+    static constexpr uint32_t pitch = D + 8, matrix = kChunk * pitch * 2;
+    static constexpr uint32_t lam = 2 * matrix, ql = lam + D * 4, a = ql + 2 * matrix, bytes = a + 2 * kChunk * kChunk * 2;
+    static constexpr uint32_t state_part = ql;           // what a pass without outputs needs
+};
+
+struct Chunks {
+    const float *q, *k, *v, *w;
+    float *o, *state, *segments;
+    uint8_t *records;
+    uint32_t rows, heads, dim, vdim, chunks;
+    uint32_t seg_len, phase;                             // chunks per segment; 0: one pass, 1: end states, 2: outputs behind the first segment
+    float qscale;
+};
+
+__device__ __forceinline__ void split2(float x, float y, uint32_t &hi, uint32_t &lo)
+{
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    const float2 f = __bfloat1622float2(h);
+    const __nv_bfloat162 l = __floats2bfloat162_rn(x - f.x, y - f.y);
+    hi = *reinterpret_cast<const uint32_t *>(&h);
+    lo = *reinterpret_cast<const uint32_t *>(&l);
+}
+
+template <int D>
+__global__ void __launch_bounds__(256) gla_prepare_kernel(const __grid_constant__ Chunks p)
+{
+    constexpr uint32_t P = D + 4, SLICES = D / 4 < 16 ? D / 4 : 16;
+    using R = Record<D>;
+    extern __shared__ __align__(16) float smem[];        // q, k, w [16][P], partial sums of A [SLICES][16 t][16 s]
+    float *sq = smem, *sk = sq + kChunk * P, *sw = sk + kChunk * P, *sa = sw + kChunk * P;
+    const uint32_t t = threadIdx.x, chunk = blockIdx.x, head = blockIdx.y, row0 = chunk * kChunk, kpitch = p.heads * p.dim;
+    pdl_launch_dependents();
+    pdl_wait();
+    for (uint32_t i = t; i < kChunk * D; i += 256) {
+        const uint32_t r = i / D, d = i % D;
+        const bool in = row0 + r < p.rows && d < p.dim;  // beyond the portion: nothing decays and nothing is added
+        const size_t at = (size_t)(row0 + r) * kpitch + head * p.dim + d;
+        sq[r * P + d] = in ? p.q[at] * p.qscale : 0.f;
+        sk[r * P + d] = in ? p.k[at] : 0.f;
+        sw[r * P + d] = in ? p.w[at] : 1.f;
+    }
+    __syncthreads();
+    uint8_t *rec = p.records + ((size_t)head * p.chunks + chunk) * R::bytes;
+    // A: thread = key token s x a share of the channels; the key decays from token to token
+    {
+        const uint32_t s = t & 15u, slice = t >> 4;
+        float acc[kChunk];
+#pragma unroll
+        for (int i = 0; i < (int)kChunk; i++) acc[i] = 0.f;
+        for (uint32_t d = slice * 4; d < (uint32_t)D; d += 64) {
+            const float4 k4 = *reinterpret_cast<const float4 *>(sk + s * P + d);
+            float4 r = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int i = 0; i < (int)kChunk; i++) {
+                const float4 w4 = *reinterpret_cast<const float4 *>(sw + i * P + d), q4 = *reinterpret_cast<const float4 *>(sq + i * P + d);
+                const bool own = (uint32_t)i == s;
+                r.x = own ? k4.x : r.x * w4.x; r.y = own ? k4.y : r.y * w4.y; r.z = own ? k4.z : r.z * w4.z; r.w = own ? k4.w : r.w * w4.w;
+                acc[i] = fmaf(r.x, q4.x, acc[i]); acc[i] = fmaf(r.y, q4.y, acc[i]); acc[i] = fmaf(r.z, q4.z, acc[i]); acc[i] = fmaf(r.w, q4.w, acc[i]);
+            }
+        }
+        if (slice < SLICES)
+#pragma unroll
+            for (int i = 0; i < (int)kChunk; i++) sa[(slice * kChunk + i) * kChunk + s] = acc[i];
+    }
+    // L q by the first half of the threads, G k and L_16 by the second, two channels each
+    {
+        const uint32_t d = (t & 127u) * 2;
+        if (d < (uint32_t)D) {
+            float2 f = make_float2(1.f, 1.f);
+            if (t < 128) {
+#pragma unroll
+                for (int i = 0; i < (int)kChunk; i++) {
+                    const float2 w2 = *reinterpret_cast<const float2 *>(sw + i * P + d), x = *reinterpret_cast<const float2 *>(sq + i * P + d);
+                    f.x *= w2.x; f.y *= w2.y;
+                    uint32_t hi, lo;
+                    split2(x.x * f.x, x.y * f.y, hi, lo);
+                    *reinterpret_cast<uint32_t *>(rec + R::ql + (i * R::pitch + d) * 2) = hi;
+                    *reinterpret_cast<uint32_t *>(rec + R::ql + R::matrix + (i * R::pitch + d) * 2) = lo;
+                }
+            } else {
+#pragma unroll
+                for (int i = (int)kChunk - 1; i >= 0; i--) {
+                    const float2 w2 = *reinterpret_cast<const float2 *>(sw + i * P + d), x = *reinterpret_cast<const float2 *>(sk + i * P + d);
+                    uint32_t hi, lo;
+                    split2(x.x * f.x, x.y * f.y, hi, lo);
+                    *reinterpret_cast<uint32_t *>(rec + (i * R::pitch + d) * 2) = hi;
+                    *reinterpret_cast<uint32_t *>(rec + R::matrix + (i * R::pitch + d) * 2) = lo;
+                    f.x *= w2.x; f.y *= w2.y;
+                }
+                *reinterpret_cast<float2 *>(rec + R::lam + d * 4) = f;
+            }
+        }
+    }
+    __syncthreads();
+    if (t < 128) {                                       // two neighbouring keys of one query
+        float2 x = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < (int)SLICES; i++) {
+            const float2 y = *reinterpret_cast<const float2 *>(sa + i * kChunk * kChunk + 2 * t);
+            x.x += y.x; x.y += y.y;
+        }
+        uint32_t hi, lo;
+        split2(x.x, x.y, hi, lo);
+        *reinterpret_cast<uint32_t *>(rec + R::a + 4 * t) = hi;
+        *reinterpret_cast<uint32_t *>(rec + R::a + kChunk * kChunk * 2 + 4 * t) = lo;
+    }
+}
+
+__device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldmatrix4(uint32_t addr, uint32_t (&r)[4])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldmatrix4_t(uint32_t addr, uint32_t (&r)[4])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
+{
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// a . b with both as sums of a high and a low part (the product of the low parts is below f32's rounding of the sum)
+__device__ __forceinline__ void mma_split(float (&c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0, uint32_t bh1, uint32_t bl0, uint32_t bl1)
+{
+    mma16816(c, ah, bl0, bl1);
+    mma16816(c, al, bh0, bh1);
+    mma16816(c, ah, bh0, bh1);
+}
+
+// CTA = head (x) x value columns (y), 16 per warp, x segment (z).
+template <int D>
+__global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constant__ Chunks p)
+{
+    using R = Record<D>;
+    extern __shared__ __align__(16) uint8_t ring[];      // kStages records
+    __shared__ float s_f[D];
+    const uint32_t t = threadIdx.x, threads = blockDim.x, lane = t & 31u, warp = t >> 5, g = lane >> 2, tq = lane & 3u;
+    const uint32_t head = blockIdx.x, v0 = (blockIdx.y * (threads >> 5) + warp) * 16, kp = (p.dim + 3u) & ~3u, vpitch = p.heads * p.vdim;
+    const uint32_t seg = p.phase == 2 ? blockIdx.z + 1 : blockIdx.z, c0 = seg * p.seg_len, c1 = min(c0 + p.seg_len, p.chunks);
+    const bool outputs = p.phase != 1 || seg == 0;
+    const uint32_t vr[2] = {v0 + g, v0 + g + 8};         // this thread's value columns
+    const bool live[2] = {vr[0] < p.vdim, vr[1] < p.vdim};
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint8_t *records = p.records + (size_t)head * p.chunks * R::bytes;
+    auto stage = [&](uint32_t c) {                       // always one commit
+        if (c < c1) {
+            const uint8_t *src = records + (size_t)c * R::bytes;
+            const uint32_t dst = smem_addr(ring + (c - c0) % kStages * R::bytes), bytes = outputs ? R::bytes : R::state_part;
+            for (uint32_t i = t * 16; i < bytes; i += threads * 16)
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst + i), "l"(src + i) : "memory");
+        }
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+    };
+    stage(c0);
+    stage(c0 + 1);
+    const float *vbase = p.v + head * p.vdim;
+    float v[8];
+    auto load_values = [&](uint32_t c) {                 // [token pair low / high half][column], two tokens each
+#pragma unroll
+        for (int h = 0; h < 2; h++)
+#pragma unroll
+            for (int i = 0; i < 2; i++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    const uint32_t row = c * kChunk + h * 8 + tq * 2 + e;
+                    v[(h * 2 + i) * 2 + e] = c < c1 && row < p.rows && live[i] ? vbase[(size_t)row * vpitch + vr[i]] : 0.f;
+                }
+    };
+    load_values(c0);
+
+    // S^T: rows are value columns, columns are keys
+    float S[D / 8][4];
+#pragma unroll
+    for (int n = 0; n < D / 8; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) S[n][e] = 0.f;
+    if (seg == 0) {
+#pragma unroll
+        for (int n = 0; n < D / 8; n++)
+#pragma unroll
+            for (int i = 0; i < 2; i++) {
+                const uint32_t d = n * 8 + tq * 2;
+                if (d < kp && live[i]) {
+                    const float2 x = *reinterpret_cast<const float2 *>(p.state + ((size_t)head * p.vdim + vr[i]) * kp + d);
+                    S[n][2 * i] = x.x; S[n][2 * i + 1] = x.y;
+                }
+            }
+    } else if (outputs) {
+        for (uint32_t s = 0; s < seg; s++) {             // the end states of the segments before this one, put together in order
+            if (s > 0) {
+                for (uint32_t d = t; d < (uint32_t)D; d += threads) {
+                    float f = 1.f;
+#pragma unroll 8
+                    for (uint32_t c = s * p.seg_len; c < (s + 1) * p.seg_len; c++) f *= *reinterpret_cast<const float *>(records + (size_t)c * R::bytes + R::lam + d * 4);
+                    s_f[d] = f;
+                }
+            }
+            __syncthreads();
+            const float *end = p.segments + ((size_t)s * p.heads + head) * p.vdim * D;
+#pragma unroll
+            for (int n = 0; n < D / 8; n++) {
+                const uint32_t d = n * 8 + tq * 2;
+                const float2 f = s > 0 ? *reinterpret_cast<const float2 *>(s_f + d) : make_float2(0.f, 0.f);
+#pragma unroll
+                for (int i = 0; i < 2; i++) {
+                    const float2 x = live[i] ? *reinterpret_cast<const float2 *>(end + (size_t)vr[i] * D + d) : make_float2(0.f, 0.f);
+                    S[n][2 * i] = fmaf(f.x, S[n][2 * i], x.x);
+                    S[n][2 * i + 1] = fmaf(f.y, S[n][2 * i + 1], x.y);
+                }
+            }
+            __syncthreads();
+        }
+    }
+
+    const uint32_t q_off = R::ql + (((lane & 7u) + (lane >> 4) * 8) * R::pitch + ((lane >> 3) & 1u) * 8) * 2;
+    const uint32_t k_off = (((lane & 7u) + ((lane >> 3) & 1u) * 8) * R::pitch + (lane >> 4) * 8) * 2;
+    for (uint32_t c = c0; c < c1; c++) {
+        asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+        __syncthreads();                                 // everyone's copies, and everyone has left the buffer that is filled now
+        stage(c + 2);
+        const uint8_t *rec = ring + (c - c0) % kStages * R::bytes;
+        const uint32_t base = smem_addr(rec);
+        uint32_t vh[4], vl[4];                           // V^T as left operand: rows value columns, columns tokens
+#pragma unroll
+        for (int i = 0; i < 4; i++) split2(v[2 * i], v[2 * i + 1], vh[i], vl[i]);
+        load_values(c + 1);
+        float o[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};          // o^T: rows value columns, columns tokens
+#pragma unroll
+        for (int j = 0; j < D / 16; j++) {
+            if (outputs) {
+                uint32_t sh[4], sl[4], qh[4], ql[4];
+                split2(S[2 * j][0], S[2 * j][1], sh[0], sl[0]);
+                split2(S[2 * j][2], S[2 * j][3], sh[1], sl[1]);
+                split2(S[2 * j + 1][0], S[2 * j + 1][1], sh[2], sl[2]);
+                split2(S[2 * j + 1][2], S[2 * j + 1][3], sh[3], sl[3]);
+                ldmatrix4(base + q_off + j * 32, qh);
+                ldmatrix4(base + q_off + R::matrix + j * 32, ql);
+                mma_split(o[0], sh, sl, qh[0], qh[1], ql[0], ql[1]);
+                mma_split(o[1], sh, sl, qh[2], qh[3], ql[2], ql[3]);
+            }
+            uint32_t kh[4], kl[4];
+            ldmatrix4_t(base + k_off + j * 32, kh);
+            ldmatrix4_t(base + k_off + R::matrix + j * 32, kl);
+#pragma unroll
+            for (int n = 0; n < 2; n++) {
+                const float2 f = *reinterpret_cast<const float2 *>(rec + R::lam + (j * 16 + n * 8 + tq * 2) * 4);
+                float (&x)[4] = S[2 * j + n];
+                x[0] *= f.x; x[1] *= f.y; x[2] *= f.x; x[3] *= f.y;
+                mma_split(x, vh, vl, kh[2 * n], kh[2 * n + 1], kl[2 * n], kl[2 * n + 1]);
+            }
+        }
+        if (!outputs) continue;
+#pragma unroll
+        for (int n = 0; n < 2; n++) {                    // tokens n * 8 + g as columns, keys of the chunk as the sum
+            const uint8_t *a = rec + R::a + ((n * 8 + g) * kChunk + tq * 2) * 2;
+            const uint32_t ah0 = *reinterpret_cast<const uint32_t *>(a), ah1 = *reinterpret_cast<const uint32_t *>(a + 16);
+            const uint32_t al0 = *reinterpret_cast<const uint32_t *>(a + kChunk * kChunk * 2), al1 = *reinterpret_cast<const uint32_t *>(a + kChunk * kChunk * 2 + 16);
+            mma_split(o[n], vh, vl, ah0, ah1, al0, al1);
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const uint32_t row = c * kChunk + n * 8 + tq * 2 + (e & 1);
+                if (row < p.rows && live[e >> 1]) p.o[(size_t)row * vpitch + head * p.vdim + vr[e >> 1]] = o[n][e];
+            }
+        }
+    }
+    const bool last = c1 == p.chunks;
+    if (p.phase == 2 && !last) return;                   // later segments may still be reading this one's end state
+#pragma unroll
+    for (int n = 0; n < D / 8; n++)
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const uint32_t d = n * 8 + tq * 2;
+            if (!live[i]) continue;
+            const float2 x = make_float2(S[n][2 * i], S[n][2 * i + 1]);
+            if (!last)       *reinterpret_cast<float2 *>(p.segments + (((size_t)seg * p.heads + head) * p.vdim + vr[i]) * D + d) = x;
+            else if (d < kp) *reinterpret_cast<float2 *>(p.state + ((size_t)head * p.vdim + vr[i]) * kp + d) = x;
+        }
+}
+
+uint32_t padded(uint32_t dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
+uint32_t warps_for(uint32_t vdim) { return std::min(kMaxWarps, (vdim + 15) / 16); }
+size_t align256(size_t n) { return (n + 255) & ~(size_t)255; }
+size_t record_bytes(uint32_t dim)
+{
+    const uint32_t d = padded(dim);
+    return d == 32 ? Record<32>::bytes : d == 64 ? Record<64>::bytes : d == 128 ? Record<128>::bytes : Record<256>::bytes;
+}
+
+// Chunks per segment; all of them: one pass.  Two launches pay from three segments on.
+uint32_t segment_chunks(uint32_t chunks, uint32_t heads, uint32_t vdim)
+{
+    const uint32_t w = warps_for(vdim), ctas = heads * ((vdim + 16 * w - 1) / (16 * w)), want = std::min(kMaxSegs, 148u / ctas + 1);
+    if (want < 3 || chunks < 12) return chunks;
+    const uint32_t len = std::max(4u, (chunks + want - 1) / want);
+    return (chunks + len - 1) / len < 3 ? chunks : len;
+}
+
+template <int D>
+int launch_sized(Chunks p, cudaStream_t st)
+{
+    const size_t prep = (size_t)(3 * kChunk * (D + 4) + std::min(D / 4, 16) * kChunk * kChunk) * 4, smem = (size_t)kStages * Record<D>::bytes;
+    if (int rc = allow_smem(gla_prepare_kernel<D>, prep)) return rc;
+    if (int rc = allow_smem(gla_chunks_kernel<D>, smem)) return rc;
+    if (int rc = launch(gla_prepare_kernel<D>, dim3(p.chunks, p.heads), dim3(256), prep, st, p)) return rc;
+    const uint32_t w = warps_for(p.vdim), segs = (p.chunks + p.seg_len - 1) / p.seg_len;
+    dim3 grid(p.heads, (p.vdim + 16 * w - 1) / (16 * w), 1);
+    if (segs == 1) {
+        gla_chunks_kernel<D><<<grid, w * 32, smem, st>>>(p);
+        MGQ_CUDA(cudaGetLastError());
+        return MGQ_OK;
+    }
+    grid.z = segs - 1;
+    p.phase = 1;
+    gla_chunks_kernel<D><<<grid, w * 32, smem, st>>>(p);
+    MGQ_CUDA(cudaGetLastError());
+    p.phase = 2;
+    gla_chunks_kernel<D><<<grid, w * 32, smem, st>>>(p);
+    MGQ_CUDA(cudaGetLastError());
+    return MGQ_OK;
+}
+
+}  // namespace
+
+size_t gla_chunks_workspace(uint32_t max_rows, uint32_t heads, uint32_t dim, uint32_t vdim)
+{
+    if (max_rows < kPrefillRows) return 0;
+    const size_t chunks = (max_rows + kChunk - 1) / kChunk;
+    return align256(chunks * heads * record_bytes(dim)) + (size_t)(kMaxSegs - 1) * heads * vdim * padded(dim) * 4;
+}
+
+int launch_gla_chunks(const ChannelDecay &a, void *stream)
+{
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (a.u || a.dim > kMaxStateDim || !a.workspace) return fail(MGQ_ERR_STATE, "gla chunks: not this recurrence");
+    Chunks p{};
+    p.q = a.q; p.k = a.k; p.v = a.v; p.w = a.d.out; p.o = a.o; p.state = a.state;
+    p.rows = a.rows; p.heads = a.heads; p.dim = a.dim; p.vdim = a.vdim; p.chunks = (a.rows + kChunk - 1) / kChunk;
+    p.records = static_cast<uint8_t *>(a.workspace);
+    p.segments = reinterpret_cast<float *>(p.records + align256((size_t)p.chunks * a.heads * record_bytes(a.dim)));
+    p.seg_len = segment_chunks(p.chunks, a.heads, a.vdim);
+    p.qscale = (float)(1.0 / sqrt((double)a.dim));
+    switch (padded(a.dim)) {
+        case 32: return launch_sized<32>(p, st);
+        case 64: return launch_sized<64>(p, st);
+        case 128: return launch_sized<128>(p, st);
+        default: return launch_sized<256>(p, st);
+    }
+}
+
+}  // namespace mgq

@@ -8,6 +8,7 @@ namespace mgq {
 
 constexpr int kMaxShifts = 8;
 constexpr uint32_t kMaxStateDim = 256;         // key dimensions of a recurrent head
+constexpr uint32_t kPrefillRows = 64;          // from here on a step takes the kernels for many rows
 
 // out[r] = table[ids[r]] * scale (+ sinusoidal vector of position pos + r); copy: a second, bf16 output or null.
 // sinusoid: (width + 1) / 2 frequencies as sums of two f32 (null: no position vector); column 2i is the sine
@@ -90,9 +91,13 @@ struct ChannelDecay {
     float *o, *state, *shift_state;
     uint32_t rows, heads, dim, vdim, shift_width;
     void *workspace;                       // scan_workspace bytes, or null (long portions then run in one piece)
+    bool split_products;                   // gated linear, kPrefillRows or more rows: chunks on the tensor cores (mgq_gla_chunks.cu),
+                                           // whose workspace is gla_chunks_workspace bytes
 };
 size_t channel_decay_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim);
 int launch_channel_decay_scan(const ChannelDecay &a, void *stream);
+size_t gla_chunks_workspace(uint32_t max_rows, uint32_t heads, uint32_t dim, uint32_t vdim);
+int launch_gla_chunks(const ChannelDecay &a, void *stream);
 int launch_channel_decay_step(const ChannelDecay &a, const HeadGate &hg, void *stream);      // rows == 1: decay, recurrence, head gate in one launch
 
 // mLSTM recurrence.  q, k [rows, heads * dim], v, o [rows, heads * vdim], gate pre-activations
@@ -137,7 +142,6 @@ size_t latent_attention_workspace(uint32_t max_rows, uint32_t heads, uint32_t di
 int launch_latent_attention(const LatentAttention &a, void *stream);
 // Many rows, bf16 cache, sizes in multiples of 8 (mgq_prefill_attention.cu): keys and values are expanded
 // from the latents once per step and the softmax runs tile by tile on the tensor cores.
-constexpr uint32_t kPrefillRows = 64;      // fewer rows take the absorbed form
 bool latent_prefill_eligible(uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t rank, bool cache_bf16);
 size_t latent_prefill_workspace(uint32_t heads, uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t slots);
 int launch_latent_prefill(const LatentAttention &a, void *stream);

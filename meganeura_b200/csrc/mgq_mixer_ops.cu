@@ -36,14 +36,15 @@ template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16 
 }
 
 // ---------------------------------------------------------------- embedding, rows, element-wise
-// Sine and cosine of p * f for f = f.x + f.y: the product's rounding error and the low part of f enter to first order.
+// Sine and cosine of p * f for f = f.x + f.y: the product's rounding error and the low part of f enter as a small angle.
 __device__ __forceinline__ void sincos_product(float p, float2 f, float &s, float &c)
 {
     const float hi = p * f.x, lo = fmaf(p, f.y, fmaf(p, f.x, -hi));
     float s0, c0;
     sincosf(hi, &s0, &c0);
-    s = fmaf(lo, c0, s0);
-    c = fmaf(-lo, s0, c0);
+    const float h = -0.5f * lo * lo;
+    s = fmaf(h, s0, fmaf(lo, c0, s0));
+    c = fmaf(h, c0, fmaf(-lo, s0, c0));
 }
 
 template <typename T>
@@ -840,10 +841,11 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_cons
     }
     const bool last = row0 + rows == p.rows;
     float *end = last ? p.state : p.segments + seg * stride;
+    const bool store = p.phase != 2 || last;             // in phase 2 later segments may still be reading the end states
 #pragma unroll
     for (int c = 0; c < C; c++)
-        if (col + c < vdim) store_keys<RPT>(end + ((size_t)head * vdim + col + c) * kp, ks, kp, S[c]);
-    if (MODE == kMlstm || !last) {
+        if (store && col + c < vdim) store_keys<RPT>(end + ((size_t)head * vdim + col + c) * kp, ks, kp, S[c]);
+    if (store && (MODE == kMlstm || !last)) {
         float *nb = normalizer(p, end, head, block);
         if (t < 8) store_keys<RPT>(nb, ks, kp, n);
         if (MODE == kMlstm && t == 0) {
@@ -1151,6 +1153,7 @@ int launch_channel_decay_scan(const ChannelDecay &a, void *stream)
 {
     const Scan p = channel_decay_args(a);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (a.split_products && a.rows >= kPrefillRows) return launch_gla_chunks(a, stream);
     return a.u ? launch_scan<kWkv>(p, a.workspace, st) : launch_scan<kGla>(p, a.workspace, st);
 }
 int launch_mlstm_scan(const Mlstm &a, void *stream) { return launch_scan<kMlstm>(mlstm_args(a), a.workspace, static_cast<cudaStream_t>(stream)); }

@@ -79,6 +79,7 @@ struct Dispatch {
     int weight_format;
     float f0;
     void *workspace;
+    bool scratch = false;         // workspace is the session's shared scratch
     std::vector<int> members;     // linear group: the node of each layer
     int exchange = -1;            // all_gather: which exchange; GEMV: the exchange it pushes its columns to (-1: none)
     bool push_done = false;       // all_gather: the producing GEMV has pushed the slice already
@@ -199,6 +200,7 @@ struct mgq_session {
     std::vector<ConcatWeight> concats;
     std::vector<Dispatch> dispatches;
     std::vector<void *> workspaces;
+    size_t scratch_bytes = 0;                  // shared by the dispatches that say so
     std::vector<uint8_t> staging;              // host scratch for quantize-on-upload
     cudaStream_t stream = nullptr;
     cudaGraph_t graph = nullptr;
@@ -636,7 +638,7 @@ int mgq_graph_lora_sigmoid_decay(mgq_graph *g, int low, int w2, int bias, float 
     return id;
 }
 
-int mgq_graph_gla(mgq_graph *g, int q, int k, int v, int decay, int state, uint32_t heads)
+int mgq_graph_gla(mgq_graph *g, int q, int k, int v, int decay, int state, uint32_t heads, int product_dtype)
 {
     if (!g) return -fail(MGQ_ERR_NULL, "null graph");
     if (!all_valid(g, {q, k, v, decay, state})) return -fail(MGQ_ERR_NAME, "gla: node id out of range");
@@ -648,8 +650,9 @@ int mgq_graph_gla(mgq_graph *g, int q, int k, int v, int decay, int state, uint3
         if (!is_act(g, id, nq.shape[0], nq.shape[1], nq.rows)) return -fail(MGQ_ERR_SHAPE, "gla: q, k and the decay must be f32 of one shape");
     if (!is_act(g, v, nq.shape[0], nv.shape[1], nq.rows)) return -fail(MGQ_ERR_SHAPE, "gla: v must be f32 rows like q");
     if (!is_param(g, state, MGQ_FMT_F32, mgq_gla_state_elements(heads, dim, vdim))) return -fail(MGQ_ERR_SHAPE, "gla: state must be an f32 parameter of %zu elements", mgq_gla_state_elements(heads, dim, vdim));
+    if (!operand_dtype(product_dtype)) return -fail(MGQ_ERR_FORMAT, "gla: products of f32, or of sums of two bf16");
     Node nd{Op::Gla, "", nv.shape, MGQ_FMT_F32, {q, k, v, decay, -1, state, -1}};         // laid out like Wkv
-    nd.at = {heads, dim, vdim};
+    nd.at = {heads, dim, vdim, product_dtype == MGQ_FMT_BF16};
     nd.rows = nq.rows;
     return push_node(g, std::move(nd));
 }
@@ -1122,18 +1125,27 @@ int sinusoid_table(mgq_session *s, uint32_t width, float base, Dispatch &d)
     return mgq_buffer_upload(d.workspace, freq.data(), freq.size() * 4, s->stream);
 }
 
+// Scratch that one dispatch fills and leaves behind; dispatches run one after the other, so they share it.
+void shared_scratch(mgq_session *s, size_t bytes, Dispatch &d)
+{
+    s->scratch_bytes = std::max(s->scratch_bytes, bytes);
+    d.scratch = bytes > 0;
+}
+
 int attention_scratch(mgq_session *s, const Node &nd, Dispatch &d)
 {
     const std::vector<uint32_t> &a = nd.at;
-    const size_t bytes = mgq::attention_workspace((uint32_t)nd.shape[0], a[0], a[1], a[2], a[3], a[4], s->nodes[nd.inputs[1]].dtype == MGQ_FMT_F16);
-    if (int rc = mgq_buffer_create(bytes, &d.workspace)) return rc;
-    s->workspaces.push_back(d.workspace);
+    shared_scratch(s, mgq::attention_workspace((uint32_t)nd.shape[0], a[0], a[1], a[2], a[3], a[4], s->nodes[nd.inputs[1]].dtype == MGQ_FMT_F16), d);
     return MGQ_OK;
 }
 
 int recurrence_workspace(mgq_session *s, const Node &nd, Dispatch &d)
 {
-    const size_t bytes = mgq::scan_workspace((uint32_t)nd.shape[0], nd.at[0], nd.at[1], nd.at.back());
+    if (nd.op == Op::Gla && nd.at[3]) {
+        shared_scratch(s, mgq::gla_chunks_workspace((uint32_t)nd.shape[0], nd.at[0], nd.at[1], nd.at[2]), d);
+        return MGQ_OK;
+    }
+    const size_t bytes = mgq::scan_workspace((uint32_t)nd.shape[0], nd.at[0], nd.at[1], nd.at[2]);
     if (bytes == 0) return MGQ_OK;
     if (int rc = mgq_buffer_create(bytes, &d.workspace)) return rc;
     s->workspaces.push_back(d.workspace);
@@ -1491,6 +1503,14 @@ int mgq_build_inference_session(const mgq_graph *g, mgq_session **out)
             default: continue;           // Input, Parameter, View, Slot, Nop: nothing to run
         }
         s->dispatches.push_back(d);
+    }
+    if (s->scratch_bytes) {
+        void *p = nullptr;
+        rc = mgq_buffer_create(s->scratch_bytes, &p);
+        if (rc) { mgq_session_free(s); return rc; }
+        s->workspaces.push_back(p);
+        for (Dispatch &d : s->dispatches)
+            if (d.scratch) d.workspace = p;
     }
     if (g_fuse_rope_cache) merge_rope_cache(s);
     if (g_fuse_mixer) merge_attention_inputs(s);
@@ -1854,6 +1874,7 @@ static int run_mixer(mgq_session *s, const Dispatch &d)
         const Node &dn = s->nodes[did];
         a.rows = a.d.rows = rows;
         a.workspace = d.workspace;
+        a.split_products = o.op == Op::Gla && o.at[3];
         a.d.out = f(did);
         if (dn.op == Op::Decay) {
             a.d.low = f(dn.inputs[0]); a.d.w2 = s->ptr(dn.inputs[1]); a.d.w0 = f(dn.inputs[2]);

@@ -1,6 +1,6 @@
-"""Prefill and decode throughput of the Petotar design at sizes of real models' layers (seeded random
+"""Prefill and decode throughput of a row-dynamic design at sizes of real models' layers (seeded random
 weights), the kernels' distance from their rooflines, and the closest decoder of this package at equal
-width, layer count and vocabulary (bench.py --design petotar)."""
+width, layer count and vocabulary (bench.py --design petotar|tobovik)."""
 from __future__ import annotations
 
 import time
@@ -12,6 +12,7 @@ from ._lib import ROWS_PICKED, ROWS_TOKENS
 from .engine import Engine
 from .graph import ShaderEntry as S
 from .petotar import Petotar, PetotarConfig
+from .tobovik import Tobovik, TobovikConfig, gla_prefixes
 from .weights import to_bf16
 
 
@@ -24,24 +25,44 @@ def _layers(kind, ff, wkv, mlstm, latent):
     return out
 
 
-# name -> (config, rank of the decay projection, decoder of the package it stands beside)
-def sizes():
-    def cfg(vocab, width, layers):
-        return {"architecture": "Petotar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": layers}
-    latent2 = dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, mask={"size": 2048}, rot={"base": 1e6, "dims": 64}, scale=192 ** -0.5)
-    latent4 = dict(latent2, heads=32)
-    a = cfg(32768, 2048, _layers("wamwsm", 6144, dict(heads=32, dim=64), dict(heads=8, dim=128, vdim=256, gate_cap=15.0), latent2))
-    b = cfg(151936, 4096, _layers("wamwsm", 12288, dict(heads=64, dim=64), dict(heads=16, dim=128, vdim=256, gate_cap=15.0), latent4))
-    like_a = M.DecoderConfig("decoder-2048", 32768, 2048, 6, 16, 4, 128, 6144, 1e-6, 1e6, M.FMT_Q4, M.FMT_Q4, M.FMT_Q4)
-    like_b = M.replace(M.QWEN3_8B, name="decoder-4096", num_hidden_layers=6)
-    return {"2048": (a, 64, like_a), "4096": (b, 64, like_b)}
+def _tobovik_layers(kind, ff, left, right, gla):
+    out = []
+    for k in kind:
+        m = dict(type="gla", mixer=dict(gla)) if k == "g" else dict(type="parallel", mixer=dict(left=left, right=right, left_scale=0.8, right_scale=0.9))
+        out.append(dict(m, mlp={"kind": "dense", "ff": ff}))
+    return out
 
 
-def random_model(config, rank, **kw) -> Petotar:
-    cfg = PetotarConfig.from_dict(config)
-    model = Petotar(cfg, lora_rank={i: rank for i, layer in enumerate(cfg.layers) if layer.type == "wkv"}, **kw)
+# design -> name -> (config, rank of the decay projection, what it stands beside: a design, or a decoder of the package)
+def sizes(design):
+    def cfg(architecture, vocab, width, layers, **more):
+        return dict({"architecture": architecture, "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": layers}, **more)
+    if design == "petotar":
+        latent2 = dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, mask={"size": 2048}, rot={"base": 1e6, "dims": 64}, scale=192 ** -0.5)
+        latent4 = dict(latent2, heads=32)
+        one = {"embedding": {"scale": 1.0}}
+        a = cfg("Petotar", 32768, 2048, _layers("wamwsm", 6144, dict(heads=32, dim=64), dict(heads=8, dim=128, vdim=256, gate_cap=15.0), latent2), **one)
+        b = cfg("Petotar", 151936, 4096, _layers("wamwsm", 12288, dict(heads=64, dim=64), dict(heads=16, dim=128, vdim=256, gate_cap=15.0), latent4), **one)
+        like_a = M.DecoderConfig("decoder-2048", 32768, 2048, 6, 16, 4, 128, 6144, 1e-6, 1e6, M.FMT_Q4, M.FMT_Q4, M.FMT_Q4)
+        like_b = M.replace(M.QWEN3_8B, name="decoder-4096", num_hidden_layers=6)
+        return {"2048": (a, 64, like_a), "4096": (b, 64, like_b)}
+    def mixers(heads):
+        left = dict(heads=heads, kv_heads=heads // 4, dim=128, vdim=128, scale=128 ** -0.5, q_temp={"coef": 0.1, "every": 8192})
+        return left, dict(heads=heads // 2, dim=128, vdim=256, tau=16.0), dict(heads=heads // 4, dim=256, vdim=512, tau=16.0)
+    return {"2048": (cfg("Tobovik", 32768, 2048, _tobovik_layers("pgppgp", 6144, *mixers(16))), 16, "petotar"),
+            "4096": (cfg("Tobovik", 151936, 4096, _tobovik_layers("pgppgp", 12288, *mixers(32))), 16, "petotar")}
+
+
+def random_model(config, rank, **kw):
+    if config["architecture"] == "Tobovik":
+        cfg = TobovikConfig.from_dict(config)
+        model = Tobovik(cfg, lora_rank={p: rank for p in gla_prefixes(cfg)}, **kw)
+    else:
+        cfg = PetotarConfig.from_dict(config)
+        model = Petotar(cfg, lora_rank={i: rank for i, layer in enumerate(cfg.layers) if layer.type == "wkv"}, **kw)
     rng = np.random.Generator(np.random.PCG64(5))
     noise = rng.standard_normal(1 << 22, dtype=np.float32)
+    around_one = isinstance(model, Tobovik)                  # norm weights: stored plain, or around zero
     for idx, (name, shape, bf16) in enumerate(model.parameters()):
         n = int(np.prod(shape))
         start = (idx * 7919) % 65536
@@ -50,22 +71,40 @@ def random_model(config, rank, **kw) -> Petotar:
             model.session.upload_param(name, to_bf16(a * np.float32(shape[1] ** -0.5)))
         elif ".mu." in name:
             model.session.set_parameter(name, 1.0 / (1.0 + np.exp(-a)))
-        elif name.endswith((".w0", ".norm")) and ".mix." in name:
-            model.session.set_parameter(name, a * 0.1 + (1.0 if name.endswith(".norm") else -3.0))
+        elif name.endswith(".a2.b"):
+            model.session.set_parameter(name, a * 1.5 + 2.0)
+        elif "norm" in name.rsplit(".", 1)[-1] and (around_one or ".mix." in name):
+            model.session.set_parameter(name, a * 0.1 + 1.0)
+        elif name.endswith(".w0") and ".mix." in name:
+            model.session.set_parameter(name, a * 0.1 - 3.0)
         else:
             model.session.set_parameter(name, a * 0.1 + (3.0 if name.endswith(".f.b") else 0.0))
     return model
 
 
-def work(model: Petotar, d, rows: int, pos: int):
+def work(model, d, rows: int, pos: int):
     """(algorithmic bytes, flops) of one dispatch for `rows` tokens that start at position `pos`."""
     p, shader = d.params, d.shader
     act = 2 if model.dtype == "bfloat16" else 4
     if shader in (S.Linear, S.LinearGLU):
         r = 1 if p[2] == model.cfg.vocab else rows
-        w = 2 if shader == S.LinearGLU else 1
+        weights = 2 * p[1] * p[2] if shader == S.LinearGLU else p[3]
         out = act if shader == S.LinearGLU else 8 if d.label.endswith("+Add") else 4
-        return 2 * w * p[1] * p[2] + r * (act * p[1] + out * p[2]), 2 * w * r * p[1] * p[2]
+        return 2 * weights + r * (act * p[1] + out * p[2]), 2 * r * weights
+    if shader == S.Gla:
+        h, vdim, dim = p[1:4]                # what one pass needs: q, k, v, the gate, the state in and out (the decay comes from its low-rank input)
+        return 8 * h * dim * vdim + rows * h * (8 * dim + vdim * (8 + act)), rows * h * dim * vdim * 5
+    if shader == S.Attention:
+        h, vdim, dim = p[1:4]
+        kv = next(x.attention.kv_heads for x in model.cfg.layers if x.attention and (x.attention.heads, x.attention.dim, x.attention.vdim) == (h, dim, vdim))
+        keys = rows * pos + rows * (rows + 1) // 2
+        return act * (pos + rows) * kv * (dim + vdim) + rows * h * (4 * dim + vdim * (4 + act)), 2 * h * keys * (dim + vdim)
+    if shader == S.AttentionInputs:
+        a = next(x.attention for x in model.cfg.layers if x.attention)
+        return rows * (a.heads * a.dim * 8 + a.kv_heads * (a.dim + a.vdim) * (4 + act)), 0
+    if shader == S.ResidualNorm:
+        two = any(x.attention for x in model.cfg.layers)
+        return rows * model.cfg.width * (12 + act + (2 if two else 0)), rows * model.cfg.width * 6
     if shader == S.Wkv:
         h, dim = p[1], p[2]
         return 8 * h * dim * dim + rows * h * dim * (4 * 5 + act), rows * h * dim * dim * 7
@@ -93,7 +132,7 @@ def work(model: Petotar, d, rows: int, pos: int):
     return rows * width * 6, 0
 
 
-def kernel_table(model: Petotar, step, rows: int, pos: int, peaks, repeats: int = 5):
+def kernel_table(model, step, rows: int, pos: int, peaks, repeats: int = 5):
     """Median microseconds of every dispatch (events around each) merged by label, with its roofline share."""
     s = model.session
     s.set_profiling(True)
@@ -120,8 +159,7 @@ def kernel_table(model: Petotar, step, rows: int, pos: int, peaks, repeats: int 
     return out
 
 
-def measure(name: str, peaks, prefill: int = 2048, context: int = 2048, steps: int = 64, tables: bool = True) -> dict:
-    config, rank, like = sizes()[name]
+def row_model_numbers(label, config, rank, peaks, prefill, context, steps, tables) -> dict:
     limit = context + prefill + 2 * steps + 32
     model = random_model(config, rank, dtype="bfloat16", max_rows=prefill, max_picked=1, max_tokens=limit)
     e, s = Engine(model, greedy=True), model.session
@@ -138,7 +176,7 @@ def measure(name: str, peaks, prefill: int = 2048, context: int = 2048, steps: i
         prompt()
     prefill_s = (time.perf_counter() - t0) / 5
     finite = bool(np.isfinite(s.read_output(model.cfg.vocab)).all())
-    out = {"model": f"petotar-{name}", "width": model.cfg.width, "layers": len(model.cfg.layers), "vocab": model.cfg.vocab, "dtype": "bfloat16",
+    out = {"model": label, "width": model.cfg.width, "layers": len(model.cfg.layers), "vocab": model.cfg.vocab, "dtype": "bfloat16",
            "prefill_tokens": prefill, "prefill_tokens_per_s": round(prefill / prefill_s), "prefill_ms": round(prefill_s * 1e3, 3), "logits_finite": finite}
     if tables:
         out["prefill_kernels"] = kernel_table(model, prompt, prefill, 0, peaks)
@@ -155,7 +193,20 @@ def measure(name: str, peaks, prefill: int = 2048, context: int = 2048, steps: i
                weight_gb=round(weights / 1e9, 3), decode_weight_gbs=round(weights / dt / 1e9, 1), first_tokens=[int(t) for t in first])
     if tables:
         out["decode_kernels"] = kernel_table(model, lambda: (s.step(), s.wait()), 1, context + 5 + steps, peaks)
-    del e, model, s
+    return out
+
+
+def measure(design: str, name: str, peaks, prefill: int = 2048, context: int = 2048, steps: int = 64, tables: bool = True) -> dict:
+    config, rank, like = sizes(design)[name]
+    out = row_model_numbers(f"{design}-{name}", config, rank, peaks, prefill, context, steps, tables)
+    if isinstance(like, str):
+        out["closest"] = row_model_numbers(f"{like}-{name}", *sizes(like)[name][:2], peaks, prefill, context, steps, tables)
+    else:
+        out["closest"] = decoder_numbers(like, peaks, context, steps, tables)
+    return out
+
+
+def decoder_numbers(like, peaks, context, steps, tables) -> dict:
     dec = M.DecodeSession(like, context + steps + 16, seed=3, greedy_history=context + steps + 16)
     dec.fill_caches(context)
     ds = dec.session
@@ -173,9 +224,9 @@ def measure(name: str, peaks, prefill: int = 2048, context: int = 2048, steps: i
     ds.wait()
     dt = (time.perf_counter() - t0) / steps
     wb = M.packed_weight_bytes(like)
-    out["closest"] = {"model": like.name, "weights": "Q4", "decode_context": context, "decode_tokens_per_s": round(1 / dt, 1), "decode_ms": round(dt * 1e3, 4),
-                      "decode_launches": len(ds.plan().dispatches) + 1, "weight_gb": round(wb / 1e9, 3), "decode_weight_gbs": round(wb / dt / 1e9, 1),
-                      "prefill": "token by token (the model has no multi-row step): the decode rate"}
+    out = {"model": like.name, "weights": "Q4", "decode_context": context, "decode_tokens_per_s": round(1 / dt, 1), "decode_ms": round(dt * 1e3, 4),
+           "decode_launches": len(ds.plan().dispatches) + 1, "weight_gb": round(wb / 1e9, 3), "decode_weight_gbs": round(wb / dt / 1e9, 1),
+           "prefill": "token by token (the model has no multi-row step): the decode rate"}
     if tables:
         ds.set_profiling(True)
         runs = []
@@ -198,5 +249,5 @@ def measure(name: str, peaks, prefill: int = 2048, context: int = 2048, steps: i
             elif d.shader == S.CachedAttention:
                 nb = 2 * (context + 1) * like.kv_dim * 4
             rows.append({"kernel": label, "dispatches": n, "us_each": round(t / n, 2), "roofline": round(nb * n / peaks[0] / 1e3 / t, 4) if nb else None})
-        out["closest"]["decode_kernels"] = rows
+        out["decode_kernels"] = rows
     return out

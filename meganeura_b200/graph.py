@@ -197,8 +197,8 @@ class Graph:
     def lora_sigmoid_decay(self, low: int, w2: int, bias: int, tau: float) -> int:
         return _node(lib.mgq_graph_lora_sigmoid_decay(self._h, low, w2, bias, tau))
 
-    def gla(self, q: int, k: int, v: int, decay: int, state: int, heads: int) -> int:
-        return _node(lib.mgq_graph_gla(self._h, q, k, v, decay, state, heads))
+    def gla(self, q: int, k: int, v: int, decay: int, state: int, heads: int, product_dtype: int = FMT_F32) -> int:
+        return _node(lib.mgq_graph_gla(self._h, q, k, v, decay, state, heads, product_dtype))
 
     def query_temperature(self, x: int, pos: int, coef: float, every: float) -> int:
         return _node(lib.mgq_graph_query_temperature(self._h, x, pos, coef, every))

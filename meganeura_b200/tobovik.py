@@ -165,7 +165,7 @@ class Tobovik(RowModel):
         n = m.heads * m.dim
         decay = g.lora_sigmoid_decay(low, self._mat(f"{p}.a2", n, self.lora_rank[p]), self._vec(f"{p}.a2.b", n), m.tau)
         state = g.parameter(f"l{i}.gla_state", [lib.mgq_gla_state_elements(m.heads, m.dim, m.vdim)])
-        o = g.gla(q, k, v, decay, state, m.heads)
+        o = g.gla(q, k, v, decay, state, m.heads, self._operand)
         return g.head_gate(o, gate, m.heads, self._vec(f"{p}.norm", m.vdim), self.cfg.eps, GATE_SILU, self._operand)
 
     @staticmethod
