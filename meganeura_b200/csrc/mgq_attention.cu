@@ -45,7 +45,63 @@ __global__ void cache_append_kernel(const float *x, CT *cache, const uint32_t *p
     if (slot < slots) cache[(size_t)slot * cols + (i - (size_t)row * cols)] = from_f32<CT>(x[i]);
 }
 
-// CTA = row x {query, key, value}.
+__device__ __forceinline__ void store4(float *p, const float4 &x) { *reinterpret_cast<float4 *>(p) = x; }
+__device__ __forceinline__ void store4(__half *p, const float4 &x)
+{
+    const __half2 a = __halves2half2(from_f32<__half>(x.x), from_f32<__half>(x.y)), b = __halves2half2(from_f32<__half>(x.z), from_f32<__half>(x.w));
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+}
+
+// CTA = row; widths in multiples of 4, at most 1024 * NV.
+template <typename CT, int NV>
+__global__ void __launch_bounds__(256) attention_inputs_vec_kernel(const __grid_constant__ AttentionInputs a)
+{
+    __shared__ float s_part[2][8];
+    const uint32_t t = threadIdx.x, row = blockIdx.x, nq = a.q_cols / 4, nk = a.k_cols / 4, nv = a.v_cols / 4;
+    float4 q[NV], k[NV], v[NV];
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint32_t p = a.pos[0] + row;
+    const float4 *qs = reinterpret_cast<const float4 *>(a.q + (size_t)row * a.q_cols), *ks = reinterpret_cast<const float4 *>(a.k + (size_t)row * a.k_cols),
+                 *vs = reinterpret_cast<const float4 *>(a.v + (size_t)row * a.v_cols);
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const uint32_t j = t + 256u * i;
+        q[i] = j < nq ? qs[j] : zero;
+        k[i] = j < nk ? ks[j] : zero;
+        v[i] = j < nv ? vs[j] : zero;
+    }
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        sq += q[i].x * q[i].x + q[i].y * q[i].y + q[i].z * q[i].z + q[i].w * q[i].w;
+        sk += k[i].x * k[i].x + k[i].y * k[i].y + k[i].z * k[i].z + k[i].w * k[i].w;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((t & 31u) == 0) { s_part[0][t >> 5] = sq; s_part[1][t >> 5] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; i++) { sq += s_part[0][i]; sk += s_part[1][i]; }
+    const float rq = 1.0f / sqrtf(sq / (float)a.q_cols + a.q_eps), rk = 1.0f / sqrtf(sk / (float)a.k_cols + a.k_eps), f = temperature(p, a.coef, a.every);
+    auto normed = [](const float4 &x, const float4 &w, float r, float offset, float f) {
+        return make_float4(x.x * r * (offset + w.x) * f, x.y * r * (offset + w.y) * f, x.z * r * (offset + w.z) * f, x.w * r * (offset + w.w) * f);
+    };
+    float *qd = a.q_out + (size_t)row * a.q_cols;
+    CT *kd = static_cast<CT *>(a.keys) + (size_t)p * a.k_cols, *vd = static_cast<CT *>(a.values) + (size_t)p * a.v_cols;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const uint32_t j = t + 256u * i;
+        if (j < nq) store4(qd + 4 * j, normed(q[i], __ldg(reinterpret_cast<const float4 *>(a.q_weight) + j), rq, a.q_offset, f));
+        if (p >= a.slots) continue;
+        if (j < nk) store4(kd + 4 * j, normed(k[i], __ldg(reinterpret_cast<const float4 *>(a.k_weight) + j), rk, a.k_offset, 1.f));
+        if (j < nv) store4(vd + 4 * j, v[i]);
+    }
+}
+
+// CTA = row x {query, key, value}; any width.
 template <typename CT>
 __global__ void __launch_bounds__(256) attention_inputs_kernel(const __grid_constant__ AttentionInputs a)
 {
@@ -504,6 +560,12 @@ int launch_cache_append(const float *x, void *cache, bool half, const uint32_t *
 int launch_attention_inputs(const AttentionInputs &a, void *stream)
 {
     cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const uint32_t widest = std::max(a.q_cols, std::max(a.k_cols, a.v_cols));
+    if ((a.q_cols | a.k_cols | a.v_cols) % 4 == 0 && widest <= 4096) {
+        if (widest <= 2048)
+            return a.half ? launch(attention_inputs_vec_kernel<__half, 2>, dim3(a.rows), dim3(256), 0, st, a) : launch(attention_inputs_vec_kernel<float, 2>, dim3(a.rows), dim3(256), 0, st, a);
+        return a.half ? launch(attention_inputs_vec_kernel<__half, 4>, dim3(a.rows), dim3(256), 0, st, a) : launch(attention_inputs_vec_kernel<float, 4>, dim3(a.rows), dim3(256), 0, st, a);
+    }
     if (a.half) return launch(attention_inputs_kernel<__half>, dim3(a.rows, 3), dim3(256), 0, st, a);
     return launch(attention_inputs_kernel<float>, dim3(a.rows, 3), dim3(256), 0, st, a);
 }

@@ -142,17 +142,9 @@ __device__ __forceinline__ void ldmatrix4_t(uint32_t addr, uint32_t (&r)[4])
 }
 __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
 {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-// a . b with both as sums of a high and a low part (the product of the low parts is below f32's rounding of the sum)
-__device__ __forceinline__ void mma_split(float (&c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0, uint32_t bh1, uint32_t bl0, uint32_t bl1)
-{
-    mma16816(c, ah, bl0, bl1);
-    mma16816(c, al, bh0, bh1);
-    mma16816(c, ah, bh0, bh1);
-}
-
 // CTA = head (x) x value columns (y), 16 per warp, x segment (z).
 template <int D>
 __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constant__ Chunks p)
@@ -254,18 +246,15 @@ __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constan
         float o[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};          // o^T: rows value columns, columns tokens
 #pragma unroll
         for (int j = 0; j < D / 16; j++) {
+            uint32_t sh[4], sl[4], qh[4], ql[4], kh[4], kl[4];
             if (outputs) {
-                uint32_t sh[4], sl[4], qh[4], ql[4];
                 split2(S[2 * j][0], S[2 * j][1], sh[0], sl[0]);
                 split2(S[2 * j][2], S[2 * j][3], sh[1], sl[1]);
                 split2(S[2 * j + 1][0], S[2 * j + 1][1], sh[2], sl[2]);
                 split2(S[2 * j + 1][2], S[2 * j + 1][3], sh[3], sl[3]);
                 ldmatrix4(base + q_off + j * 32, qh);
                 ldmatrix4(base + q_off + R::matrix + j * 32, ql);
-                mma_split(o[0], sh, sl, qh[0], qh[1], ql[0], ql[1]);
-                mma_split(o[1], sh, sl, qh[2], qh[3], ql[2], ql[3]);
             }
-            uint32_t kh[4], kl[4];
             ldmatrix4_t(base + k_off + j * 32, kh);
             ldmatrix4_t(base + k_off + R::matrix + j * 32, kl);
 #pragma unroll
@@ -273,7 +262,17 @@ __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constan
                 const float2 f = *reinterpret_cast<const float2 *>(rec + R::lam + (j * 16 + n * 8 + tq * 2) * 4);
                 float (&x)[4] = S[2 * j + n];
                 x[0] *= f.x; x[1] *= f.y; x[2] *= f.x; x[3] *= f.y;
-                mma_split(x, vh, vl, kh[2 * n], kh[2 * n + 1], kl[2 * n], kl[2 * n + 1]);
+            }
+            // high . low, low . high, high . high of four independent sums (low . low is below the rounding of the sum)
+#pragma unroll
+            for (int part = 0; part < 3; part++) {
+                const uint32_t (&qb)[4] = part == 0 ? ql : qh, (&kb)[4] = part == 0 ? kl : kh, (&sa)[4] = part == 1 ? sl : sh, (&va)[4] = part == 1 ? vl : vh;
+                if (outputs) {
+                    mma16816(o[0], sa, qb[0], qb[1]);
+                    mma16816(o[1], sa, qb[2], qb[3]);
+                }
+                mma16816(S[2 * j], va, kb[0], kb[1]);
+                mma16816(S[2 * j + 1], va, kb[2], kb[3]);
             }
         }
         if (!outputs) continue;
@@ -282,7 +281,9 @@ __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constan
             const uint8_t *a = rec + R::a + ((n * 8 + g) * kChunk + tq * 2) * 2;
             const uint32_t ah0 = *reinterpret_cast<const uint32_t *>(a), ah1 = *reinterpret_cast<const uint32_t *>(a + 16);
             const uint32_t al0 = *reinterpret_cast<const uint32_t *>(a + kChunk * kChunk * 2), al1 = *reinterpret_cast<const uint32_t *>(a + kChunk * kChunk * 2 + 16);
-            mma_split(o[n], vh, vl, ah0, ah1, al0, al1);
+            mma16816(o[n], vh, al0, al1);
+            mma16816(o[n], vl, ah0, ah1);
+            mma16816(o[n], vh, ah0, ah1);
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 const uint32_t row = c * kChunk + n * 8 + tq * 2 + (e & 1);

@@ -14,21 +14,46 @@ namespace mgq {
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;\n" ::: "memory"); }
 __device__ __forceinline__ void pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory"); }
 
+// cluster_y: CTAs along y that form a cluster.
 template <typename... Params, typename... Args>
-int launch(void (*kernel)(Params...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args... args)
+int launch_clustered(void (*kernel)(Params...), dim3 grid, dim3 block, uint32_t cluster_y, size_t smem, cudaStream_t stream, Args... args)
 {
     cudaLaunchConfig_t lc{};
     lc.gridDim = grid;
     lc.blockDim = block;
     lc.dynamicSmemBytes = smem;
     lc.stream = stream;
-    cudaLaunchAttribute attr[1];
+    cudaLaunchAttribute attr[2];
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
     attr[0].val.programmaticStreamSerializationAllowed = 1;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = 1;
+    attr[1].val.clusterDim.y = cluster_y;
+    attr[1].val.clusterDim.z = 1;
     lc.attrs = attr;
-    lc.numAttrs = 1;
+    lc.numAttrs = cluster_y > 1 ? 2 : 1;
     MGQ_CUDA(cudaLaunchKernelEx(&lc, kernel, static_cast<Params>(args)...));
     return MGQ_OK;
+}
+template <typename... Params, typename... Args>
+int launch(void (*kernel)(Params...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args... args)
+{
+    return launch_clustered(kernel, grid, block, 1, smem, stream, static_cast<Params>(args)...);
+}
+
+// All CTAs of the cluster: arrive and wait, shared-memory writes before are visible behind.
+__device__ __forceinline__ void cluster_sync()
+{
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;\n" ::: "memory");
+}
+// A float of the same shared variable in CTA `rank` of the cluster.
+__device__ __forceinline__ float cluster_load(const float *p, uint32_t rank)
+{
+    uint32_t addr;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(addr) : "r"((uint32_t)__cvta_generic_to_shared(p)), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
+    return v;
 }
 
 // Opts a kernel into more than 48 KB of shared memory, static part included (a no-op for the driver when repeated).

@@ -7,8 +7,9 @@
 // register arithmetic plus a short shuffle reduction; keys beyond `dim` are zero.
 //   scan_kernel  several tokens: CTA = head x a block of value columns (x a segment of a long portion),
 //                state in registers, the tokens' vectors staged through a double-buffered cp.async ring.
-//   step_kernel  one token: CTA = head; the decay projection (or the gates), the recurrence, the
-//                per-head norm and the output gate in one launch, state streamed once.
+//   step_kernel  one token: a cluster per head, its CTAs share out the value columns; the decay projection (or
+//                the gates), the recurrence, the per-head norm (the CTAs' sums of squares meet through distributed
+//                shared memory) and the output gate in one launch, state streamed once.
 #include <algorithm>
 
 #include "mgq_mixer.cuh"
@@ -859,7 +860,7 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const __grid_cons
 }
 
 // ---------------------------------------------------------------- one token: decay / gates, recurrence, head norm, gate
-constexpr uint32_t kStepThreads = 512, kStepCols = kStepThreads / 8;
+constexpr uint32_t kStepThreads = 512, kStepCols = kStepThreads / 8, kStepCluster = 8;
 
 template <int MODE, int RPT, typename OT>
 __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constant__ Scan p, const __grid_constant__ HeadGate hg,
@@ -867,8 +868,8 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
 {
     constexpr int KS = RPT * 8;
     extern __shared__ __align__(16) float smem[];        // q, k, w [KS] each; o [vdim]; the decay's low-rank input [rank]
-    __shared__ float s_part[kStepThreads / 32], s_gate[3];
-    const uint32_t t = threadIdx.x, head = blockIdx.x, ks = t & 7u, dim = p.dim, vdim = p.vdim, kp = pad4(dim);
+    __shared__ float s_part[kStepThreads / 32], s_gate[3], s_squares;
+    const uint32_t t = threadIdx.x, head = blockIdx.x, part = blockIdx.y, parts = gridDim.y, ks = t & 7u, dim = p.dim, vdim = p.vdim, kp = pad4(dim);
     float *sq = smem, *sk = sq + KS, *sw = sk + KS, *so = sw + KS, *s_low = so + vdim;
     float u[RPT], n[RPT];
 #pragma unroll
@@ -884,7 +885,9 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
         sk[i] = i < dim ? p.k[head * dim + i] : 0.f;
         sw[i] = 0.f;
     }
-    float *nrow = normalizer(p, p.state, head, 0);
+    // mlstm: every CTA reads and advances the copies of n and m that belong to its columns
+    const uint32_t blocks_per_part = kStepCols / block_cols(dim);
+    float *nrow = normalizer(p, p.state, head, part * blocks_per_part);
     if (MODE != kMlstm) {
         const __nv_bfloat16 *w2 = static_cast<const __nv_bfloat16 *>(d.w2);
         const uint32_t rank = d.rank;
@@ -913,7 +916,8 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
     float ss = 0.f, n_out[RPT];
 #pragma unroll
     for (int i = 0; i < RPT; i++) n_out[i] = 0.f;
-    for (uint32_t col = t / 8; col < (vdim + kStepCols - 1) / kStepCols * kStepCols; col += kStepCols) {
+    for (uint32_t c0 = part * kStepCols; c0 < vdim; c0 += parts * kStepCols) {
+        const uint32_t col = c0 + t / 8;
         const bool live = col < vdim;
         float *srow = p.state + ((size_t)head * vdim + (live ? col : 0)) * kp;
         float S[1][RPT], nn[RPT], out1[1], den;
@@ -934,19 +938,29 @@ __global__ void __launch_bounds__(kStepThreads) step_kernel(const __grid_constan
             if (ks == 0) { so[col] = out; ss = fmaf(out, out, ss); }
         }
     }
-    const float r = 1.0f / sqrtf(block_sum(ss, s_part) / (float)vdim + hg.eps);     // its barriers also publish so[] and order the reads of n and m
+    ss = block_sum(ss, s_part);                          // its barriers also publish so[] and order the reads of n and m
+    if (parts > 1) {
+        if (t == 0) s_squares = ss;
+        cluster_sync();
+        ss = 0.f;
+        for (uint32_t i = 0; i < parts; i++) ss += cluster_load(&s_squares, i);
+        cluster_sync();                                  // no CTA leaves while its sum may still be read
+    }
+    const float r = 1.0f / sqrtf(ss / (float)vdim + hg.eps);
     OT *dst = static_cast<OT *>(hg.out) + head * vdim;
     for (uint32_t j = t; j < vdim; j += kStepThreads) {
+        if (j / kStepCols % parts != part) continue;
         const float g = hg.gate[head * vdim + j], s = sigmoid_f(g);
         dst[j] = from_f32<OT>(so[j] * r * hg.weight[hg.shared ? j : head * vdim + j] * (hg.silu ? g * s : s));
     }
     if (MODE == kMlstm) {
         for (uint32_t blk = t / 8; blk < value_blocks(dim, vdim); blk += kStepCols) {
+            if (blk / blocks_per_part % parts != part) continue;
             float *nb = normalizer(p, p.state, head, blk);
             store_keys<RPT>(nb, ks, kp, n_out);
             if (ks == 0) nb[kp] = m_new;
         }
-    } else if (p.shift_state) {
+    } else if (p.shift_state && part == 0) {
         for (uint32_t j = head * kStepThreads + t; j < p.shift_width; j += p.heads * kStepThreads) p.shift_state[j] = p.shift_state[p.shift_width + j];
     }
 }
@@ -1002,12 +1016,14 @@ template <int MODE, int RPT>
 int launch_step_rpt(const Scan &p, const HeadGate &hg, const Decay &d, cudaStream_t stream)
 {
     const size_t smem = (size_t)(3 * RPT * 8 + p.vdim + d.rank) * sizeof(float);
+    const uint32_t parts = std::min(kStepCluster, (p.vdim + kStepCols - 1) / kStepCols);
+    const dim3 grid(p.heads, parts);
     if (hg.out_bf16) {
         if (int rc = allow_smem(step_kernel<MODE, RPT, __nv_bfloat16>, smem)) return rc;
-        return launch(step_kernel<MODE, RPT, __nv_bfloat16>, dim3(p.heads), dim3(kStepThreads), smem, stream, p, hg, d);
+        return launch_clustered(step_kernel<MODE, RPT, __nv_bfloat16>, grid, dim3(kStepThreads), parts, smem, stream, p, hg, d);
     }
     if (int rc = allow_smem(step_kernel<MODE, RPT, float>, smem)) return rc;
-    return launch(step_kernel<MODE, RPT, float>, dim3(p.heads), dim3(kStepThreads), smem, stream, p, hg, d);
+    return launch_clustered(step_kernel<MODE, RPT, float>, grid, dim3(kStepThreads), parts, smem, stream, p, hg, d);
 }
 
 template <int MODE>
