@@ -5,13 +5,15 @@
 //     o_t = S^T (L_t q_t) + sum_(s <= t) A_ts v_s,      A_ts = sum_d q_t k_s a_(s+1) .. a_t
 //     S'  = diag(L_16) S + sum_s (G_s k_s) v_s^T
 // Only products of decays appear, never a quotient, so nothing overflows however strong the decay is.
-//   gla_prepare_kernel  CTA = chunk x head: A, L q, G k and L_16 into a record that the next kernel copies as it is
+//   gla_prepare_kernel  CTA = chunk x head: the decays from their low-rank projection, then A, L q, G k and L_16
+//                       into a record that the next kernel copies as it is
 //   gla_chunks_kernel   a warp keeps S^T for 16 value columns and all keys in registers, as f32 accumulators of
 //                       mma.sync whose layout is also that of the products' left operand, and walks the chunks;
 //                       the records come through a ring of cp.async copies
 // State and sums are f32.  The products' operands (state, decayed queries and keys, A, values) enter as sums of two
-// bf16, three products each: 16 to 17 significant bits with the range of f32.  A long portion is cut into segments
-// that run in two launches, like in the token-by-token scan (mgq_mixer_ops.cu).
+// bf16, three products each: 16 to 17 significant bits with the range of f32.  A long portion is cut into segments:
+// a first pass leaves the end state of every segment but the last, each started from nothing, gla_combine_kernel
+// turns them into the segments' start states, and a second pass runs all segments with outputs.
 #include <algorithm>
 
 #include "mgq_mixer.cuh"
@@ -29,11 +31,12 @@ template <int D> struct Record {
 };
 
 struct Chunks {
-    const float *q, *k, *v, *w;
-    float *o, *state, *segments;
+    const float *q, *k, *v, *w;                          // w: decays, or null: from d
+    Decay d;
+    float *o, *state, *segments, *products;              // products: of a segment's decays, [segment][heads][D]
     uint8_t *records;
     uint32_t rows, heads, dim, vdim, chunks;
-    uint32_t seg_len, phase;                             // chunks per segment; 0: one pass, 1: end states, 2: outputs behind the first segment
+    uint32_t seg_len, segs, states_only;                 // chunks per segment; the first pass leaves end states only
     float qscale;
 };
 
@@ -56,13 +59,64 @@ __global__ void __launch_bounds__(256) gla_prepare_kernel(const __grid_constant_
     const uint32_t t = threadIdx.x, chunk = blockIdx.x, head = blockIdx.y, row0 = chunk * kChunk, kpitch = p.heads * p.dim;
     pdl_launch_dependents();
     pdl_wait();
-    for (uint32_t i = t; i < kChunk * D; i += 256) {
-        const uint32_t r = i / D, d = i % D;
-        const bool in = row0 + r < p.rows && d < p.dim;  // beyond the portion: nothing decays and nothing is added
-        const size_t at = (size_t)(row0 + r) * kpitch + head * p.dim + d;
-        sq[r * P + d] = in ? p.q[at] * p.qscale : 0.f;
-        sk[r * P + d] = in ? p.k[at] : 0.f;
-        sw[r * P + d] = in ? p.w[at] : 1.f;
+    // beyond the portion and beyond the head's channels: nothing decays and nothing is added
+    if (p.dim % 4 == 0) {
+#pragma unroll
+        for (uint32_t j = 0; j < (kChunk * D / 4 + 255) / 256; j++) {
+            const uint32_t i = t + 256 * j, r = i / (D / 4), d = i % (D / 4) * 4;
+            if (i >= kChunk * D / 4) break;
+            const bool in = row0 + r < p.rows && d < p.dim;
+            const size_t at = (size_t)(row0 + r) * kpitch + head * p.dim + d;
+            float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q;
+            if (in) { q = *reinterpret_cast<const float4 *>(p.q + at); k = *reinterpret_cast<const float4 *>(p.k + at); }
+            *reinterpret_cast<float4 *>(sq + r * P + d) = make_float4(q.x * p.qscale, q.y * p.qscale, q.z * p.qscale, q.w * p.qscale);
+            *reinterpret_cast<float4 *>(sk + r * P + d) = k;
+        }
+    } else {
+#pragma unroll 4
+        for (uint32_t i = t; i < kChunk * D; i += 256) {
+            const uint32_t r = i / D, d = i % D;
+            const bool in = row0 + r < p.rows && d < p.dim;
+            const size_t at = (size_t)(row0 + r) * kpitch + head * p.dim + d;
+            sq[r * P + d] = in ? p.q[at] * p.qscale : 0.f;
+            sk[r * P + d] = in ? p.k[at] : 0.f;
+        }
+    }
+    if (p.w) {
+#pragma unroll 4
+        for (uint32_t i = t; i < kChunk * D; i += 256) {
+            const uint32_t r = i / D, d = i % D;
+            const bool in = row0 + r < p.rows && d < p.dim;
+            sw[r * P + d] = in ? p.w[(size_t)(row0 + r) * kpitch + head * p.dim + d] : 1.f;
+        }
+    } else {
+        // thread = channel x a share of the tokens; the low-rank inputs lie where the partial sums of A go later
+        constexpr uint32_t GROUPS = 256 / D, PER = kChunk / GROUPS;
+        const uint32_t d = t % D, r0 = t / D * PER, ranks = p.d.rank;
+        float z[PER];
+        for (uint32_t j0 = 0; j0 < ranks; j0 += 128) {
+            const uint32_t nj = min(128u, ranks - j0);
+            __syncthreads();
+            for (uint32_t i = t; i < kChunk * nj; i += 256) {
+                const uint32_t r = i / nj, j = i % nj;
+                sa[r * 128 + j] = row0 + r < p.rows ? decay_input(p.d.low[(size_t)(row0 + r) * ranks + j0 + j], p.d.inv_tau) : 0.f;
+            }
+            __syncthreads();
+            if (d < p.dim) {
+                if (j0 == 0)
+#pragma unroll
+                    for (int i = 0; i < (int)PER; i++) z[i] = p.d.w0[head * p.dim + d];
+                const __nv_bfloat16 *w2 = static_cast<const __nv_bfloat16 *>(p.d.w2) + (size_t)(head * p.dim + d) * ranks + j0;
+#pragma unroll 8
+                for (uint32_t j = 0; j < nj; j++) {
+                    const float x = __bfloat162float(w2[j]);
+#pragma unroll
+                    for (int i = 0; i < (int)PER; i++) z[i] = fmaf(x, sa[(r0 + i) * 128 + j], z[i]);
+                }
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < (int)PER; i++) sw[(r0 + i) * P + d] = d < p.dim && row0 + r0 + i < p.rows ? decay_value(z[i], p.d.inv_tau) : 1.f;
     }
     __syncthreads();
     uint8_t *rec = p.records + ((size_t)head * p.chunks + chunk) * R::bytes;
@@ -151,11 +205,11 @@ __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constan
 {
     using R = Record<D>;
     extern __shared__ __align__(16) uint8_t ring[];      // kStages records
-    __shared__ float s_f[D];
+    __shared__ float s_f[D];                             // product of the decays so far (first pass)
     const uint32_t t = threadIdx.x, threads = blockDim.x, lane = t & 31u, warp = t >> 5, g = lane >> 2, tq = lane & 3u;
     const uint32_t head = blockIdx.x, v0 = (blockIdx.y * (threads >> 5) + warp) * 16, kp = (p.dim + 3u) & ~3u, vpitch = p.heads * p.vdim;
-    const uint32_t seg = p.phase == 2 ? blockIdx.z + 1 : blockIdx.z, c0 = seg * p.seg_len, c1 = min(c0 + p.seg_len, p.chunks);
-    const bool outputs = p.phase != 1 || seg == 0;
+    const uint32_t seg = blockIdx.z, c0 = seg * p.seg_len, c1 = min(c0 + p.seg_len, p.chunks);
+    const bool outputs = !p.states_only;
     const uint32_t vr[2] = {v0 + g, v0 + g + 8};         // this thread's value columns
     const bool live[2] = {vr[0] < p.vdim, vr[1] < p.vdim};
     pdl_launch_dependents();
@@ -193,44 +247,25 @@ __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constan
     for (int n = 0; n < D / 8; n++)
 #pragma unroll
         for (int e = 0; e < 4; e++) S[n][e] = 0.f;
-    if (seg == 0) {
+    if (seg == 0 || outputs) {                           // start state: the sequence's, or what the combination left
+        const bool own = seg == 0 && (p.segs == 1 || !outputs);
+        const uint32_t slot = seg == 0 ? p.segs - 1 : seg - 1, pitch = own ? kp : D;
+        const float *start = own ? p.state + (size_t)head * p.vdim * kp : p.segments + ((size_t)slot * p.heads + head) * p.vdim * D;
 #pragma unroll
         for (int n = 0; n < D / 8; n++)
 #pragma unroll
             for (int i = 0; i < 2; i++) {
                 const uint32_t d = n * 8 + tq * 2;
-                if (d < kp && live[i]) {
-                    const float2 x = *reinterpret_cast<const float2 *>(p.state + ((size_t)head * p.vdim + vr[i]) * kp + d);
+                if (d < pitch && live[i]) {
+                    const float2 x = *reinterpret_cast<const float2 *>(start + (size_t)vr[i] * pitch + d);
                     S[n][2 * i] = x.x; S[n][2 * i + 1] = x.y;
                 }
             }
-    } else if (outputs) {
-        for (uint32_t s = 0; s < seg; s++) {             // the end states of the segments before this one, put together in order
-            if (s > 0) {
-                for (uint32_t d = t; d < (uint32_t)D; d += threads) {
-                    float f = 1.f;
-#pragma unroll 8
-                    for (uint32_t c = s * p.seg_len; c < (s + 1) * p.seg_len; c++) f *= *reinterpret_cast<const float *>(records + (size_t)c * R::bytes + R::lam + d * 4);
-                    s_f[d] = f;
-                }
-            }
-            __syncthreads();
-            const float *end = p.segments + ((size_t)s * p.heads + head) * p.vdim * D;
-#pragma unroll
-            for (int n = 0; n < D / 8; n++) {
-                const uint32_t d = n * 8 + tq * 2;
-                const float2 f = s > 0 ? *reinterpret_cast<const float2 *>(s_f + d) : make_float2(0.f, 0.f);
-#pragma unroll
-                for (int i = 0; i < 2; i++) {
-                    const float2 x = live[i] ? *reinterpret_cast<const float2 *>(end + (size_t)vr[i] * D + d) : make_float2(0.f, 0.f);
-                    S[n][2 * i] = fmaf(f.x, S[n][2 * i], x.x);
-                    S[n][2 * i + 1] = fmaf(f.y, S[n][2 * i + 1], x.y);
-                }
-            }
-            __syncthreads();
-        }
     }
 
+    const bool product = !outputs && blockIdx.y == 0;
+    if (product)
+        for (uint32_t d = t; d < (uint32_t)D; d += threads) s_f[d] = 1.f;      // a thread only ever touches its own entries
     const uint32_t q_off = R::ql + (((lane & 7u) + (lane >> 4) * 8) * R::pitch + ((lane >> 3) & 1u) * 8) * 2;
     const uint32_t k_off = (((lane & 7u) + ((lane >> 3) & 1u) * 8) * R::pitch + (lane >> 4) * 8) * 2;
     for (uint32_t c = c0; c < c1; c++) {
@@ -275,6 +310,8 @@ __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constan
                 mma16816(S[2 * j + 1], va, kb[2], kb[3]);
             }
         }
+        if (product)
+            for (uint32_t d = t; d < (uint32_t)D; d += threads) s_f[d] *= *reinterpret_cast<const float *>(rec + R::lam + d * 4);
         if (!outputs) continue;
 #pragma unroll
         for (int n = 0; n < 2; n++) {                    // tokens n * 8 + g as columns, keys of the chunk as the sum
@@ -291,8 +328,9 @@ __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constan
             }
         }
     }
-    const bool last = c1 == p.chunks;
-    if (p.phase == 2 && !last) return;                   // later segments may still be reading this one's end state
+    if (outputs && c1 != p.chunks) return;
+    if (product)
+        for (uint32_t d = t; d < (uint32_t)D; d += threads) p.products[((size_t)seg * p.heads + head) * D + d] = s_f[d];
 #pragma unroll
     for (int n = 0; n < D / 8; n++)
 #pragma unroll
@@ -300,9 +338,37 @@ __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constan
             const uint32_t d = n * 8 + tq * 2;
             if (!live[i]) continue;
             const float2 x = make_float2(S[n][2 * i], S[n][2 * i + 1]);
-            if (!last)       *reinterpret_cast<float2 *>(p.segments + (((size_t)seg * p.heads + head) * p.vdim + vr[i]) * D + d) = x;
+            if (!outputs)    *reinterpret_cast<float2 *>(p.segments + (((size_t)seg * p.heads + head) * p.vdim + vr[i]) * D + d) = x;
             else if (d < kp) *reinterpret_cast<float2 *>(p.state + ((size_t)head * p.vdim + vr[i]) * kp + d) = x;
         }
+}
+
+// End states of segments that started from nothing (the first one: from the state) -> states behind them, in place.
+// The last slot receives a copy of the sequence's state, which the last segment of the second pass overwrites.
+// CTA = head x kCombineCols value columns; thread = 4 keys of a share of the columns.
+constexpr uint32_t kCombineCols = 16;
+template <int D>
+__global__ void __launch_bounds__(256) gla_combine_kernel(const __grid_constant__ Chunks p)
+{
+    const uint32_t t = threadIdx.x, head = blockIdx.x, v0 = blockIdx.y * kCombineCols;
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t step = (size_t)p.heads * p.vdim * D;
+    const uint32_t kp = (p.dim + 3u) & ~3u;
+    for (uint32_t i = t; i < kCombineCols * D / 4; i += 256) {
+        const uint32_t v = v0 + i / (D / 4), d = i % (D / 4) * 4;
+        if (v >= p.vdim) break;
+        float *at = p.segments + ((size_t)head * p.vdim + v) * D + d;
+        float4 S = *reinterpret_cast<const float4 *>(at);
+        *reinterpret_cast<float4 *>(at + (p.segs - 1) * step) =
+            d < kp ? *reinterpret_cast<const float4 *>(p.state + ((size_t)head * p.vdim + v) * kp + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+        for (uint32_t s = 1; s + 1 < p.segs; s++) {
+            const float4 x = *reinterpret_cast<const float4 *>(at + s * step), f = *reinterpret_cast<const float4 *>(p.products + ((size_t)s * p.heads + head) * D + d);
+            S = make_float4(fmaf(f.x, S.x, x.x), fmaf(f.y, S.y, x.y), fmaf(f.z, S.z, x.z), fmaf(f.w, S.w, x.w));
+            *reinterpret_cast<float4 *>(at + s * step) = S;
+        }
+    }
 }
 
 uint32_t padded(uint32_t dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
@@ -314,10 +380,10 @@ size_t record_bytes(uint32_t dim)
     return d == 32 ? Record<32>::bytes : d == 64 ? Record<64>::bytes : d == 128 ? Record<128>::bytes : Record<256>::bytes;
 }
 
-// Chunks per segment; all of them: one pass.  Two launches pay from three segments on.
+// Chunks per segment; all of them: one pass.  Two passes pay from three segments on.
 uint32_t segment_chunks(uint32_t chunks, uint32_t heads, uint32_t vdim)
 {
-    const uint32_t w = warps_for(vdim), ctas = heads * ((vdim + 16 * w - 1) / (16 * w)), want = std::min(kMaxSegs, 148u / ctas + 1);
+    const uint32_t w = warps_for(vdim), ctas = heads * ((vdim + 16 * w - 1) / (16 * w)), want = std::min(kMaxSegs, 148u / ctas);
     if (want < 3 || chunks < 12) return chunks;
     const uint32_t len = std::max(4u, (chunks + want - 1) / want);
     return (chunks + len - 1) / len < 3 ? chunks : len;
@@ -326,25 +392,21 @@ uint32_t segment_chunks(uint32_t chunks, uint32_t heads, uint32_t vdim)
 template <int D>
 int launch_sized(Chunks p, cudaStream_t st)
 {
-    const size_t prep = (size_t)(3 * kChunk * (D + 4) + std::min(D / 4, 16) * kChunk * kChunk) * 4, smem = (size_t)kStages * Record<D>::bytes;
+    const size_t prep = (size_t)(3 * kChunk * (D + 4) + std::max(std::min(D / 4, 16) * kChunk * kChunk, kChunk * 128)) * 4, smem = (size_t)kStages * Record<D>::bytes;
     if (int rc = allow_smem(gla_prepare_kernel<D>, prep)) return rc;
     if (int rc = allow_smem(gla_chunks_kernel<D>, smem)) return rc;
     if (int rc = launch(gla_prepare_kernel<D>, dim3(p.chunks, p.heads), dim3(256), prep, st, p)) return rc;
-    const uint32_t w = warps_for(p.vdim), segs = (p.chunks + p.seg_len - 1) / p.seg_len;
-    dim3 grid(p.heads, (p.vdim + 16 * w - 1) / (16 * w), 1);
-    if (segs == 1) {
-        gla_chunks_kernel<D><<<grid, w * 32, smem, st>>>(p);
-        MGQ_CUDA(cudaGetLastError());
-        return MGQ_OK;
+    const uint32_t w = warps_for(p.vdim);
+    dim3 grid(p.heads, (p.vdim + 16 * w - 1) / (16 * w), p.segs);
+    if (p.segs > 1) {
+        grid.z = p.segs - 1;
+        p.states_only = 1;
+        if (int rc = launch(gla_chunks_kernel<D>, grid, dim3(w * 32), smem, st, p)) return rc;
+        if (int rc = launch(gla_combine_kernel<D>, dim3(p.heads, (p.vdim + kCombineCols - 1) / kCombineCols), dim3(256), 0, st, p)) return rc;
+        grid.z = p.segs;
+        p.states_only = 0;
     }
-    grid.z = segs - 1;
-    p.phase = 1;
-    gla_chunks_kernel<D><<<grid, w * 32, smem, st>>>(p);
-    MGQ_CUDA(cudaGetLastError());
-    p.phase = 2;
-    gla_chunks_kernel<D><<<grid, w * 32, smem, st>>>(p);
-    MGQ_CUDA(cudaGetLastError());
-    return MGQ_OK;
+    return launch(gla_chunks_kernel<D>, grid, dim3(w * 32), smem, st, p);
 }
 
 }  // namespace
@@ -353,7 +415,7 @@ size_t gla_chunks_workspace(uint32_t max_rows, uint32_t heads, uint32_t dim, uin
 {
     if (max_rows < kPrefillRows) return 0;
     const size_t chunks = (max_rows + kChunk - 1) / kChunk;
-    return align256(chunks * heads * record_bytes(dim)) + (size_t)(kMaxSegs - 1) * heads * vdim * padded(dim) * 4;
+    return align256(chunks * heads * record_bytes(dim)) + (size_t)kMaxSegs * heads * (vdim + 1) * padded(dim) * 4;
 }
 
 int launch_gla_chunks(const ChannelDecay &a, void *stream)
@@ -361,11 +423,13 @@ int launch_gla_chunks(const ChannelDecay &a, void *stream)
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     if (a.u || a.dim > kMaxStateDim || !a.workspace) return fail(MGQ_ERR_STATE, "gla chunks: not this recurrence");
     Chunks p{};
-    p.q = a.q; p.k = a.k; p.v = a.v; p.w = a.d.out; p.o = a.o; p.state = a.state;
+    p.q = a.q; p.k = a.k; p.v = a.v; p.w = a.decay_pending ? nullptr : a.d.out; p.d = a.d; p.o = a.o; p.state = a.state;
     p.rows = a.rows; p.heads = a.heads; p.dim = a.dim; p.vdim = a.vdim; p.chunks = (a.rows + kChunk - 1) / kChunk;
     p.records = static_cast<uint8_t *>(a.workspace);
     p.segments = reinterpret_cast<float *>(p.records + align256((size_t)p.chunks * a.heads * record_bytes(a.dim)));
+    p.products = p.segments + (size_t)kMaxSegs * a.heads * a.vdim * padded(a.dim);
     p.seg_len = segment_chunks(p.chunks, a.heads, a.vdim);
+    p.segs = (p.chunks + p.seg_len - 1) / p.seg_len;
     p.qscale = (float)(1.0 / sqrt((double)a.dim));
     switch (padded(a.dim)) {
         case 32: return launch_sized<32>(p, st);

@@ -80,6 +80,13 @@ struct Decay {
     float inv_tau;
 };
 int launch_decay(const Decay &a, void *stream);
+__device__ __forceinline__ float log_sigmoid(float z) { return z < 0.f ? z - log1pf(expf(z)) : -log1pf(expf(-z)); }
+__device__ __forceinline__ float decay_input(float low, float inv_tau) { return inv_tau == 0.f ? tanhf(low) : low; }
+__device__ __forceinline__ float decay_value(float z, float inv_tau)
+{
+    if (inv_tau == 0.f) return expf(-expf(z));
+    return expf((fminf(z, 0.f) - logf(1.0f + expf(-fabsf(z)))) * inv_tau);       // close to 1 only the absolute error of the logarithm counts
+}
 
 // Recurrences with a decay per key channel.  q, k, d.out [rows, heads * dim], v, o [rows, heads * vdim].
 //   u set (RWKV-style):        o = (S + diag(u) k v^T)^T q, then S = diag(decay) S + k v^T
@@ -93,6 +100,7 @@ struct ChannelDecay {
     void *workspace;                       // scan_workspace bytes, or null (long portions then run in one piece)
     bool split_products;                   // gated linear, kPrefillRows or more rows: chunks on the tensor cores (mgq_gla_chunks.cu),
                                            // whose workspace is gla_chunks_workspace bytes
+    bool decay_pending;                    // d.out is not computed yet (only with that form, which computes the decay itself)
 };
 size_t channel_decay_state_elements(uint32_t heads, uint32_t dim, uint32_t vdim);
 int launch_channel_decay_scan(const ChannelDecay &a, void *stream);

@@ -433,10 +433,6 @@ __global__ void __launch_bounds__(256) head_gate_vec_kernel(const float *o, cons
 }
 
 // ---------------------------------------------------------------- decays, 64 rows x 64 channels per CTA
-__device__ __forceinline__ float log_sigmoid(float z) { return z < 0.f ? z - log1pf(expf(z)) : -log1pf(expf(-z)); }
-__device__ __forceinline__ float decay_input(float low, float inv_tau) { return inv_tau == 0.f ? tanhf(low) : low; }
-__device__ __forceinline__ float decay_value(float z, float inv_tau) { return inv_tau == 0.f ? expf(-expf(z)) : expf(log_sigmoid(z) * inv_tau); }
-
 constexpr uint32_t kDecayTile = 64, kDecayK = 16;
 __global__ void __launch_bounds__(256) decay_kernel(const __grid_constant__ Decay a)
 {

@@ -1889,7 +1889,9 @@ static int run_mixer(mgq_session *s, const Dispatch &d)
         a.shift_width = o.inputs[6] >= 0 ? (uint32_t)(s->nodes[o.inputs[6]].elements() / 2) : 0;
         if (!fused) return mgq::launch_channel_decay_scan(a, s->stream);
         if (rows == 1) return mgq::launch_channel_decay_step(a, hg, s->stream);
-        if (int rc = mgq::launch_decay(a.d, s->stream)) return rc;
+        a.decay_pending = a.split_products && rows >= mgq::kPrefillRows;
+        if (!a.decay_pending)
+            if (int rc = mgq::launch_decay(a.d, s->stream)) return rc;
         if (int rc = mgq::launch_channel_decay_scan(a, s->stream)) return rc;
         return mgq::launch_head_gate(a.o, hg, rows, o.at[0], o.at[2], s->stream);
     }
