@@ -10,8 +10,9 @@
 //   gla_chunks_kernel   a warp keeps S^T for 16 value columns and all keys in registers, as f32 accumulators of
 //                       mma.sync whose layout is also that of the products' left operand, and walks the chunks;
 //                       the records come through a ring of cp.async copies
-// State and sums are f32.  The products' operands (state, decayed queries and keys, A, values) enter as sums of two
-// bf16, three products each: 16 to 17 significant bits with the range of f32.  A long portion is cut into segments:
+// State, decays and sums are f32.  Where the state is read it enters as the sum of three bf16, i.e. with all its
+// bits; the decayed queries and keys, A and the values as sums of two, three products each: 16 to 17 significant bits
+// of numbers whose factors are projections, with the range of f32.  A long portion is cut into segments:
 // a first pass leaves the end state of every segment but the last, each started from nothing, gla_combine_kernel
 // turns them into the segments' start states, and a second pass runs all segments with outputs.
 #include <algorithm>
@@ -47,6 +48,13 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t &hi, uint32_t 
     const __nv_bfloat162 l = __floats2bfloat162_rn(x - f.x, y - f.y);
     hi = *reinterpret_cast<const uint32_t *>(&h);
     lo = *reinterpret_cast<const uint32_t *>(&l);
+}
+__device__ __forceinline__ void split3(float x, float y, uint32_t &hi, uint32_t &mid, uint32_t &lo)
+{
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    const float2 f = __bfloat1622float2(h);
+    hi = *reinterpret_cast<const uint32_t *>(&h);
+    split2(x - f.x, y - f.y, mid, lo);
 }
 
 template <int D>
@@ -281,12 +289,12 @@ __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constan
         float o[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};          // o^T: rows value columns, columns tokens
 #pragma unroll
         for (int j = 0; j < D / 16; j++) {
-            uint32_t sh[4], sl[4], qh[4], ql[4], kh[4], kl[4];
+            uint32_t sh[4], sm[4], sl[4], qh[4], ql[4], kh[4], kl[4];
             if (outputs) {
-                split2(S[2 * j][0], S[2 * j][1], sh[0], sl[0]);
-                split2(S[2 * j][2], S[2 * j][3], sh[1], sl[1]);
-                split2(S[2 * j + 1][0], S[2 * j + 1][1], sh[2], sl[2]);
-                split2(S[2 * j + 1][2], S[2 * j + 1][3], sh[3], sl[3]);
+                split3(S[2 * j][0], S[2 * j][1], sh[0], sm[0], sl[0]);
+                split3(S[2 * j][2], S[2 * j][3], sh[1], sm[1], sl[1]);
+                split3(S[2 * j + 1][0], S[2 * j + 1][1], sh[2], sm[2], sl[2]);
+                split3(S[2 * j + 1][2], S[2 * j + 1][3], sh[3], sm[3], sl[3]);
                 ldmatrix4(base + q_off + j * 32, qh);
                 ldmatrix4(base + q_off + R::matrix + j * 32, ql);
             }
@@ -298,14 +306,16 @@ __global__ void __launch_bounds__(256, 1) gla_chunks_kernel(const __grid_constan
                 float (&x)[4] = S[2 * j + n];
                 x[0] *= f.x; x[1] *= f.y; x[2] *= f.x; x[3] *= f.y;
             }
-            // high . low, low . high, high . high of four independent sums (low . low is below the rounding of the sum)
+            // small products first; the sums are independent of each other
 #pragma unroll
-            for (int part = 0; part < 3; part++) {
-                const uint32_t (&qb)[4] = part == 0 ? ql : qh, (&kb)[4] = part == 0 ? kl : kh, (&sa)[4] = part == 1 ? sl : sh, (&va)[4] = part == 1 ? vl : vh;
+            for (int part = 0; part < 5; part++) {
+                const uint32_t (&sa)[4] = part == 0 ? sl : part == 1 || part == 3 ? sm : sh, (&qb)[4] = part == 1 || part == 2 ? ql : qh;
                 if (outputs) {
                     mma16816(o[0], sa, qb[0], qb[1]);
                     mma16816(o[1], sa, qb[2], qb[3]);
                 }
+                if (part >= 3) continue;
+                const uint32_t (&va)[4] = part == 1 ? vl : vh, (&kb)[4] = part == 0 ? kl : kh;
                 mma16816(S[2 * j], va, kb[0], kb[1]);
                 mma16816(S[2 * j + 1], va, kb[2], kb[3]);
             }
