@@ -28,7 +28,7 @@ def _layers(kind, ff, wkv, mlstm, latent):
 def _tobovik_layers(kind, ff, left, right, gla):
     out = []
     for k in kind:
-        m = dict(type="gla", mixer=dict(gla)) if k == "g" else dict(type="parallel", mixer=dict(left=left, right=right, left_scale=0.8, right_scale=0.9))
+        m = dict(type="gla", mixer=dict(gla)) if k == "g" else dict(type="parallel", mixer=dict(left=left, right=right, left_scale=0.7, right_scale=1.0))
         out.append(dict(m, mlp={"kind": "dense", "ff": ff}))
     return out
 
